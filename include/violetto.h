@@ -47,6 +47,7 @@ typedef struct {
     uint32_t flags;            /* VLT_FLAG_* */
 } VltEngineConfig;
 #define VLT_FLAG_HOST_ONLY 1u /* plan only: no device memory, steps cannot run */
+#define VLT_FLAG_FP32 2u      /* everything in 32-bit (model folders of the Lonasun architecture; others refuse it) */
 
 /* engine/src/engine.rs:59-95 `Tuning`. The reference's Apple-GPU knobs (gpu_cores,
  * splitk_target, decode_split, verify_ki) are replaced by B200 ones; the rows policy is kept. 0 = default. */
@@ -109,7 +110,8 @@ const char* vlt_last_error(void);
 
 /* Engine::new, engine/src/engine.rs:221-250. `tuning` may be NULL. The weight file is a plain decoder's (its `meta` tensor
  * describes it: the benchmark's models) or one of the reference's own architecture as tools/convert.py:64-114 writes it (no
- * `meta`; engine/src/model.rs:6-20, with the shapes read off the file). */
+ * `meta`; engine/src/model.rs:6-20, with the shapes read off the file). A folder with config.json and model.safetensors is
+ * loaded by the architecture config.json names (Lonasun; nothing in the reference corresponds to it). */
 int vlt_engine_new(const char* weights_path, const VltEngineConfig* cfg, const VltTuning* tuning, VltEngine** out);
 /* Drop for Engine. */
 void vlt_engine_free(VltEngine* e);
@@ -123,16 +125,21 @@ uint32_t vlt_seq_len(VltEngine* e, uint32_t seq);
 int vlt_seq_set_sampling(VltEngine* e, uint32_t seq, const VltSampling* s);
 /* Engine::step, engine.rs:310-314: one synchronous step of CPU-fed runs. */
 int vlt_step(VltEngine* e, const VltRun* runs, uint32_t n_runs, const VltStepOptions* opts, VltStepOutput* out);
+/* The same with each run's own head rows: want[i] lists n_want[i] of run i's tokens by their place in the run (opts->head is
+ * not read). The reference takes none, the last or all of a run's rows (engine.rs:140-150). */
+int vlt_step_rows(VltEngine* e, const VltRun* runs, uint32_t n_runs, const uint32_t* const* want, const uint32_t* n_want, const VltStepOptions* opts, VltStepOutput* out);
 /* Engine::step_capture, engine.rs:318-355, with LayerCapture, engine.rs:175-188: a synchronous step that stops after
  * every layer and hands that layer's intermediates (host memory, valid during the call) to `fn`: n rows each of
  * resid_in [d_model] (the residual stream entering the layer), attn_in [d_model] (its RMS-normed rows), qkv [qkv_width]
  * (q | k | v after the folded norm and RoPE, fp32: before the rounding to bf16 and q's softmax scale), sdpa_out
  * [attn_width] (the attention's output), attn_out [d_model] (the o projection's output before the residual add), mlp_in
  * [d_model] (the RMS-normed stream after attention), mlp_out [d_model] (the down projection's output before the residual
- * add); resid_base is the reference's MUDD base (NULL for a plain decoder). */
+ * add); resid_base is the reference's MUDD base (NULL for a plain decoder). A Lonasun model hands out resid_in, sdpa_out (the
+ * gated attention, attn_width columns) and resid_out (the stream leaving the layer run); the others are NULL there, and
+ * resid_out is NULL for a plain decoder. */
 typedef struct {
     uint32_t layer, n, d_model, qkv_width, attn_width;
-    const float *resid_in, *attn_in, *qkv, *sdpa_out, *attn_out, *mlp_in, *mlp_out, *resid_base;
+    const float *resid_in, *attn_in, *qkv, *sdpa_out, *attn_out, *mlp_in, *mlp_out, *resid_base, *resid_out;
 } VltLayerCapture;
 typedef void (*VltCaptureFn)(const VltLayerCapture* layer, void* user);
 int vlt_step_capture(VltEngine* e, const VltRun* runs, uint32_t n_runs, const VltStepOptions* opts, VltCaptureFn fn, void* user, VltStepOutput* out);

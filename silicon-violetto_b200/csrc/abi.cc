@@ -73,6 +73,7 @@ int vlt_engine_new(const char* weights_path, const VltEngineConfig* cfg, const V
         c.max_head_rows = cfg->max_head_rows;
         c.device = cfg->device_ordinal;
         c.host_only = (cfg->flags & VLT_FLAG_HOST_ONLY) != 0;
+        c.fp32 = (cfg->flags & VLT_FLAG_FP32) != 0;
         Tuning t;
         if (tuning) {
             if (tuning->spec_tokens) t.spec_tokens = tuning->spec_tokens;
@@ -118,7 +119,7 @@ int vlt_model_desc(VltEngine* e, VltModelDesc* out) {
     return guard([&] {
         const Engine& en = eng(e);
         const ModelDesc& m = en.model.md;
-        *out = VltModelDesc{m.n_layers, m.d, m.n_heads, m.n_kv, m.hd, m.ffn, m.vocab, m.vocab_real, m.page, m.eps, m.attn_scale, en.model.layers[0].qkv.int8 ? 1u : 0u};
+        *out = VltModelDesc{m.n_layers, m.d, m.n_heads, m.n_kv, m.hd, m.ffn, m.vocab, m.vocab_real, m.page, m.eps, m.attn_scale, !en.model.layers.empty() && en.model.layers[0].qkv.int8 ? 1u : 0u};
     });
 }
 
@@ -150,18 +151,35 @@ static void fill_output(Engine& en, const StepOutput& r, VltStepOutput* out) {
     out->gpu_seconds = r.gpu_seconds;
 }
 
+static void step_with(VltEngine* e, const VltRun* runs, uint32_t n_runs, const uint32_t* const* want, const uint32_t* n_want, const VltStepOptions* opts, VltStepOutput* out) {
+    Engine& en = eng(e);
+    no_step_in_flight(e);
+    std::vector<PlanRun> rs;
+    for (uint32_t i = 0; i < n_runs; i++) {
+        for (uint32_t j = 0; j < runs[i].n_tokens; j++)
+            if (runs[i].tokens[j] >= en.model.md.vocab) throw Error("token id out of range");  // engine.rs:346-348
+        if (n_want) rs.push_back(PlanRun{runs[i].seq, runs[i].tokens, runs[i].n_tokens, Rows::Listed, false, want[i], n_want[i]});
+        else rs.push_back(PlanRun{runs[i].seq, runs[i].tokens, runs[i].n_tokens, Rows(opts->head), false});
+    }
+    StepOptions o{n_want ? Rows::Listed : Rows(opts->head), Rows(opts->hidden), opts->read_logits != 0, opts->read_taps != 0};
+    fill_output(en, en.step(rs, o), out);
+}
+static void no_listed_rows(uint32_t r) {
+    if (r > VLT_ROWS_ALL) throw Error("unknown rows option " + std::to_string(r));
+}
+
 int vlt_step(VltEngine* e, const VltRun* runs, uint32_t n_runs, const VltStepOptions* opts, VltStepOutput* out) {
     return guard([&] {
-        Engine& en = eng(e);
-        no_step_in_flight(e);
-        std::vector<PlanRun> rs;
-        for (uint32_t i = 0; i < n_runs; i++) {
-            for (uint32_t j = 0; j < runs[i].n_tokens; j++)
-                if (runs[i].tokens[j] >= en.model.md.vocab) throw Error("token id out of range");  // engine.rs:346-348
-            rs.push_back(PlanRun{runs[i].seq, runs[i].tokens, runs[i].n_tokens, Rows(opts->head), false});
-        }
-        StepOptions o{Rows(opts->head), Rows(opts->hidden), opts->read_logits != 0, opts->read_taps != 0};
-        fill_output(en, en.step(rs, o), out);
+        no_listed_rows(opts->head);
+        no_listed_rows(opts->hidden);
+        step_with(e, runs, n_runs, nullptr, nullptr, opts, out);
+    });
+}
+int vlt_step_rows(VltEngine* e, const VltRun* runs, uint32_t n_runs, const uint32_t* const* want, const uint32_t* n_want, const VltStepOptions* opts, VltStepOutput* out) {
+    return guard([&] {
+        if (!want || !n_want) throw Error("vlt_step_rows: null argument");
+        no_listed_rows(opts->hidden);
+        step_with(e, runs, n_runs, want, n_want, opts, out);
     });
 }
 
@@ -183,7 +201,8 @@ int vlt_step_capture(VltEngine* e, const VltRun* runs, uint32_t n_runs, const Vl
         StepOptions o{Rows(opts->head), Rows(opts->hidden), opts->read_logits != 0, opts->read_taps != 0};
         const ModelDesc& md = en.model.md;
         fill_output(en, en.step_capture(rs, o, [&](const LayerCapture& c) {
-            const VltLayerCapture v{c.layer, c.n, md.d, md.qkv_w(), md.n_heads * md.hd, c.resid_in, c.attn_in, c.qkv, c.sdpa_out, c.attn_out, c.mlp_in, c.mlp_out, nullptr};
+            const VltLayerCapture v{c.layer, c.n, md.d, md.qkv_w(), c.attn_width ? c.attn_width : md.n_heads * md.hd, c.resid_in, c.attn_in, c.qkv, c.sdpa_out, c.attn_out,
+                                    c.mlp_in, c.mlp_out, nullptr, c.resid_out};
             fn(&v, user);
         }), out);
     });

@@ -15,14 +15,21 @@ void Sampling::check() const {
 }
 
 // ------------------------------------------------------------------ KV cache
-void KvCache::init(const EngineConfig& cfg, const ModelDesc& md, uint32_t n_layers, bool with_pool) {
-    page = md.page;
+void KvCache::init(const EngineConfig& cfg, uint32_t page_size, std::vector<KvShape> layers, uint32_t elem_bytes, bool with_pool) {
+    page = page_size;
     n_pages = (cfg.global_kv_tokens + page - 1) / page;
     max_pages = (cfg.max_seq_len + page - 1) / page;
-    const size_t bytes = size_t(n_layers) * n_pages * page * md.n_kv * md.hd * 2;
+    shapes = std::move(layers);
+    size_t ks = 0, vs = 0;
+    for (const KvShape& l : shapes) {
+        k_off.push_back(ks);
+        v_off.push_back(vs);
+        ks += size_t(n_pages) * page * l.n_kv * l.dk;
+        vs += size_t(n_pages) * page * l.n_kv * l.dv;
+    }
     if (with_pool) {
-        k.alloc(bytes, false);
-        v.alloc(bytes, false);
+        k.alloc(ks * elem_bytes, false);
+        v.alloc(vs * elem_bytes, false);
     }
     page_table.alloc(size_t(cfg.max_seqs) * max_pages * 4, !with_pool);
     free_pages.clear();
@@ -123,7 +130,17 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
     if (cfg.max_seqs == 0 || cfg.max_step_tokens == 0 || cfg.max_chunk == 0 || cfg.max_head_rows == 0) throw Error("engine config: zero capacity");
     model.load(weights, cfg.host_only);
     const ModelDesc& md = model.md;
-    kv.init(cfg, md, model.limite ? model.n_global : md.n_layers, !cfg.host_only);  // (the reference's architecture pages its global layers only)
+    if (cfg.fp32 && !model.lonasun) throw Error(weights + ": this architecture has no fp32 path");
+    if (model.lonasun) {
+        std::vector<KvShape> shapes;
+        for (const LayerRun& r : model.lonasun->runs) {
+            const GatedAttention& m = model.lonasun->layers[r.layer].mix;
+            shapes.push_back({m.kv_heads, m.dim, m.vdim});
+        }
+        kv.init(cfg, md.page, shapes, cfg.fp32 ? 4 : 2, !cfg.host_only);
+    } else {
+        kv.init(cfg, md.page, std::vector<KvShape>(model.limite ? model.n_global : md.n_layers, {md.n_kv, md.hd, md.hd}), 2, !cfg.host_only);  // (the reference's architecture pages its global layers only)
+    }
     seqs.resize(cfg.max_seqs);
     for (auto& st : sets) st.init(cfg);
 
@@ -131,23 +148,25 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
     const size_t n = cfg.max_step_tokens, hr = cfg.max_head_rows, ms = cfg.max_seqs;
     auto f = [&](Buffer& b, size_t floats) { b.alloc(floats * 4, ho); };
     if (!ho) {
+        const size_t n16 = (n + 15) / 16 * 16, hr16 = (hr + 15) / 16 * 16;
         f(s.h, n * md.d);
-        f(s.qkv, n * md.qkv_w());
-        f(s.attn, n * md.n_heads * md.hd);
-        f(s.act, n * md.ffn);
-        f(s.part, n * 16 * md.n_heads * ATTN_PART);  // buffers.rs:9: 16 partial slots per token of a full step
         f(s.hfin_head, hr * md.d);
         f(s.hfin_all, n * md.d);
         f(s.logits, hr * md.vocab);
         f(s.inv, n);
-        const size_t n16 = (n + 15) / 16 * 16, hr16 = (hr + 15) / 16 * 16;
         s.h_b.alloc(n16 * md.d * 2, false);
+        s.hfin_b.alloc(hr16 * md.d * 2, false);
+        f(s.inv_head, hr);
+        if (!model.lonasun) {  // (its layers' scratch is its own)
+        f(s.qkv, n * md.qkv_w());
+        f(s.attn, n * md.n_heads * md.hd);
+        f(s.act, n * md.ffn);
+        f(s.part, n * 16 * md.n_heads * ATTN_PART);  // buffers.rs:9: 16 partial slots per token of a full step
         s.attn_b.alloc(n16 * md.n_heads * md.hd * 2, false);
         s.q_b.alloc(n16 * md.n_heads * md.hd * 2, false);
         s.ssq.alloc(size_t(md.d / 128 + 1) * n16 * 4, false);
         s.act_b.alloc(n16 * md.ffn * 2, false);
-        s.hfin_b.alloc(hr16 * md.d * 2, false);
-        f(s.inv_head, hr);
+        }
     }
     f(s.meta, 2 * n);
     f(s.lens, ms);
@@ -169,7 +188,10 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
     std::vector<GenState> open(ms, gen_open());
     s.gen.write_vec(0, open);
 
-    if (!ho) {
+    if (!ho && model.lonasun) {
+        init_lonasun();
+        VLT_CUDA(cudaDeviceSynchronize());
+    } else if (!ho) {
         // engine.rs:392-421 `rope_table`: theta = float32(pos) * frequency, cos and sin rounded to bf16.
         const uint32_t npos = cfg.max_seq_len + FEED_W, half = uint32_t(model.rope_freq.size());  // hd / 2; 32 pairs for a head of 128 of the reference's architecture
         std::vector<float> tab(size_t(npos) * half * 2);
@@ -368,6 +390,11 @@ Plan Engine::plan(uint32_t set, const std::vector<PlanRun>& runs, Rows hidden) {
         auto rows = [&](Rows r, std::vector<uint32_t>& v) {
             if (r == Rows::Last) v.push_back(first_row + count - 1);
             if (r == Rows::All) for (uint32_t x = first_row; x < first_row + count; x++) v.push_back(x);
+            if (r == Rows::Listed)
+                for (uint32_t j = 0; j < run.n_want; j++) {
+                    if (run.want[j] >= count) throw Error("row " + std::to_string(run.want[j]) + " of a run of " + std::to_string(count));
+                    v.push_back(first_row + run.want[j]);
+                }
         };
         const uint32_t first_head = uint32_t(head_rows.size());
         rows(run.verify ? Rows::All : run.head, head_rows);
@@ -402,7 +429,8 @@ Plan Engine::plan(uint32_t set, const std::vector<PlanRun>& runs, Rows hidden) {
     p.ctiles = uint32_t(ctiles.size() / 2);
     p.n = n;
     p.n_head = uint32_t(head_rows.size());
-    p.head_all = p.n_head == n;  // (rows are listed in step order, each once)
+    p.head_all = p.n_head == n;  // (rows are in step order, each once, unless a caller lists them)
+    for (uint32_t i = 0; i < p.n_head && p.head_all; i++) p.head_all = head_rows[i] == i;
     p.n_hidden = uint32_t(hidden_rows.size());
     p.n_runs = uint32_t(runs.size());
     p.tiles = uint32_t(tiles.size() / 2);
@@ -890,6 +918,7 @@ void Engine::encode_forward_limite(uint32_t set, const Plan& p) {
 
 // engine/src/engine/encode.rs:99-105 `encode_forward`, after the step set's upload.
 void Engine::encode_forward(uint32_t set, const Plan& p) {
+    if (model.lonasun) { encode_forward_lonasun(set, p); return; }
     if (model.limite) { encode_forward_limite(set, p); return; }
     begin_step(set, p);
     for (uint32_t li = 0; li < model.md.n_layers; li++) encode_layer(set, p, li);
@@ -906,7 +935,7 @@ void Engine::begin_step(uint32_t set, const Plan& p) {
     VLT_CUDA(cudaEventRecord(st.uploaded, copy_in));
     VLT_CUDA(cudaEventRecord(st.start, stream));
     VLT_CUDA(cudaStreamWaitEvent(stream, st.uploaded, 0));
-    launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
+    launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), lz ? lz->x0.as<float>() : s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
                  s.feed.as<uint32_t>(), s.tree.as<uint32_t>(), st.in<uint32_t>(st.o_vis), p.n, model.md.d, model.md.vocab, stream);
 }
 
@@ -965,6 +994,7 @@ void Engine::upload_set(uint32_t set) {
 void Engine::load_drafter(const std::string& path) {
     for (const auto& q : seqs)
         if (q) throw Error("load the drafter before the first sequence (it changes how many pages a step reserves)");
+    if (model.lonasun) throw Error(path + ": the drafters are built for the other architectures' hidden states");
     auto dr = std::make_unique<Drafter>();
     const ModelDesc& md = model.md;
     dr->w.load(path, cfg.host_only);
@@ -1395,7 +1425,15 @@ StepOutput Engine::read_output(const Plan& p, const StepOptions& opts, double gp
 // engine/src/engine.rs:318-355 `step_capture`.
 StepOutput Engine::step_capture(const std::vector<PlanRun>& runs, const StepOptions& opts, const std::function<void(const LayerCapture&)>& f) {
     if (cfg.host_only) throw Error("this engine was created host-only: it plans steps but cannot run them (no CPU path)");
-    if (model.limite) throw Error("step_capture is built for the plain decoder");
+    if (model.limite) throw Error("step_capture is not built for the reference's own architecture");
+    if (model.lonasun) {
+        Plan p = plan(0, runs, opts.hidden);
+        encode_forward_lonasun(0, p, &f);
+        commit(0);
+        const double secs = wait(0);
+        check_device_error(0);
+        return read_output(p, opts, secs);
+    }
     const ModelDesc& md = model.md;
     if (!cap) {
         cap = std::make_unique<CaptureBufs>();
@@ -1431,6 +1469,11 @@ void Engine::bench_fill(uint32_t id, uint32_t len, uint32_t seed) {
     sq.len += len;
     s.lens.write(id * 4, &sq.len, 4);
     kv.reserve(id, sq.pages, sq.len);
+    if (seed && model.lonasun && !cfg.host_only) {
+        launch_mixer_fill(lz->caches.as<MixerCache>(), model.md.n_layers, id, from, sq.len, seed, cfg.fp32, stream);
+        VLT_CUDA(cudaStreamSynchronize(stream));
+        return;
+    }
     if (seed && model.limite) throw Error("bench_fill with values fills a plain decoder's paged pool; a model of the reference's own architecture is filled by computing it");
     if (seed && !cfg.host_only) {
         launch_kv_fill(kv.k.as<uint16_t>(), kv.v.as<uint16_t>(), kv.page_table.as<uint32_t>(), kv_args(), model.md.n_layers, id, from, sq.len, seed, stream);
@@ -1539,6 +1582,7 @@ void Engine::draft_trees(const float* logits, uint32_t n_rows, uint32_t nv, cons
 void Engine::bench_matmul(const std::string& kind, uint32_t n, uint32_t variant, uint32_t reps, double* seconds, uint64_t* bytes) {
     if (cfg.host_only) throw Error("this engine was created host-only: it cannot run kernels");
     const bool head = kind == "head";
+    if (model.lonasun) throw Error("bench_matmul times the other architectures' projections");
     if (!head && kind != "qkv" && kind != "o" && kind != "gate_up" && kind != "down") throw Error("unknown matmul " + kind);
     if (n == 0 || n > (head ? cfg.max_head_rows : cfg.max_step_tokens)) throw Error(kind + " can't take " + std::to_string(n) + " tokens");
     cudaEvent_t e0, e1;

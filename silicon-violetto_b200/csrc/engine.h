@@ -10,7 +10,7 @@
 
 #include "common.h"
 #include "kernels.h"
-#include "weights.h"
+#include "model.h"
 
 namespace vlt {
 
@@ -19,6 +19,7 @@ struct EngineConfig {
     uint32_t max_seqs = 8, max_step_tokens = 512, max_chunk = 512, global_kv_tokens = 65536, max_seq_len = 131072, max_head_rows = 64;
     int device = 0;
     bool host_only = false;
+    bool fp32 = false;  // activations, caches and products in fp32 (architectures that have such a path)
 };
 
 // engine/src/engine.rs:59-95, with B200 knobs in place of the Apple-GPU ones.
@@ -38,7 +39,7 @@ struct Sampling {
     SampleRow row_of(uint32_t tok) const { SampleRow r = row_at(0); r.tok = tok; return r; }
 };
 
-enum class Rows : uint32_t { None = 0, Last = 1, All = 2 };
+enum class Rows : uint32_t { None = 0, Last = 1, All = 2, Listed = 3 };
 
 // engine/src/engine/plan.rs:8-18.
 struct PlanRun {
@@ -47,6 +48,8 @@ struct PlanRun {
     uint32_t count;
     Rows head;
     bool verify;
+    const uint32_t* want = nullptr;  // Rows::Listed: these rows of the run, in this order
+    uint32_t n_want = 0;
 };
 
 // engine/src/engine/plan.rs:20-37.
@@ -66,12 +69,19 @@ struct Seq {
     Sampling sampling;
 };
 
-// engine/src/engine/kv.rs:9-90, every layer paged.
+// One layer's heads in the paged pool.
+struct KvShape {
+    uint32_t n_kv, dk, dv;
+};
+// engine/src/engine/kv.rs:9-90, every layer paged: all layers share the page table, each has its own slice of the pools
+// ([page][kv head][position in page][dk or dv]), from k_off / v_off elements on.
 struct KvCache {
     Buffer k, v, page_table;
+    std::vector<KvShape> shapes;
+    std::vector<size_t> k_off, v_off;
     std::vector<uint32_t> free_pages;
     uint32_t n_pages = 0, max_pages = 0, page = 16;
-    void init(const EngineConfig& cfg, const ModelDesc& md, uint32_t n_layers, bool with_pool);
+    void init(const EngineConfig& cfg, uint32_t page_size, std::vector<KvShape> layers, uint32_t elem_bytes, bool with_pool);
     void reserve(uint32_t slot, std::vector<uint32_t>& pages, uint32_t len);
     void release(const std::vector<uint32_t>& pages);
 };
@@ -115,6 +125,8 @@ struct StepOutput {
 struct LayerCapture {
     uint32_t layer, n;
     const float *resid_in, *attn_in, *qkv, *sdpa_out, *attn_out, *mlp_in, *mlp_out;
+    const float* resid_out = nullptr;  // the stream leaving the layer (Lonasun, which hands out this, resid_in and sdpa_out only)
+    uint32_t attn_width = 0;           // sdpa_out's columns, where layers differ
 };
 
 class Engine {
@@ -233,6 +245,23 @@ class Engine {
         Buffer k_local, v_local;  // [local layer][slot][kv head][ring][128] bf16
         Buffer hist0, hist12, hist23, xattn, base, mixed, vdir, gates, part;  // part: the attention's partials per (token, head, key split)
     };
+    // The Lonasun design (model.lonasun): a ring of projected rows per (layer run, slot) beside the paged pool, and scratch.
+    struct LonasunState {
+        Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding; a norm's rows; (stream ; embedding)
+        Buffer proj, q_f, q_b, attn_f, attn_b;    // q | k | v | gate as projected; rotated q; the gated attention
+        Buffer moe_x, moe_xb, ids, weights, src, place, tiles, n_tiles, hid_f, hid_b, rows, sh_f, sh_b, shared;
+        Buffer rings, caches;                     // caches: MixerCache per layer run, on the device
+        std::vector<Buffer> rope;                 // per distinct rotation: [position][dims / 2] (cos, sin), fp32
+        std::vector<MixerCache> run;              // the host's copy of caches
+    };
+    static constexpr uint32_t EXPERT_TILE_MIN = 16;  // rows of an expert per tile, at least
+    std::unique_ptr<LonasunState> lz;
+    void init_lonasun();
+    void encode_experts(const LonasunLayer& l, uint32_t n, const uint16_t* norm);
+    void encode_forward_lonasun(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
+    // Y = epilogue(W x) in the engine's precision: xf in an fp32 engine, else xb through the GEMM, the streamed matmul or,
+    // for sizes neither takes, the CUDA cores.
+    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr);
     std::unique_ptr<LimiteState> lim;
     LimiteKv limite_kv(const LimiteLayer& x) const;
     void encode_forward_limite(uint32_t set, const Plan& p);

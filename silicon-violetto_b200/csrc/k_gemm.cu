@@ -452,6 +452,7 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
             else if (EPI == EPI_RESID) y[j] = m.ra * base[j] + m.rb * (m.scale * x);  // (1, 1, 1 for a plain decoder: the same bits as base + x)
             else if (EPI == EPI_HEAD) y[j] = row < m.vocab_real ? x * inv[j] : -INFINITY;
             else if (EPI == EPI_HEAD_CAP) y[j] = row < m.vocab_real ? 23.0f * (1.0f / (1.0f + __expf(-(x + 5.0f) / 7.5f))) : -INFINITY;  // kernels.metal:196-199
+            else if (EPI == EPI_RELU2) y[j] = x > 0.0f ? x * x : 0.0f;
             else y[j] = x;
         }
         if (EPI == EPI_RESID && m.ssq_out) {
@@ -627,6 +628,7 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
     case EPI_HEAD: return int8 ? gemm::gemm_kernel<true, EPI_HEAD> : gemm::gemm_kernel<false, EPI_HEAD>;
     case EPI_QKV: return int8 ? gemm::gemm_kernel<true, EPI_QKV> : gemm::gemm_kernel<false, EPI_QKV>;
     case EPI_HEAD_CAP: return int8 ? gemm::gemm_kernel<true, EPI_HEAD_CAP> : gemm::gemm_kernel<false, EPI_HEAD_CAP>;
+    case EPI_RELU2: return int8 ? gemm::gemm_kernel<true, EPI_RELU2> : gemm::gemm_kernel<false, EPI_RELU2>;
     default: return int8 ? gemm::gemm_kernel<true, EPI_RAW> : gemm::gemm_kernel<false, EPI_RAW>;
     }
 }
@@ -634,7 +636,7 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
 bool gemm_supported(const MatArgs& a) {
     const bool grouped = a.int8 && a.group < a.k;  // scale groups: powers of two from 8
     return a.n >= 1 && a.n <= 256 && a.m % gemm::BM == 0 && a.k % gemm::BK == 0 && (!grouped || (a.group >= 8 && !(a.group & (a.group - 1)))) && a.Xb != nullptr &&
-           (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.inv_in != nullptr || a.ssq_in != nullptr);
+           (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.epi == EPI_RELU2 || a.inv_in != nullptr || a.ssq_in != nullptr);
 }
 
 void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaStream_t s, bool allow_paired) {
@@ -677,7 +679,7 @@ void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaSt
     const size_t smem = paired ? need : std::max<size_t>(need, 116 * 1024);
     configured.once([] {
         for (int i8 = 0; i8 < 2; i8++)
-            for (uint32_t epi = EPI_NORM; epi <= EPI_HEAD_CAP; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            for (uint32_t epi = EPI_NORM; epi <= EPI_RELU2; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
     });
@@ -686,7 +688,7 @@ void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaSt
     static thread_local std::map<std::tuple<bool, uint32_t, uint32_t>, uint32_t> wave;  // (int8, smem, cluster size) -> clusters one wave holds
     uint32_t splits = std::max(1u, std::min(8u, std::min(sm_count / tiles, nkb)));  // (1 for a paired launch: more tiles than SMs)
     for (; splits > 1; splits--) {
-        auto wk = std::make_tuple(a.int8, uint32_t(smem) * 8 + a.epi, splits);
+        auto wk = std::make_tuple(a.int8, uint32_t(smem) * 16 + a.epi, splits);
         auto w = wave.find(wk);
         if (w == wave.end()) {
             cudaLaunchConfig_t q = {};

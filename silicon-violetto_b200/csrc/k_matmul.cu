@@ -23,9 +23,10 @@ __device__ __forceinline__ void store_out(const MatArgs& a, uint32_t t, uint32_t
     case EPI_RESID: y = a.ra * a.base[o] + a.rb * (a.scale * acc); break;
     case EPI_HEAD: y = row < a.vocab_real ? acc * inv : -INFINITY; break;
     case EPI_HEAD_CAP: y = row < a.vocab_real ? 23.0f * (1.0f / (1.0f + expf(-(acc + 5.0f) / 7.5f))) : -INFINITY; break;
+    case EPI_RELU2: y = acc > 0.0f ? acc * acc : 0.0f; break;
     default: y = acc; break;
     }
-    a.Y[o] = y;
+    if (a.Y) a.Y[o] = y;
     if (a.Yb) a.Yb[o] = f32_to_bf16(y);
 }
 __device__ __forceinline__ void store_swiglu(const MatArgs& a, uint32_t t, uint32_t row, float g, float u, float inv) {

@@ -1,0 +1,238 @@
+// The attention mixer's work between its projections and its attention, as parameterised kernels: a short causal
+// convolution over time on q, k and v, rotation of pairs (i, i + dims / 2), K and V into a paged cache whose heads may have
+// different key and value sizes; the convolution's state -- the projected rows before the step -- in a ring per sequence
+// slot; and a scalar form of the chunked attention for any head sizes and for fp32 caches.
+#include <algorithm>
+
+#include "kernels.h"
+
+namespace vlt {
+
+namespace mixer {
+
+__device__ __forceinline__ void store_kv(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_kv(uint16_t* p, float v) { *p = f32_to_bf16(v); }
+__device__ __forceinline__ float load_kv(const float* p) { return *p; }
+__device__ __forceinline__ float load_kv(const uint16_t* p) { return bf16_to_f32(*p); }
+
+__device__ __forceinline__ size_t page_row(const PagedKv& kv, uint32_t slot, uint32_t g, uint32_t pos) {
+    const uint32_t page = kv.page_table[size_t(slot) * kv.max_pages + (pos >> kv.page_shift)], psize = 1u << kv.page_shift;
+    return (size_t(page) * kv.n_kv + g) * psize + (pos & (psize - 1));
+}
+
+// Where the projected row `back` positions before token t lies: among the rows of its own tile of 8 that it descends from
+// (its `vis` mask names them: a chain's all, a draft tree's its ancestors), then among the run's earlier rows, then in the
+// slot's ring of rows that earlier steps left; none before the sequence's start.
+__device__ __forceinline__ const float* row_before(const ConvArgs& a, uint32_t t, uint32_t back) {
+    const uint32_t row = a.tin[2 * t + 1], i = row % 8;
+    if (back == 0) return a.u + size_t(t) * a.ldu;
+    uint32_t anc = a.vis[t] & ((1u << i) - 1);
+    const uint32_t n = __popc(anc);
+    if (back <= n) {
+        uint32_t bit = 0;
+        for (uint32_t k = 0; k < back; k++) {
+            bit = 31 - __clz(anc);
+            anc &= ~(1u << bit);
+        }
+        return a.u + size_t(t - i + bit) * a.ldu;
+    }
+    const uint32_t over = back - n;  // positions before the tile
+    if (over <= row - i) return a.u + size_t(t - i - over) * a.ldu;
+    const uint32_t before = over - (row - i), start = a.meta[2 * (t - row) + 1];  // positions before the run
+    if (before > start) return nullptr;
+    return a.ring + (size_t(a.tin[2 * t]) * a.ring_len + (start - before) % a.ring_len) * a.conv_channels;
+}
+
+// grid (tokens, heads + 2 kv heads): one q, k or v head of one token a block.
+template <typename T>
+__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a) {
+    pdl_start();
+    extern __shared__ float y[];  // the head after its convolution
+    __shared__ const float* from[32];
+    const uint32_t t = blockIdx.x, unit = blockIdx.y, tid = threadIdx.x;
+    const uint32_t kind = unit < a.heads ? 0u : unit < a.heads + a.kv.n_kv ? 1u : 2u;
+    const uint32_t head = kind == 0 ? unit : kind == 1 ? unit - a.heads : unit - a.heads - a.kv.n_kv, width = kind == 2 ? a.kv.dv : a.kv.dk;
+    const uint32_t c0 = kind == 2 ? (a.heads + a.kv.n_kv) * a.kv.dk + head * a.kv.dv : unit * a.kv.dk;
+    const uint32_t slot = a.meta[2 * t], pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], cpos = a.meta[2 * (t - row) + 1] + row;
+    if (tid < a.taps) from[tid] = row_before(a, t, tid);
+    __syncthreads();
+    for (uint32_t c = tid; c < width; c += 128) {
+        const uint16_t* w = a.w + size_t(c0 + c) * a.taps;
+        float s = 0.0f;
+        for (uint32_t j = 0; j < a.taps; j++) {
+            const float* u = from[a.taps - 1 - j];
+            if (u) s = fmaf(bf16_to_f32(w[j]), u[c0 + c], s);
+        }
+        y[c] = s;
+        if (a.write_ring) a.ring[(size_t(slot) * a.ring_len + cpos % a.ring_len) * a.conv_channels + c0 + c] = from[0][c0 + c];
+    }
+    __syncthreads();
+    T* cache = nullptr;
+    if (kind) cache = static_cast<T*>(kind == 1 ? a.kv.k : a.kv.v) + page_row(a.kv, slot, head, cpos) * width;
+    const float2* cs = reinterpret_cast<const float2*>(a.rope) + size_t(pos) * (a.rot_dims / 2);
+    for (uint32_t c = tid; c < width; c += 128) {
+        float v = y[c];
+        if (kind < 2 && c < a.rot_dims) {
+            const uint32_t half = a.rot_dims / 2;
+            if (c < half) v = y[c] * cs[c].x - y[c + half] * cs[c].y;
+            else v = y[c] * cs[c - half].x + y[c - half] * cs[c - half].y;
+        }
+        if (kind == 0) {
+            const size_t o = (size_t(t) * a.heads + head) * width + c;
+            if (a.q_f) a.q_f[o] = v;
+            if (a.q_b) a.q_b[o] = f32_to_bf16(v * a.q_scale);
+        } else {
+            store_kv(cache + c, v);
+        }
+    }
+}
+
+// The last rows of every run into its slot's ring, for steps whose runs are long enough to wrap it (a run's first rows must
+// have read the ring before its last ones overwrite it). grid (runs, rows of the ring).
+__global__ void __launch_bounds__(256) conv_state_kernel(const ConvArgs a, const RunIn* __restrict__ runs) {
+    pdl_start();
+    const RunIn ru = runs[blockIdx.x];
+    if (blockIdx.y >= ru.count) return;
+    const uint32_t row = ru.count - 1 - blockIdx.y, pos = a.meta[2 * ru.first + 1] + row;
+    const float* src = a.u + size_t(ru.first + row) * a.ldu;
+    float* dst = a.ring + (size_t(ru.slot) * a.ring_len + pos % a.ring_len) * a.conv_channels;
+    for (uint32_t c = threadIdx.x; c < a.conv_channels; c += 256) dst[c] = src[c];
+}
+
+// Attention of one token and query head per block: the cached keys from the chunk's first position (or the sequence's) up to
+// the token's tile of 8, then the tile's rows its `vis` names that lie in the same chunk; softmax in fp32 with a running
+// maximum over blocks of 128 keys; the gate on the result.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) {
+    pdl_start();
+    extern __shared__ float sm[];
+    float *q = sm, *o = sm + a.kv.dk, *p = o + a.kv.dv;
+    __shared__ uint32_t rows[128];  // (a key's row in the pool; pools of more than 2^32 rows do not exist)
+    __shared__ float red[8];
+    const uint32_t t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, g = h / (a.heads / a.kv.n_kv);
+    const uint32_t slot = a.meta[2 * t], pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], mask = a.vis[t];
+    const uint32_t tile0 = t - row % 8, p_tile = a.meta[2 * (t - row) + 1] + row - row % 8;  // the tile's first token and cache position
+    const uint32_t lo = a.chunk ? pos / a.chunk * a.chunk : 0, n_old = p_tile > lo ? p_tile - lo : 0;
+    const T* K = static_cast<const T*>(a.kv.k);
+    const T* V = static_cast<const T*>(a.kv.v);
+    for (uint32_t c = tid; c < a.kv.dk; c += 128) q[c] = a.q_f[(size_t(t) * a.heads + h) * a.kv.dk + c];
+    for (uint32_t c = tid; c < a.kv.dv; c += 128) o[c] = 0.0f;
+    float m = -INFINITY, l = 0.0f;
+    __syncthreads();
+    for (uint32_t i0 = 0; i0 < n_old + 8; i0 += 128) {
+        const uint32_t i = i0 + tid;
+        float s = -INFINITY;
+        bool seen = i < n_old;
+        uint32_t kp = lo + i;
+        if (!seen && i < n_old + 8) {
+            const uint32_t j = i - n_old;
+            kp = p_tile + j;
+            seen = ((mask >> j) & 1u) && (!a.chunk || a.meta[2 * (tile0 + j) + 1] / a.chunk == pos / a.chunk);
+        }
+        if (seen) {
+            const size_t r = page_row(a.kv, slot, g, kp);
+            rows[tid] = uint32_t(r);
+            const T* k = K + r * a.kv.dk;
+            float d = 0.0f;
+            for (uint32_t c = 0; c < a.kv.dk; c++) d = fmaf(q[c], load_kv(k + c), d);
+            s = d * a.scale;
+        }
+        float mx = warp_max(s);
+        if (tid % 32 == 0) red[tid / 32] = mx;
+        __syncthreads();
+        mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+        const float mn = fmaxf(m, mx), corr = m == -INFINITY ? 0.0f : expf(m - mn), w = s == -INFINITY ? 0.0f : expf(s - mn);
+        p[tid] = w;
+        const float sum = warp_sum(w);
+        if (tid % 32 == 0) red[4 + tid / 32] = sum;
+        __syncthreads();
+        if (mx != -INFINITY) {
+            l = l * corr + ((red[4] + red[5]) + (red[6] + red[7]));
+            m = mn;
+            const uint32_t n = min(128u, n_old + 8 - i0);
+            for (uint32_t c = tid; c < a.kv.dv; c += 128) {
+                float acc = o[c] * corr;
+                for (uint32_t j = 0; j < n; j++)
+                    if (p[j] != 0.0f) acc = fmaf(p[j], load_kv(V + size_t(rows[j]) * a.kv.dv + c), acc);
+                o[c] = acc;
+            }
+        }
+        __syncthreads();
+    }
+    for (uint32_t c = tid; c < a.kv.dv; c += 128) {
+        const float gt = 1.0f / (1.0f + expf(-a.gate[size_t(t) * a.ldg + h * a.kv.dv + c])), y = o[c] / l * gt;
+        const size_t at = (size_t(t) * a.heads + h) * a.kv.dv + c;
+        if (a.out) a.out[at] = y;
+        if (a.out_b) a.out_b[at] = f32_to_bf16(y);
+    }
+}
+
+// The accepted path's rows of a verified draft tree, from where they were computed to where they belong: K and V in every
+// layer run's pages, and the convolution's ring rows. grid (runs, layer runs); a thread keeps to its own columns.
+template <typename T>
+__global__ void __launch_bounds__(256) mixer_compact_kernel(const RunIn* __restrict__ runs, const uint32_t* __restrict__ path, const uint32_t* __restrict__ path_len,
+                                                            const uint32_t* __restrict__ lens, const MixerCache* __restrict__ caches) {
+    pdl_start();
+    const uint32_t r = blockIdx.x, k = path_len[r];
+    if (k < 2) return;
+    const MixerCache mc = caches[blockIdx.y];
+    const uint32_t slot = runs[r].slot, p0 = lens[slot] - k;
+    for (uint32_t j = 1; j < k; j++) {
+        const uint32_t from = path[r * FEED_W + j];
+        if (from == j) continue;
+        for (uint32_t g = 0; g < mc.kv.n_kv; g++) {
+            const size_t src = page_row(mc.kv, slot, g, p0 + from), dst = page_row(mc.kv, slot, g, p0 + j);
+            for (uint32_t c = threadIdx.x; c < mc.kv.dk; c += 256) static_cast<T*>(mc.kv.k)[dst * mc.kv.dk + c] = static_cast<const T*>(mc.kv.k)[src * mc.kv.dk + c];
+            for (uint32_t c = threadIdx.x; c < mc.kv.dv; c += 256) static_cast<T*>(mc.kv.v)[dst * mc.kv.dv + c] = static_cast<const T*>(mc.kv.v)[src * mc.kv.dv + c];
+        }
+        float* ring = mc.ring + size_t(slot) * mc.ring_len * mc.channels;
+        for (uint32_t c = threadIdx.x; c < mc.channels; c += 256) ring[size_t((p0 + j) % mc.ring_len) * mc.channels + c] = ring[size_t((p0 + from) % mc.ring_len) * mc.channels + c];
+    }
+}
+
+// Small pseudo-random keys and values for positions that are not computed (benchmarks). grid (positions, layer runs).
+template <typename T>
+__global__ void __launch_bounds__(256) mixer_fill_kernel(const MixerCache* __restrict__ caches, uint32_t slot, uint32_t from, uint32_t seed) {
+    const MixerCache mc = caches[blockIdx.y];
+    const uint32_t pos = from + blockIdx.x;
+    for (uint32_t g = 0; g < mc.kv.n_kv; g++) {
+        const size_t r = page_row(mc.kv, slot, g, pos);
+        for (uint32_t c = threadIdx.x; c < mc.kv.dk + mc.kv.dv; c += 256) {
+            const float v = (float(philox(make_uint4(pos, blockIdx.y * 131 + g, c, slot), seed, 0xf111u).x >> 8) * 0x1p-24f - 0.5f) * 0.5f;
+            if (c < mc.kv.dk) store_kv(static_cast<T*>(mc.kv.k) + r * mc.kv.dk + c, v);
+            else store_kv(static_cast<T*>(mc.kv.v) + r * mc.kv.dv + c - mc.kv.dk, v);
+        }
+    }
+}
+
+}  // namespace mixer
+
+void launch_conv_qkv(const ConvArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
+    const dim3 grid(n, a.heads + 2 * a.kv.n_kv);
+    const size_t smem = std::max(a.kv.dk, a.kv.dv) * 4;
+    if (fp32) launch_pdl(mixer::conv_qkv_kernel<float>, grid, 128, smem, s, a);
+    else launch_pdl(mixer::conv_qkv_kernel<uint16_t>, grid, 128, smem, s, a);
+}
+void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cudaStream_t s) {
+    if (n_runs) launch_pdl(mixer::conv_state_kernel, dim3(n_runs, a.ring_len), 256, 0, s, a, runs);
+}
+void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
+    const size_t smem = (a.kv.dk + a.kv.dv + 128) * 4;
+    if (fp32) launch_pdl(mixer::attn_any_kernel<float>, dim3(n, a.heads), 128, smem, s, a);
+    else launch_pdl(mixer::attn_any_kernel<uint16_t>, dim3(n, a.heads), 128, smem, s, a);
+}
+void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_layers,
+                          bool fp32, cudaStream_t s) {
+    if (!n_runs) return;
+    if (fp32) launch_pdl(mixer::mixer_compact_kernel<float>, dim3(n_runs, n_layers), 256, 0, s, runs, path, path_len, lens, caches);
+    else launch_pdl(mixer::mixer_compact_kernel<uint16_t>, dim3(n_runs, n_layers), 256, 0, s, runs, path, path_len, lens, caches);
+}
+void launch_mixer_fill(const MixerCache* caches, uint32_t n_layers, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s) {
+    if (to <= from) return;
+    const dim3 grid(to - from, n_layers);
+    if (fp32) mixer::mixer_fill_kernel<float><<<grid, 256, 0, s>>>(caches, slot, from, seed);
+    else mixer::mixer_fill_kernel<uint16_t><<<grid, 256, 0, s>>>(caches, slot, from, seed);
+    launch_counter()++;
+}
+
+}  // namespace vlt

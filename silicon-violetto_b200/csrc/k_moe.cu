@@ -1,0 +1,211 @@
+// A mixture of experts: the router (fp32 scores over the experts and the identity experts, a correction that moves the
+// choice but not the weights), the tokens sorted by expert, and the weighted sum of what the experts left. The experts' own
+// matrices are grouped linear layers (k_linear.cu, k_grouped.cu).
+#include <algorithm>
+
+#include "kernels.h"
+
+namespace vlt {
+
+namespace moe {
+
+constexpr uint32_t ROUTER_THREADS = 256;
+
+// One block per TOK tokens: the RMS norm of their rows (kept for the experts), the scores' logits with a warp per output,
+// softmax and the choice with a warp per token. Ties go to the lower index.
+template <uint32_t TOK>
+__global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs a) {
+    pdl_start();
+    extern __shared__ float sm[];
+    constexpr uint32_t NW = ROUTER_THREADS / 32;
+    const uint32_t t0 = blockIdx.x * TOK, tid = threadIdx.x, warp = tid / 32, lane = tid % 32, nt = min(TOK, a.n - t0);
+    float *x = sm, *z = sm + TOK * a.d;  // the normed rows, the scores
+    __shared__ float red[TOK][NW];
+#pragma unroll
+    for (uint32_t j = 0; j < TOK; j++) {
+        float ss = 0.0f;
+        if (j < nt)
+            for (uint32_t i = tid; i < a.d; i += ROUTER_THREADS) {
+                const float v = a.x[size_t(t0 + j) * a.d + i];
+                x[j * a.d + i] = v;
+                ss += v * v;
+            }
+        ss = warp_sum(ss);
+        if (lane == 0) red[j][warp] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (uint32_t j = 0; j < TOK; j++) {
+        if (j >= nt) break;
+        float tot = 0.0f;
+        for (uint32_t w = 0; w < NW; w++) tot += red[j][w];
+        const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
+        for (uint32_t i = tid; i < a.d; i += ROUTER_THREADS) {
+            const float v = x[j * a.d + i] * inv * (1.0f + bf16_to_f32(a.norm[i]));
+            x[j * a.d + i] = v;
+            const size_t o = size_t(t0 + j) * a.d + i;
+            if (a.xn) a.xn[o] = v;
+            if (a.xn_b) a.xn_b[o] = f32_to_bf16(v);
+        }
+    }
+    __syncthreads();
+    const uint32_t all = a.experts + a.identity;
+    for (uint32_t e = warp; e < all; e += NW) {
+        float s[TOK] = {};
+        const uint16_t* w = a.router + size_t(e) * a.d;
+        for (uint32_t i = lane; i < a.d; i += 32) {
+            const float wv = bf16_to_f32(w[i]);
+#pragma unroll
+            for (uint32_t j = 0; j < TOK; j++)
+                if (j < nt) s[j] = fmaf(wv, x[j * a.d + i], s[j]);
+        }
+#pragma unroll
+        for (uint32_t j = 0; j < TOK; j++) {
+            s[j] = warp_sum(s[j]);
+            if (lane == 0) z[j * all + e] = s[j];
+        }
+    }
+    __syncthreads();
+    if (warp >= nt) return;
+    for (uint32_t j = warp; j < nt; j += NW) {
+        float* zt = z + j * all;
+        const uint32_t t = t0 + j;
+        float m = -INFINITY, sum = 0.0f;
+        for (uint32_t e = lane; e < all; e += 32) m = fmaxf(m, zt[e]);
+        m = warp_max(m);
+        for (uint32_t e = lane; e < all; e += 32) {
+            const float p = expf(zt[e] - m);
+            zt[e] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        for (uint32_t e = lane; e < all; e += 32) zt[e] = zt[e] / sum;
+        __syncwarp();
+        // The choice: the largest score + correction, `top` times; a chosen score is marked by its sign bit (scores are >= 0).
+        float total = 0.0f;
+        for (uint32_t k = 0; k < a.top; k++) {
+            float bv = -INFINITY;
+            uint32_t bi = 0xffffffffu;
+            for (uint32_t e = lane; e < all; e += 32) {
+                if (signbit(zt[e])) continue;
+                better(bv, bi, zt[e] + bf16_to_f32(a.correction[e]), e);
+            }
+            warp_best(bv, bi);
+            if (bi >= all) bi = 0;  // (only if the logits are not numbers)
+            const float s = fabsf(zt[bi]);
+            total += s;
+            __syncwarp();
+            if (lane == 0) {
+                zt[bi] = -s;
+                a.ids[size_t(t) * a.top + k] = bi;
+                a.weights[size_t(t) * a.top + k] = s;
+            }
+            __syncwarp();
+        }
+        const float inv = 1.0f / (total + 1e-20f);
+        for (uint32_t k = lane; k < a.top; k += 32) a.weights[size_t(t) * a.top + k] *= inv;
+    }
+}
+
+// The (token, choice) pairs in expert order, by one block: counts, their prefix sums, the pairs' places, and the table of
+// (expert, first row, rows <= tile) tiles the grouped linear layers run over. Which of an expert's rows a token gets is left
+// to the atomics; nothing depends on it.
+__global__ void __launch_bounds__(1024) sort_kernel(const SortArgs a) {
+    pdl_start();
+    extern __shared__ uint32_t sh[];
+    uint32_t *cnt = sh, *cur = sh + a.experts, *tile0 = cur + a.experts;
+    __shared__ uint32_t n_tiles;
+    const uint32_t tid = threadIdx.x, pairs = a.n * a.top;
+    for (uint32_t e = tid; e < a.experts; e += 1024) cnt[e] = 0;
+    __syncthreads();
+    for (uint32_t i = tid; i < pairs; i += 1024) {
+        const uint32_t e = a.ids[i];
+        if (e < a.experts) atomicAdd(cnt + e, 1u);
+    }
+    __syncthreads();
+    if (tid < 32) {
+        uint32_t rows = 0, tiles = 0;
+        for (uint32_t e0 = 0; e0 < a.experts; e0 += 32) {
+            const uint32_t e = e0 + tid, c = e < a.experts ? cnt[e] : 0, k = (c + a.tile - 1) / a.tile;
+            uint32_t sc = c, sk = k;
+#pragma unroll
+            for (uint32_t o = 1; o < 32; o *= 2) {
+                const uint32_t pc = __shfl_up_sync(0xffffffffu, sc, o), pk = __shfl_up_sync(0xffffffffu, sk, o);
+                if (tid >= o) { sc += pc; sk += pk; }
+            }
+            if (e < a.experts) { cur[e] = rows + sc - c; tile0[e] = tiles + sk - k; }
+            rows += __shfl_sync(0xffffffffu, sc, 31);
+            tiles += __shfl_sync(0xffffffffu, sk, 31);
+        }
+        if (tid == 0) { n_tiles = tiles; *a.n_tiles = tiles; }
+    }
+    __syncthreads();
+    for (uint32_t e = tid; e < a.experts; e += 1024)
+        for (uint32_t k = 0, at = tile0[e]; k < cnt[e]; k += a.tile, at++) {
+            a.tiles[3 * at] = e;
+            a.tiles[3 * at + 1] = cur[e] + k;
+            a.tiles[3 * at + 2] = min(a.tile, cnt[e] - k);
+        }
+    __syncthreads();
+    for (uint32_t i = tid; i < pairs; i += 1024) {
+        const uint32_t e = a.ids[i];
+        if (e < a.experts) {
+            const uint32_t p = atomicAdd(cur + e, 1u);
+            a.src[p] = i / a.top;
+            a.place[i] = p;
+        }
+    }
+}
+
+// out[t] = x[t] + sum_k weight_k (expert k's row, or the token's own normed row for an identity expert) + the shared
+// expert's row, in the order of the choice; and, if asked, the next layer's RMS norm of it. A block per token.
+__global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
+    pdl_start();
+    __shared__ float red[8];
+    const uint32_t t = blockIdx.x, tid = threadIdx.x;
+    float ss = 0.0f;
+    for (uint32_t i = tid; i < a.d; i += 256) {
+        const size_t o = size_t(t) * a.d + i;
+        float y = 0.0f;
+        for (uint32_t k = 0; k < a.top; k++) {
+            const uint32_t e = a.ids[size_t(t) * a.top + k];
+            const float w = a.weights[size_t(t) * a.top + k];
+            y = fmaf(w, e < a.experts ? a.y[size_t(a.place[size_t(t) * a.top + k]) * a.d + i] : a.xn[o], y);
+        }
+        if (a.shared) y += a.shared[o];
+        y += a.x[o];
+        a.out[o] = y;
+        ss += y * y;
+    }
+    if (!a.norm) return;
+    ss = warp_sum(ss);
+    if (tid % 32 == 0) red[tid / 32] = ss;
+    __syncthreads();
+    float tot = 0.0f;
+    for (uint32_t w = 0; w < 8; w++) tot += red[w];
+    const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
+    for (uint32_t i = tid; i < a.d; i += 256) {
+        const size_t o = size_t(t) * a.d + i;
+        const float v = a.out[o] * inv * (1.0f + bf16_to_f32(a.norm[i]));
+        if (a.next) a.next[o] = v;
+        if (a.next_b) a.next_b[o] = f32_to_bf16(v);
+    }
+}
+
+}  // namespace moe
+
+void launch_router(const RouterArgs& a, cudaStream_t s) {
+    const uint32_t all = a.experts + a.identity;
+    static PerDevice configured;
+    configured.once([] {
+        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    // Many tokens share a read of the router's matrix, four a block; few spread over the SMs one by one.
+    if (a.n >= 592 && (size_t(a.d) + all) * 16 <= 100 * 1024) launch_pdl(moe::router_kernel<4>, (a.n + 3) / 4, moe::ROUTER_THREADS, (size_t(a.d) + all) * 16, s, a);
+    else launch_pdl(moe::router_kernel<1>, a.n, moe::ROUTER_THREADS, (size_t(a.d) + all) * 4, s, a);
+}
+void launch_expert_sort(const SortArgs& a, cudaStream_t s) { launch_pdl(moe::sort_kernel, 1, 1024, size_t(a.experts) * 12, s, a); }
+void launch_combine(const CombineArgs& a, uint32_t n, cudaStream_t s) { launch_pdl(moe::combine_kernel, n, 256, 0, s, a); }
+
+}  // namespace vlt

@@ -9,7 +9,7 @@
 namespace vlt {
 
 // Epilogues of a matmul, engine/src/engine/kernels.rs:3-9 and kernels.metal:154-209.
-enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI_RAW = 5, EPI_QKV = 6, EPI_HEAD_CAP = 7 };  // 7: 23 sigmoid((acc + 5) / 7.5), kernels.metal:196-199
+enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI_RAW = 5, EPI_QKV = 6, EPI_HEAD_CAP = 7, EPI_RELU2 = 8 };  // 7: 23 sigmoid((acc + 5) / 7.5), kernels.metal:196-199; 8: max(acc, 0)^2
 
 // What the tensor-core GEMM's EPI_QKV epilogue needs to finish the qkv projection the way `qkv_post` does
 // (kernels.metal:749-801): RoPE on q and k, q scaled and rounded to bf16 for the attention, k and v rounded
@@ -197,6 +197,100 @@ void launch_matmul_rows(const MatArgs& a, cudaStream_t s);                      
 // out[r] = in[rows ? rows[r] : r] as fp32 (and bf16); inv[r] = 1 / rms (kernels.metal:117-148).
 void launch_prep_rows(const float* in, const uint32_t* rows, uint32_t n, uint32_t k, float eps, float* out_f32, uint16_t* out_bf16, float* inv,
                       bool normalize, bool round_out, cudaStream_t s);
+
+// Linear layers of any shape on the CUDA cores (k_linear.cu): bf16 weights, activations in fp32 or bf16, fp32 products and
+// sums. With `tiles`, a grouped layer: tile j multiplies rows p0 .. p0 + count - 1 by group g's matrix W + g m k.
+struct LinearArgs {
+    const uint16_t* W;
+    const void* X;           // [rows][k] fp32 or bf16
+    const uint32_t* src;     // optional: the row of X that row p multiplies
+    const float* base;       // EPI_RESID
+    float* Y;                // optional, as is
+    uint16_t* Yb;            // its bf16 copy
+    uint32_t n, m, k, epi;   // EPI_RAW, EPI_RESID or EPI_RELU2
+    const uint32_t* tiles;   // [.][3]: (group, first row, rows)
+    const uint32_t* n_tiles;
+    uint32_t max_tiles;      // at most so many tiles (the grid)
+};
+void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s);
+void launch_norm_rows(const float* in, const uint32_t* rows, uint32_t n, uint32_t k, float eps, const uint16_t* w, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
+void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
+
+// One layer run's pages: [page][kv head][position in page][dk or dv] for K and for V, bf16 or fp32.
+struct PagedKv {
+    void *k, *v;
+    const uint32_t* page_table;
+    uint32_t max_pages, page_shift, n_kv, dk, dv;
+};
+// A layer run's cache as the path compaction and the benchmark's fill see it.
+struct MixerCache {
+    PagedKv kv;
+    float* ring;
+    uint32_t ring_len, channels;
+};
+// The work between an attention mixer's projections and its attention (k_mixer.cu).
+struct ConvArgs {
+    const float* u;                       // projected rows, q | k | v | ... [n][ldu]
+    const uint16_t* w;                    // [channels][taps]
+    float* ring;                          // [slot][ring_len][channels]: the projected rows of the positions before the step
+    const uint32_t *meta, *tin, *vis;
+    const float* rope;                    // [position][rot_dims / 2] (cos, sin)
+    PagedKv kv;
+    float* q_f;                           // optional: [n][heads][dk]
+    uint16_t* q_b;                        // optional: the same times q_scale, bf16
+    float q_scale;
+    uint32_t ldu, taps, ring_len, conv_channels, heads, rot_dims;
+    bool write_ring;                      // false: launch_conv_state does it afterwards
+};
+void launch_conv_qkv(const ConvArgs& a, uint32_t n, bool fp32, cudaStream_t s);
+void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cudaStream_t s);
+struct ChunkedAttnArgs {
+    const float* q_f;                     // the scalar kernel's q
+    const uint16_t* q_b;                  // the tensor-core kernels' q, scale * log2(e) folded in
+    const uint32_t *meta, *tin, *vis;
+    PagedKv kv;
+    const float* gate;                    // [n][ldg]: the output is multiplied by sigmoid(gate)
+    uint32_t ldg, heads, chunk;           // chunk 0: every position before
+    float scale;
+    float* out;                           // optional [n][heads][dv]
+    uint16_t* out_b;                      // optional
+};
+void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s);
+void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_layers,
+                          bool fp32, cudaStream_t s);
+void launch_mixer_fill(const MixerCache* caches, uint32_t n_layers, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s);
+
+// A mixture of experts (k_moe.cu).
+struct RouterArgs {
+    const float* x;                       // the stream [n][d]
+    const uint16_t *norm, *router, *correction;
+    float* xn;                            // optional: its normed rows
+    uint16_t* xn_b;                       // optional, bf16
+    uint32_t* ids;                        // [n][top]; experts and beyond: an identity expert
+    float* weights;                       // [n][top]
+    uint32_t n, d, experts, identity, top;
+    float eps;
+};
+void launch_router(const RouterArgs& a, cudaStream_t s);
+struct SortArgs {
+    const uint32_t* ids;
+    uint32_t *src, *place;                // row -> token, (token, choice) -> row
+    uint32_t *tiles, *n_tiles;
+    uint32_t n, top, experts, tile;
+};
+void launch_expert_sort(const SortArgs& a, cudaStream_t s);
+struct CombineArgs {
+    const float *x, *y, *xn, *shared;     // the stream, the experts' rows, the normed stream, the shared expert's rows (optional)
+    const uint32_t *ids, *place;
+    const float* weights;
+    float* out;                           // may be x
+    const uint16_t* norm;                 // optional: the next layer's norm, into next / next_b
+    float* next;
+    uint16_t* next_b;
+    uint32_t d, experts, top;
+    float eps;
+};
+void launch_combine(const CombineArgs& a, uint32_t n, cudaStream_t s);
 
 // row_skip (optional): rows marked 1 are left untouched (another rule decides them).
 void launch_sample(const float* logits, const SampleRow* rows, uint32_t* out, const uint32_t* meta, uint32_t n_rows, uint32_t vocab, cudaStream_t s,

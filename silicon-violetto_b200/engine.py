@@ -22,6 +22,7 @@ FEED_W = 16
 NO_TOK = 0xFFFFFFFF
 VERIFY_T = 8
 FLAG_HOST_ONLY = 1
+FLAG_FP32 = 2
 
 
 class EngineError(RuntimeError):
@@ -62,7 +63,7 @@ class _StepOutput(C.Structure):
 
 class _LayerCapture(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("layer", "n", "d_model", "qkv_width", "attn_width")] + \
-               [(n, C.POINTER(C.c_float)) for n in ("resid_in", "attn_in", "qkv", "sdpa_out", "attn_out", "mlp_in", "mlp_out", "resid_base")]
+               [(n, C.POINTER(C.c_float)) for n in ("resid_in", "attn_in", "qkv", "sdpa_out", "attn_out", "mlp_in", "mlp_out", "resid_base", "resid_out")]
 
 
 _CAPTURE_FN = C.CFUNCTYPE(None, C.POINTER(_LayerCapture), C.c_void_p)
@@ -126,6 +127,7 @@ class EngineConfig:
     max_head_rows: int = 64
     device_ordinal: int = 0
     host_only: bool = False
+    fp32: bool = False  # everything in 32-bit (architectures that have such a path)
 
 
 @dataclass
@@ -187,7 +189,7 @@ class Engine:
         cfg = cfg or EngineConfig()
         t = tuning or Tuning()
         c = _Config(cfg.max_seqs, cfg.max_step_tokens, cfg.max_chunk, cfg.global_kv_tokens, cfg.max_seq_len, cfg.max_head_rows, cfg.device_ordinal,
-                    FLAG_HOST_ONLY if cfg.host_only else 0)
+                    (FLAG_HOST_ONLY if cfg.host_only else 0) | (FLAG_FP32 if cfg.fp32 else 0))
         ct = _Tuning(t.spec_tokens, t.spec_tokens_short, t.spec_kv, t.spec_rows_long, int(t.spec_policy_off), t.sm_count, t.attn_keys_per_cta,
                      t.gemm_min_rows, int(t.plain_attention), int(t.gemm_unpaired))
         self.h = C.c_void_p()
@@ -293,6 +295,19 @@ class Engine:
         _check(lib().vlt_step(self.h, arr, C.c_uint32(len(runs)), C.byref(co), C.byref(out)))
         return self._result(out, bufs, n, opts)
 
+    def step_rows(self, runs, want, opts: StepOptions | None = None) -> StepOutput:
+        """A synchronous step whose head rows are listed per run: want[i] holds places among run i's tokens."""
+        opts = opts or StepOptions()
+        arr, keep = self._runs(runs)
+        n = sum(len(k) for k in keep)
+        rows = [_u32(w) for w in want]
+        ptrs = (C.POINTER(C.c_uint32) * len(rows))(*[_ptr(r) for r in rows])
+        counts = _u32([r.size for r in rows])
+        co = _StepOptions(0, opts.hidden, int(opts.read_logits), int(opts.read_taps))
+        out, bufs = self._out(n, opts)
+        _check(lib().vlt_step_rows(self.h, arr, C.c_uint32(len(runs)), ptrs, _ptr(counts), C.byref(co), C.byref(out)))
+        return self._result(out, bufs, n, opts)
+
     def step_capture(self, runs, opts: StepOptions | None = None):
         """engine.rs:318-355: a step that hands every layer's intermediates back. Returns (StepOutput, [layer dicts]) with
         each dict's arrays shaped [n][width]."""
@@ -305,8 +320,9 @@ class Engine:
 
         def take(pc, _user):
             c = pc.contents
-            widths = dict(resid_in=c.d_model, attn_in=c.d_model, qkv=c.qkv_width, sdpa_out=c.attn_width, attn_out=c.d_model, mlp_in=c.d_model, mlp_out=c.d_model)
-            layers.append({"layer": c.layer, **{k: np.ctypeslib.as_array(getattr(c, k), shape=(c.n, w)).copy() for k, w in widths.items()}})
+            widths = dict(resid_in=c.d_model, attn_in=c.d_model, qkv=c.qkv_width, sdpa_out=c.attn_width, attn_out=c.d_model, mlp_in=c.d_model, mlp_out=c.d_model,
+                          resid_out=c.d_model)
+            layers.append({"layer": c.layer, **{k: np.ctypeslib.as_array(getattr(c, k), shape=(c.n, w)).copy() for k, w in widths.items() if getattr(c, k)}})
 
         cb = _CAPTURE_FN(take)
         _check(lib().vlt_step_capture(self.h, arr, C.c_uint32(len(runs)), C.byref(co), cb, None, C.byref(out)))

@@ -114,6 +114,7 @@ pub struct VltLayerCapture {
     pub mlp_in: *const f32,
     pub mlp_out: *const f32,
     pub resid_base: *const f32,
+    pub resid_out: *const f32,
 }
 pub type VltCaptureFn = extern "C" fn(layer: *const VltLayerCapture, user: *mut c_void);
 #[repr(C)]
