@@ -314,6 +314,100 @@ def limite_figure(E, local, ctx, steps=30, stream_counts=(1, 8, 32), keys_per_bl
     return out
 
 
+LONASUN = dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=8192, experts=64, top=8, ff=1024, shared=1024, vocab=32768, layers=4)
+
+
+def lonasun_files():
+    """A Lonasun model whose layers resemble a real model's (width 2048, 16 / 4 heads of 128, 64 experts of 1024 with 8 a
+    token, a shared one), four of them, and the plain decoder of equal size beside it: the same query and key / value widths
+    (32 / 8 heads of 64) and a dense feed-forward with the parameters one token uses (two matrices of 9 x 1024 there are three
+    of 6144 here). Random-init, bf16."""
+    from silicon_violetto_b200 import lonasun, synth
+    CACHE.mkdir(parents=True, exist_ok=True)
+    c = LONASUN
+    moe = dict(experts=c["experts"], top=c["top"], ff=c["ff"], shared=c["shared"], identity=0)
+    cfg = lonasun.config(c["width"], c["vocab"], [lonasun.layer(c["heads"], c["kv_heads"], c["dim"], c["vdim"], c["chunk"], conv=4, rot_dims=64, base=500000.0, moe=moe)] * c["layers"])
+    folder = CACHE / "lonasun_4x2048"
+    if not (folder / "ok").exists():
+        lonasun.write_model(folder, cfg, lonasun.random_weights(cfg))
+        (folder / "ok").write_text("ok")
+    plain = CACHE / "plain_4x2048.vlt"
+    if not plain.with_suffix(".ok").exists():
+        synth.write_target(plain, dict(n_layers=c["layers"], d=c["width"], n_heads=32, n_kv=8, hd=64, ffn=6144, vocab=c["vocab"], eps=1e-5, theta=500000.0, page=16), seed=0)
+        plain.with_suffix(".ok").write_text("ok")
+    return folder, plain
+
+
+def lonasun_figure(E, local, ctx, steps, stream_counts, hbm_peak, tc_peak):
+    """Decoding over a filled context of `ctx` positions and a `ctx`-token prompt in chunks of 512, the Lonasun model and the
+    plain decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their
+    own) the fraction of the measured copy bandwidth or bf16 throughput its algorithmic bytes or FLOPs make."""
+    c, L = LONASUN, LONASUN["layers"]
+    folder, plain = lonasun_files()
+    attn_w = (c["heads"] + c["kv_heads"]) * c["dim"] + c["kv_heads"] * c["vdim"]
+    o_p = c["heads"] * c["vdim"] * c["width"]
+    expert_p = 2 * c["ff"] * c["width"]
+    weights = {"lonasun": lambda touched: L * ((attn_w + c["heads"] * c["vdim"]) * c["width"] + o_p + (touched + 1) * expert_p),
+               "plain": lambda touched: L * (attn_w * c["width"] + o_p + 3 * 6144 * c["width"])}
+    kv_row = c["kv_heads"] * (c["dim"] + c["vdim"]) * 2
+    out = {"workload": f"{L} layers x {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in chunks of 512"}
+    for name, path in (("lonasun", folder), ("plain", plain)):
+        res = out[name] = {}
+        for n_s in stream_counts:
+            eng = E.Engine(path, E.EngineConfig(max_seqs=n_s, max_step_tokens=max(64, n_s), max_chunk=32, global_kv_tokens=n_s * (ctx + 192), max_seq_len=ctx + 128,
+                                                max_head_rows=max(8, n_s), device_ordinal=local), E.Tuning(spec_policy_off=True))
+            seqs = [eng.new_seq() for _ in range(n_s)]
+            for i, s_ in enumerate(seqs):
+                eng.bench_fill(s_, ctx, seed=1 + i)
+            with eng.generator() as g, Clocks(local) as clocks:
+                for j, s_ in enumerate(seqs):
+                    g.submit(E.Request(("resume", s_, 100 + j), 2 * steps + 16, sampling=E.Sampling(0.6, 0.95, 1 + j)))
+                for _ in range(5):
+                    g.step()
+                eng.mark(0)
+                for _ in range(steps):
+                    g.step()
+                eng.mark(1)
+                g.step()
+                ms = eng.mark_elapsed_ms() / steps
+                eng.profile_read()
+                eng.set_profile(True)
+                for _ in range(steps):
+                    g.step()
+                prof = eng.profile_read()
+                eng.set_profile(False)
+            eng.close()
+            touched = c["experts"] * (1 - (1 - c["top"] / c["experts"]) ** n_s)  # experts a step of n_s tokens reads, on average
+            wb, kb = 2 * weights[name](touched), n_s * ctx * kv_row * L
+            gms = {k: v["ms"] / steps for k, v in prof.items()}
+            res[f"decode_{n_s}"] = {"ms_per_step": ms, "tokens_per_s": n_s / (ms * 1e-3), "groups_ms": gms, "weight_bytes": wb, "kv_bytes": kb, "clocks": clocks.summary(),
+                                    "matmul_frac_hbm": wb / (gms["matmul"] * 1e-3) / 1e9 / hbm_peak, "attention_frac_hbm": kb / (gms["attention"] * 1e-3) / 1e9 / hbm_peak,
+                                    "step_frac_hbm": (wb + kb) / (ms * 1e-3) / 1e9 / hbm_peak}
+        eng = E.Engine(path, E.EngineConfig(max_seqs=1, max_step_tokens=512, max_chunk=512, global_kv_tokens=ctx + 128, max_seq_len=ctx + 64, max_head_rows=8, device_ordinal=local),
+                       E.Tuning(spec_policy_off=True))
+        prompt = [int(x) for x in np.random.default_rng(7).integers(0, eng.desc.vocab, ctx)]
+        for turn in ("warm", "timed", "groups"):
+            if turn == "groups":
+                eng.profile_read()
+                eng.set_profile(True)
+            with eng.generator() as g:
+                g.submit(E.Request(prompt, 1))
+                eng.mark(0)
+                while not g.is_idle():
+                    g.step()
+                eng.mark(1)
+                if turn == "timed":
+                    ms = eng.mark_elapsed_ms()
+            if turn == "groups":
+                gms = {k: v["ms"] for k, v in eng.profile_read().items()}
+                eng.set_profile(False)
+        eng.close()
+        mm, at = 2.0 * ctx * weights[name](c["top"]), L * 2.0 * c["heads"] * (c["dim"] + c["vdim"]) * ctx * ctx / 2
+        res["prefill"] = {"ms": ms, "tokens_per_s": ctx / (ms * 1e-3), "groups_ms": gms, "matmul_frac_tc": mm / (gms["matmul"] * 1e-3) / 1e12 / tc_peak,
+                          "attention_frac_tc": at / (gms["attention"] * 1e-3) / 1e12 / tc_peak}
+    return out
+
+
 def prefill_figure(E, path, ctx, local, chunk=512):
     """A `ctx`-token prompt of the reference's LCG ids computed in chunks of `chunk` tokens through the generator (the
     tensor-core GEMM in blocks of 256 tokens, the chunk attention kernel), one stream; device time from the first chunk's
@@ -362,11 +456,11 @@ def main():
     ap.add_argument("--attn-keys", type=int, default=0, help="keys per attention block (0: the engine's own choice)")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers: a profiler-size case, not a bench value")
     ap.add_argument("--no-limite", action="store_true", help="skip the reference-architecture pass of the extras (it writes a 2 GB file first)")
-    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite")
+    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite and --only lonasun")
     ap.add_argument("--limite-drafter", action="store_true", help="--only limite: with the reference's block drafter loaded (tree drafts of up to 8 rows)")
     ap.add_argument("--limite-int8", action="store_true", help="--only limite: int8 weights in the reference converter's default groups (64; the head 8)")
     ap.add_argument("--limite-keys", type=int, default=0, help="--only limite: keys per attention block (VltTuning.attn_keys_per_cta); 0 = the library's choice")
-    ap.add_argument("--only", default="", help="'prefill', 'acceptance' or 'limite' (the reference's own architecture at its shapes, decoding): run that one pass alone and print its figure (not the bench line)")
+    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) or 'lonasun' (a Lonasun model beside a plain decoder of equal size): run that one pass alone and print its figure (not the bench line)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank, world, local = int(os.environ.get("RANK", 0)), int(os.environ.get("WORLD_SIZE", 1)), int(os.environ.get("LOCAL_RANK", 0))
@@ -412,6 +506,10 @@ def main():
     solo = lambda: torch.cuda.synchronize(local)
     _package()
     from silicon_violetto_b200 import engine as E
+    if args.only == "lonasun":
+        peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+        print(json.dumps(lonasun_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], hbm_peak, peaks.get("bf16_tflops", 1590.0))))
+        return
     path = model_file("1b", not args.bf16, rank, args.layers)
     if args.only:
         if args.only == "prefill":
@@ -422,7 +520,7 @@ def main():
         elif args.only == "limite":
             print(json.dumps(limite_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], args.limite_keys, args.limite_drafter, args.limite_int8)))
         else:
-            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance' or 'limite'")
+            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite' or 'lonasun'")
         return
     total = args.warmup + args.steps + 6
     # The headline pass, on every rank: the int8 target with the chain drafter loaded (1 layer + fc + a head over 16 384 draft

@@ -176,13 +176,18 @@ void Engine::encode_forward_lonasun(uint32_t set, const Plan& p, const std::func
         c.heads = a.heads;
         c.rot_dims = a.rot.dims;
         c.write_ring = short_runs;
-        c.q_f = z.q_f.as<float>();
+        const bool fast_attn = !f32 && !tuning.plain_attention && chunk_attn_fits(a.dim, a.vdim, md.page);
+        if (fast_attn) c.q_b = z.q_b.as<uint16_t>();
+        else c.q_f = z.q_f.as<float>();
+        c.q_scale = a.scale * LOG2E;
         sp = span_begin(G_SMALL);
         launch_conv_qkv(c, n, f32, stream);
         if (!short_runs) launch_conv_state(c, st.in<RunIn>(st.o_runs), p.n_runs, stream);
         span_end(sp);
         ChunkedAttnArgs at{};
         at.q_f = z.q_f.as<float>();
+        at.q_b = z.q_b.as<uint16_t>();
+        at.ctiles = st.in<uint32_t>(st.o_ctiles);
         at.meta = c.meta;
         at.tin = c.tin;
         at.vis = c.vis;
@@ -195,7 +200,8 @@ void Engine::encode_forward_lonasun(uint32_t set, const Plan& p, const std::func
         at.out = f32 || capture ? z.attn_f.as<float>() : nullptr;
         at.out_b = z.attn_b.as<uint16_t>();
         sp = span_begin(G_ATTN);
-        launch_attn_any(at, n, f32, stream);
+        if (fast_attn) launch_attn_chunked(at, n, p.chunked ? p.ctiles : 0, a.chunk ? std::min(p.max_keys, a.chunk) : p.max_keys, sm_count, tuning.attn_keys_per_cta, stream);
+        else launch_attn_any(at, n, f32, stream);
         span_end(sp);
         if (capture) sdpa = host(z.attn_f.as<float>(), size_t(n) * a.out_w());
         sp = span_begin(G_MATMUL);
@@ -271,7 +277,12 @@ void Engine::encode_experts(const LonasunLayer& l, uint32_t n, const uint16_t* n
     so.n = n;
     so.top = e.top;
     so.experts = e.experts;
-    so.tile = EXPERT_TILE_MIN;
+    // The experts' matrices on the tensor cores where their sizes fit: tiles as long as an expert's rows on average, so that
+    // its weights are read once. On the CUDA cores a tile has 64.
+    const bool fast = !f32 && grouped_fits(e.ff, d) && grouped_fits(d, e.ff);
+    so.tile = 64;
+    if (fast)
+        for (so.tile = EXPERT_TILE_MIN; so.tile < 128 && so.tile < 2 * pairs / (e.experts + e.identity);) so.tile *= 2;
     int sp = span_begin(G_SMALL);
     launch_router(r, stream);
     launch_expert_sort(so, stream);
@@ -289,7 +300,8 @@ void Engine::encode_experts(const LonasunLayer& l, uint32_t n, const uint16_t* n
     up.tiles = so.tiles;
     up.n_tiles = so.n_tiles;
     up.max_tiles = pairs / so.tile + std::min(e.experts, pairs);
-    launch_linear(up, !f32, stream);
+    if (fast) launch_grouped(up, e.experts, so.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(up, !f32, stream);
     LinearArgs down = up;
     down.W = reinterpret_cast<const uint16_t*>(e.down.w);
     down.X = f32 ? static_cast<const void*>(z.hid_f.as<float>()) : z.hid_b.as<uint16_t>();
@@ -299,7 +311,8 @@ void Engine::encode_experts(const LonasunLayer& l, uint32_t n, const uint16_t* n
     down.m = d;
     down.k = e.ff;
     down.epi = EPI_RAW;
-    launch_linear(down, !f32, stream);
+    if (fast) launch_grouped(down, e.experts, so.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(down, !f32, stream);
     if (e.shared_ff) {
         project(e.shared_up, n, z.moe_x.as<float>(), z.moe_xb.as<uint16_t>(), z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), EPI_RELU2);
         project(e.shared_down, n, z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), z.shared.as<float>(), nullptr, EPI_RAW);

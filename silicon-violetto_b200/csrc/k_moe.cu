@@ -9,14 +9,12 @@ namespace vlt {
 
 namespace moe {
 
-constexpr uint32_t ROUTER_THREADS = 256;
-
 // One block per TOK tokens: the RMS norm of their rows (kept for the experts), the scores' logits with a warp per output,
 // softmax and the choice with a warp per token. Ties go to the lower index.
-template <uint32_t TOK>
+template <uint32_t TOK, uint32_t ROUTER_THREADS>
 __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs a) {
     pdl_start();
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     constexpr uint32_t NW = ROUTER_THREADS / 32;
     const uint32_t t0 = blockIdx.x * TOK, tid = threadIdx.x, warp = tid / 32, lane = tid % 32, nt = min(TOK, a.n - t0);
     float *x = sm, *z = sm + TOK * a.d;  // the normed rows, the scores
@@ -30,6 +28,8 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
                 x[j * a.d + i] = v;
                 ss += v * v;
             }
+        else
+            for (uint32_t i = tid; i < a.d; i += ROUTER_THREADS) x[j * a.d + i] = 0.0f;
         ss = warp_sum(ss);
         if (lane == 0) red[j][warp] = ss;
     }
@@ -53,7 +53,30 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
     for (uint32_t e = warp; e < all; e += NW) {
         float s[TOK] = {};
         const uint16_t* w = a.router + size_t(e) * a.d;
-        for (uint32_t i = lane; i < a.d; i += 32) {
+        uint32_t done = 0;
+        if (a.d % 8 == 0) {  // eight weights a load, several loads together
+            const uint4* w8 = reinterpret_cast<const uint4*>(w);
+            const uint32_t groups = a.d / 8;
+            constexpr uint32_t U = TOK == 1 ? 8 : 4;
+            for (uint32_t g0 = lane; g0 < groups; g0 += 32 * U) {
+                uint4 v[U];
+#pragma unroll
+                for (uint32_t u = 0; u < U; u++) v[u] = g0 + 32 * u < groups ? __ldg(w8 + g0 + 32 * u) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                for (uint32_t u = 0; u < U; u++) {
+                    if (g0 + 32 * u >= groups) break;
+#pragma unroll
+                    for (uint32_t j = 0; j < TOK; j++) {
+                        const float4* xp = reinterpret_cast<const float4*>(x + j * a.d + (g0 + 32 * u) * 8);
+                        const float4 xa = xp[0], xb = xp[1];
+                        s[j] = fmaf(bf16lo(v[u].x), xa.x, fmaf(bf16hi(v[u].x), xa.y, fmaf(bf16lo(v[u].y), xa.z, fmaf(bf16hi(v[u].y), xa.w, s[j]))));
+                        s[j] = fmaf(bf16lo(v[u].z), xb.x, fmaf(bf16hi(v[u].z), xb.y, fmaf(bf16lo(v[u].w), xb.z, fmaf(bf16hi(v[u].w), xb.w, s[j]))));
+                    }
+                }
+            }
+            done = a.d;
+        }
+        for (uint32_t i = done + lane; i < a.d; i += 32) {
             const float wv = bf16_to_f32(w[i]);
 #pragma unroll
             for (uint32_t j = 0; j < TOK; j++)
@@ -158,24 +181,55 @@ __global__ void __launch_bounds__(1024) sort_kernel(const SortArgs a) {
 }
 
 // out[t] = x[t] + sum_k weight_k (expert k's row, or the token's own normed row for an identity expert) + the shared
-// expert's row, in the order of the choice; and, if asked, the next layer's RMS norm of it. A block per token.
+// expert's row, in the order of the choice; and, if asked, the next layer's RMS norm of it. A block per token; V: the
+// columns a thread takes at a time.
+template <typename V>
+__device__ __forceinline__ void fma_v(V& y, float w, const V& v);
+template <>
+__device__ __forceinline__ void fma_v<float>(float& y, float w, const float& v) { y = fmaf(w, v, y); }
+template <>
+__device__ __forceinline__ void fma_v<float4>(float4& y, float w, const float4& v) {
+    y.x = fmaf(w, v.x, y.x);
+    y.y = fmaf(w, v.y, y.y);
+    y.z = fmaf(w, v.z, y.z);
+    y.w = fmaf(w, v.w, y.w);
+}
+__device__ __forceinline__ float square(float y) { return y * y; }
+__device__ __forceinline__ float square(const float4& y) { return (y.x * y.x + y.y * y.y) + (y.z * y.z + y.w * y.w); }
+
+template <typename V>
 __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     pdl_start();
+    extern __shared__ __align__(16) float row[];  // the new row, then the choices' weights and rows
+    constexpr uint32_t W = sizeof(V) / 4;
     __shared__ float red[8];
-    const uint32_t t = blockIdx.x, tid = threadIdx.x;
+    const uint32_t t = blockIdx.x, tid = threadIdx.x, dv = a.d / W;
+    float* wt = row + (a.d + 3) / 4 * 4;
+    const float** src = reinterpret_cast<const float**>(wt + (a.top + 1) / 2 * 2);
+    for (uint32_t k = tid; k < a.top; k += 256) {
+        const size_t i = size_t(t) * a.top + k;
+        wt[k] = a.weights[i];
+        src[k] = a.ids[i] < a.experts ? a.y + size_t(a.place[i]) * a.d : a.xn + size_t(t) * a.d;
+    }
+    __syncthreads();
+    const V one{};
     float ss = 0.0f;
-    for (uint32_t i = tid; i < a.d; i += 256) {
-        const size_t o = size_t(t) * a.d + i;
-        float y = 0.0f;
-        for (uint32_t k = 0; k < a.top; k++) {
-            const uint32_t e = a.ids[size_t(t) * a.top + k];
-            const float w = a.weights[size_t(t) * a.top + k];
-            y = fmaf(w, e < a.experts ? a.y[size_t(a.place[size_t(t) * a.top + k]) * a.d + i] : a.xn[o], y);
+    for (uint32_t i = tid; i < dv; i += 256) {
+        V y = one, x = reinterpret_cast<const V*>(a.x + size_t(t) * a.d)[i], sh = one;
+        if (a.shared) sh = reinterpret_cast<const V*>(a.shared + size_t(t) * a.d)[i];
+        for (uint32_t k0 = 0; k0 < a.top; k0 += 8) {
+            V v[8];
+#pragma unroll
+            for (uint32_t u = 0; u < 8; u++) v[u] = k0 + u < a.top ? reinterpret_cast<const V*>(src[k0 + u])[i] : one;
+#pragma unroll
+            for (uint32_t u = 0; u < 8; u++)
+                if (k0 + u < a.top) fma_v(y, wt[k0 + u], v[u]);
         }
-        if (a.shared) y += a.shared[o];
-        y += a.x[o];
-        a.out[o] = y;
-        ss += y * y;
+        fma_v(y, 1.0f, sh);
+        fma_v(y, 1.0f, x);
+        reinterpret_cast<V*>(a.out + size_t(t) * a.d)[i] = y;
+        reinterpret_cast<V*>(row)[i] = y;
+        ss += square(y);
     }
     if (!a.norm) return;
     ss = warp_sum(ss);
@@ -186,7 +240,7 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
     for (uint32_t i = tid; i < a.d; i += 256) {
         const size_t o = size_t(t) * a.d + i;
-        const float v = a.out[o] * inv * (1.0f + bf16_to_f32(a.norm[i]));
+        const float v = row[i] * inv * (1.0f + bf16_to_f32(a.norm[i]));
         if (a.next) a.next[o] = v;
         if (a.next_b) a.next_b[o] = f32_to_bf16(v);
     }
@@ -198,14 +252,26 @@ void launch_router(const RouterArgs& a, cudaStream_t s) {
     const uint32_t all = a.experts + a.identity;
     static PerDevice configured;
     configured.once([] {
-        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<1, 1024>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<1, 512>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<4, 512>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     });
     // Many tokens share a read of the router's matrix, four a block; few spread over the SMs one by one.
-    if (a.n >= 592 && (size_t(a.d) + all) * 16 <= 100 * 1024) launch_pdl(moe::router_kernel<4>, (a.n + 3) / 4, moe::ROUTER_THREADS, (size_t(a.d) + all) * 16, s, a);
-    else launch_pdl(moe::router_kernel<1>, a.n, moe::ROUTER_THREADS, (size_t(a.d) + all) * 4, s, a);
+    const size_t one = (size_t(a.d) + all) * 4;
+    if (a.n >= 256 && one <= 25 * 1024) launch_pdl(moe::router_kernel<4, 512>, (a.n + 3) / 4, 512, 4 * one, s, a);
+    else if (a.n > 148) launch_pdl(moe::router_kernel<1, 512>, a.n, 512, one, s, a);
+    else launch_pdl(moe::router_kernel<1, 1024>, a.n, 1024, one, s, a);
 }
 void launch_expert_sort(const SortArgs& a, cudaStream_t s) { launch_pdl(moe::sort_kernel, 1, 1024, size_t(a.experts) * 12, s, a); }
-void launch_combine(const CombineArgs& a, uint32_t n, cudaStream_t s) { launch_pdl(moe::combine_kernel, n, 256, 0, s, a); }
+void launch_combine(const CombineArgs& a, uint32_t n, cudaStream_t s) {
+    const size_t smem = (size_t(a.d) + 3) / 4 * 16 + (size_t(a.top) + 1) / 2 * 8 + size_t(a.top) * 8;
+    static PerDevice configured;
+    configured.once([] {
+        VLT_CUDA(cudaFuncSetAttribute(moe::combine_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        VLT_CUDA(cudaFuncSetAttribute(moe::combine_kernel<float4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    if (a.d % 4 == 0) launch_pdl(moe::combine_kernel<float4>, n, 256, smem, s, a);
+    else launch_pdl(moe::combine_kernel<float>, n, 256, smem, s, a);
+}
 
 }  // namespace vlt

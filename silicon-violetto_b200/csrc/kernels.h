@@ -213,6 +213,8 @@ struct LinearArgs {
     uint32_t max_tiles;      // at most so many tiles (the grid)
 };
 void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s);
+bool grouped_fits(uint32_t m, uint32_t k);  // the tensor-core form (k_grouped.cu): bf16 activations, EPI_RAW or EPI_RELU2
+void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint32_t* err_flag, cudaStream_t s);
 void launch_norm_rows(const float* in, const uint32_t* rows, uint32_t n, uint32_t k, float eps, const uint16_t* w, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
 
@@ -248,6 +250,7 @@ struct ChunkedAttnArgs {
     const float* q_f;                     // the scalar kernel's q
     const uint16_t* q_b;                  // the tensor-core kernels' q, scale * log2(e) folded in
     const uint32_t *meta, *tin, *vis;
+    const uint32_t* ctiles;               // the prefill kernel's (first token, rows <= 64) tiles
     PagedKv kv;
     const float* gate;                    // [n][ldg]: the output is multiplied by sigmoid(gate)
     uint32_t ldg, heads, chunk;           // chunk 0: every position before
@@ -255,6 +258,8 @@ struct ChunkedAttnArgs {
     float* out;                           // optional [n][heads][dv]
     uint16_t* out_b;                      // optional
 };
+bool chunk_attn_fits(uint32_t dk, uint32_t dv, uint32_t page);  // k_chunk_attn.cu's kernels, bf16 caches; else launch_attn_any
+void launch_attn_chunked(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s);
 void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_layers,
                           bool fp32, cudaStream_t s);
