@@ -125,6 +125,7 @@ class GenerateArgs:
     temperature: float = 0.6
     top_p: float = 0.95
     seed: int = 0
+    fp32: bool = False  # everything in 32-bit, for architectures that have such a path
 
 
 def generate(weights, a: GenerateArgs, tuning: E.Tuning | None = None) -> dict:
@@ -146,7 +147,7 @@ def generate(weights, a: GenerateArgs, tuning: E.Tuning | None = None) -> dict:
     drafts = bool(a.replay or a.drafter)
     cfg = E.EngineConfig(max_seqs=max_seqs, max_step_tokens=max(a.chunk, max_seqs), max_chunk=a.chunk,
                          global_kv_tokens=a.kv_tokens or max_seqs * (-(-longest // 128) * 128 + (16 if a.drafter else 0)), max_seq_len=longest,
-                         max_head_rows=max_seqs * (a.spec_rows if drafts else 1))
+                         max_head_rows=max_seqs * (a.spec_rows if drafts else 1), fp32=a.fp32)
     eng = E.Engine(weights, cfg, tuning)
     if a.drafter:
         eng.load_drafter(a.drafter)
