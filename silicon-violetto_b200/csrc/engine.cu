@@ -479,9 +479,9 @@ void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint3
 }
 
 // Whether the streamed kernel itself (not its scalar stand-in) takes this matrix.
-bool Engine::stream_fits(const Matrix& w) const {
+bool Engine::stream_fits(const Matrix& w, uint32_t n) const {
     MatArgs a{};
-    a.n = 1;
+    a.n = n;
     a.k = w.k;
     a.m = w.m;
     a.group = w.group;

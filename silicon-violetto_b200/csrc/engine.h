@@ -307,7 +307,7 @@ class Engine {
     KvArgs kv_args() const;
     void matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint32_t epi, const float* base, float* inv_out, uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr,
                 const uint16_t* xb = nullptr, uint16_t* yb = nullptr, float scale = 1.0f, float ra = 1.0f, float rb = 1.0f);
-    bool stream_fits(const Matrix& w) const;
+    bool stream_fits(const Matrix& w, uint32_t n = 1) const;
     // The tensor-core GEMM: xb is x in bf16, inv the rows' 1/rms (normed epilogues), yb an optional bf16 copy of y.
     void matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, const float* inv,
                      uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr, float* ssq_out = nullptr, const float* ssq_in = nullptr, float scale = 1.0f, float ra = 1.0f,

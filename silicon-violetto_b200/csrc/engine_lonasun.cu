@@ -100,7 +100,7 @@ void Engine::init_lonasun() {
 void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base) {
     if (!cfg.fp32 && gemm_fits(w, n)) {
         matmul_gemm(w, n, xb, y, yb, epi, base, nullptr);
-    } else if (!cfg.fp32 && n <= 8 && stream_fits(w)) {
+    } else if (!cfg.fp32 && stream_fits(w, n)) {
         matmul(w, n, nullptr, y, epi, base, nullptr, 0, nullptr, xb, yb);
     } else {
         LinearArgs a{};

@@ -7,7 +7,8 @@
 //                         copies; a row's keys may be split over a cluster of blocks, whose first adds up what the others
 //                         store into its shared memory.
 //   chunk_prefill_kernel  64 rows of a run and one query head per block: the rows are the M side, the keys come a page at a
-//                         time; the softmax stays in registers.
+//                         time, every other page to each of two groups of four warps, which meet at the end (a prompt's portion
+//                         has few blocks for its SMs); the softmax stays in registers.
 //
 // Both take q rotated, scaled by scale * log2(e) and rounded to bf16, keep scores and softmax in fp32, and finish the mixer:
 // the output times sigmoid(gate), bf16 for the projection after it.
@@ -266,19 +267,22 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
     }
 }
 
-constexpr uint32_t CQ = 64, CK = PAGE;
+constexpr uint32_t CK = PAGE, GROUPS = 2;
 template <uint32_t DK, uint32_t DV>
 constexpr uint32_t prefill_stages() { return DK + DV > 128 ? 2 : 3; }
-
-// grid (chunk tiles, query heads), 128 threads: warp w has rows 16 w .. 16 w + 15 of the tile.
 template <uint32_t DK, uint32_t DV>
-__global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const ChunkedAttnArgs a) {
+constexpr uint32_t prefill_smem() { return GROUPS * prefill_stages<DK, DV>() * CK * (DK + DV) * 2; }
+
+// grid (chunk tiles, query heads), 256 threads: warp w of a group has rows 16 w .. 16 w + 15 of the tile.
+template <uint32_t DK, uint32_t DV>
+__global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(const ChunkedAttnArgs a) {
     pdl_start();
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr uint32_t KB = CK * DK * 2, VB = CK * DV * 2, KS = DK / 16, ND = DV / 8, KC = DK / 8, VC = DV / 8, ST = prefill_stages<DK, DV>();
     __shared__ uint32_t lows[WARPS], ends[WARPS];
+    static_assert(64 * (DV + 4) * 4 <= prefill_smem<DK, DV>() / GROUPS, "the second group's sums must fit in a ring");
     const uint32_t tile = blockIdx.x, h = blockIdx.y, kvh = h / (a.heads / a.kv.n_kv);
-    const uint32_t tid = threadIdx.x, warp = tid / 32, lane = tid % 32, g = lane >> 2, tq = lane & 3;
+    const uint32_t grp = threadIdx.x / (WARPS * 32), tid = threadIdx.x % (WARPS * 32), warp = tid / 32, lane = tid % 32, g = lane >> 2, tq = lane & 3;
     const uint32_t t0 = a.ctiles[2 * tile], rows = a.ctiles[2 * tile + 1];
     uint32_t tok[2], low = 0xffffffffu, end = 0;
     bool live[2];
@@ -299,17 +303,18 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const Chunked
         low = min(low, __shfl_xor_sync(0xffffffffu, low, o));
         end = max(end, __shfl_xor_sync(0xffffffffu, end, o));
     }
-    if (lane == 0) { lows[warp] = low; ends[warp] = end; }
+    if (lane == 0 && grp == 0) { lows[warp] = low; ends[warp] = end; }
     __syncthreads();
-    const uint32_t b0 = min(min(lows[0], lows[1]), min(lows[2], lows[3])) / CK, b1 = (max(max(ends[0], ends[1]), max(ends[2], ends[3])) + CK - 1) / CK;
+    const uint32_t b0 = min(min(lows[0], lows[1]), min(lows[2], lows[3])) / CK + grp, b1 = (max(max(ends[0], ends[1]), max(ends[2], ends[3])) + CK - 1) / CK;
 
     const uint32_t* pages = a.kv.page_table + size_t(v[0].slot) * a.kv.max_pages;
     const uint16_t* K = static_cast<const uint16_t*>(a.kv.k);
     const uint16_t* V = static_cast<const uint16_t*>(a.kv.v);
-    const uint32_t ring = smem_u32(smem);
+    const uint32_t ring = smem_u32(smem) + grp * ST * (KB + VB);
+    auto group_sync = [&] { asm volatile("bar.sync %0, %1;" ::"r"(1 + grp), "n"(WARPS * 32) : "memory"); };
     auto issue = [&](uint32_t b) {  // a page of keys
         const size_t r0 = (size_t(pages[b]) * a.kv.n_kv + kvh) << PAGE_SHIFT;
-        const uint32_t dst = ring + (b - b0) % ST * (KB + VB);
+        const uint32_t dst = ring + (b - b0) / GROUPS % ST * (KB + VB);
 #pragma unroll
         for (uint32_t c = tid; c < CK * KC; c += WARPS * 32) {
             const uint32_t key = c / KC, piece = c % KC;
@@ -323,7 +328,7 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const Chunked
     };
 #pragma unroll
     for (uint32_t i = 0; i < ST; i++) {
-        if (b0 + i < b1) issue(b0 + i);
+        if (b0 + i * GROUPS < b1) issue(b0 + i * GROUPS);
         cp_async_commit();
     }
     uint32_t qa[KS][4];
@@ -343,10 +348,10 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const Chunked
 #pragma unroll
     for (uint32_t j = 0; j < ND; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
     const uint32_t lo_max = max(v[0].lo, v[1].lo), first_min = min(v[0].first, v[1].first);
-    for (uint32_t b = b0; b < b1; b++) {
+    for (uint32_t b = b0; b < b1; b += GROUPS) {
         cp_async_wait<ST - 1>();
-        __syncthreads();  // everybody's copies of the page are in
-        const uint32_t kbase = ring + (b - b0) % ST * (KB + VB), vbase = kbase + KB, key0 = b * CK;
+        group_sync();  // everybody's copies of the page are in
+        const uint32_t kbase = ring + (b - b0) / GROUPS % ST * (KB + VB), vbase = kbase + KB, key0 = b * CK;
         if (key0 < ends[warp] && key0 + CK > lows[warp]) {  // (a warp whose rows see nothing of the page skips the arithmetic, not the barriers)
             float s[8][4];
 #pragma unroll
@@ -412,16 +417,41 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const Chunked
                 }
             }
         }
-        __syncthreads();  // every warp is done with the stage
-        if (b + ST < b1) issue(b + ST);
+        group_sync();  // every warp of the group is done with the stage
+        if (b + ST * GROUPS < b1) issue(b + ST * GROUPS);
         cp_async_commit();
     }
     cp_async_wait<0>();
 #pragma unroll
     for (int r = 0; r < 2; r++) {
-        float l = l_run[r];
-        l += __shfl_xor_sync(0xffffffffu, l, 1);
-        l += __shfl_xor_sync(0xffffffffu, l, 2);
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+    }
+    // The second group's (m, l, o) to the first through its own ring: a row's o, then m and l.
+    constexpr uint32_t OS = DV + 4;
+    float* sums = reinterpret_cast<float*>(smem + ST * (KB + VB));
+    if (grp) {
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            float* row = sums + (warp * 16 + g + 8 * r) * OS;
+#pragma unroll
+            for (uint32_t j = 0; j < ND; j++) *reinterpret_cast<float2*>(row + 8 * j + 2 * tq) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
+            if (tq == 0) { row[DV] = m_run[r]; row[DV + 1] = l_run[r]; }
+        }
+    }
+    __syncthreads();
+    if (grp) return;
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const float* row = sums + (warp * 16 + g + 8 * r) * OS;
+        const float m1 = row[DV], m = fmaxf(m_run[r], m1), w0 = m_run[r] == -INFINITY ? 0.0f : fast_exp2(m_run[r] - m), w1 = m1 == -INFINITY ? 0.0f : fast_exp2(m1 - m);
+        const float l = l_run[r] * w0 + row[DV + 1] * w1;
+#pragma unroll
+        for (uint32_t j = 0; j < ND; j++) {
+            const float2 other = *reinterpret_cast<const float2*>(row + 8 * j + 2 * tq);
+            o[j][2 * r] = o[j][2 * r] * w0 + other.x * w1;
+            o[j][2 * r + 1] = o[j][2 * r + 1] * w0 + other.y * w1;
+        }
         if (!live[r]) continue;
         const float inv = l > 0.0f ? 1.0f / l : 0.0f;
         const size_t at = (size_t(tok[r]) * a.heads + h) * DV;
@@ -439,14 +469,14 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_prefill_kernel(const Chunked
 template <uint32_t DK, uint32_t DV>
 void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t splits, cudaStream_t s) {
     static PerDevice configured;
-    constexpr uint32_t dsm = decode_smem<DK, DV>(), psm = prefill_stages<DK, DV>() * CK * (DK + DV) * 2;
+    constexpr uint32_t dsm = decode_smem<DK, DV>(), psm = prefill_smem<DK, DV>();
     configured.once([] {
         VLT_CUDA(cudaFuncSetAttribute(chunk_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(dsm)));
         VLT_CUDA(cudaFuncSetAttribute(chunk_decode_kernel<DK, DV>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
         VLT_CUDA(cudaFuncSetAttribute(chunk_prefill_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(psm)));
     });
     if (n_ctiles) {
-        launch_pdl(chunk_prefill_kernel<DK, DV>, dim3(n_ctiles, a.heads), WARPS * 32, psm, s, a);
+        launch_pdl(chunk_prefill_kernel<DK, DV>, dim3(n_ctiles, a.heads), GROUPS * WARPS * 32, psm, s, a);
         return;
     }
     const uint32_t groups = (a.heads / a.kv.n_kv + 7) / 8;

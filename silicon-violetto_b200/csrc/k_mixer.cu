@@ -88,7 +88,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a) {
 }
 
 // The last rows of every run into its slot's ring, for steps whose runs are long enough to wrap it (a run's first rows must
-// have read the ring before its last ones overwrite it). grid (runs, rows of the ring).
+// have read the ring before its last ones overwrite it). grid (runs, rows of the ring, spans of 1024 channels).
 __global__ void __launch_bounds__(256) conv_state_kernel(const ConvArgs a, const RunIn* __restrict__ runs) {
     pdl_start();
     const RunIn ru = runs[blockIdx.x];
@@ -96,7 +96,12 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const ConvArgs a, const
     const uint32_t row = ru.count - 1 - blockIdx.y, pos = a.meta[2 * ru.first + 1] + row;
     const float* src = a.u + size_t(ru.first + row) * a.ldu;
     float* dst = a.ring + (size_t(ru.slot) * a.ring_len + pos % a.ring_len) * a.conv_channels;
-    for (uint32_t c = threadIdx.x; c < a.conv_channels; c += 256) dst[c] = src[c];
+    const uint32_t end = min(a.conv_channels, (blockIdx.z + 1) * 1024);
+#pragma unroll
+    for (uint32_t u = 0; u < 4; u++) {
+        const uint32_t c = blockIdx.z * 1024 + u * 256 + threadIdx.x;
+        if (c < end) dst[c] = src[c];
+    }
 }
 
 // Attention of one token and query head per block: the cached keys from the chunk's first position (or the sequence's) up to
@@ -214,7 +219,7 @@ void launch_conv_qkv(const ConvArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
     else launch_pdl(mixer::conv_qkv_kernel<uint16_t>, grid, 128, smem, s, a);
 }
 void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cudaStream_t s) {
-    if (n_runs) launch_pdl(mixer::conv_state_kernel, dim3(n_runs, a.ring_len), 256, 0, s, a, runs);
+    if (n_runs) launch_pdl(mixer::conv_state_kernel, dim3(n_runs, a.ring_len, (a.conv_channels + 1023) / 1024), 256, 0, s, a, runs);
 }
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
     const size_t smem = (a.kv.dk + a.kv.dv + 128) * 4;

@@ -50,43 +50,49 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
     }
     __syncthreads();
     const uint32_t all = a.experts + a.identity;
-    for (uint32_t e = warp; e < all; e += NW) {
-        float s[TOK] = {};
-        const uint16_t* w = a.router + size_t(e) * a.d;
+    // A warp takes EX outputs at a time over all the block's tokens, four neighbouring columns a lane and round: one read of x
+    // serves EX outputs, one of the weights TOK tokens, and the loads of U rounds go out together.
+    constexpr uint32_t EX = TOK == 1 ? 1 : 4, U = TOK == 1 ? 16 : 2;
+    for (uint32_t e0 = warp * EX; e0 < all; e0 += NW * EX) {
+        float s[EX][TOK] = {};
         uint32_t done = 0;
-        if (a.d % 8 == 0) {  // eight weights a load, several loads together
-            const uint4* w8 = reinterpret_cast<const uint4*>(w);
-            const uint32_t groups = a.d / 8;
-            constexpr uint32_t U = TOK == 1 ? 8 : 4;
+        if (a.d % 4 == 0) {
+            const uint32_t groups = a.d / 4;
             for (uint32_t g0 = lane; g0 < groups; g0 += 32 * U) {
-                uint4 v[U];
+                uint2 v[U][EX];
 #pragma unroll
-                for (uint32_t u = 0; u < U; u++) v[u] = g0 + 32 * u < groups ? __ldg(w8 + g0 + 32 * u) : make_uint4(0, 0, 0, 0);
+                for (uint32_t u = 0; u < U; u++)
+#pragma unroll
+                    for (uint32_t k = 0; k < EX; k++)
+                        v[u][k] = g0 + 32 * u < groups && e0 + k < all ? __ldg(reinterpret_cast<const uint2*>(a.router + size_t(e0 + k) * a.d) + g0 + 32 * u) : make_uint2(0, 0);
 #pragma unroll
                 for (uint32_t u = 0; u < U; u++) {
                     if (g0 + 32 * u >= groups) break;
 #pragma unroll
                     for (uint32_t j = 0; j < TOK; j++) {
-                        const float4* xp = reinterpret_cast<const float4*>(x + j * a.d + (g0 + 32 * u) * 8);
-                        const float4 xa = xp[0], xb = xp[1];
-                        s[j] = fmaf(bf16lo(v[u].x), xa.x, fmaf(bf16hi(v[u].x), xa.y, fmaf(bf16lo(v[u].y), xa.z, fmaf(bf16hi(v[u].y), xa.w, s[j]))));
-                        s[j] = fmaf(bf16lo(v[u].z), xb.x, fmaf(bf16hi(v[u].z), xb.y, fmaf(bf16lo(v[u].w), xb.z, fmaf(bf16hi(v[u].w), xb.w, s[j]))));
+                        const float4 xv = *reinterpret_cast<const float4*>(x + j * a.d + (g0 + 32 * u) * 4);
+#pragma unroll
+                        for (uint32_t k = 0; k < EX; k++)
+                            s[k][j] = fmaf(bf16lo(v[u][k].x), xv.x, fmaf(bf16hi(v[u][k].x), xv.y, fmaf(bf16lo(v[u][k].y), xv.z, fmaf(bf16hi(v[u][k].y), xv.w, s[k][j]))));
                     }
                 }
             }
             done = a.d;
         }
-        for (uint32_t i = done + lane; i < a.d; i += 32) {
-            const float wv = bf16_to_f32(w[i]);
+        for (uint32_t i = done + lane; i < a.d; i += 32)
 #pragma unroll
-            for (uint32_t j = 0; j < TOK; j++)
-                if (j < nt) s[j] = fmaf(wv, x[j * a.d + i], s[j]);
-        }
+            for (uint32_t k = 0; k < EX; k++) {
+                const float wv = e0 + k < all ? bf16_to_f32(a.router[size_t(e0 + k) * a.d + i]) : 0.0f;
 #pragma unroll
-        for (uint32_t j = 0; j < TOK; j++) {
-            s[j] = warp_sum(s[j]);
-            if (lane == 0) z[j * all + e] = s[j];
-        }
+                for (uint32_t j = 0; j < TOK; j++) s[k][j] = fmaf(wv, x[j * a.d + i], s[k][j]);
+            }
+#pragma unroll
+        for (uint32_t k = 0; k < EX; k++)
+#pragma unroll
+            for (uint32_t j = 0; j < TOK; j++) {
+                const float sum = warp_sum(s[k][j]);
+                if (lane == 0 && e0 + k < all) z[j * all + e0 + k] = sum;
+            }
     }
     __syncthreads();
     if (warp >= nt) return;

@@ -30,11 +30,15 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
     // An id past the vocabulary can only come from the device (a row of NaN logits has no argmax): read it as 0
     // rather than index out of the table.
     if (tok >= vocab) tok = 0;
-    const uint32_t* row = reinterpret_cast<const uint32_t*>(table + size_t(tok) * d);
-    float2* o = reinterpret_cast<float2*>(out + size_t(t) * d);
-    for (uint32_t i = tid; i < d / 2; i += blockDim.x) {
-        const uint32_t w = row[i];
-        o[i] = make_float2(bf16lo(w), bf16hi(w));
+    if (d % 2 == 0) {
+        const uint32_t* row = reinterpret_cast<const uint32_t*>(table + size_t(tok) * d);
+        float2* o = reinterpret_cast<float2*>(out + size_t(t) * d);
+        for (uint32_t i = tid; i < d / 2; i += blockDim.x) {
+            const uint32_t w = row[i];
+            o[i] = make_float2(bf16lo(w), bf16hi(w));
+        }
+    } else {
+        for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]);
     }
     __syncthreads();  // every thread has read tokens[t]
     if (tid == 0) {

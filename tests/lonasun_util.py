@@ -77,6 +77,31 @@ def standing_keys(special):
     return change
 
 
+def decided_routing(cfg, bits):
+    """An edit after which no choice of experts is a close one, so that bf16 and 32-bit choose alike: the routers read
+    directions that nothing but the embeddings writes, and every token has its own order of them with even steps."""
+    d, rng = cfg["width"], np.random.default_rng(11)
+    most = max(lc["mlp"]["router"]["experts"] + lc["mlp"]["router"]["identity"] for lc in cfg["layers"] if lc.get("mlp"))
+    R = np.linalg.qr(rng.standard_normal((d, most)))[0].T  # [directions][d]
+    off = lambda w: w - R.T @ (R @ w)  # a matrix that writes the stream, without the directions
+    get = lambda n: lonasun.from_bf16(bits[n]).reshape(bits[n].shape).astype(np.float64)
+    put = lambda n, w: bits.__setitem__(n, lonasun.to_bf16(w.astype(np.float32)).reshape(w.shape))
+    order = np.stack([rng.permutation(most) for _ in range(cfg["vocab"])]) - (most - 1) / 2
+    put("embed", off(get("embed").T).T + 24.0 / most * order @ R)
+    if cfg.get("loop"):
+        a, b = get("loop.in")[:, :d], get("loop.in")[:, d:]
+        put("loop.in", np.concatenate([0.6 * np.eye(d) + off(off(a).T).T * 0.5, 0.4 * np.eye(d) + off(off(b).T).T * 0.5], axis=1))
+    for name in list(bits):
+        if name.endswith(".mix.o") or name.endswith(".down"):
+            put(name, off(get(name)))
+        elif name.endswith("norm2"):
+            put(name, np.zeros(d))
+        elif name.endswith(".router"):
+            put(name, 0.4 * R[:bits[name].shape[0]])
+        elif name.endswith(".correction"):
+            put(name, get(name) * 0.01)
+
+
 def engine(folder, fp32: bool, tokens: int = 512, seqs: int = 4, head_rows: int | None = None, kv_tokens: int | None = None, tuning=None) -> E.Engine:
     return E.Engine(folder, E.EngineConfig(max_seqs=seqs, max_step_tokens=tokens, max_chunk=tokens, global_kv_tokens=kv_tokens or tokens * 2, max_seq_len=max(tokens, 1024),
                                            max_head_rows=head_rows or tokens, fp32=fp32), tuning)
@@ -121,4 +146,4 @@ def error(got, want) -> np.ndarray:
     return np.sqrt((d * d).mean(axis=1)) / want.std()
 
 
-LIMIT = {True: 2e-5, False: 0.04}  # fp32 engine, bf16 engine
+LIMIT = {True: 2e-5, False: 0.05}  # fp32 engine, bf16 engine
