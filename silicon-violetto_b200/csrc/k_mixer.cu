@@ -43,46 +43,81 @@ __device__ __forceinline__ const float* row_before(const ConvArgs& a, uint32_t t
     return a.ring + (size_t(a.tin[2 * t]) * a.ring_len + (start - before) % a.ring_len) * a.conv_channels;
 }
 
-// grid (tokens, heads + 2 kv heads): one q, k or v head of one token a block.
-template <typename T>
-__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a) {
+// grid (tokens / TB, heads + 2 kv heads): one q, k or v head of TB tokens a block (a step of many tokens: the tokens' chains of
+// dependent loads run side by side).
+template <typename T, uint32_t TB>
+__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_t n) {
     pdl_start();
-    extern __shared__ float y[];  // the head after its convolution
-    __shared__ const float* from[32];
-    const uint32_t t = blockIdx.x, unit = blockIdx.y, tid = threadIdx.x;
+    extern __shared__ float y[];  // [TB][width]: the head after its convolution
+    __shared__ const float* from[TB][32];
+    __shared__ uint32_t pos_s[TB], cpos_s[TB], slot_s[TB];
+    __shared__ size_t row_s[TB];  // where the head's key or value goes in the cache
+    const uint32_t t0 = blockIdx.x * TB, unit = blockIdx.y, tid = threadIdx.x, nt = min(TB, n - t0);
     const uint32_t kind = unit < a.heads ? 0u : unit < a.heads + a.kv.n_kv ? 1u : 2u;
     const uint32_t head = kind == 0 ? unit : kind == 1 ? unit - a.heads : unit - a.heads - a.kv.n_kv, width = kind == 2 ? a.kv.dv : a.kv.dk;
     const uint32_t c0 = kind == 2 ? (a.heads + a.kv.n_kv) * a.kv.dk + head * a.kv.dv : unit * a.kv.dk;
-    const uint32_t slot = a.meta[2 * t], pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], cpos = a.meta[2 * (t - row) + 1] + row;
-    if (tid < a.taps) from[tid] = row_before(a, t, tid);
+    // (a block's last tokens past the step repeat its first: their rows exist, and are not stored)
+    const uint32_t mine = tid / 32, back = tid % 32;  // a warp per token works out where its rows lie
+    if (mine < TB) {
+        const uint32_t t = t0 + (mine < nt ? mine : 0);
+        if (back < a.taps) from[mine][back] = row_before(a, t, back);
+        if (back == 0) {
+            const uint32_t row = a.tin[2 * t + 1];
+            slot_s[mine] = a.meta[2 * t];
+            pos_s[mine] = a.meta[2 * t + 1];
+            cpos_s[mine] = a.meta[2 * (t - row) + 1] + row;
+            row_s[mine] = kind ? page_row(a.kv, slot_s[mine], head, cpos_s[mine]) : 0;
+        }
+    }
     __syncthreads();
     for (uint32_t c = tid; c < width; c += 128) {
         const uint16_t* w = a.w + size_t(c0 + c) * a.taps;
-        float s = 0.0f;
-        for (uint32_t j = 0; j < a.taps; j++) {
-            const float* u = from[a.taps - 1 - j];
-            if (u) s = fmaf(bf16_to_f32(w[j]), u[c0 + c], s);
+        float s[TB] = {}, last[TB] = {};
+        for (uint32_t j0 = 0; j0 < a.taps; j0 += 4) {  // four taps' loads together
+            float wj[4], u[4][TB];
+#pragma unroll
+            for (uint32_t k = 0; k < 4; k++) {
+                const bool real = j0 + k < a.taps;
+                wj[k] = real ? bf16_to_f32(w[j0 + k]) : 0.0f;
+#pragma unroll
+                for (uint32_t i = 0; i < TB; i++) {
+                    const float* p = real ? from[i][a.taps - 1 - j0 - k] : nullptr;
+                    u[k][i] = p ? p[c0 + c] : 0.0f;
+                }
+            }
+#pragma unroll
+            for (uint32_t k = 0; k < 4; k++)
+#pragma unroll
+                for (uint32_t i = 0; i < TB; i++) {
+                    s[i] = fmaf(wj[k], u[k][i], s[i]);
+                    if (j0 + k + 1 == a.taps) last[i] = u[k][i];
+                }
         }
-        y[c] = s;
-        if (a.write_ring) a.ring[(size_t(slot) * a.ring_len + cpos % a.ring_len) * a.conv_channels + c0 + c] = from[0][c0 + c];
+#pragma unroll
+        for (uint32_t i = 0; i < TB; i++) {
+            y[i * width + c] = s[i];
+            if (a.write_ring && i < nt) a.ring[(size_t(slot_s[i]) * a.ring_len + cpos_s[i] % a.ring_len) * a.conv_channels + c0 + c] = last[i];
+        }
     }
     __syncthreads();
-    T* cache = nullptr;
-    if (kind) cache = static_cast<T*>(kind == 1 ? a.kv.k : a.kv.v) + page_row(a.kv, slot, head, cpos) * width;
-    const float2* cs = reinterpret_cast<const float2*>(a.rope) + size_t(pos) * (a.rot_dims / 2);
+    const uint32_t half = a.rot_dims / 2;
     for (uint32_t c = tid; c < width; c += 128) {
-        float v = y[c];
-        if (kind < 2 && c < a.rot_dims) {
-            const uint32_t half = a.rot_dims / 2;
-            if (c < half) v = y[c] * cs[c].x - y[c + half] * cs[c].y;
-            else v = y[c] * cs[c - half].x + y[c - half] * cs[c - half].y;
-        }
-        if (kind == 0) {
-            const size_t o = (size_t(t) * a.heads + head) * width + c;
-            if (a.q_f) a.q_f[o] = v;
-            if (a.q_b) a.q_b[o] = f32_to_bf16(v * a.q_scale);
-        } else {
-            store_kv(cache + c, v);
+#pragma unroll
+        for (uint32_t i = 0; i < TB; i++) {
+            if (i >= nt) break;
+            const float* yi = y + i * width;
+            float v = yi[c];
+            if (kind < 2 && c < a.rot_dims) {
+                const float2 cs = reinterpret_cast<const float2*>(a.rope)[size_t(pos_s[i]) * half + (c < half ? c : c - half)];
+                v = c < half ? yi[c] * cs.x - yi[c + half] * cs.y : yi[c] * cs.x + yi[c - half] * cs.y;
+            }
+            if (kind == 0) {
+                const size_t o = (size_t(t0 + i) * a.heads + head) * width + c;
+                if (a.q_f) a.q_f[o] = v;
+                if (a.q_b) a.q_b[o] = f32_to_bf16(v * a.q_scale);
+            } else {
+                store_kv(static_cast<T*>(kind == 1 ? a.kv.k : a.kv.v) + row_s[i] * width + c, v);
+            }
         }
     }
 }
@@ -213,10 +248,13 @@ __global__ void __launch_bounds__(256) mixer_fill_kernel(const MixerCache* __res
 }  // namespace mixer
 
 void launch_conv_qkv(const ConvArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
-    const dim3 grid(n, a.heads + 2 * a.kv.n_kv);
-    const size_t smem = std::max(a.kv.dk, a.kv.dv) * 4;
-    if (fp32) launch_pdl(mixer::conv_qkv_kernel<float>, grid, 128, smem, s, a);
-    else launch_pdl(mixer::conv_qkv_kernel<uint16_t>, grid, 128, smem, s, a);
+    const uint32_t units = a.heads + 2 * a.kv.n_kv, tb = n >= 64 ? 4 : 1;
+    const dim3 grid((n + tb - 1) / tb, units);
+    const size_t smem = size_t(tb) * std::max(a.kv.dk, a.kv.dv) * 4;
+    if (tb == 1 && fp32) launch_pdl(mixer::conv_qkv_kernel<float, 1>, grid, 128, smem, s, a, n);
+    else if (tb == 1) launch_pdl(mixer::conv_qkv_kernel<uint16_t, 1>, grid, 128, smem, s, a, n);
+    else if (fp32) launch_pdl(mixer::conv_qkv_kernel<float, 4>, grid, 128, smem, s, a, n);
+    else launch_pdl(mixer::conv_qkv_kernel<uint16_t, 4>, grid, 128, smem, s, a, n);
 }
 void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cudaStream_t s) {
     if (n_runs) launch_pdl(mixer::conv_state_kernel, dim3(n_runs, a.ring_len, (a.conv_channels + 1023) / 1024), 256, 0, s, a, runs);

@@ -110,29 +110,36 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
         sum = warp_sum(sum);
         for (uint32_t e = lane; e < all; e += 32) zt[e] = zt[e] / sum;
         __syncwarp();
-        // The choice: the largest score + correction, `top` times; a chosen score is marked by its sign bit (scores are >= 0).
-        float total = 0.0f;
+        // The choice: the largest score + correction, `top` times, ties to the lower index. Kept as integers that order as
+        // the numbers do (0: chosen already), so that a warp's maximum is one instruction.
+        uint32_t* ct = reinterpret_cast<uint32_t*>(z + TOK * all) + j * all;
+        for (uint32_t e = lane; e < all; e += 32) {
+            const uint32_t u = __float_as_uint(zt[e] + bf16_to_f32(a.correction[e]));
+            ct[e] = max(u & 0x80000000u ? ~u : u | 0x80000000u, 1u);
+        }
+        __syncwarp();
+        float total = 0.0f, kept = 0.0f;  // lane k keeps choice k's score (past 32 they wait in memory)
         for (uint32_t k = 0; k < a.top; k++) {
-            float bv = -INFINITY;
-            uint32_t bi = 0xffffffffu;
-            for (uint32_t e = lane; e < all; e += 32) {
-                if (signbit(zt[e])) continue;
-                better(bv, bi, zt[e] + bf16_to_f32(a.correction[e]), e);
-            }
-            warp_best(bv, bi);
-            if (bi >= all) bi = 0;  // (only if the logits are not numbers)
-            const float s = fabsf(zt[bi]);
+            uint32_t bv = 0, bi = all;
+            for (uint32_t e = lane; e < all; e += 32)
+                if (ct[e] > bv) { bv = ct[e]; bi = e; }
+            const uint32_t best = __reduce_max_sync(0xffffffffu, bv);
+            bi = __reduce_min_sync(0xffffffffu, bv == best ? bi : all);
+            if (bi >= all) bi = 0;  // (never: there are at least `top` outputs)
+            const float s = zt[bi];
             total += s;
             __syncwarp();
             if (lane == 0) {
-                zt[bi] = -s;
+                ct[bi] = 0;
                 a.ids[size_t(t) * a.top + k] = bi;
-                a.weights[size_t(t) * a.top + k] = s;
+                if (k >= 32) a.weights[size_t(t) * a.top + k] = s;
             }
+            if (lane == k) kept = s;
             __syncwarp();
         }
         const float inv = 1.0f / (total + 1e-20f);
-        for (uint32_t k = lane; k < a.top; k += 32) a.weights[size_t(t) * a.top + k] *= inv;
+        if (lane < a.top) a.weights[size_t(t) * a.top + lane] = kept * inv;
+        for (uint32_t k = 32 + lane; k < a.top; k += 32) a.weights[size_t(t) * a.top + k] *= inv;
     }
 }
 
@@ -263,7 +270,7 @@ void launch_router(const RouterArgs& a, cudaStream_t s) {
         VLT_CUDA(cudaFuncSetAttribute(moe::router_kernel<4, 512>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     });
     // Many tokens share a read of the router's matrix, four a block; few spread over the SMs one by one.
-    const size_t one = (size_t(a.d) + all) * 4;
+    const size_t one = (size_t(a.d) + 2 * all) * 4;  // the normed row, the scores, what the choice goes by
     if (a.n >= 256 && one <= 25 * 1024) launch_pdl(moe::router_kernel<4, 512>, (a.n + 3) / 4, 512, 4 * one, s, a);
     else if (a.n > 148) launch_pdl(moe::router_kernel<1, 512>, a.n, 512, one, s, a);
     else launch_pdl(moe::router_kernel<1, 1024>, a.n, 1024, one, s, a);
