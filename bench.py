@@ -314,43 +314,48 @@ def limite_figure(E, local, ctx, steps=30, stream_counts=(1, 8, 32), keys_per_bl
     return out
 
 
-LONASUN = dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=8192, experts=64, top=8, ff=1024, shared=1024, vocab=32768, layers=4)
+# Layers of real models' sizes; `plain` sizes the plain decoder beside each: the same query and key / value widths in heads of 64
+# and a dense feed-forward with the parameters one token uses (three matrices there, two here).
+LONASUN_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=8192, experts=64, top=8, ff=1024, shared=1024, vocab=32768, layers=4, ctx=8000,
+                 plain=dict(n_heads=32, n_kv=8, ffn=6144)),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, chunk=2048, experts=32, top=4, ff=1536, shared=1536, vocab=32768, layers=2, ctx=1900,
+                 plain=dict(n_heads=64, n_kv=16, ffn=5120)),
+}
 
 
-def lonasun_files():
-    """A Lonasun model whose layers resemble a real model's (width 2048, 16 / 4 heads of 128, 64 experts of 1024 with 8 a
-    token, a shared one), four of them, and the plain decoder of equal size beside it: the same query and key / value widths
-    (32 / 8 heads of 64) and a dense feed-forward with the parameters one token uses (two matrices of 9 x 1024 there are three
-    of 6144 here). Random-init, bf16."""
+def lonasun_files(size):
+    """A Lonasun model and the plain decoder of equal size (LONASUN_SIZES), random-init, bf16, written once per box."""
     from silicon_violetto_b200 import lonasun, synth
     CACHE.mkdir(parents=True, exist_ok=True)
-    c = LONASUN
+    c = LONASUN_SIZES[size]
     moe = dict(experts=c["experts"], top=c["top"], ff=c["ff"], shared=c["shared"], identity=0)
     cfg = lonasun.config(c["width"], c["vocab"], [lonasun.layer(c["heads"], c["kv_heads"], c["dim"], c["vdim"], c["chunk"], conv=4, rot_dims=64, base=500000.0, moe=moe)] * c["layers"])
-    folder = CACHE / "lonasun_4x2048"
+    folder = CACHE / f"lonasun_{size}"
     if not (folder / "ok").exists():
         lonasun.write_model(folder, cfg, lonasun.random_weights(cfg))
         (folder / "ok").write_text("ok")
-    plain = CACHE / "plain_4x2048.vlt"
+    plain = CACHE / f"plain_{size}.vlt"
     if not plain.with_suffix(".ok").exists():
-        synth.write_target(plain, dict(n_layers=c["layers"], d=c["width"], n_heads=32, n_kv=8, hd=64, ffn=6144, vocab=c["vocab"], eps=1e-5, theta=500000.0, page=16), seed=0)
+        synth.write_target(plain, dict(n_layers=c["layers"], d=c["width"], hd=64, vocab=c["vocab"], eps=1e-5, theta=500000.0, page=16, **c["plain"]), seed=0)
         plain.with_suffix(".ok").write_text("ok")
     return folder, plain
 
 
-def lonasun_figure(E, local, ctx, steps, stream_counts, hbm_peak, tc_peak):
-    """Decoding over a filled context of `ctx` positions and a `ctx`-token prompt in chunks of 512, the Lonasun model and the
+def lonasun_figure(E, local, size, steps, stream_counts, hbm_peak, tc_peak):
+    """Decoding over a filled context and a prompt of the same length (all in one chunk of positions) in portions of 512, the Lonasun model and the
     plain decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their
     own) the fraction of the measured copy bandwidth or bf16 throughput its algorithmic bytes or FLOPs make."""
-    c, L = LONASUN, LONASUN["layers"]
-    folder, plain = lonasun_files()
+    c = LONASUN_SIZES[size]
+    L, ctx = c["layers"], c["ctx"]
+    folder, plain = lonasun_files(size)
     attn_w = (c["heads"] + c["kv_heads"]) * c["dim"] + c["kv_heads"] * c["vdim"]
     o_p = c["heads"] * c["vdim"] * c["width"]
     expert_p = 2 * c["ff"] * c["width"]
     weights = {"lonasun": lambda touched: L * ((attn_w + c["heads"] * c["vdim"]) * c["width"] + o_p + (touched + 1) * expert_p),
-               "plain": lambda touched: L * (attn_w * c["width"] + o_p + 3 * 6144 * c["width"])}
+               "plain": lambda touched: L * (attn_w * c["width"] + o_p + 3 * c["plain"]["ffn"] * c["width"])}
     kv_row = c["kv_heads"] * (c["dim"] + c["vdim"]) * 2
-    out = {"workload": f"{L} layers x {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in chunks of 512"}
+    out = {"workload": f"{L} layers x {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in portions of 512"}
     for name, path in (("lonasun", folder), ("plain", plain)):
         res = out[name] = {}
         for n_s in stream_counts:
@@ -460,7 +465,7 @@ def main():
     ap.add_argument("--limite-drafter", action="store_true", help="--only limite: with the reference's block drafter loaded (tree drafts of up to 8 rows)")
     ap.add_argument("--limite-int8", action="store_true", help="--only limite: int8 weights in the reference converter's default groups (64; the head 8)")
     ap.add_argument("--limite-keys", type=int, default=0, help="--only limite: keys per attention block (VltTuning.attn_keys_per_cta); 0 = the library's choice")
-    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) or 'lonasun' (a Lonasun model beside a plain decoder of equal size): run that one pass alone and print its figure (not the bench line)")
+    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) or 'lonasun' (Lonasun models beside plain decoders of equal size): run that one pass alone and print its figure (not the bench line)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank, world, local = int(os.environ.get("RANK", 0)), int(os.environ.get("WORLD_SIZE", 1)), int(os.environ.get("LOCAL_RANK", 0))
@@ -508,7 +513,8 @@ def main():
     from silicon_violetto_b200 import engine as E
     if args.only == "lonasun":
         peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
-        print(json.dumps(lonasun_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], hbm_peak, peaks.get("bf16_tflops", 1590.0))))
+        print(json.dumps({n: lonasun_figure(E, local, n, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], hbm_peak, peaks.get("bf16_tflops", 1590.0))
+                          for n in LONASUN_SIZES}))
         return
     path = model_file("1b", not args.bf16, rank, args.layers)
     if args.only:

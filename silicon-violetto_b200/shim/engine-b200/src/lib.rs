@@ -114,6 +114,7 @@ pub struct LayerCapture<'a> {
     pub mlp_in: &'a [f32],
     pub mlp_out: &'a [f32],
     pub resid_base: Option<&'a [f32]>,
+    pub resid_out: Option<&'a [f32]>,
 }
 
 /// engine/src/engine/hooks.rs:9-19.
@@ -259,7 +260,8 @@ impl Engine {
     pub fn step_capture(&mut self, runs: &[Run], opts: &StepOptions, f: &mut dyn FnMut(&LayerCapture)) -> Result<StepOutput, String> {
         extern "C" fn tramp(c: *const ffi::VltLayerCapture, user: *mut c_void) {
             let (c, f) = unsafe { (&*c, &mut *(user as *mut &mut dyn FnMut(&LayerCapture))) };
-            let s = |p: *const f32, w: u32| unsafe { std::slice::from_raw_parts(p, (c.n * w) as usize) };
+            // (an intermediate that the model's architecture does not hand out is an empty slice)
+            let s = |p: *const f32, w: u32| -> &[f32] { if p.is_null() { &[] } else { unsafe { std::slice::from_raw_parts(p, (c.n * w) as usize) } } };
             f(&LayerCapture {
                 layer: c.layer as usize,
                 n: c.n as usize,
@@ -271,6 +273,7 @@ impl Engine {
                 mlp_in: s(c.mlp_in, c.d_model),
                 mlp_out: s(c.mlp_out, c.d_model),
                 resid_base: if c.resid_base.is_null() { None } else { Some(s(c.resid_base, c.d_model)) },
+                resid_out: if c.resid_out.is_null() { None } else { Some(s(c.resid_out, c.d_model)) },
             });
         }
         let mut f = f;
