@@ -130,13 +130,13 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
     if (cfg.max_seqs == 0 || cfg.max_step_tokens == 0 || cfg.max_chunk == 0 || cfg.max_head_rows == 0) throw Error("engine config: zero capacity");
     model.load(weights, cfg.host_only);
     const ModelDesc& md = model.md;
-    if (cfg.fp32 && !model.lonasun) throw Error(weights + ": this architecture has no fp32 path");
-    if (model.lonasun) {
-        std::vector<KvShape> shapes;
-        for (const LayerRun& r : model.lonasun->runs) {
-            const GatedAttention& m = model.lonasun->layers[r.layer].mix;
-            shapes.push_back({m.kv_heads, m.dim, m.vdim});
-        }
+    if (cfg.fp32 && !model.layered) throw Error(weights + ": this architecture has no fp32 path");
+    if (model.layered) {
+        if (model.layered->positions) cfg.max_seq_len = std::min(cfg.max_seq_len, model.layered->n_positions);
+        std::vector<KvShape> shapes;  // a slice per (layer run, mixer), of no bytes for one without keys
+        for (const LayerRun& r : model.layered->runs)
+            for (const Mixer& x : model.layered->layers[r.layer].mix)
+                shapes.push_back(x.kind == MixerKind::Attention ? KvShape{x.attn.kv_heads, x.attn.dim, x.attn.vdim} : KvShape{0, 0, 0});
         kv.init(cfg, md.page, shapes, cfg.fp32 ? 4 : 2, !cfg.host_only);
     } else {
         kv.init(cfg, md.page, std::vector<KvShape>(model.limite ? model.n_global : md.n_layers, {md.n_kv, md.hd, md.hd}), 2, !cfg.host_only);  // (the reference's architecture pages its global layers only)
@@ -157,7 +157,7 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
         s.h_b.alloc(n16 * md.d * 2, false);
         s.hfin_b.alloc(hr16 * md.d * 2, false);
         f(s.inv_head, hr);
-        if (!model.lonasun) {  // (its layers' scratch is its own)
+        if (!model.layered) {  // (its layers' scratch is its own)
         f(s.qkv, n * md.qkv_w());
         f(s.attn, n * md.n_heads * md.hd);
         f(s.act, n * md.ffn);
@@ -188,8 +188,8 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
     std::vector<GenState> open(ms, gen_open());
     s.gen.write_vec(0, open);
 
-    if (!ho && model.lonasun) {
-        init_lonasun();
+    if (!ho && model.layered) {
+        init_layered();
         VLT_CUDA(cudaDeviceSynchronize());
     } else if (!ho) {
         // engine.rs:392-421 `rope_table`: theta = float32(pos) * frequency, cos and sin rounded to bf16.
@@ -412,6 +412,7 @@ Plan Engine::plan(uint32_t set, const std::vector<PlanRun>& runs, Rows hidden) {
         max_keys = std::max(max_keys, new_len);
         max_count = std::max(max_count, count);
         p.branches = p.branches || (run.verify && count > 2);
+        p.verified = p.verified || (run.verify && count > 1);
         sq.len = new_len;
     }
     if (head_rows.size() > cfg.max_head_rows) throw Error(std::to_string(head_rows.size()) + " head rows (max " + std::to_string(cfg.max_head_rows) + ")");
@@ -918,7 +919,7 @@ void Engine::encode_forward_limite(uint32_t set, const Plan& p) {
 
 // engine/src/engine/encode.rs:99-105 `encode_forward`, after the step set's upload.
 void Engine::encode_forward(uint32_t set, const Plan& p) {
-    if (model.lonasun) { encode_forward_lonasun(set, p); return; }
+    if (model.layered) { encode_forward_layered(set, p); return; }
     if (model.limite) { encode_forward_limite(set, p); return; }
     begin_step(set, p);
     for (uint32_t li = 0; li < model.md.n_layers; li++) encode_layer(set, p, li);
@@ -935,8 +936,10 @@ void Engine::begin_step(uint32_t set, const Plan& p) {
     VLT_CUDA(cudaEventRecord(st.uploaded, copy_in));
     VLT_CUDA(cudaEventRecord(st.start, stream));
     VLT_CUDA(cudaStreamWaitEvent(stream, st.uploaded, 0));
-    launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), lz ? lz->x0.as<float>() : s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
-                 s.feed.as<uint32_t>(), s.tree.as<uint32_t>(), st.in<uint32_t>(st.o_vis), p.n, model.md.d, model.md.vocab, stream);
+    const LayeredModel* lm = model.layered.get();
+    launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), lm ? lay->x0.as<float>() : s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
+                 s.feed.as<uint32_t>(), s.tree.as<uint32_t>(), st.in<uint32_t>(st.o_vis), p.n, model.md.d, model.md.vocab, stream, lm ? lm->positions : nullptr,
+                 lm ? lm->n_positions : 0);
 }
 
 // engine/src/engine/encode.rs:439-451 `encode_replay`.
@@ -994,7 +997,7 @@ void Engine::upload_set(uint32_t set) {
 void Engine::load_drafter(const std::string& path) {
     for (const auto& q : seqs)
         if (q) throw Error("load the drafter before the first sequence (it changes how many pages a step reserves)");
-    if (model.lonasun) throw Error(path + ": the drafters are built for the other architectures' hidden states");
+    if (model.layered) throw Error(path + ": the drafters are built for the other architectures' hidden states");
     auto dr = std::make_unique<Drafter>();
     const ModelDesc& md = model.md;
     dr->w.load(path, cfg.host_only);
@@ -1426,9 +1429,9 @@ StepOutput Engine::read_output(const Plan& p, const StepOptions& opts, double gp
 StepOutput Engine::step_capture(const std::vector<PlanRun>& runs, const StepOptions& opts, const std::function<void(const LayerCapture&)>& f) {
     if (cfg.host_only) throw Error("this engine was created host-only: it plans steps but cannot run them (no CPU path)");
     if (model.limite) throw Error("step_capture is not built for the reference's own architecture");
-    if (model.lonasun) {
+    if (model.layered) {
         Plan p = plan(0, runs, opts.hidden);
-        encode_forward_lonasun(0, p, &f);
+        encode_forward_layered(0, p, &f);
         commit(0);
         const double secs = wait(0);
         check_device_error(0);
@@ -1469,8 +1472,9 @@ void Engine::bench_fill(uint32_t id, uint32_t len, uint32_t seed) {
     sq.len += len;
     s.lens.write(id * 4, &sq.len, 4);
     kv.reserve(id, sq.pages, sq.len);
-    if (seed && model.lonasun && !cfg.host_only) {
-        launch_mixer_fill(lz->caches.as<MixerCache>(), model.md.n_layers, id, from, sq.len, seed, cfg.fp32, stream);
+    if (seed && model.layered && !cfg.host_only) {
+        launch_mixer_fill(lay->caches.as<MixerCache>(), uint32_t(lay->run.size()), id, from, sq.len, seed, cfg.fp32, stream);
+        launch_recurrent_fill(lay->recurrent_dev.as<RecurrentCache>(), uint32_t(lay->recurrent.size()), id, seed, stream);
         VLT_CUDA(cudaStreamSynchronize(stream));
         return;
     }
@@ -1582,7 +1586,7 @@ void Engine::draft_trees(const float* logits, uint32_t n_rows, uint32_t nv, cons
 void Engine::bench_matmul(const std::string& kind, uint32_t n, uint32_t variant, uint32_t reps, double* seconds, uint64_t* bytes) {
     if (cfg.host_only) throw Error("this engine was created host-only: it cannot run kernels");
     const bool head = kind == "head";
-    if (model.lonasun) throw Error("bench_matmul times the other architectures' projections");
+    if (model.layered) throw Error("bench_matmul times the other architectures' projections");
     if (!head && kind != "qkv" && kind != "o" && kind != "gate_up" && kind != "down") throw Error("unknown matmul " + kind);
     if (n == 0 || n > (head ? cfg.max_head_rows : cfg.max_step_tokens)) throw Error(kind + " can't take " + std::to_string(n) + " tokens");
     cudaEvent_t e0, e1;

@@ -56,6 +56,7 @@ struct PlanRun {
 struct Plan {
     uint32_t n = 0, n_head = 0, n_hidden = 0, n_runs = 0, tiles = 0, max_run = 0;
     bool branches = false;
+    bool verified = false;  // some run is a verified one of several rows
     bool head_all = false;  // every row of the step goes through the head, in order
     uint32_t ctiles = 0;   // chunk tiles of at most 64 rows (the prefill attention's blocks)
     bool chunked = false;  // some run is longer than VERIFY_T rows: the step's attention is the chunk kernel (encode.rs:299-355)
@@ -125,7 +126,7 @@ struct StepOutput {
 struct LayerCapture {
     uint32_t layer, n;
     const float *resid_in, *attn_in, *qkv, *sdpa_out, *attn_out, *mlp_in, *mlp_out;
-    const float* resid_out = nullptr;  // the stream leaving the layer (Lonasun, which hands out this, resid_in and sdpa_out only)
+    const float* resid_out = nullptr;  // the stream leaving the layer (model folders, which hand out this, resid_in and, for an attention, sdpa_out only)
     uint32_t attn_width = 0;           // sdpa_out's columns, where layers differ
 };
 
@@ -245,20 +246,32 @@ class Engine {
         Buffer k_local, v_local;  // [local layer][slot][kv head][ring][128] bf16
         Buffer hist0, hist12, hist23, xattn, base, mixed, vdir, gates, part;  // part: the attention's partials per (token, head, key split)
     };
-    // The Lonasun design (model.lonasun): a ring of projected rows per (layer run, slot) beside the paged pool, and scratch.
-    struct LonasunState {
+    // A model folder's layers (model.layered): caches per (layer run, mixer) beside the paged pool, and scratch.
+    struct LayeredState {
         Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding; a norm's rows; (stream ; embedding)
-        Buffer proj, q_f, q_b, attn_f, attn_b;    // q | k | v | gate as projected; rotated q; the gated attention
+        Buffer proj, q_f, q_b, attn_f, attn_b;    // a mixer's projections; finished q; what the output projection reads
         Buffer moe_x, moe_xb, ids, weights, src, place, tiles, n_tiles, hid_f, hid_b, rows, sh_f, sh_b, shared;
-        Buffer rings, caches;                     // caches: MixerCache per layer run, on the device
+        Buffer ff_f, ff_b, branch;                // a dense layer's hidden rows; the outputs of mixers side by side
+        Buffer conv, steps, y, mix_f, mix_b, low, decay;  // a recurrence's inputs and outputs
+        Buffer rings, states, caches, recurrent_dev;      // caches, recurrent_dev: MixerCache, RecurrentCache on the device
         std::vector<Buffer> rope;                 // per distinct rotation: [position][dims / 2] (cos, sin), fp32
         std::vector<MixerCache> run;              // the host's copy of caches
+        std::vector<uint32_t> first;              // a layer run's first entry in it
+        std::vector<RecurrentCache> recurrent;
+        uint32_t max_heads = 0;                   // of a recurrence
     };
     static constexpr uint32_t EXPERT_TILE_MIN = 16;  // rows of an expert per tile, at least
-    std::unique_ptr<LonasunState> lz;
-    void init_lonasun();
-    void encode_experts(const LonasunLayer& l, uint32_t n, const uint16_t* norm);
-    void encode_forward_lonasun(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
+    static constexpr uint32_t SHIFT_TILE_MIN = 16;   // tokens of a mix per tile, at least
+    std::unique_ptr<LayeredState> lay;
+    void init_layered();
+    void encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm);
+    ConvArgs conv_args(StepSet& st, const Plan& p, const MixerCache& mc, const float* u, uint32_t ldu, uint32_t taps);
+    void mixer_out(const Matrix& o, uint32_t n, const float* cur, float* alone);
+    void encode_attention(StepSet& st, const Plan& p, const Attention& a, const MixerCache& mc, const float* cur, float* alone, bool capture);
+    void encode_recurrence(StepSet& st, const Plan& p, ScanArgs& a, GatedNormArgs& g);
+    void encode_state_space(StepSet& st, const Plan& p, const StateSpace& x, const MixerCache& mc, const float* cur, float* alone);
+    void encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const MixerCache& mc, const float* cur, float* alone);
+    void encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
     // Y = epilogue(W x) in the engine's precision: xf in an fp32 engine, else xb through the GEMM, the streamed matmul or,
     // for sizes neither takes, the CUDA cores.
     void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr);

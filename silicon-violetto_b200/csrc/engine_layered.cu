@@ -1,0 +1,636 @@
+// The step of a model folder: its layer runs in order over the engine's planner, page table, sampler and acceptance.
+#include <algorithm>
+#include <cmath>
+
+#include "engine.h"
+
+namespace vlt {
+
+void Engine::init_layered() {
+    const LayeredModel& m = *model.layered;
+    const ModelDesc& md = model.md;
+    lay = std::make_unique<LayeredState>();
+    LayeredState& z = *lay;
+    const bool f32 = cfg.fp32;
+    const size_t n = cfg.max_step_tokens, n16 = (n + 15) / 16 * 16, d = md.d;
+    size_t proj = 0, q = 0, out = 0, pairs = 0, hid = 0, sff = 0, tiles = 0, top = 0, rows = 0, ff = 0, branch = 0, channels = 0, y = 0, inner = 0, heads = 0, low = 0;
+    bool shift = false;
+    for (const FolderLayer& l : m.layers) {
+        if (l.mix.size() > 1) branch = 2 * d;
+        for (const Mixer& x : l.mix) {
+            if (x.kind == MixerKind::Attention) {
+                proj = std::max<size_t>(proj, x.attn.proj.m);
+                q = std::max<size_t>(q, x.attn.heads * x.attn.dim);
+                out = std::max<size_t>(out, x.attn.out_w());
+            } else if (x.kind == MixerKind::StateSpace) {
+                proj = std::max<size_t>(proj, x.ssm.in.m);
+                channels = std::max<size_t>(channels, x.ssm.channels());
+                y = std::max<size_t>(y, x.ssm.inner());
+                out = std::max<size_t>(out, x.ssm.inner());
+                heads = std::max<size_t>(heads, 2 * x.ssm.heads);
+            } else {
+                shift = true;
+                proj = std::max<size_t>(proj, 4 * x.tmix.inner());
+                inner = std::max<size_t>(inner, x.tmix.inner());
+                y = std::max<size_t>(y, x.tmix.inner());
+                out = std::max<size_t>(out, x.tmix.inner());
+                heads = std::max<size_t>(heads, x.tmix.heads);
+                low = std::max<size_t>(low, x.tmix.w1.m);
+                tiles = std::max<size_t>(tiles, 4 * (n / SHIFT_TILE_MIN + 1));
+            }
+        }
+        if (l.mlp == MlpKind::Dense) ff = std::max<size_t>(ff, l.dense.up.m);
+        if (l.mlp != MlpKind::Experts) continue;
+        const ExpertLayer& e = l.experts;
+        const size_t p = n * e.top;
+        top = std::max<size_t>(top, e.top);
+        pairs = std::max(pairs, p);
+        hid = std::max(hid, p * e.ff);
+        rows = std::max(rows, p * d);
+        sff = std::max<size_t>(sff, e.shared_ff);
+        tiles = std::max(tiles, p / EXPERT_TILE_MIN + std::min<size_t>(e.experts, p) + 1);
+    }
+    auto f = [](Buffer& b, size_t floats) { b.alloc(floats * 4, false); };
+    auto h = [&](Buffer& b, size_t halves) { if (!f32) b.alloc(halves * 2, false); };  // the 16-bit copies
+    auto w = [&](Buffer& b, size_t floats) { if (f32) b.alloc(floats * 4, false); };   // their 32-bit counterparts
+    f(z.x0, n * d);
+    if (shift) f(z.xn_f, n * d);  // (rows are mixed in 32-bit)
+    else w(z.xn_f, n * d);
+    h(z.xn_b, n16 * d);
+    if (m.loop_in.m) {
+        w(z.cat_f, n * 2 * d);
+        h(z.cat_b, n16 * 2 * d);
+    }
+    f(z.proj, n * proj);
+    f(z.q_f, n * q);
+    h(z.q_b, n16 * q);
+    f(z.attn_f, n * out);
+    h(z.attn_b, n16 * out);
+    if (pairs) {
+        f(z.moe_x, n * d);
+        h(z.moe_xb, n16 * d);
+        f(z.ids, n * top);
+        f(z.weights, n * top);
+        f(z.src, pairs);
+        f(z.place, pairs);
+        w(z.hid_f, hid);
+        h(z.hid_b, hid + 256);
+        f(z.rows, rows);
+        w(z.sh_f, n * sff);
+        h(z.sh_b, n16 * sff);
+        f(z.shared, n * d);
+    }
+    f(z.tiles, 3 * tiles);
+    f(z.n_tiles, 1);
+    w(z.ff_f, n * ff);
+    h(z.ff_b, n16 * ff);
+    f(z.branch, n * branch);
+    f(z.conv, n * channels);
+    f(z.steps, n * heads);
+    f(z.y, n * y);
+    if (shift) {
+        w(z.mix_f, 5 * n * d);
+        h(z.mix_b, 5 * n * d + 16 * d);
+        f(z.low, n * low);
+        f(z.decay, n * inner);
+    }
+    // Angles in double, the table in fp32: positions up to the longest sequence and a verified tree past it.
+    for (const Rotation& r : m.rotations) {
+        const uint32_t npos = cfg.max_seq_len + FEED_W, half = r.dims / 2;
+        std::vector<float> tab(size_t(npos) * half * 2);
+        for (uint32_t i = 0; i < half; i++) {
+            const double freq = std::pow(r.base, -2.0 * i / r.dims);
+            for (uint32_t p = 0; p < npos; p++) {
+                tab[(size_t(p) * half + i) * 2] = float(std::cos(p * freq));
+                tab[(size_t(p) * half + i) * 2 + 1] = float(std::sin(p * freq));
+            }
+        }
+        z.rope.emplace_back();
+        z.rope.back().alloc(std::max<size_t>(tab.size() * 4, 16), false);
+        z.rope.back().write_vec(0, tab);
+    }
+    // Per (layer run, mixer): its pages; a ring per slot of the rows a convolution or shift reaches back over, and room for a
+    // verified run past them; a recurrence's state per slot and what a verified run leaves for it.
+    uint32_t page_shift = 0;
+    while ((1u << page_shift) < md.page) page_shift++;
+    const size_t es = f32 ? 4 : 2;
+    size_t ring = 0, state = 0;
+    for (int pass = 0; pass < 2; pass++) {  // sizes, then addresses
+        float *rings = z.rings.as<float>(), *states = z.states.as<float>();
+        ring = state = 0;
+        uint32_t i = 0;
+        auto take = [&](size_t floats) {
+            float* p = states + state;
+            state += (floats + 31) / 32 * 32;
+            return p;
+        };
+        z.run.clear();
+        z.first.clear();
+        z.recurrent.clear();
+        for (const LayerRun& r : m.runs) {
+            z.first.push_back(i);
+            for (const Mixer& x : m.layers[r.layer].mix) {
+                MixerCache c{};
+                if (x.kind == MixerKind::Attention) {
+                    const Attention& a = x.attn;
+                    c.kv = PagedKv{kv.k.as<uint8_t>() + kv.k_off[i] * es, kv.v.as<uint8_t>() + kv.v_off[i] * es, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, a.kv_heads, a.dim, a.vdim};
+                    if (a.conv.w) { c.channels = a.conv.channels; c.ring_len = a.conv.taps - 1 + VERIFY_T; }
+                } else {
+                    const bool tm = x.kind == MixerKind::TimeMix;
+                    c.channels = tm ? md.d : x.ssm.channels();
+                    c.ring_len = (tm ? 2 : x.ssm.conv.taps) - 1 + VERIFY_T;
+                    RecurrentCache rc{};
+                    rc.heads = tm ? x.tmix.heads : x.ssm.heads;
+                    rc.per = tm ? 1 : x.ssm.heads / x.ssm.groups;
+                    rc.N = tm ? x.tmix.dim : x.ssm.state;
+                    rc.Np = recurrent_pitch(rc.N);
+                    rc.P = tm ? x.tmix.dim : x.ssm.vdim;
+                    rc.channel_decay = tm;
+                    const size_t kept = size_t(cfg.max_seqs) * VERIFY_T;
+                    rc.state = take(size_t(cfg.max_seqs) * rc.heads * rc.P * rc.Np);
+                    rc.keep_k = take(kept * (rc.heads / rc.per) * rc.N);
+                    rc.keep_d = take(kept * rc.heads * (tm ? rc.N : 2));
+                    rc.keep_v = take(kept * rc.heads * rc.P);
+                    c.recurrent = uint32_t(z.recurrent.size());
+                    z.recurrent.push_back(rc);
+                    z.max_heads = std::max(z.max_heads, rc.heads);
+                }
+                c.ring = rings + ring;
+                ring += size_t(cfg.max_seqs) * c.ring_len * c.channels;
+                z.run.push_back(c);
+                i++;
+            }
+        }
+        if (pass == 0) {
+            f(z.rings, ring);
+            f(z.states, state);
+        }
+    }
+    z.caches.alloc(z.run.size() * sizeof(MixerCache), false);
+    z.caches.write_vec(0, z.run);
+    if (z.recurrent.empty()) return;
+    z.recurrent_dev.alloc(z.recurrent.size() * sizeof(RecurrentCache), false);
+    z.recurrent_dev.write_vec(0, z.recurrent);
+}
+
+void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base) {
+    if (!cfg.fp32 && gemm_fits(w, n)) {
+        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr);
+    } else if (!cfg.fp32 && stream_fits(w, n)) {
+        matmul(w, n, nullptr, y, epi, base, nullptr, 0, nullptr, xb, yb);
+    } else {
+        LinearArgs a{};
+        a.W = reinterpret_cast<const uint16_t*>(w.w);
+        a.X = cfg.fp32 ? static_cast<const void*>(xf) : xb;
+        a.base = base;
+        a.Y = y;
+        a.Yb = yb;
+        a.n = n;
+        a.m = w.m;
+        a.k = w.k;
+        a.epi = epi;
+        launch_linear(a, !cfg.fp32, stream);
+    }
+}
+
+// A mixer's output: onto the stream (from `cur`, the residual added) or, as one of several, into a place of its own.
+void Engine::mixer_out(const Matrix& o, uint32_t n, const float* cur, float* alone) {
+    LayeredState& z = *lay;
+    const int sp = span_begin(G_MATMUL);
+    project(o, n, z.attn_f.as<float>(), z.attn_b.as<uint16_t>(), alone ? alone : s.h.as<float>(), nullptr, alone ? EPI_RAW : EPI_RESID, alone ? nullptr : cur);
+    span_end(sp);
+}
+
+// What a convolution or shift over rows u needs to find the rows before them, and to leave its own.
+ConvArgs Engine::conv_args(StepSet& st, const Plan& p, const MixerCache& mc, const float* u, uint32_t ldu, uint32_t taps) {
+    ConvArgs c{};
+    c.u = u;
+    c.ldu = ldu;
+    c.taps = taps;
+    c.ring = mc.ring;
+    c.ring_len = mc.ring_len;
+    c.conv_channels = mc.channels;
+    c.write_ring = mc.channels && p.max_run <= VERIFY_T;  // a step whose runs all fit a verified run leaves the rows as it goes
+    c.meta = s.meta.as<uint32_t>();
+    c.tin = st.in<uint32_t>(st.o_tin);
+    c.vis = st.in<uint32_t>(st.o_vis);
+    return c;
+}
+
+void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, const MixerCache& mc, const float* cur, float* alone, bool capture) {
+    LayeredState& z = *lay;
+    const uint32_t n = p.n;
+    const bool f32 = cfg.fp32;
+    int sp = span_begin(G_MATMUL);
+    project(a.proj, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), z.proj.as<float>(), nullptr, EPI_RAW);
+    span_end(sp);
+    ConvArgs c = conv_args(st, p, mc, z.proj.as<float>(), a.proj.m, a.conv.w ? a.conv.taps : 1);
+    c.w = a.conv.w;
+    c.rope = a.rot.dims ? z.rope[a.rot.table].as<float>() : nullptr;
+    c.kv = mc.kv;
+    c.heads = a.heads;
+    c.rot_dims = a.rot.dims;
+    c.unit_qk = a.unit_qk;
+    c.unit_eps = model.md.eps;
+    c.temp = a.temp;
+    const bool fast_attn = !f32 && !tuning.plain_attention && chunk_attn_fits(a.dim, a.vdim, model.md.page);
+    if (fast_attn) c.q_b = z.q_b.as<uint16_t>();
+    else c.q_f = z.q_f.as<float>();
+    c.q_scale = a.scale * LOG2E;
+    sp = span_begin(G_SMALL);
+    launch_conv_qkv(c, n, f32, stream);
+    if (mc.channels && !c.write_ring) launch_conv_state(c, st.in<RunIn>(st.o_runs), p.n_runs, stream);
+    span_end(sp);
+    ChunkedAttnArgs at{};
+    at.q_f = z.q_f.as<float>();
+    at.q_b = z.q_b.as<uint16_t>();
+    at.ctiles = st.in<uint32_t>(st.o_ctiles);
+    at.meta = c.meta;
+    at.tin = c.tin;
+    at.vis = c.vis;
+    at.kv = mc.kv;
+    at.gate = a.gated ? z.proj.as<float>() + a.qkv_w() : nullptr;
+    at.ldg = a.proj.m;
+    at.heads = a.heads;
+    at.chunk = a.chunk;
+    at.window = a.window;
+    at.scale = a.scale;
+    at.out = f32 || capture ? z.attn_f.as<float>() : nullptr;
+    at.out_b = z.attn_b.as<uint16_t>();
+    uint32_t most = p.max_keys;  // keys a row may see
+    for (uint32_t bound : {a.chunk, a.window})
+        if (bound) most = std::min(most, bound);
+    sp = span_begin(G_ATTN);
+    if (fast_attn) launch_attn_chunked(at, n, p.chunked ? p.ctiles : 0, most, sm_count, tuning.attn_keys_per_cta, stream);
+    else launch_attn_any(at, n, f32, stream);
+    span_end(sp);
+    mixer_out(a.o, n, cur, alone);
+}
+
+// The recurrence itself and the norm and gate of its outputs, from the rows that the mixer has prepared.
+void Engine::encode_recurrence(StepSet& st, const Plan& p, ScanArgs& a, GatedNormArgs& g) {
+    LayeredState& z = *lay;
+    a.runs = st.in<RunIn>(st.o_runs);
+    a.gen = s.gen.as<GenState>();
+    a.meta = s.meta.as<uint32_t>();
+    a.vis = st.in<uint32_t>(st.o_vis);
+    a.n_runs = p.n_runs;
+    a.max_run = p.max_run;
+    a.y = z.y.as<float>();
+    g.y = a.y;
+    g.width = a.c.heads * a.c.P;
+    g.eps = model.md.eps;
+    g.out_f32 = cfg.fp32 ? z.attn_f.as<float>() : nullptr;
+    g.out_bf16 = z.attn_b.as<uint16_t>();
+    int sp = span_begin(G_ATTN);
+    launch_scan(a, stream);
+    span_end(sp);
+    sp = span_begin(G_SMALL);
+    launch_gated_norm(g, p.n, stream);
+    span_end(sp);
+}
+
+void Engine::encode_state_space(StepSet& st, const Plan& p, const StateSpace& x, const MixerCache& mc, const float* cur, float* alone) {
+    LayeredState& z = *lay;
+    const uint32_t n = p.n, inner = x.inner(), ld = x.in.m;
+    float* proj = z.proj.as<float>();
+    int sp = span_begin(G_MATMUL);
+    project(x.in, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), proj, nullptr, EPI_RAW);
+    span_end(sp);
+    ConvArgs c = conv_args(st, p, mc, proj + inner, ld, x.conv.taps);
+    c.w = x.conv.w;
+    c.bias = x.conv.b;
+    sp = span_begin(G_SMALL);
+    launch_conv_silu(c, StepSizeArgs{proj + inner + x.channels(), ld, x.heads, x.dt_bias, x.a_log, z.steps.as<float>()}, n, z.conv.as<float>(), stream);
+    if (!c.write_ring) launch_conv_state(c, st.in<RunIn>(st.o_runs), p.n_runs, stream);
+    span_end(sp);
+    ScanArgs a{};
+    a.c = z.recurrent[mc.recurrent];
+    a.v = z.conv.as<float>();
+    a.k = a.v + inner;
+    a.q = a.k + x.groups * x.state;
+    a.ldq = a.ldk = a.ldv = x.channels();
+    a.decay = z.steps.as<float>();
+    a.skip = x.skip;
+    GatedNormArgs g{};
+    g.gate = proj;
+    g.ldg = ld;
+    g.w = x.norm;
+    g.groups = x.norm_groups;
+    g.gate_first = true;
+    encode_recurrence(st, p, a, g);
+    mixer_out(x.o, n, cur, alone);
+}
+
+void Engine::encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const MixerCache& mc, const float* cur, float* alone) {
+    LayeredState& z = *lay;
+    const uint32_t n = p.n, d = model.md.d, K = x.inner();
+    const bool f32 = cfg.fp32;
+    // r, k, v and g are one grouped product over the four mixes they read.
+    const bool fast = !f32 && grouped_fits(K, d);
+    ShiftArgs sh{};
+    sh.c = conv_args(st, p, mc, z.xn_f.as<float>(), d, 2);
+    for (int i = 0; i < 5; i++) sh.mu[i] = x.mu[i];
+    sh.out_f32 = z.mix_f.as<float>();
+    sh.out_bf16 = z.mix_b.as<uint16_t>();
+    sh.tiles = z.tiles.as<uint32_t>();
+    sh.n_tiles = z.n_tiles.as<uint32_t>();
+    sh.tile = 64;
+    if (fast)
+        for (sh.tile = SHIFT_TILE_MIN; sh.tile < 128 && sh.tile < n;) sh.tile *= 2;
+    int sp = span_begin(G_SMALL);
+    launch_token_shift(sh, n, stream);
+    if (!sh.c.write_ring) launch_conv_state(sh.c, st.in<RunIn>(st.o_runs), p.n_runs, stream);
+    span_end(sp);
+    sp = span_begin(G_MATMUL);
+    LinearArgs l{};
+    l.W = reinterpret_cast<const uint16_t*>(x.rkvg.w);
+    const size_t one = size_t(n) * d;  // (the decay's mix lies first, at an address that does not depend on n)
+    l.X = f32 ? static_cast<const void*>(sh.out_f32 + one) : sh.out_bf16 + one;
+    l.Y = z.proj.as<float>();
+    l.m = K;
+    l.k = d;
+    l.epi = EPI_RAW;
+    l.tiles = sh.tiles;
+    l.n_tiles = sh.n_tiles;
+    l.max_tiles = 4 * ((n + sh.tile - 1) / sh.tile);
+    if (fast) launch_grouped(l, 4, sh.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(l, !f32, stream);
+    project(x.w1, n, sh.out_f32, sh.out_bf16, z.low.as<float>(), nullptr, EPI_RAW);
+    span_end(sp);
+    const size_t rows = size_t(n) * K;
+    DecayArgs dc{};
+    dc.hid = z.low.as<float>();
+    dc.ldh = x.w1.m;
+    dc.r = l.Y;
+    dc.k = l.Y + rows;
+    dc.w2 = x.w2;
+    dc.w0 = x.w0;
+    dc.u = x.bonus;
+    dc.rank = x.rank;
+    dc.heads = x.heads;
+    dc.dim = x.dim;
+    dc.decay = z.decay.as<float>();
+    dc.bonus = z.steps.as<float>();
+    sp = span_begin(G_SMALL);
+    launch_decay(dc, n, stream);
+    span_end(sp);
+    ScanArgs a{};
+    a.c = z.recurrent[mc.recurrent];
+    a.q = dc.r;
+    a.k = dc.k;
+    a.v = l.Y + 2 * rows;
+    a.ldq = a.ldk = a.ldv = K;
+    a.decay = dc.decay;
+    a.bonus = dc.bonus;
+    GatedNormArgs g{};
+    g.gate = l.Y + 3 * rows;
+    g.ldg = K;
+    g.w = x.norm;
+    g.groups = x.heads;
+    encode_recurrence(st, p, a, g);
+    mixer_out(x.o, n, cur, alone);
+}
+
+void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture) {
+    const LayeredModel& m = *model.layered;
+    const ModelDesc& md = model.md;
+    begin_step(set, p);  // upload; the embedding into x0
+    LayeredState& z = *lay;
+    StepSet& st = sets[set];
+    const bool f32 = cfg.fp32;
+    const uint32_t n = p.n, d = md.d;
+    float* h = s.h.as<float>();
+    const float* cur = z.x0.as<float>();  // the stream; h from the first layer on
+    bool normed = false;  // the layer before has left norm1's rows
+    auto host = [&](const float* dev, size_t count) {
+        std::vector<float> v(count);
+        VLT_CUDA(cudaMemcpyAsync(v.data(), dev, count * 4, cudaMemcpyDeviceToHost, stream));
+        VLT_CUDA(cudaStreamSynchronize(stream));
+        return v;
+    };
+    NormArgs na{};
+    na.n = n;
+    na.k = d;
+    na.eps = md.eps;
+    na.scale = 1.0f;
+    na.out_f32 = z.xn_f.as<float>();
+    na.out_bf16 = z.xn_b.as<uint16_t>();
+    for (uint32_t ri = 0; ri < m.runs.size(); ri++) {
+        const FolderLayer& l = m.layers[m.runs[ri].layer];
+        int sp;
+        if (m.runs[ri].loop_in) {
+            sp = span_begin(G_SMALL);
+            launch_concat_rows(cur, z.x0.as<float>(), n, d, z.cat_f.as<float>(), z.cat_b.as<uint16_t>(), stream);
+            span_end(sp);
+            sp = span_begin(G_MATMUL);
+            project(m.loop_in, n, z.cat_f.as<float>(), z.cat_b.as<uint16_t>(), h, nullptr, EPI_RAW);
+            span_end(sp);
+            cur = h;
+        }
+        std::vector<float> resid_in, sdpa;
+        uint32_t attn_width = 0;
+        if (!normed) {
+            na.in = cur;
+            na.add = m.runs[ri].add_embed ? z.x0.as<float>() : nullptr;
+            na.sum = h;
+            na.norm = l.norm1;
+            sp = span_begin(G_SMALL);
+            launch_norm_rows(na, stream);
+            span_end(sp);
+            if (na.add) cur = h;
+            na.add = nullptr;
+        }
+        if (capture) resid_in = host(cur, size_t(n) * d);
+        const bool several = l.mix.size() > 1;
+        for (uint32_t b = 0; b < l.mix.size(); b++) {
+            const Mixer& x = l.mix[b];
+            const MixerCache& mc = z.run[z.first[ri] + b];
+            float* alone = several ? z.branch.as<float>() + size_t(b) * n * d : nullptr;
+            switch (x.kind) {
+            case MixerKind::Attention: encode_attention(st, p, x.attn, mc, cur, alone, capture != nullptr); break;
+            case MixerKind::StateSpace: encode_state_space(st, p, x.ssm, mc, cur, alone); break;
+            case MixerKind::TimeMix: encode_time_mix(st, p, x.tmix, mc, cur, alone); break;
+            }
+            if (capture && x.kind == MixerKind::Attention) {
+                attn_width = x.attn.out_w();
+                sdpa = host(z.attn_f.as<float>(), size_t(n) * attn_width);
+            }
+        }
+        if (several) {
+            MergeArgs mg{};
+            mg.x = cur;
+            mg.a = z.branch.as<float>();
+            mg.b = mg.a + size_t(n) * d;
+            mg.norm_a = l.mix[0].out;
+            mg.norm_b = l.mix[1].out;
+            if (l.mlp == MlpKind::Dense) mg.norm = l.norm2;
+            mg.out = h;
+            mg.next = na.out_f32;
+            mg.next_b = na.out_bf16;
+            mg.n = n;
+            mg.d = d;
+            mg.eps = md.eps;
+            sp = span_begin(G_SMALL);
+            launch_merge_rows(mg, stream);
+            span_end(sp);
+        }
+        cur = h;
+        normed = false;
+        if (l.mlp == MlpKind::Experts) {
+            const bool next_norm = ri + 1 < m.runs.size() && !m.runs[ri + 1].loop_in && !m.runs[ri + 1].add_embed;
+            encode_experts(l, n, next_norm ? m.layers[m.runs[ri + 1].layer].norm1 : RowNorm{});
+            normed = next_norm;
+        } else if (l.mlp == MlpKind::Dense) {
+            if (!several) {
+                na.in = h;
+                na.norm = l.norm2;
+                sp = span_begin(G_SMALL);
+                launch_norm_rows(na, stream);
+                span_end(sp);
+            }
+            sp = span_begin(G_MATMUL);
+            project(l.dense.up, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), EPI_RELU2);
+            project(l.dense.down, n, z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), h, nullptr, EPI_RESID, h);
+            span_end(sp);
+        }
+        if (capture) {
+            const std::vector<float> resid_out = host(h, size_t(n) * d);
+            LayerCapture lc{ri, n, resid_in.data(), nullptr, nullptr, attn_width ? sdpa.data() : nullptr, nullptr, nullptr, nullptr};
+            lc.resid_out = resid_out.data();
+            lc.attn_width = attn_width;
+            (*capture)(lc);
+        }
+        // (kernels.metal:133-148 `tap_rows`, as the other architectures' taps)
+        auto tap = std::find(tap_layers.begin(), tap_layers.end(), ri);
+        if (tap != tap_layers.end()) launch_prep_rows(h, nullptr, n, d, md.eps, tap_bufs[tap - tap_layers.begin()].as<float>(), nullptr, nullptr, true, true, stream);
+    }
+    // The tail: the final norm of the hidden and head rows, the head, sampling, accept, compaction.
+    const int sp = span_begin(G_TAIL);
+    na.in = h;
+    na.norm = m.final_norm;
+    na.rows = st.in<uint32_t>(st.o_hidden_rows);
+    na.n = p.n_hidden;
+    na.out_f32 = s.hfin_all.as<float>();
+    na.out_bf16 = nullptr;
+    launch_norm_rows(na, stream);
+    if (p.n_head) {
+        na.rows = st.in<uint32_t>(st.o_head_rows);
+        na.n = p.n_head;
+        na.scale = m.logit_scale;  // (the head is linear)
+        na.out_f32 = s.hfin_head.as<float>();
+        na.out_bf16 = f32 ? nullptr : s.hfin_b.as<uint16_t>();
+        launch_norm_rows(na, stream);
+        project(model.head, p.n_head, s.hfin_head.as<float>(), s.hfin_b.as<uint16_t>(), s.logits.as<float>(), nullptr, EPI_RAW);
+        if (!forced_logits.empty()) {
+            if (forced_logits.size() != size_t(p.n_head) * md.vocab) throw Error("forced logits: wrong size");
+            VLT_CUDA(cudaMemcpyAsync(s.logits.dev, forced_logits.data(), forced_logits.size() * 4, cudaMemcpyHostToDevice, stream));
+        }
+        launch_sample(s.logits.as<float>(), st.in<SampleRow>(st.o_sample_rows), st.out<uint32_t>(st.o_out_ids), s.meta.as<uint32_t>(), p.n_head, md.vocab, stream, nullptr);
+    }
+    launch_accept(st.in<RunIn>(st.o_runs), st.in<uint32_t>(st.o_tokens), st.out<uint32_t>(st.o_out_ids), s.lens.as<uint32_t>(), s.feed.as<uint32_t>(), s.gen.as<GenState>(),
+                  st.out<uint32_t>(st.o_emitted), p.n_runs, s.tree.as<uint32_t>(), s.path.as<uint32_t>(), s.path_len.as<uint32_t>(), s.on_path.as<uint32_t>(), stream, nullptr);
+    if (p.branches)
+        launch_mixer_compact(st.in<RunIn>(st.o_runs), s.path.as<uint32_t>(), s.path_len.as<uint32_t>(), s.lens.as<uint32_t>(), z.caches.as<MixerCache>(), p.n_runs,
+                             uint32_t(z.run.size()), f32, stream);
+    if (p.verified)
+        launch_recurrent_commit(st.in<RunIn>(st.o_runs), s.path.as<uint32_t>(), s.path_len.as<uint32_t>(), s.lens.as<uint32_t>(), z.recurrent_dev.as<RecurrentCache>(), p.n_runs,
+                                uint32_t(z.recurrent.size()), z.max_heads, stream);
+    span_end(sp);
+}
+
+// h += the experts' weighted rows + the shared expert's, on norm2's rows of h; norm: the norm the next layer run begins
+// with, whose rows are then left as well.
+void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
+    LayeredState& z = *lay;
+    const ExpertLayer& e = l.experts;
+    const bool f32 = cfg.fp32;
+    const uint32_t d = model.md.d, pairs = n * e.top;
+    float* h = s.h.as<float>();
+    RouterArgs r{};
+    r.x = h;
+    r.norm = l.norm2;
+    r.router = e.router;
+    r.correction = e.correction;
+    r.xn = f32 || e.identity ? z.moe_x.as<float>() : nullptr;
+    r.xn_b = z.moe_xb.as<uint16_t>();
+    r.ids = z.ids.as<uint32_t>();
+    r.weights = z.weights.as<float>();
+    r.n = n;
+    r.d = d;
+    r.experts = e.experts;
+    r.identity = e.identity;
+    r.top = e.top;
+    r.eps = model.md.eps;
+    SortArgs so{};
+    so.ids = r.ids;
+    so.src = z.src.as<uint32_t>();
+    so.place = z.place.as<uint32_t>();
+    so.tiles = z.tiles.as<uint32_t>();
+    so.n_tiles = z.n_tiles.as<uint32_t>();
+    so.n = n;
+    so.top = e.top;
+    so.experts = e.experts;
+    // The experts' matrices on the tensor cores where their sizes fit: tiles as long as an expert's rows on average, so that
+    // its weights are read once. On the CUDA cores a tile has 64.
+    const bool fast = !f32 && grouped_fits(e.ff, d) && grouped_fits(d, e.ff);
+    so.tile = 64;
+    if (fast)
+        for (so.tile = EXPERT_TILE_MIN; so.tile < 128 && so.tile < 2 * pairs / (e.experts + e.identity);) so.tile *= 2;
+    int sp = span_begin(G_SMALL);
+    launch_router(r, stream);
+    launch_expert_sort(so, stream);
+    span_end(sp);
+    sp = span_begin(G_MATMUL);
+    LinearArgs up{};
+    up.W = reinterpret_cast<const uint16_t*>(e.up.w);
+    up.X = f32 ? static_cast<const void*>(z.moe_x.as<float>()) : z.moe_xb.as<uint16_t>();
+    up.src = so.src;
+    up.Y = z.hid_f.as<float>();
+    up.Yb = z.hid_b.as<uint16_t>();
+    up.m = e.ff;
+    up.k = d;
+    up.epi = EPI_RELU2;
+    up.tiles = so.tiles;
+    up.n_tiles = so.n_tiles;
+    up.max_tiles = pairs / so.tile + std::min(e.experts, pairs);
+    if (fast) launch_grouped(up, e.experts, so.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(up, !f32, stream);
+    LinearArgs down = up;
+    down.W = reinterpret_cast<const uint16_t*>(e.down.w);
+    down.X = f32 ? static_cast<const void*>(z.hid_f.as<float>()) : z.hid_b.as<uint16_t>();
+    down.src = nullptr;
+    down.Y = z.rows.as<float>();
+    down.Yb = nullptr;
+    down.m = d;
+    down.k = e.ff;
+    down.epi = EPI_RAW;
+    if (fast) launch_grouped(down, e.experts, so.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(down, !f32, stream);
+    if (e.shared_ff) {
+        project(e.shared_up, n, z.moe_x.as<float>(), z.moe_xb.as<uint16_t>(), z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), EPI_RELU2);
+        project(e.shared_down, n, z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), z.shared.as<float>(), nullptr, EPI_RAW);
+    }
+    span_end(sp);
+    CombineArgs c{};
+    c.x = h;
+    c.y = z.rows.as<float>();
+    c.xn = z.moe_x.as<float>();
+    c.shared = e.shared_ff ? z.shared.as<float>() : nullptr;
+    c.ids = r.ids;
+    c.place = so.place;
+    c.weights = r.weights;
+    c.out = h;
+    c.norm = norm;
+    c.next = z.xn_f.as<float>();
+    c.next_b = z.xn_b.as<uint16_t>();
+    c.d = d;
+    c.experts = e.experts;
+    c.top = e.top;
+    c.eps = model.md.eps;
+    sp = span_begin(G_SMALL);
+    launch_combine(c, n, stream);
+    span_end(sp);
+}
+
+}  // namespace vlt

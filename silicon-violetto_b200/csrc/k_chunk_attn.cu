@@ -1,6 +1,6 @@
-// Chunked, gated attention over paged keys on the tensor cores, for head sizes that are instantiated below (other sizes and
-// fp32 caches: k_mixer.cu's scalar kernel). A position sees the keys of its own chunk of positions only, so what a row walks
-// is bounded by the chunk, and starts wherever the chunk does, in the middle of a page or not.
+// Attention over paged keys on the tensor cores, chunked, windowed or over everything before, for head sizes that are instantiated
+// below (other sizes and fp32 caches: k_mixer.cu's scalar kernel). What a row walks begins wherever its chunk or window does, in
+// the middle of a page or not, and is bounded by it.
 //
 //   chunk_decode_kernel   a row (token) and up to 8 query heads of one kv head per block: the keys are the MMAs' M side, the
 //                         heads its columns; four warps take tiles of 16 keys in turn, each with its own ring of asynchronous
@@ -11,7 +11,7 @@
 //                         has few blocks for its SMs); the softmax stays in registers.
 //
 // Both take q rotated, scaled by scale * log2(e) and rounded to bf16, keep scores and softmax in fp32, and finish the mixer:
-// the output times sigmoid(gate), bf16 for the projection after it.
+// the output times sigmoid(gate) where there is a gate, bf16 for the projection after it.
 #include <algorithm>
 
 #include "kernels.h"
@@ -38,7 +38,7 @@ __device__ __forceinline__ float gated(float y, float gate) { return y / (1.0f +
 constexpr uint32_t PAGE_SHIFT = 6, PAGE = 1u << PAGE_SHIFT;
 
 // What token t sees: cached keys [lo, first) and, of its tile of 8 rows that starts at cache position `first`, those `mask`
-// names (its `vis`, less the rows of another chunk: siblings of a draft tree may lie on both sides of an edge).
+// names (its `vis`, less the rows of an earlier chunk or out of the window: the rows of a draft tree may lie on both sides of an edge).
 struct View {
     uint32_t slot, lo, first, mask;
 };
@@ -47,16 +47,14 @@ __device__ __forceinline__ View view_of(const ChunkedAttnArgs& a, uint32_t t) {
     View v;
     v.slot = a.meta[2 * t];
     v.first = a.meta[2 * (t - row) + 1] + row - i;
-    v.lo = 0;
+    v.lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0;
     v.mask = a.vis[t];
-    if (a.chunk) {
-        const uint32_t c = pos / a.chunk;
-        v.lo = c * a.chunk;
+    if (v.lo) {
         uint32_t seen = 0;
         for (uint32_t m = v.mask; m;) {
             const uint32_t j = __ffs(m) - 1;
             m &= m - 1;
-            if (a.meta[2 * (t - i + j) + 1] / a.chunk == c) seen |= 1u << j;
+            if (a.meta[2 * (t - i + j) + 1] >= v.lo) seen |= 1u << j;
         }
         v.mask = seen;
     }
@@ -259,7 +257,8 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
 #pragma unroll
         for (uint32_t j = 0; j < PER; j++) {
             const uint32_t c = lane + 32 * j;
-            const float y = gated(oo[c2][j] / ll[c2], a.gate[size_t(t) * a.ldg + (h0 + col) * DV + c]);
+            float y = oo[c2][j] / ll[c2];
+            if (a.gate) y = gated(y, a.gate[size_t(t) * a.ldg + (h0 + col) * DV + c]);
             const size_t at = (size_t(t) * a.heads + h0 + col) * DV + c;
             if (a.out) a.out[at] = y;
             a.out_b[at] = f32_to_bf16(y);
@@ -455,11 +454,12 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
         if (!live[r]) continue;
         const float inv = l > 0.0f ? 1.0f / l : 0.0f;
         const size_t at = (size_t(tok[r]) * a.heads + h) * DV;
-        const float* gate = a.gate + size_t(tok[r]) * a.ldg + h * DV;
+        const float* gate = a.gate ? a.gate + size_t(tok[r]) * a.ldg + h * DV : nullptr;
 #pragma unroll
         for (uint32_t j = 0; j < ND; j++) {
             const uint32_t c = 8 * j + 2 * tq;
-            const float x = gated(o[j][2 * r] * inv, gate[c]), y = gated(o[j][2 * r + 1] * inv, gate[c + 1]);
+            float x = o[j][2 * r] * inv, y = o[j][2 * r + 1] * inv;
+            if (gate) { x = gated(x, gate[c]); y = gated(y, gate[c + 1]); }
             if (a.out) { a.out[at + c] = x; a.out[at + c + 1] = y; }
             *reinterpret_cast<uint32_t*>(a.out_b + at + c) = pack_bf16(x, y);
         }

@@ -1,6 +1,6 @@
 // Linear layers on the CUDA cores, for what the tensor-core kernels do not take: activations in fp32 throughout (true fp32
 // products and sums: bf16 weights are exact in fp32), and matrices whose sizes fit neither the streamed kernel nor the GEMM.
-// Also the row passes in front of a projection: RMS norm with a weight stored around zero, and two streams side by side.
+// Also the row passes in front of a projection: RMS norms, two streams side by side, and two mixers' outputs onto the stream.
 #include <algorithm>
 
 #include "kernels.h"
@@ -72,25 +72,66 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
     }
 }
 
-// out[r] = x / sqrt(mean(x^2) + eps) (1 + w) for row rows[r] (or r), fp32 and / or bf16. A block per row.
-__global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict__ in, const uint32_t* __restrict__ rows, uint32_t k, float eps, const uint16_t* __restrict__ w,
-                                                        float* out_f32, uint16_t* out_bf16) {
-    pdl_start();
-    __shared__ float red[8];
-    const uint32_t r = blockIdx.x, tid = threadIdx.x;
-    const float* x = in + size_t(rows ? rows[r] : r) * k;
-    float ss = 0.0f;
-    for (uint32_t i = tid; i < k; i += 256) ss += x[i] * x[i];
-    ss = warp_sum(ss);
-    if (tid % 32 == 0) red[tid / 32] = ss;
+__device__ __forceinline__ float block_sum(float v, float* red) {  // 256 threads; `red` of 8, free to use again after the next barrier
+    v = warp_sum(v);
+    if (threadIdx.x % 32 == 0) red[threadIdx.x / 32] = v;
     __syncthreads();
     float tot = 0.0f;
     for (uint32_t i = 0; i < 8; i++) tot += red[i];
-    const float inv = 1.0f / sqrtf(tot / float(k) + eps);
-    for (uint32_t i = tid; i < k; i += 256) {
-        const float v = x[i] * inv * (1.0f + bf16_to_f32(w[i]));
-        if (out_f32) out_f32[size_t(r) * k + i] = v;
-        if (out_bf16) out_bf16[size_t(r) * k + i] = f32_to_bf16(v);
+    return tot;
+}
+// See NormArgs. A block per row, which it keeps in shared memory.
+__global__ void __launch_bounds__(256) norm_rows_kernel(const NormArgs a) {
+    pdl_start();
+    extern __shared__ float row[];
+    __shared__ float red[8];
+    const uint32_t r = blockIdx.x, tid = threadIdx.x;
+    const size_t from = size_t(a.rows ? a.rows[r] : r) * a.k;
+    float ss = 0.0f;
+    for (uint32_t i = tid; i < a.k; i += 256) {
+        float x = a.in[from + i];
+        if (a.add) {
+            x += a.add[from + i];
+            a.sum[from + i] = x;
+        }
+        row[i] = x;
+        ss += x * x;
+    }
+    const float inv = a.scale / sqrtf(block_sum(ss, red) / float(a.k) + a.eps);
+    for (uint32_t i = tid; i < a.k; i += 256) {
+        const float v = row[i] * inv * weight_of(a.norm, i);
+        if (a.out_f32) a.out_f32[size_t(r) * a.k + i] = v;
+        if (a.out_bf16) a.out_bf16[size_t(r) * a.k + i] = f32_to_bf16(v);
+    }
+}
+
+// See MergeArgs. A block per row.
+__global__ void __launch_bounds__(256) merge_rows_kernel(const MergeArgs a) {
+    pdl_start();
+    extern __shared__ float row[];
+    __shared__ float red[3][8];
+    const uint32_t tid = threadIdx.x;
+    const size_t from = size_t(blockIdx.x) * a.d;
+    float sa = 0.0f, sb = 0.0f;
+    for (uint32_t i = tid; i < a.d; i += 256) {
+        const float p = a.a[from + i], q = a.b[from + i];
+        sa += p * p;
+        sb += q * q;
+    }
+    const float ia = 0.5f / sqrtf(block_sum(sa, red[0]) / float(a.d) + a.eps), ib = 0.5f / sqrtf(block_sum(sb, red[1]) / float(a.d) + a.eps);
+    float ss = 0.0f;
+    for (uint32_t i = tid; i < a.d; i += 256) {
+        const float y = a.x[from + i] + (a.a[from + i] * ia * weight_of(a.norm_a, i) + a.b[from + i] * ib * weight_of(a.norm_b, i));
+        a.out[from + i] = y;
+        row[i] = y;
+        ss += y * y;
+    }
+    if (!a.norm.w) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red[2]) / float(a.d) + a.eps);
+    for (uint32_t i = tid; i < a.d; i += 256) {
+        const float v = row[i] * inv * weight_of(a.norm, i);
+        if (a.next) a.next[from + i] = v;
+        if (a.next_b) a.next_b[from + i] = f32_to_bf16(v);
     }
 }
 
@@ -114,8 +155,15 @@ void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s) {
     if (x_bf16) launch_pdl(linear::linear_kernel<uint16_t>, grid, 256, 0, s, a);
     else launch_pdl(linear::linear_kernel<float>, grid, 256, 0, s, a);
 }
-void launch_norm_rows(const float* in, const uint32_t* rows, uint32_t n, uint32_t k, float eps, const uint16_t* w, float* out_f32, uint16_t* out_bf16, cudaStream_t s) {
-    if (n) launch_pdl(linear::norm_rows_kernel, n, 256, 0, s, in, rows, k, eps, w, out_f32, out_bf16);
+void launch_norm_rows(const NormArgs& a, cudaStream_t s) {
+    static PerDevice configured;
+    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(linear::norm_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); });
+    if (a.n) launch_pdl(linear::norm_rows_kernel, a.n, 256, size_t(a.k) * 4, s, a);
+}
+void launch_merge_rows(const MergeArgs& a, cudaStream_t s) {
+    static PerDevice configured;
+    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(linear::merge_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); });
+    if (a.n) launch_pdl(linear::merge_rows_kernel, a.n, 256, size_t(a.d) * 4, s, a);
 }
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s) {
     if (n) launch_pdl(linear::concat_rows_kernel, n, 256, 0, s, a, b, d, out_f32, out_bf16);

@@ -1,7 +1,8 @@
 // The attention mixer's work between its projections and its attention, as parameterised kernels: a short causal
-// convolution over time on q, k and v, rotation of pairs (i, i + dims / 2), K and V into a paged cache whose heads may have
+// convolution over time on q, k and v, rotation of pairs (i, i + dims / 2), q and k heads of unit length, queries that grow with
+// their position (each of them optional), K and V into a paged cache whose heads may have
 // different key and value sizes; the convolution's state -- the projected rows before the step -- in a ring per sequence
-// slot; and a scalar form of the chunked attention for any head sizes and for fp32 caches.
+// slot; and a scalar form of the chunked or windowed attention for any head sizes and for fp32 caches.
 #include <algorithm>
 
 #include "kernels.h"
@@ -20,29 +21,6 @@ __device__ __forceinline__ size_t page_row(const PagedKv& kv, uint32_t slot, uin
     return (size_t(page) * kv.n_kv + g) * psize + (pos & (psize - 1));
 }
 
-// Where the projected row `back` positions before token t lies: among the rows of its own tile of 8 that it descends from
-// (its `vis` mask names them: a chain's all, a draft tree's its ancestors), then among the run's earlier rows, then in the
-// slot's ring of rows that earlier steps left; none before the sequence's start.
-__device__ __forceinline__ const float* row_before(const ConvArgs& a, uint32_t t, uint32_t back) {
-    const uint32_t row = a.tin[2 * t + 1], i = row % 8;
-    if (back == 0) return a.u + size_t(t) * a.ldu;
-    uint32_t anc = a.vis[t] & ((1u << i) - 1);
-    const uint32_t n = __popc(anc);
-    if (back <= n) {
-        uint32_t bit = 0;
-        for (uint32_t k = 0; k < back; k++) {
-            bit = 31 - __clz(anc);
-            anc &= ~(1u << bit);
-        }
-        return a.u + size_t(t - i + bit) * a.ldu;
-    }
-    const uint32_t over = back - n;  // positions before the tile
-    if (over <= row - i) return a.u + size_t(t - i - over) * a.ldu;
-    const uint32_t before = over - (row - i), start = a.meta[2 * (t - row) + 1];  // positions before the run
-    if (before > start) return nullptr;
-    return a.ring + (size_t(a.tin[2 * t]) * a.ring_len + (start - before) % a.ring_len) * a.conv_channels;
-}
-
 // grid (tokens / TB, heads + 2 kv heads): one q, k or v head of TB tokens a block (a step of many tokens: the tokens' chains of
 // dependent loads run side by side).
 template <typename T, uint32_t TB>
@@ -52,6 +30,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
     __shared__ const float* from[TB][32];
     __shared__ uint32_t pos_s[TB], cpos_s[TB], slot_s[TB];
     __shared__ size_t row_s[TB];  // where the head's key or value goes in the cache
+    __shared__ float factor[TB];  // what multiplies the head of a query or key
     const uint32_t t0 = blockIdx.x * TB, unit = blockIdx.y, tid = threadIdx.x, nt = min(TB, n - t0);
     const uint32_t kind = unit < a.heads ? 0u : unit < a.heads + a.kv.n_kv ? 1u : 2u;
     const uint32_t head = kind == 0 ? unit : kind == 1 ? unit - a.heads : unit - a.heads - a.kv.n_kv, width = kind == 2 ? a.kv.dv : a.kv.dk;
@@ -60,25 +39,26 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
     const uint32_t mine = tid / 32, back = tid % 32;  // a warp per token works out where its rows lie
     if (mine < TB) {
         const uint32_t t = t0 + (mine < nt ? mine : 0);
-        if (back < a.taps) from[mine][back] = row_before(a, t, back);
+        if (back < a.taps) from[mine][back] = row_before(a, t, back);  // (without a convolution: the row itself)
         if (back == 0) {
             const uint32_t row = a.tin[2 * t + 1];
             slot_s[mine] = a.meta[2 * t];
             pos_s[mine] = a.meta[2 * t + 1];
             cpos_s[mine] = a.meta[2 * (t - row) + 1] + row;
             row_s[mine] = kind ? page_row(a.kv, slot_s[mine], head, cpos_s[mine]) : 0;
+            factor[mine] = kind == 0 && a.temp.every > 0 ? 1.0f + a.temp.coef * logf(float(floor(double(pos_s[mine] + 1) / a.temp.every)) + 1.0f) : 1.0f;
         }
     }
     __syncthreads();
     for (uint32_t c = tid; c < width; c += 128) {
-        const uint16_t* w = a.w + size_t(c0 + c) * a.taps;
+        const uint16_t* w = a.w ? a.w + size_t(c0 + c) * a.taps : nullptr;
         float s[TB] = {}, last[TB] = {};
         for (uint32_t j0 = 0; j0 < a.taps; j0 += 4) {  // four taps' loads together
             float wj[4], u[4][TB];
 #pragma unroll
             for (uint32_t k = 0; k < 4; k++) {
                 const bool real = j0 + k < a.taps;
-                wj[k] = real ? bf16_to_f32(w[j0 + k]) : 0.0f;
+                wj[k] = !real ? 0.0f : w ? bf16_to_f32(w[j0 + k]) : 1.0f;
 #pragma unroll
                 for (uint32_t i = 0; i < TB; i++) {
                     const float* p = real ? from[i][a.taps - 1 - j0 - k] : nullptr;
@@ -100,6 +80,15 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
         }
     }
     __syncthreads();
+    if (a.unit_qk && kind < 2) {  // a warp per token
+        if (mine < TB) {
+            float ss = 0.0f;
+            for (uint32_t c = back; c < width; c += 32) ss += y[mine * width + c] * y[mine * width + c];
+            ss = warp_sum(ss);
+            if (back == 0) factor[mine] *= 1.0f / sqrtf(ss / float(width) + a.unit_eps);
+        }
+        __syncthreads();
+    }
     const uint32_t half = a.rot_dims / 2;
     for (uint32_t c = tid; c < width; c += 128) {
 #pragma unroll
@@ -111,6 +100,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
                 const float2 cs = reinterpret_cast<const float2*>(a.rope)[size_t(pos_s[i]) * half + (c < half ? c : c - half)];
                 v = c < half ? yi[c] * cs.x - yi[c + half] * cs.y : yi[c] * cs.x + yi[c - half] * cs.y;
             }
+            if (kind < 2) v *= factor[i];
             if (kind == 0) {
                 const size_t o = (size_t(t0 + i) * a.heads + head) * width + c;
                 if (a.q_f) a.q_f[o] = v;
@@ -139,9 +129,9 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const ConvArgs a, const
     }
 }
 
-// Attention of one token and query head per block: the cached keys from the chunk's first position (or the sequence's) up to
-// the token's tile of 8, then the tile's rows its `vis` names that lie in the same chunk; softmax in fp32 with a running
-// maximum over blocks of 128 keys; the gate on the result.
+// Attention of one token and query head per block: the cached keys from the chunk's or window's first position (or the
+// sequence's) up to the token's tile of 8, then the tile's rows its `vis` names that lie no further back than that; softmax in fp32 with a running
+// maximum over blocks of 128 keys; the gate, if there is one, on the result.
 template <typename T>
 __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) {
     pdl_start();
@@ -152,7 +142,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
     const uint32_t t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, g = h / (a.heads / a.kv.n_kv);
     const uint32_t slot = a.meta[2 * t], pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], mask = a.vis[t];
     const uint32_t tile0 = t - row % 8, p_tile = a.meta[2 * (t - row) + 1] + row - row % 8;  // the tile's first token and cache position
-    const uint32_t lo = a.chunk ? pos / a.chunk * a.chunk : 0, n_old = p_tile > lo ? p_tile - lo : 0;
+    const uint32_t lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0, n_old = p_tile > lo ? p_tile - lo : 0;
     const T* K = static_cast<const T*>(a.kv.k);
     const T* V = static_cast<const T*>(a.kv.v);
     for (uint32_t c = tid; c < a.kv.dk; c += 128) q[c] = a.q_f[(size_t(t) * a.heads + h) * a.kv.dk + c];
@@ -167,7 +157,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
         if (!seen && i < n_old + 8) {
             const uint32_t j = i - n_old;
             kp = p_tile + j;
-            seen = ((mask >> j) & 1u) && (!a.chunk || a.meta[2 * (tile0 + j) + 1] / a.chunk == pos / a.chunk);
+            seen = ((mask >> j) & 1u) && a.meta[2 * (tile0 + j) + 1] >= lo;
         }
         if (seen) {
             const size_t r = page_row(a.kv, slot, g, kp);
@@ -200,7 +190,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
         __syncthreads();
     }
     for (uint32_t c = tid; c < a.kv.dv; c += 128) {
-        const float gt = 1.0f / (1.0f + expf(-a.gate[size_t(t) * a.ldg + h * a.kv.dv + c])), y = o[c] / l * gt;
+        const float gt = a.gate ? 1.0f / (1.0f + expf(-a.gate[size_t(t) * a.ldg + h * a.kv.dv + c])) : 1.0f, y = o[c] / l * gt;
         const size_t at = (size_t(t) * a.heads + h) * a.kv.dv + c;
         if (a.out) a.out[at] = y;
         if (a.out_b) a.out_b[at] = f32_to_bf16(y);
@@ -208,7 +198,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
 }
 
 // The accepted path's rows of a verified draft tree, from where they were computed to where they belong: K and V in every
-// layer run's pages, and the convolution's ring rows. grid (runs, layer runs); a thread keeps to its own columns.
+// layer run's pages, and the convolution's ring rows. grid (runs, mixers' caches); a thread keeps to its own columns.
 template <typename T>
 __global__ void __launch_bounds__(256) mixer_compact_kernel(const RunIn* __restrict__ runs, const uint32_t* __restrict__ path, const uint32_t* __restrict__ path_len,
                                                             const uint32_t* __restrict__ lens, const MixerCache* __restrict__ caches) {
@@ -230,7 +220,7 @@ __global__ void __launch_bounds__(256) mixer_compact_kernel(const RunIn* __restr
     }
 }
 
-// Small pseudo-random keys and values for positions that are not computed (benchmarks). grid (positions, layer runs).
+// Small pseudo-random keys and values for positions that are not computed (benchmarks). grid (positions, mixers' caches).
 template <typename T>
 __global__ void __launch_bounds__(256) mixer_fill_kernel(const MixerCache* __restrict__ caches, uint32_t slot, uint32_t from, uint32_t seed) {
     const MixerCache mc = caches[blockIdx.y];
@@ -264,15 +254,15 @@ void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream
     if (fp32) launch_pdl(mixer::attn_any_kernel<float>, dim3(n, a.heads), 128, smem, s, a);
     else launch_pdl(mixer::attn_any_kernel<uint16_t>, dim3(n, a.heads), 128, smem, s, a);
 }
-void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_layers,
+void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_caches,
                           bool fp32, cudaStream_t s) {
     if (!n_runs) return;
-    if (fp32) launch_pdl(mixer::mixer_compact_kernel<float>, dim3(n_runs, n_layers), 256, 0, s, runs, path, path_len, lens, caches);
-    else launch_pdl(mixer::mixer_compact_kernel<uint16_t>, dim3(n_runs, n_layers), 256, 0, s, runs, path, path_len, lens, caches);
+    if (fp32) launch_pdl(mixer::mixer_compact_kernel<float>, dim3(n_runs, n_caches), 256, 0, s, runs, path, path_len, lens, caches);
+    else launch_pdl(mixer::mixer_compact_kernel<uint16_t>, dim3(n_runs, n_caches), 256, 0, s, runs, path, path_len, lens, caches);
 }
-void launch_mixer_fill(const MixerCache* caches, uint32_t n_layers, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s) {
+void launch_mixer_fill(const MixerCache* caches, uint32_t n_caches, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s) {
     if (to <= from) return;
-    const dim3 grid(to - from, n_layers);
+    const dim3 grid(to - from, n_caches);
     if (fp32) mixer::mixer_fill_kernel<float><<<grid, 256, 0, s>>>(caches, slot, from, seed);
     else mixer::mixer_fill_kernel<uint16_t><<<grid, 256, 0, s>>>(caches, slot, from, seed);
     launch_counter()++;

@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
         for (uint32_t w = 0; w < NW; w++) tot += red[j][w];
         const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
         for (uint32_t i = tid; i < a.d; i += ROUTER_THREADS) {
-            const float v = x[j * a.d + i] * inv * (1.0f + bf16_to_f32(a.norm[i]));
+            const float v = x[j * a.d + i] * inv * weight_of(a.norm, i);
             x[j * a.d + i] = v;
             const size_t o = size_t(t0 + j) * a.d + i;
             if (a.xn) a.xn[o] = v;
@@ -244,7 +244,7 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
         reinterpret_cast<V*>(row)[i] = y;
         ss += square(y);
     }
-    if (!a.norm) return;
+    if (!a.norm.w) return;
     ss = warp_sum(ss);
     if (tid % 32 == 0) red[tid / 32] = ss;
     __syncthreads();
@@ -253,7 +253,7 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
     for (uint32_t i = tid; i < a.d; i += 256) {
         const size_t o = size_t(t) * a.d + i;
-        const float v = row[i] * inv * (1.0f + bf16_to_f32(a.norm[i]));
+        const float v = row[i] * inv * weight_of(a.norm, i);
         if (a.next) a.next[o] = v;
         if (a.next_b) a.next_b[o] = f32_to_bf16(v);
     }

@@ -4,6 +4,7 @@
 
 #include "common.h"
 #include "device.cuh"
+#include "layered.h"
 #include "weights.h"
 
 namespace vlt {
@@ -27,6 +28,8 @@ struct QkvEpilogue {
     uint16_t* k_cache;
     uint16_t* v_cache;
 };
+
+__device__ __forceinline__ float weight_of(const RowNorm& n, uint32_t i) { return (n.around_zero ? 1.0f : 0.0f) + bf16_to_f32(n.w[i]); }
 
 // Y[t][row] = epilogue(W[row] . bf16(X[t])). X fp32 [n][k]; Y fp32 (SWIGLU: [n][m/2]).
 struct MatArgs {
@@ -58,7 +61,8 @@ struct MatArgs {
 };
 
 void launch_embed(const uint16_t* table, uint32_t* tokens, float* out, const uint32_t* tin, uint32_t* meta, const uint32_t* lens,
-                  const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s);
+                  const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s,
+                  const uint16_t* positions = nullptr, uint32_t n_positions = 0);  // positions: [n_positions][d], a vector per position to add
 void launch_qkv_post(const float* qkv, const uint32_t* meta, const uint32_t* tin, const float* rope, uint16_t* k_cache, uint16_t* v_cache,
                      const uint32_t* page_table, KvArgs kv, uint32_t layer, uint32_t n, uint32_t n_heads, float scale_log2, uint16_t* q_b, const uint32_t* cpos, cudaStream_t s);
 // q | k | v rows as the attention sees them before rounding (RoPE on q and k, kernels.metal:727-736), for step_capture.
@@ -215,7 +219,33 @@ struct LinearArgs {
 void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s);
 bool grouped_fits(uint32_t m, uint32_t k);  // the tensor-core form (k_grouped.cu): bf16 activations, EPI_RAW or EPI_RELU2
 void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint32_t* err_flag, cudaStream_t s);
-void launch_norm_rows(const float* in, const uint32_t* rows, uint32_t n, uint32_t k, float eps, const uint16_t* w, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
+// out[r] = x / sqrt(mean x^2 + eps) times the weight times `scale`, x being row rows[r] (or r) of `in`, plus that of `add`, the
+// sum then left in `sum`.
+struct NormArgs {
+    const float* in;
+    const uint32_t* rows;    // optional
+    const float* add;        // optional
+    float* sum;              // with add
+    uint32_t n, k;
+    float eps;
+    RowNorm norm;
+    float scale;
+    float* out_f32;          // optional
+    uint16_t* out_bf16;      // optional
+};
+void launch_norm_rows(const NormArgs& a, cudaStream_t s);
+// x[r] += the mean of two rows, each divided by its root mean square and times its weight; norm.w (optional): the normed rows of
+// the sum as well.
+struct MergeArgs {
+    const float *x, *a, *b;
+    RowNorm norm_a, norm_b, norm;
+    float* out;              // may be x
+    float* next;             // optional
+    uint16_t* next_b;        // optional
+    uint32_t n, d;
+    float eps;
+};
+void launch_merge_rows(const MergeArgs& a, cudaStream_t s);
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
 
 // One layer run's pages: [page][kv head][position in page][dk or dv] for K and for V, bf16 or fp32.
@@ -224,16 +254,18 @@ struct PagedKv {
     const uint32_t* page_table;
     uint32_t max_pages, page_shift, n_kv, dk, dv;
 };
-// A layer run's cache as the path compaction and the benchmark's fill see it.
+// A mixer's cache as the path compaction and the benchmark's fill see it (kv.n_kv 0: no pages; channels 0: no ring).
 struct MixerCache {
     PagedKv kv;
     float* ring;
     uint32_t ring_len, channels;
+    uint32_t recurrent;  // a recurrence's index among the model's (see RecurrentCache)
 };
 // The work between an attention mixer's projections and its attention (k_mixer.cu).
 struct ConvArgs {
     const float* u;                       // projected rows, q | k | v | ... [n][ldu]
-    const uint16_t* w;                    // [channels][taps]
+    const uint16_t* w;                    // [channels][taps]; NULL: no convolution (taps is 1, and there is no ring)
+    const uint16_t* bias;                 // [channels] (launch_conv_silu), optional
     float* ring;                          // [slot][ring_len][channels]: the projected rows of the positions before the step
     const uint32_t *meta, *tin, *vis;
     const float* rope;                    // [position][rot_dims / 2] (cos, sin)
@@ -243,7 +275,32 @@ struct ConvArgs {
     float q_scale;
     uint32_t ldu, taps, ring_len, conv_channels, heads, rot_dims;
     bool write_ring;                      // false: launch_conv_state does it afterwards
+    float unit_eps;                       // with unit_qk: q's and k's heads over sqrt(mean square + unit_eps)
+    bool unit_qk;
+    QueryTemperature temp;
 };
+// Where the row `back` positions before token t lies: among the rows of its own tile of 8 that it descends from (its `vis` mask
+// names them: a chain's all, a draft tree's its ancestors), then among the run's earlier rows, then in the slot's ring of rows
+// that earlier steps left; none before the sequence's start.
+__device__ __forceinline__ const float* row_before(const ConvArgs& a, uint32_t t, uint32_t back) {
+    const uint32_t row = a.tin[2 * t + 1], i = row % 8;
+    if (back == 0) return a.u + size_t(t) * a.ldu;
+    uint32_t anc = a.vis[t] & ((1u << i) - 1);
+    const uint32_t n = __popc(anc);
+    if (back <= n) {
+        uint32_t bit = 0;
+        for (uint32_t k = 0; k < back; k++) {
+            bit = 31 - __clz(anc);
+            anc &= ~(1u << bit);
+        }
+        return a.u + size_t(t - i + bit) * a.ldu;
+    }
+    const uint32_t over = back - n;  // positions before the tile
+    if (over <= row - i) return a.u + size_t(t - i - over) * a.ldu;
+    const uint32_t before = over - (row - i), start = a.meta[2 * (t - row) + 1];  // positions before the run
+    if (before > start) return nullptr;
+    return a.ring + (size_t(a.tin[2 * t]) * a.ring_len + (start - before) % a.ring_len) * a.conv_channels;
+}
 void launch_conv_qkv(const ConvArgs& a, uint32_t n, bool fp32, cudaStream_t s);
 void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cudaStream_t s);
 struct ChunkedAttnArgs {
@@ -252,8 +309,8 @@ struct ChunkedAttnArgs {
     const uint32_t *meta, *tin, *vis;
     const uint32_t* ctiles;               // the prefill kernel's (first token, rows <= 64) tiles
     PagedKv kv;
-    const float* gate;                    // [n][ldg]: the output is multiplied by sigmoid(gate)
-    uint32_t ldg, heads, chunk;           // chunk 0: every position before
+    const float* gate;                    // optional [n][ldg]: the output is multiplied by sigmoid(gate)
+    uint32_t ldg, heads, chunk, window;   // what a position sees (see Attention); both 0: every position before
     float scale;
     float* out;                           // optional [n][heads][dv]
     uint16_t* out_b;                      // optional
@@ -261,14 +318,85 @@ struct ChunkedAttnArgs {
 bool chunk_attn_fits(uint32_t dk, uint32_t dv, uint32_t page);  // k_chunk_attn.cu's kernels, bf16 caches; else launch_attn_any
 void launch_attn_chunked(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s);
-void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_layers,
+void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_caches,
                           bool fp32, cudaStream_t s);
-void launch_mixer_fill(const MixerCache* caches, uint32_t n_layers, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s);
+void launch_mixer_fill(const MixerCache* caches, uint32_t n_caches, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s);
+
+// Linear recurrences (k_recurrent.cu): per head S_t = D_t S_(t-1) + k_t v_t^T over a state of [N key channels][P value channels]
+// in fp32, D_t a number per head (the state space) or one per key channel (time mixing). The state lies as [slot][head][P][Np],
+// Np being N rounded up to a multiple of 32 (recurrent_pitch) with zeros behind.
+struct RecurrentCache {
+    float* state;
+    // The rows of a verified run, kept until it is known which of them stand: keys [slot][8][heads / per][N], decays
+    // [slot][8][heads][N] or (key scale, decay) [slot][8][heads][2], values [slot][8][heads][P].
+    float *keep_k, *keep_d, *keep_v;
+    uint32_t heads, per, N, Np, P;  // per: heads that share a key row
+    bool channel_decay;
+};
+struct ScanArgs {
+    const float *q, *k, *v;  // row t's of head h at q + t ldq + (h / per) N, k likewise, v + t ldv + h P
+    uint32_t ldq, ldk, ldv;
+    const float* decay;      // per channel: [n][heads][N]; else [n][heads][2] (the key's factor, the decay)
+    const float* bonus;      // per channel: [n][heads], what of v is added to the output, which is read before the update; ...
+    const uint16_t* skip;    // ... else per head bf16, the output being read after it
+    RecurrentCache c;
+    const RunIn* runs;
+    const GenState* gen;     // a sequence that has ended keeps its state
+    const uint32_t *meta, *vis;
+    uint32_t n_runs, max_run;
+    float* y;                // [n][heads P]
+};
+uint32_t recurrent_pitch(uint32_t N);  // Np
+void launch_scan(const ScanArgs& a, cudaStream_t s);
+// After acceptance: the states of the verified runs advance over the accepted path's rows.
+void launch_recurrent_commit(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const RecurrentCache* caches, uint32_t n_runs,
+                             uint32_t n_caches, uint32_t max_heads, cudaStream_t s);
+void launch_recurrent_fill(const RecurrentCache* caches, uint32_t n_caches, uint32_t slot, uint32_t seed, cudaStream_t s);
+// y[t][c] = silu(bias + convolution) for a.conv_channels channels, and per head softplus(dt + dt_bias) and exp(-exp(a_log) of that).
+struct StepSizeArgs {
+    const float* dt;         // [n][ld]
+    uint32_t ld, heads;
+    const uint16_t *bias, *a_log;
+    float* out;              // [n][heads][2]
+};
+void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, float* y, cudaStream_t s);
+// Row t's mixes with the row before it, h + (h' - h) mu, five of them: [mix][n][channels], fp32 and / or bf16, the last mu's
+// first. tiles: the grouped projection's table over the four behind it (group, first row, rows), `tile` rows at most.
+struct ShiftArgs {
+    ConvArgs c;              // u: the normed rows; the ring
+    const uint16_t* mu[5];
+    float* out_f32;
+    uint16_t* out_bf16;
+    uint32_t *tiles, *n_tiles;
+    uint32_t tile;
+};
+void launch_token_shift(const ShiftArgs& a, uint32_t n, cudaStream_t s);
+// exp(-exp(w0 + w2 tanh(hid))) per key channel, and per head the sum of r k u over its channels.
+struct DecayArgs {
+    const float* hid;        // [n][ldh]: w1's product
+    const float *r, *k;      // [n][heads dim]
+    const uint16_t *w2, *w0, *u;
+    uint32_t ldh, rank, heads, dim;
+    float *decay, *bonus;    // [n][heads][dim], [n][heads]
+};
+void launch_decay(const DecayArgs& a, uint32_t n, cudaStream_t s);
+// Rows of `groups` equal parts, each over its own root mean square, times w; silu(gate) goes on before the norm or at the end.
+struct GatedNormArgs {
+    const float *y, *gate;   // [n][width], [n][ldg]
+    const uint16_t* w;
+    uint32_t width, ldg, groups;
+    bool gate_first;
+    float eps;
+    float* out_f32;          // optional
+    uint16_t* out_bf16;      // optional
+};
+void launch_gated_norm(const GatedNormArgs& a, uint32_t n, cudaStream_t s);
 
 // A mixture of experts (k_moe.cu).
 struct RouterArgs {
     const float* x;                       // the stream [n][d]
-    const uint16_t *norm, *router, *correction;
+    RowNorm norm;
+    const uint16_t *router, *correction;
     float* xn;                            // optional: its normed rows
     uint16_t* xn_b;                       // optional, bf16
     uint32_t* ids;                        // [n][top]; experts and beyond: an identity expert
@@ -289,7 +417,7 @@ struct CombineArgs {
     const uint32_t *ids, *place;
     const float* weights;
     float* out;                           // may be x
-    const uint16_t* norm;                 // optional: the next layer's norm, into next / next_b
+    RowNorm norm;                         // optional: the next layer's norm, into next / next_b
     float* next;
     uint16_t* next_b;
     uint32_t d, experts, top;

@@ -1,0 +1,222 @@
+// Model folders: decoders whose config.json lists their layers one by one. This file has the mechanisms a layer can hold, each a
+// parameter struct of its own, the list of layer runs, and what the readers of the designs (lonasun.h, leduvik.h) share: the
+// tensors' places and the loop over a span of layers. A design's reader fills it; engine_layered.cu runs it.
+#pragma once
+#include <memory>
+
+#include "weights.h"
+
+namespace vlt {
+
+// Of rows: x / sqrt(mean x^2 + eps), times the weight (as stored, or stored around zero: 1 + w).
+struct RowNorm {
+    const uint16_t* w = nullptr;
+    bool around_zero = false;
+};
+// y_t = b[c] + sum_j w[c][j] u_(t - taps + 1 + j) per channel.
+struct ShortConv {
+    const uint16_t *w = nullptr, *b = nullptr;  // [channels][taps] bf16, no weights: none; [channels], optional
+    uint32_t channels = 0, taps = 1;
+};
+// Dimensions i and i + dims / 2 of a head's first `dims` turn by position * base^(-2 i / dims).
+struct Rotation {
+    uint32_t dims = 0;
+    double base = 1;
+    uint32_t table = 0;  // index among the model's rotations
+};
+// Queries are multiplied by 1 + coef ln(floor((position + 1) / every) + 1). every 0: not at all.
+struct QueryTemperature {
+    float coef = 0;
+    double every = 0;
+};
+// Attention over pages of keys. What a position sees of the positions up to its own: those of its own block of `chunk`, or the
+// last `window`, or (both 0) all.
+struct Attention {
+    uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, chunk = 0, window = 0;
+    float scale = 1;
+    bool unit_qk = false;  // q's and k's heads are divided by their root mean square
+    bool gated = false;    // the output times sigmoid(gate)
+    Rotation rot;
+    QueryTemperature temp;
+    ShortConv conv;  // over q | k | v
+    Matrix proj, o;  // proj: the rows of q, k, v and, if gated, the gate stacked
+    uint32_t qkv_w() const { return (heads + kv_heads) * dim + kv_heads * vdim; }
+    uint32_t out_w() const { return heads * vdim; }
+};
+// A selective state space: S = exp(-exp(A_h) dt) S + dt B x^T, y = S^T C + D_h x per head; x, B and C out of a short convolution
+// and silu, dt = softplus(dt + dt_bias); y silu(z) normed in equal parts.
+struct StateSpace {
+    uint32_t heads = 0, vdim = 0, state = 0, groups = 1, norm_groups = 1;
+    ShortConv conv;  // over x | B | C
+    Matrix in, o;    // in: z | x | B | C | dt
+    const uint16_t *dt_bias = nullptr, *a_log = nullptr, *skip = nullptr, *norm = nullptr;
+    uint32_t inner() const { return heads * vdim; }
+    uint32_t channels() const { return inner() + 2 * groups * state; }
+};
+// A linear recurrence with a decay per key channel: o = r^T (S + diag(u) k v^T), S = diag(w) S + k v^T per head, the inputs each
+// read from their own mix of a row and the row before it; o per head to unit rms, normed, times silu(gate).
+struct TimeMix {
+    uint32_t heads = 0, dim = 0, rank = 0;
+    const uint16_t* mu[5] = {};  // r, k, v, g, w: [d]
+    Matrix rkvg;                 // four matrices [heads dim][d] stacked
+    Matrix w1, o;                // w1 [rank][d]
+    const uint16_t *w2 = nullptr, *w0 = nullptr, *bonus = nullptr, *norm = nullptr;  // w2 [heads dim][rank], bonus [heads][dim]
+    uint32_t inner() const { return heads * dim; }
+};
+enum class MixerKind { Attention, StateSpace, TimeMix };
+struct Mixer {
+    MixerKind kind = MixerKind::Attention;
+    Attention attn;
+    StateSpace ssm;
+    TimeMix tmix;
+    RowNorm out;  // on the output, in layers of several mixers
+};
+// relu(W_up h)^2 through W_down, `top` of `experts` + `identity` per token, softmax scores, a shared expert (ff 0: none).
+struct ExpertLayer {
+    uint32_t experts = 0, identity = 0, top = 0, ff = 0, shared_ff = 0;
+    const uint16_t *router = nullptr, *correction = nullptr;  // [experts + identity][d], [experts + identity]
+    Matrix up, down;                                          // all experts': [experts * ff][d], [experts * d][ff]
+    Matrix shared_up, shared_down;
+};
+// W_down relu(W_up h)^2.
+struct DenseLayer {
+    Matrix up, down;
+};
+enum class MlpKind { None, Experts, Dense };
+struct FolderLayer {
+    RowNorm norm1, norm2;
+    std::vector<Mixer> mix;  // several: side by side on the same rows, each output normed, the mean added
+    MlpKind mlp = MlpKind::None;
+    ExpertLayer experts;
+    DenseLayer dense;
+};
+// A layer run: with a loop a layer runs several times, each with a cache of its own.
+struct LayerRun {
+    uint32_t layer;
+    bool loop_in;    // (stream ; embedding) goes through loop_in first
+    bool add_embed;  // the embedding is added to the stream first
+};
+
+inline Json read_json(const std::string& path) {
+    FILE* f = std::fopen(path.c_str(), "rb");
+    if (!f) throw Error(path + ": cannot open");
+    std::string text;
+    char buf[65536];
+    for (size_t n; (n = std::fread(buf, 1, sizeof buf, f)) > 0;) text.append(buf, n);
+    std::fclose(f);
+    return Json::parse(text.data(), text.size(), path);
+}
+
+struct LayeredModel {
+    static constexpr uint32_t PAGE = 64;       // positions per cache page
+    static constexpr uint32_t MAX_TAPS = 32;   // of a short convolution
+    static constexpr uint32_t MAX_STATE = 512; // key channels of a recurrence
+    SafeTensors w;
+    std::string where;  // for messages
+    std::vector<FolderLayer> layers;
+    std::vector<LayerRun> runs;
+    std::vector<Rotation> rotations;  // the distinct ones
+    Matrix loop_in, head;
+    const uint16_t *embed = nullptr, *positions = nullptr;  // positions: a learned vector per position (optional)
+    uint32_t n_positions = 0;                               // rows of it; sequences are no longer than that
+    RowNorm final_norm;
+    float logit_scale = 1;
+
+    // A design's reader: its own part of config.json and the tensors it names.
+    using Reader = void (*)(LayeredModel&, const Json&, ModelDesc&);
+    static std::unique_ptr<LayeredModel> load(Reader read, const Json& cfg, const std::string& dir, bool host_only, ModelDesc& md) {
+        auto m = std::make_unique<LayeredModel>();
+        m->where = dir;
+        m->w.open(dir + "/model.safetensors");
+        md.d = cfg.at("width").count("width");
+        md.vocab = md.vocab_real = cfg.at("vocab").count("vocab");
+        md.eps = float(cfg.at("norm").at("eps").number("norm.eps"));
+        md.page = PAGE;
+        m->layers.resize(cfg.at("layers").items.size());  // (their addresses are kept in `fixups` from here on)
+        if (m->layers.empty() || md.d == 0 || md.vocab == 0) throw Error(dir + ": a model needs layers, a width and a vocabulary");
+        read(*m, cfg, md);
+        m->describe(md);
+        m->w.to_device(host_only);
+        const uint8_t* base = m->w.buffer.as<uint8_t>();
+        for (auto& fix : m->fixups) *fix.first = base + fix.second;  // the tensors' addresses, now that they have one
+        m->fixups.clear();
+        m->w.unmap();
+        return m;
+    }
+
+    void point(const uint16_t*& p, size_t offset) { fixups.emplace_back(reinterpret_cast<const uint8_t**>(&p), offset); }
+    void point(const uint16_t*& p, const std::string& name, const std::vector<uint32_t>& shape) { point(p, w.place(name, shape)); }
+    void matrix(Matrix& m, uint32_t rows, uint32_t k, size_t offset) {
+        m.m = rows;
+        m.k = k;
+        fixups.emplace_back(&m.w, offset);
+    }
+    void matrix(Matrix& m, const std::string& name, uint32_t rows, uint32_t k) { matrix(m, rows, k, w.place(name, {rows, k})); }
+    // Rows of zeros after the stack placed last, up to whole tiles of the tensor-core GEMM (where its k fits it): for projections
+    // whose consumers read a part of each output row.
+    void padded(Matrix& m, uint32_t rows, uint32_t k, size_t offset) {
+        const uint32_t whole = k % 64 == 0 ? (rows + 127) / 128 * 128 : rows;
+        w.zeros(size_t(whole - rows) * k * 2);
+        matrix(m, whole, k, offset);
+    }
+    // q, k, v and, if gated, g of an attention, and its output matrix.
+    void attention_matrices(Attention& a, const std::string& pre, uint32_t d) {
+        if (a.kv_heads == 0 || a.heads == 0 || a.heads % a.kv_heads || a.dim == 0 || a.vdim == 0) throw Error(pre + ": the heads do not fit the kv heads");
+        const uint32_t qw = a.heads * a.dim, kw = a.kv_heads * a.dim, vw = a.kv_heads * a.vdim;
+        const size_t at = w.place(pre + "q", {qw, d});
+        w.place(pre + "k", {kw, d}, false);
+        w.place(pre + "v", {vw, d}, false);
+        if (a.gated) w.place(pre + "g", {a.out_w(), d}, false);
+        padded(a.proj, qw + kw + vw + (a.gated ? a.out_w() : 0), d, at);
+        matrix(a.o, pre + "o", d, a.out_w());
+    }
+    static void sizes(Attention& a, const Json& m) {
+        a.heads = m.at("heads").count("heads");
+        a.kv_heads = m.at("kv_heads").count("kv_heads");
+        a.dim = m.at("dim").count("dim");
+        a.vdim = m.at("vdim").count("vdim");
+        a.scale = float(m.at("scale").number("scale"));
+    }
+    void check_taps(const ShortConv& c, const std::string& pre) const {
+        if (c.taps == 0 || c.taps > MAX_TAPS) throw Error(pre + ": a convolution takes 1 to " + std::to_string(MAX_TAPS) + " taps");
+    }
+    // The layers' order: a span of them several times in a row. begins(pass): what a pass's first run does with the embedding.
+    template <typename F>
+    void order(const Json& loop, F&& begins) {
+        const uint32_t n = uint32_t(layers.size());
+        uint32_t start = 0, stop = 0, times = 0;
+        if (!loop.is_null()) {
+            start = loop.at("start").count("loop.start");
+            stop = loop.at("stop").count("loop.stop");
+            times = loop.at("times").count("loop.times");
+            if (start >= stop || stop > n || times == 0) throw Error(where + ": the loop does not fit the layers");
+        }
+        for (uint32_t i = 0; i < start; i++) runs.push_back({i, false, false});
+        for (uint32_t t = 0; t < times; t++)
+            for (uint32_t i = start; i < stop; i++) {
+                LayerRun r{i, false, false};
+                if (i == start) begins(r, t);
+                runs.push_back(r);
+            }
+        for (uint32_t i = stop; i < n; i++) runs.push_back({i, false, false});
+    }
+
+  private:
+    std::vector<std::pair<const uint8_t**, size_t>> fixups;
+    // What the step's shared machinery asks about: the widest layer.
+    void describe(ModelDesc& md) const {
+        md.n_layers = uint32_t(runs.size());
+        for (const FolderLayer& l : layers) {
+            for (const Mixer& x : l.mix) {
+                if (x.kind != MixerKind::Attention) continue;
+                md.n_heads = std::max(md.n_heads, x.attn.heads);
+                md.n_kv = std::max(md.n_kv, x.attn.kv_heads);
+                md.hd = std::max(md.hd, x.attn.dim);
+                if (md.attn_scale == 0) md.attn_scale = x.attn.scale;
+            }
+            md.ffn = std::max(md.ffn, std::max(l.experts.ff, l.dense.up.m));
+        }
+    }
+};
+
+}  // namespace vlt

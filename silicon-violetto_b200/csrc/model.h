@@ -2,6 +2,7 @@
 #pragma once
 #include <memory>
 
+#include "leduvik.h"
 #include "lonasun.h"
 #include "weights.h"
 
@@ -24,18 +25,21 @@ struct Model {
     const float* mudd_mix = nullptr;        // [2][2][3][33]
     uint32_t n_local = 0, n_global = 0;
 
-    std::unique_ptr<LonasunModel> lonasun;  // a model folder's own description of its layers
+    std::unique_ptr<LayeredModel> layered;  // a model folder's own description of its layers
 
-    // A model folder: config.json names the architecture, and with it the loader.
+    // A model folder: config.json names the architecture, and with it the reader.
     void load_folder(const std::string& dir, bool host_only) {
         const std::string path = dir + "/config.json";
         const Json cfg = read_json(path);
         const std::string& arch = cfg.at("architecture").text("architecture");
-        static const struct { const char* name; void (*load)(Model&, const Json&, const std::string&, bool); } registry[] = {
-            {"Lonasun", [](Model& m, const Json& c, const std::string& d, bool h) { m.lonasun = LonasunModel::load(c, d, h, m.md); m.embed = m.lonasun->embed; m.head = m.lonasun->head; }},
-        };
-        for (const auto& r : registry)
-            if (arch == r.name) { r.load(*this, cfg, dir, host_only); return; }
+        static const struct { const char* name; LayeredModel::Reader read; } registry[] = {{"Lonasun", lonasun::read}, {"Leduvik", leduvik::read}};
+        for (const auto& r : registry) {
+            if (arch != r.name) continue;
+            layered = LayeredModel::load(r.read, cfg, dir, host_only, md);
+            embed = layered->embed;
+            head = layered->head;
+            return;
+        }
         throw Error(path + ": no architecture named " + arch);
     }
 

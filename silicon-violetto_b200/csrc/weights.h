@@ -162,6 +162,7 @@ struct SafeTensors {
             const size_t size = e.dtype == "BF16" || e.dtype == "F16" ? 2 : e.dtype == "F32" || e.dtype == "I32" ? 4 : 0;
             if (size && e.nbytes != count * size) throw Error(name + ": its data does not fit its shape");
             total += e.nbytes + 256;
+            if (e.shape.size() == 2) total += size_t(128) * e.shape[1] * 2;  // (room for `zeros`; untouched pages of it cost nothing)
             entries[name] = e;
         }
         buffer.alloc(total + 256, true);  // (filled on the host, then moved to the device in one copy: see to_device)
@@ -187,6 +188,18 @@ struct SafeTensors {
         std::memcpy(buffer.as<uint8_t>() + at, e.data, e.nbytes);
         used += e.nbytes;
         return at;
+    }
+    // Zero bytes after the tensor placed last.
+    void zeros(size_t nbytes) {
+        if (used + nbytes > buffer.bytes) throw Error(path + ": no room for padding");
+        used += nbytes;  // (the buffer starts as zeros)
+    }
+    // The rows of a matrix whose number nothing but its shape says.
+    uint32_t rows(const std::string& name) const {
+        auto it = entries.find(name);
+        if (it == entries.end()) throw Error(path + ": no tensor " + name);
+        if (it->second.shape.size() != 2 || it->second.shape[0] == 0) throw Error(name + ": not a matrix");
+        return it->second.shape[0];
     }
     // The placed tensors' final home; offsets stay as they are.
     void to_device(bool host_only) {

@@ -2,11 +2,7 @@
 benchmarks. The engine reads the folders itself (csrc/lonasun.h)."""
 from __future__ import annotations
 
-import json
-import struct
-from pathlib import Path
-
-import numpy as np
+from .folders import Pool, from_bf16, to_bf16, write_model  # noqa: F401  (callers take them from here)
 
 
 def layer(heads, kv_heads, dim, vdim, chunk, conv=4, rot_dims=None, base=10000.0, scale=None, moe=None) -> dict:
@@ -58,55 +54,20 @@ def shapes(cfg: dict) -> dict:
     return out
 
 
-def to_bf16(a: np.ndarray) -> np.ndarray:
-    """fp32 -> bf16 bit patterns, round to nearest even."""
-    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
-
-
-def from_bf16(bits: np.ndarray) -> np.ndarray:
-    return (bits.astype(np.uint32) << 16).view(np.float32)
-
-
 def random_weights(cfg: dict, seed: int = 0, pool: int = 1 << 22) -> dict:
     """name -> bf16 bits. Matrices N(0, 1 / fan-in), convolutions N(0, 1 / taps) with the newest tap raised, norms and
-    corrections small. Large models repeat a pool of values (their speed does not depend on them)."""
-    rng = np.random.default_rng(seed)
-    base, at, out = rng.standard_normal(pool, dtype=np.float32), 0, {}
+    corrections small."""
+    values, out = Pool(seed, pool), {}
     for name, shape in shapes(cfg).items():
-        n = int(np.prod(shape))
-        if n <= pool - at:
-            v = base[at:at + n]
-            at += n
-        else:
-            at = int(rng.integers(0, pool // 2)) | 1
-            v = np.resize(np.roll(base, -at), n)
+        v = values.take(shape)
         if name.endswith("norm1") or name.endswith("norm2") or name == "final.norm":
             v = v * 0.1
         elif name.endswith("correction"):
             v = v * 0.02
         elif name.endswith(".conv"):
-            v = (v * 0.3).reshape(shape).copy()
+            v = v * 0.3
             v[:, -1] += 0.8
         elif name != "embed":
             v = v * (shape[-1] ** -0.5)
-        out[name] = to_bf16(v).reshape(shape)
+        out[name] = to_bf16(v)
     return out
-
-
-def write_model(folder, cfg: dict, weights: dict) -> Path:
-    """weights: name -> bf16 bits (uint16)."""
-    folder = Path(folder)
-    folder.mkdir(parents=True, exist_ok=True)
-    (folder / "config.json").write_text(json.dumps(cfg, indent=1))
-    head, at = {}, 0
-    for name, w in weights.items():
-        head[name] = {"dtype": "BF16", "shape": list(w.shape), "data_offsets": [at, at + w.nbytes]}
-        at += w.nbytes
-    text = json.dumps(head).encode()
-    text += b" " * (-len(text) % 8)
-    with open(folder / "model.safetensors", "wb") as f:
-        f.write(struct.pack("<Q", len(text)) + text)
-        for w in weights.values():
-            f.write(np.ascontiguousarray(w).tobytes())
-    return folder
