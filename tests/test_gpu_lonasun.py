@@ -17,8 +17,7 @@ BOTH = pytest.mark.parametrize("fp32", [True, False], ids=["fp32", "bf16"])
 NAMES = ["odd", "fast", "one", "one_odd", "experts"]
 
 
-def prompt(cfg, n, seed):
-    return [int(t) for t in np.random.default_rng(seed).integers(0, cfg["vocab"], n)]
+prompt = lu.prompt
 
 
 def close(got, want, fp32, factor=1.0):
