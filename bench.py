@@ -342,21 +342,73 @@ def lonasun_files(size):
     return folder, plain
 
 
-def lonasun_figure(E, local, size, steps, stream_counts, hbm_peak, tc_peak):
-    """Decoding over a filled context and a prompt of the same length (all in one chunk of positions) in portions of 512, the Lonasun model and the
-    plain decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their
-    own) the fraction of the measured copy bandwidth or bf16 throughput its algorithmic bytes or FLOPs make."""
+def lonasun_work(size):
+    """What a Lonasun model of LONASUN_SIZES and the plain decoder beside it read and compute, for folder_figure."""
     c = LONASUN_SIZES[size]
-    L, ctx = c["layers"], c["ctx"]
-    folder, plain = lonasun_files(size)
     attn_w = (c["heads"] + c["kv_heads"]) * c["dim"] + c["kv_heads"] * c["vdim"]
     o_p = c["heads"] * c["vdim"] * c["width"]
     expert_p = 2 * c["ff"] * c["width"]
-    weights = {"lonasun": lambda touched: L * ((attn_w + c["heads"] * c["vdim"]) * c["width"] + o_p + (touched + 1) * expert_p),
-               "plain": lambda touched: L * (attn_w * c["width"] + o_p + 3 * c["plain"]["ffn"] * c["width"])}
-    kv_row = c["kv_heads"] * (c["dim"] + c["vdim"]) * 2
-    out = {"workload": f"{L} layers x {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in portions of 512"}
-    for name, path in (("lonasun", folder), ("plain", plain)):
+    moe = lambda touched: c["layers"] * ((attn_w + c["heads"] * c["vdim"]) * c["width"] + o_p + (touched + 1) * expert_p)
+    dense = c["layers"] * (attn_w * c["width"] + o_p + 3 * c["plain"]["ffn"] * c["width"])
+    kv = c["layers"] * c["kv_heads"] * (c["dim"] + c["vdim"]) * 2
+    flops = c["layers"] * 2.0 * c["heads"] * (c["dim"] + c["vdim"])
+    touched = lambda n: c["experts"] * (1 - (1 - c["top"] / c["experts"]) ** n)  # experts a step of n tokens reads, on average
+    keys = lambda ctx: {"decode_weights": lambda n: dense, "prompt_weights": dense, "kv": kv * ctx, "state": 0, "attention_flops": flops * ctx * ctx / 2}
+    return c, {"lonasun": {**keys(c["ctx"]), "decode_weights": lambda n: moe(touched(n)), "prompt_weights": moe(c["top"])}, "plain": keys(c["ctx"])}
+
+
+# Layers of real models' sizes, in blocks of the design's three kinds; `plain` as above.
+LEDUVIK_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=1024, ssm=dict(heads=64, vdim=64, state=128, groups=1, norm_groups=1), right=(32, 64), rank=64, ff=8192,
+                 vocab=32768, blocks=2, ctx=8000, plain=dict(n_heads=32, n_kv=8, ffn=5376)),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=1024, ssm=dict(heads=128, vdim=64, state=128, groups=8, norm_groups=8), right=(64, 64), rank=128, ff=14336,
+                 vocab=32768, blocks=1, ctx=1900, plain=dict(n_heads=64, n_kv=16, ffn=9472)),
+}
+
+
+def leduvik_files(size):
+    """A Leduvik model and the plain decoder of equal size (LEDUVIK_SIZES), random-init, bf16, written once per box."""
+    from silicon_violetto_b200 import leduvik, synth
+    CACHE.mkdir(parents=True, exist_ok=True)
+    c = LEDUVIK_SIZES[size]
+    heads = (c["heads"], c["kv_heads"], c["dim"], c["vdim"])
+    block = [leduvik.window(*heads, c["window"], c["dim"] ** -0.5, ff=c["ff"]), leduvik.state_space(**c["ssm"], ff=c["ff"]), leduvik.parallel(*heads, *c["right"], every=1024, ff=c["ff"])]
+    folder = CACHE / f"leduvik_{size}"
+    if not (folder / "ok").exists():
+        cfg = leduvik.config(c["width"], c["vocab"], block * c["blocks"], max_positions=c["ctx"] + 256)
+        leduvik.write_model(folder, cfg, leduvik.random_weights(cfg, rank=c["rank"]))
+        (folder / "ok").write_text("ok")
+    plain = CACHE / f"plain_leduvik_{size}.vlt"
+    if not plain.with_suffix(".ok").exists():
+        synth.write_target(plain, dict(n_layers=3 * c["blocks"], d=c["width"], hd=64, vocab=c["vocab"], eps=1e-5, theta=500000.0, page=16, **c["plain"]), seed=0)
+        plain.with_suffix(".ok").write_text("ok")
+    return folder, plain
+
+
+def leduvik_work(size):
+    """What a Leduvik model of LEDUVIK_SIZES and the plain decoder beside it read and compute, for folder_figure."""
+    c = LEDUVIK_SIZES[size]
+    d, ctx, m, (rh, rd) = c["width"], c["ctx"], c["ssm"], c["right"]
+    attn_p = ((c["heads"] + c["kv_heads"]) * c["dim"] + c["kv_heads"] * c["vdim"] + c["heads"] * c["vdim"]) * d
+    inner = m["heads"] * m["vdim"]
+    ssm_p = (2 * inner + 2 * m["groups"] * m["state"] + m["heads"] + inner) * d
+    right_p = 5 * rh * rd * d + c["rank"] * (d + rh * rd)
+    ours = c["blocks"] * (2 * attn_p + ssm_p + right_p + 3 * 2 * c["ff"] * d)
+    plain = 3 * c["blocks"] * (attn_p + 3 * c["plain"]["ffn"] * d)
+    row, flops, seen = c["kv_heads"] * (c["dim"] + c["vdim"]) * 2, 2.0 * c["heads"] * (c["dim"] + c["vdim"]), min(c["window"], ctx)
+    state = c["blocks"] * 2 * 4 * (inner * m["state"] + rh * rd * rd)  # read and written
+    at = lambda keys, pairs, weights, state: {"decode_weights": lambda n: weights, "prompt_weights": weights, "kv": c["blocks"] * row * keys, "state": state,
+                                              "attention_flops": c["blocks"] * flops * pairs}
+    return c, {"leduvik": at(seen + ctx, ctx * ctx / 2 + seen * (ctx - seen / 2), ours, state), "plain": at(3 * ctx, 3 * ctx * ctx / 2, plain, 0)}
+
+
+def folder_figure(E, local, c, files, work, steps, stream_counts, hbm_peak, tc_peak):
+    """Decoding over a filled context and a prompt of the same length in portions of 512, the folder's model and the plain
+    decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their own) the
+    fraction of the measured copy bandwidth or bf16 throughput its algorithmic bytes or FLOPs make."""
+    ctx = c["ctx"]
+    out = {"workload": f"layers of width {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in portions of 512"}
+    for (name, w), path in zip(work.items(), files):
         res = out[name] = {}
         for n_s in stream_counts:
             eng = E.Engine(path, E.EngineConfig(max_seqs=n_s, max_step_tokens=max(64, n_s), max_chunk=32, global_kv_tokens=n_s * (ctx + 192), max_seq_len=ctx + 128,
@@ -382,12 +434,12 @@ def lonasun_figure(E, local, size, steps, stream_counts, hbm_peak, tc_peak):
                 prof = eng.profile_read()
                 eng.set_profile(False)
             eng.close()
-            touched = c["experts"] * (1 - (1 - c["top"] / c["experts"]) ** n_s)  # experts a step of n_s tokens reads, on average
-            wb, kb = 2 * weights[name](touched), n_s * ctx * kv_row * L
+            wb, kb, sb = 2 * w["decode_weights"](n_s), n_s * w["kv"], n_s * w["state"]
             gms = {k: v["ms"] / steps for k, v in prof.items()}
-            res[f"decode_{n_s}"] = {"ms_per_step": ms, "tokens_per_s": n_s / (ms * 1e-3), "groups_ms": gms, "weight_bytes": wb, "kv_bytes": kb, "clocks": clocks.summary(),
-                                    "matmul_frac_hbm": wb / (gms["matmul"] * 1e-3) / 1e9 / hbm_peak, "attention_frac_hbm": kb / (gms["attention"] * 1e-3) / 1e9 / hbm_peak,
-                                    "step_frac_hbm": (wb + kb) / (ms * 1e-3) / 1e9 / hbm_peak}
+            frac = lambda b, group: b / (gms[group] * 1e-3) / 1e9 / hbm_peak
+            res[f"decode_{n_s}"] = {"ms_per_step": ms, "tokens_per_s": n_s / (ms * 1e-3), "groups_ms": gms, "weight_bytes": wb, "kv_bytes": kb, "state_bytes": sb, "clocks": clocks.summary(),
+                                    "matmul_frac_hbm": frac(wb, "matmul"), "attention_frac_hbm": frac(kb, "attention"), "recurrence_frac_hbm": frac(sb, "recurrence") if sb else None,
+                                    "step_frac_hbm": (wb + kb + sb) / (ms * 1e-3) / 1e9 / hbm_peak}
         eng = E.Engine(path, E.EngineConfig(max_seqs=1, max_step_tokens=512, max_chunk=512, global_kv_tokens=ctx + 128, max_seq_len=ctx + 64, max_head_rows=8, device_ordinal=local),
                        E.Tuning(spec_policy_off=True))
         prompt = [int(x) for x in np.random.default_rng(7).integers(0, eng.desc.vocab, ctx)]
@@ -407,9 +459,8 @@ def lonasun_figure(E, local, size, steps, stream_counts, hbm_peak, tc_peak):
                 gms = {k: v["ms"] for k, v in eng.profile_read().items()}
                 eng.set_profile(False)
         eng.close()
-        mm, at = 2.0 * ctx * weights[name](c["top"]), L * 2.0 * c["heads"] * (c["dim"] + c["vdim"]) * ctx * ctx / 2
-        res["prefill"] = {"ms": ms, "tokens_per_s": ctx / (ms * 1e-3), "groups_ms": gms, "matmul_frac_tc": mm / (gms["matmul"] * 1e-3) / 1e12 / tc_peak,
-                          "attention_frac_tc": at / (gms["attention"] * 1e-3) / 1e12 / tc_peak}
+        res["prefill"] = {"ms": ms, "tokens_per_s": ctx / (ms * 1e-3), "groups_ms": gms, "matmul_frac_tc": 2.0 * ctx * w["prompt_weights"] / (gms["matmul"] * 1e-3) / 1e12 / tc_peak,
+                          "attention_frac_tc": w["attention_flops"] / (gms["attention"] * 1e-3) / 1e12 / tc_peak}
     return out
 
 
@@ -461,11 +512,11 @@ def main():
     ap.add_argument("--attn-keys", type=int, default=0, help="keys per attention block (0: the engine's own choice)")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers: a profiler-size case, not a bench value")
     ap.add_argument("--no-limite", action="store_true", help="skip the reference-architecture pass of the extras (it writes a 2 GB file first)")
-    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite and --only lonasun")
+    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite, lonasun and leduvik")
     ap.add_argument("--limite-drafter", action="store_true", help="--only limite: with the reference's block drafter loaded (tree drafts of up to 8 rows)")
     ap.add_argument("--limite-int8", action="store_true", help="--only limite: int8 weights in the reference converter's default groups (64; the head 8)")
     ap.add_argument("--limite-keys", type=int, default=0, help="--only limite: keys per attention block (VltTuning.attn_keys_per_cta); 0 = the library's choice")
-    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) or 'lonasun' (Lonasun models beside plain decoders of equal size): run that one pass alone and print its figure (not the bench line)")
+    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) 'lonasun' or 'leduvik' (models of those designs beside plain decoders of equal size): run that one pass alone and print its figure (not the bench line)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank, world, local = int(os.environ.get("RANK", 0)), int(os.environ.get("WORLD_SIZE", 1)), int(os.environ.get("LOCAL_RANK", 0))
@@ -511,10 +562,14 @@ def main():
     solo = lambda: torch.cuda.synchronize(local)
     _package()
     from silicon_violetto_b200 import engine as E
-    if args.only == "lonasun":
+    if args.only in ("lonasun", "leduvik"):
         peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
-        print(json.dumps({n: lonasun_figure(E, local, n, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], hbm_peak, peaks.get("bf16_tflops", 1590.0))
-                          for n in LONASUN_SIZES}))
+        sizes, files, work = {"lonasun": (LONASUN_SIZES, lonasun_files, lonasun_work), "leduvik": (LEDUVIK_SIZES, leduvik_files, leduvik_work)}[args.only]
+        figures = {}
+        for n in sizes:
+            c, w = work(n)
+            figures[n] = folder_figure(E, local, c, files(n), w, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], hbm_peak, peaks.get("bf16_tflops", 1590.0))
+        print(json.dumps(figures))
         return
     path = model_file("1b", not args.bf16, rank, args.layers)
     if args.only:
@@ -526,7 +581,7 @@ def main():
         elif args.only == "limite":
             print(json.dumps(limite_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], args.limite_keys, args.limite_drafter, args.limite_int8)))
         else:
-            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite' or 'lonasun'")
+            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite', 'lonasun' or 'leduvik'")
         return
     total = args.warmup + args.steps + 6
     # The headline pass, on every rank: the int8 target with the chain drafter loaded (1 layer + fc + a head over 16 384 draft

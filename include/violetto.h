@@ -333,7 +333,7 @@ int vlt_debug_mark(VltEngine* e, uint32_t which);
 int vlt_debug_mark_elapsed_ms(VltEngine* e, double* ms);
 uint64_t vlt_debug_launches(void);
 int vlt_debug_profile(VltEngine* e, uint32_t on);
-int vlt_debug_profile_read(VltEngine* e, double* ms5, uint32_t* launches5);
+int vlt_debug_profile_read(VltEngine* e, double* ms6, uint32_t* launches6);
 int vlt_debug_step_bytes(VltEngine* e, uint64_t* h2d, uint64_t* d2h);
 
 #ifdef __cplusplus

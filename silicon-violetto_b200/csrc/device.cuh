@@ -169,6 +169,46 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// The block's sum, to every thread. red: 32 floats of shared memory, free to use again after the next barrier.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    if (threadIdx.x % 32 == 0) red[threadIdx.x / 32] = v;
+    __syncthreads();
+    float tot = 0.0f;
+    for (uint32_t i = 0; i < blockDim.x / 32; i++) tot += red[i];
+    return tot;
+}
+// V consecutive floats (1 or 4, aligned) and bf16 values, for row kernels that take rows of any length.
+template <uint32_t V>
+__device__ __forceinline__ void load_f32(float (&x)[V], const float* p) {
+    if constexpr (V == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
+    } else x[0] = *p;
+}
+template <uint32_t V>
+__device__ __forceinline__ void store_f32(float* p, const float (&x)[V]) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+    else *p = x[0];
+}
+template <uint32_t V>
+__device__ __forceinline__ void load_bf16(float (&x)[V], const uint16_t* p) {
+    if constexpr (V == 4) {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        x[0] = bf16lo(v.x); x[1] = bf16hi(v.x); x[2] = bf16lo(v.y); x[3] = bf16hi(v.y);
+    } else x[0] = bf16_to_f32(*p);
+}
+template <uint32_t V>
+__device__ __forceinline__ void store_bf16(uint16_t* p, const float (&x)[V]) {
+    if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+    else *p = f32_to_bf16(x[0]);
+}
+// Threads of a block that has a row of `width`: one per V values as far as 1024 go.
+inline uint32_t row_threads(uint32_t width, uint32_t v) {
+    const uint32_t t = (width / v + 31) / 32 * 32;
+    return t < 64 ? 64 : t > 1024 ? 1024 : t;
+}
+
 // kernels.metal:1418-1427 `better`, `simd_best`: (value, id) with ties to the lowest id.
 __device__ __forceinline__ void better(float& bv, uint32_t& bi, float v, uint32_t i) {
     if (v > bv || (v == bv && i < bi)) { bv = v; bi = i; }

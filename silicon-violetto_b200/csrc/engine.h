@@ -190,9 +190,9 @@ class Engine {
 
     // Measurement: two stream marks (GPU time between them), and, while `profile` is on, the GPU
     // time of each kernel group of the queued steps (cuda events around the group's launches). The groups are disjoint:
-    // the first three are the target's layers, G_TAIL its head, sampling and acceptance, G_DRAFTER everything the
+    // the first three and G_RECURRENCE are the target's layers, G_TAIL its head, sampling and acceptance, G_DRAFTER everything the
     // drafter runs (its own projections and attention included).
-    enum Group : int { G_MATMUL = 0, G_ATTN = 1, G_SMALL = 2, G_TAIL = 3, G_DRAFTER = 4, G_COUNT = 5 };
+    enum Group : int { G_MATMUL = 0, G_ATTN = 1, G_SMALL = 2, G_TAIL = 3, G_DRAFTER = 4, G_RECURRENCE = 5, G_COUNT = 6 };
     void mark(int which);
     double mark_elapsed_ms();
     bool profile = false;

@@ -174,9 +174,10 @@ void Engine::init_layered() {
 }
 
 void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base) {
-    if (!cfg.fp32 && gemm_fits(w, n)) {
+    const bool gemm = !cfg.fp32 && w.m % 128 == 0 && w.k % 64 == 0, stream_takes = !cfg.fp32 && stream_fits(w, n);
+    if (gemm && (gemm_fits(w, n) || !stream_takes)) {  // (few rows that are too long for the streamed kernel's shared memory, too)
         matmul_gemm(w, n, xb, y, yb, epi, base, nullptr);
-    } else if (!cfg.fp32 && stream_fits(w, n)) {
+    } else if (stream_takes) {
         matmul(w, n, nullptr, y, epi, base, nullptr, 0, nullptr, xb, yb);
     } else {
         LinearArgs a{};
@@ -282,7 +283,7 @@ void Engine::encode_recurrence(StepSet& st, const Plan& p, ScanArgs& a, GatedNor
     g.eps = model.md.eps;
     g.out_f32 = cfg.fp32 ? z.attn_f.as<float>() : nullptr;
     g.out_bf16 = z.attn_b.as<uint16_t>();
-    int sp = span_begin(G_ATTN);
+    int sp = span_begin(G_RECURRENCE);
     launch_scan(a, stream);
     span_end(sp);
     sp = span_begin(G_SMALL);

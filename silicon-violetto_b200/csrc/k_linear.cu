@@ -72,66 +72,87 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
     }
 }
 
-__device__ __forceinline__ float block_sum(float v, float* red) {  // 256 threads; `red` of 8, free to use again after the next barrier
-    v = warp_sum(v);
-    if (threadIdx.x % 32 == 0) red[threadIdx.x / 32] = v;
-    __syncthreads();
-    float tot = 0.0f;
-    for (uint32_t i = 0; i < 8; i++) tot += red[i];
-    return tot;
-}
 // See NormArgs. A block per row, which it keeps in shared memory.
-__global__ void __launch_bounds__(256) norm_rows_kernel(const NormArgs a) {
+template <uint32_t V>
+__global__ void __launch_bounds__(1024) norm_rows_kernel(const NormArgs a) {
     pdl_start();
-    extern __shared__ float row[];
-    __shared__ float red[8];
-    const uint32_t r = blockIdx.x, tid = threadIdx.x;
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    const uint32_t r = blockIdx.x, tid = threadIdx.x * V, step = blockDim.x * V;
     const size_t from = size_t(a.rows ? a.rows[r] : r) * a.k;
     float ss = 0.0f;
-    for (uint32_t i = tid; i < a.k; i += 256) {
-        float x = a.in[from + i];
+    for (uint32_t i = tid; i < a.k; i += step) {
+        float x[V];
+        load_f32<V>(x, a.in + from + i);
         if (a.add) {
-            x += a.add[from + i];
-            a.sum[from + i] = x;
+            float y[V];
+            load_f32<V>(y, a.add + from + i);
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) x[j] += y[j];
+            store_f32<V>(a.sum + from + i, x);
         }
-        row[i] = x;
-        ss += x * x;
+        store_f32<V>(row + i, x);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) ss += x[j] * x[j];
     }
     const float inv = a.scale / sqrtf(block_sum(ss, red) / float(a.k) + a.eps);
-    for (uint32_t i = tid; i < a.k; i += 256) {
-        const float v = row[i] * inv * weight_of(a.norm, i);
-        if (a.out_f32) a.out_f32[size_t(r) * a.k + i] = v;
-        if (a.out_bf16) a.out_bf16[size_t(r) * a.k + i] = f32_to_bf16(v);
+    for (uint32_t i = tid; i < a.k; i += step) {
+        float x[V], w[V];
+        load_f32<V>(x, row + i);
+        weights_of<V>(w, a.norm, i);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) x[j] *= inv * w[j];
+        if (a.out_f32) store_f32<V>(a.out_f32 + size_t(r) * a.k + i, x);
+        if (a.out_bf16) store_bf16<V>(a.out_bf16 + size_t(r) * a.k + i, x);
     }
 }
 
 // See MergeArgs. A block per row.
-__global__ void __launch_bounds__(256) merge_rows_kernel(const MergeArgs a) {
+template <uint32_t V>
+__global__ void __launch_bounds__(1024) merge_rows_kernel(const MergeArgs a) {
     pdl_start();
-    extern __shared__ float row[];
-    __shared__ float red[3][8];
-    const uint32_t tid = threadIdx.x;
+    extern __shared__ __align__(16) float rows[];  // the two outputs; the first then holds the sum
+    __shared__ float red[3][32];
+    float *ra = rows, *rb = rows + a.d;
+    const uint32_t tid = threadIdx.x * V, step = blockDim.x * V;
     const size_t from = size_t(blockIdx.x) * a.d;
     float sa = 0.0f, sb = 0.0f;
-    for (uint32_t i = tid; i < a.d; i += 256) {
-        const float p = a.a[from + i], q = a.b[from + i];
-        sa += p * p;
-        sb += q * q;
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float p[V], q[V];
+        load_f32<V>(p, a.a + from + i);
+        load_f32<V>(q, a.b + from + i);
+        store_f32<V>(ra + i, p);
+        store_f32<V>(rb + i, q);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) { sa += p[j] * p[j]; sb += q[j] * q[j]; }
     }
     const float ia = 0.5f / sqrtf(block_sum(sa, red[0]) / float(a.d) + a.eps), ib = 0.5f / sqrtf(block_sum(sb, red[1]) / float(a.d) + a.eps);
     float ss = 0.0f;
-    for (uint32_t i = tid; i < a.d; i += 256) {
-        const float y = a.x[from + i] + (a.a[from + i] * ia * weight_of(a.norm_a, i) + a.b[from + i] * ib * weight_of(a.norm_b, i));
-        a.out[from + i] = y;
-        row[i] = y;
-        ss += y * y;
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float p[V], q[V], x[V], wa[V], wb[V];
+        load_f32<V>(p, ra + i);
+        load_f32<V>(q, rb + i);
+        load_f32<V>(x, a.x + from + i);
+        weights_of<V>(wa, a.norm_a, i);
+        weights_of<V>(wb, a.norm_b, i);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) {
+            x[j] += p[j] * ia * wa[j] + q[j] * ib * wb[j];
+            ss += x[j] * x[j];
+        }
+        store_f32<V>(a.out + from + i, x);
+        store_f32<V>(ra + i, x);
     }
     if (!a.norm.w) return;
     const float inv = 1.0f / sqrtf(block_sum(ss, red[2]) / float(a.d) + a.eps);
-    for (uint32_t i = tid; i < a.d; i += 256) {
-        const float v = row[i] * inv * weight_of(a.norm, i);
-        if (a.next) a.next[from + i] = v;
-        if (a.next_b) a.next_b[from + i] = f32_to_bf16(v);
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float x[V], w[V];
+        load_f32<V>(x, ra + i);
+        weights_of<V>(w, a.norm, i);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) x[j] *= inv * w[j];
+        if (a.next) store_f32<V>(a.next + from + i, x);
+        if (a.next_b) store_bf16<V>(a.next_b + from + i, x);
     }
 }
 
@@ -157,13 +178,21 @@ void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s) {
 }
 void launch_norm_rows(const NormArgs& a, cudaStream_t s) {
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(linear::norm_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); });
-    if (a.n) launch_pdl(linear::norm_rows_kernel, a.n, 256, size_t(a.k) * 4, s, a);
+    configured.once([] {
+        for (auto f : {linear::norm_rows_kernel<1>, linear::norm_rows_kernel<4>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    if (!a.n) return;
+    if (a.k % 4 == 0) launch_pdl(linear::norm_rows_kernel<4>, a.n, row_threads(a.k, 4), size_t(a.k) * 4, s, a);
+    else launch_pdl(linear::norm_rows_kernel<1>, a.n, row_threads(a.k, 1), size_t(a.k) * 4, s, a);
 }
 void launch_merge_rows(const MergeArgs& a, cudaStream_t s) {
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(linear::merge_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); });
-    if (a.n) launch_pdl(linear::merge_rows_kernel, a.n, 256, size_t(a.d) * 4, s, a);
+    configured.once([] {
+        for (auto f : {linear::merge_rows_kernel<1>, linear::merge_rows_kernel<4>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    if (!a.n) return;
+    if (a.d % 4 == 0) launch_pdl(linear::merge_rows_kernel<4>, a.n, row_threads(a.d, 4), size_t(a.d) * 8, s, a);
+    else launch_pdl(linear::merge_rows_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 8, s, a);
 }
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s) {
     if (n) launch_pdl(linear::concat_rows_kernel, n, 256, 0, s, a, b, d, out_f32, out_bf16);

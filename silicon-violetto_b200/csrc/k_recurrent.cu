@@ -2,9 +2,10 @@
 // and its step sizes, time mixing's mixes of neighbouring rows and its decays, and the gated norm of the outputs.
 //
 // The recurrence S = D S + k v^T runs token by token in fp32, the state in registers: a block has 16 value channels of one head of
-// one run, eight lanes share a value channel and hold an eighth of its key channels each, in pairs for the packed fp32
-// instructions. Rows come in by asynchronous copies, a chunk of tokens ahead; the output's sums over the eight lanes are taken
-// for eight tokens at a time, so that a token costs one exchange between lanes. A prompt's portion reads and writes the state
+// one run; 8, 16 or 32 lanes, by the number of key channels, share four value channels and hold four key channels (or a few
+// times four) of each, in pairs for the packed fp32 instructions: what a lane reads of q, k and decays serves four columns. Rows
+// come in by asynchronous copies, a chunk of tokens ahead; the output's sums over the lanes are taken for eight tokens at a time,
+// by exchanges that halve what a lane carries. A prompt's portion reads and writes the state
 // once, like a decoded token. The result of a row depends on nothing but the rows before it, however they are cut into steps.
 #include <algorithm>
 
@@ -14,7 +15,7 @@ namespace vlt {
 
 namespace recurrent {
 
-constexpr uint32_t LANES = 8, COLS = 16, THREADS = LANES * COLS;
+constexpr uint32_t PC = 4, COLS = 4 * PC;  // value channels of a thread, of a block
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(uint32_t(__cvta_generic_to_shared(dst))), "l"(src) : "memory"); }
@@ -42,67 +43,110 @@ __device__ __forceinline__ Stage stage_at(float* base, uint32_t np, uint32_t tok
     return st;
 }
 
-// The state as a thread holds it: key channels 4 lane + 32 i .. + 3 of its value channel, in two pairs each.
+// The state as a thread holds it: key channels 4 lane + 4 L i .. + 3 of PC neighbouring value channels, in two pairs each.
 template <uint32_t NV>
 struct State {
-    float2 a[NV], b[NV];
+    float2 a[NV][PC], b[NV][PC];
     __device__ __forceinline__ void clear() {
 #pragma unroll
-        for (uint32_t i = 0; i < NV; i++) a[i] = b[i] = make_float2(0.0f, 0.0f);
-    }
-    __device__ __forceinline__ void load(const float* p) {
+        for (uint32_t i = 0; i < NV; i++)
 #pragma unroll
-        for (uint32_t i = 0; i < NV; i++) {
-            const float4 x = *reinterpret_cast<const float4*>(p + 32 * i);
-            a[i] = make_float2(x.x, x.y);
-            b[i] = make_float2(x.z, x.w);
-        }
-    }
-    __device__ __forceinline__ void store(float* p) const {
-#pragma unroll
-        for (uint32_t i = 0; i < NV; i++) *reinterpret_cast<float4*>(p + 32 * i) = make_float4(a[i].x, a[i].y, b[i].x, b[i].y);
+            for (uint32_t c = 0; c < PC; c++) a[i][c] = b[i][c] = make_float2(0.0f, 0.0f);
     }
 };
-
-// One token: the state advances; the returned sum is this lane's part of q . S (before the update with channel decays, after it
-// without).
-template <uint32_t NV, bool CHANNEL>
-__device__ __forceinline__ float advance(State<NV>& S, const Stage& st, uint32_t np, uint32_t j, uint32_t n0, uint32_t col) {
-    const float factor = CHANNEL ? 1.0f : st.s[4 * j], v = st.v[j * COLS + col] * factor;
-    const float2 vv = make_float2(v, v);
-    float2 acc = make_float2(0.0f, 0.0f), d = acc;
-    if (!CHANNEL) d = make_float2(st.s[4 * j + 1], st.s[4 * j + 1]);
-    const float *q = st.q + j * np + n0, *k = st.k + j * np + n0, *w = st.w + j * np + n0;
+template <uint32_t L, uint32_t NV>
+__device__ __forceinline__ void load_state(State<NV>& S, const float* p, uint32_t cols) {  // cols: of the PC, those that exist
 #pragma unroll
-    for (uint32_t i = 0; i < NV; i++) {
-        const float4 q4 = *reinterpret_cast<const float4*>(q + 32 * i), k4 = *reinterpret_cast<const float4*>(k + 32 * i);
-        const float2 kva = __fmul2_rn(make_float2(k4.x, k4.y), vv), kvb = __fmul2_rn(make_float2(k4.z, k4.w), vv);
-        if (CHANNEL) {
-            const float4 w4 = *reinterpret_cast<const float4*>(w + 32 * i);
-            acc = __ffma2_rn(make_float2(q4.x, q4.y), S.a[i], acc);
-            acc = __ffma2_rn(make_float2(q4.z, q4.w), S.b[i], acc);
-            S.a[i] = __ffma2_rn(make_float2(w4.x, w4.y), S.a[i], kva);
-            S.b[i] = __ffma2_rn(make_float2(w4.z, w4.w), S.b[i], kvb);
-        } else {
-            S.a[i] = __ffma2_rn(d, S.a[i], kva);
-            S.b[i] = __ffma2_rn(d, S.b[i], kvb);
-            acc = __ffma2_rn(make_float2(q4.x, q4.y), S.a[i], acc);
-            acc = __ffma2_rn(make_float2(q4.z, q4.w), S.b[i], acc);
+    for (uint32_t i = 0; i < NV; i++)
+#pragma unroll
+        for (uint32_t c = 0; c < PC; c++) {
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (c < cols) x = *reinterpret_cast<const float4*>(p + (c * NV + i) * 4 * L);
+            S.a[i][c] = make_float2(x.x, x.y);
+            S.b[i][c] = make_float2(x.z, x.w);
         }
-    }
-    return acc.x + acc.y;
+}
+template <uint32_t L, uint32_t NV>
+__device__ __forceinline__ void store_state(const State<NV>& S, float* p, uint32_t cols) {
+#pragma unroll
+    for (uint32_t i = 0; i < NV; i++)
+#pragma unroll
+        for (uint32_t c = 0; c < PC; c++)
+            if (c < cols) *reinterpret_cast<float4*>(p + (c * NV + i) * 4 * L) = make_float4(S.a[i][c].x, S.a[i][c].y, S.b[i][c].x, S.b[i][c].y);
 }
 
-// grid (heads x slices of 16 value channels, runs). tc: tokens a chunk, a multiple of 8; two chunks in shared memory if a run is longer.
-template <uint32_t NV, bool CHANNEL>
-__global__ void __launch_bounds__(THREADS) scan_kernel(const ScanArgs a, uint32_t tc, bool aligned) {
+// One token: the state advances; part[c] is this lane's part of q . S (before the update with channel decays, after it without).
+template <uint32_t L, uint32_t NV, bool CHANNEL>
+__device__ __forceinline__ void advance(State<NV>& S, const Stage& st, uint32_t j, uint32_t lane, uint32_t col, float* part) {
+    constexpr uint32_t NP = 4 * L * NV;
+    const float4 v4 = *reinterpret_cast<const float4*>(st.v + j * COLS + col);
+    float v[PC] = {v4.x, v4.y, v4.z, v4.w};
+    float2 d = make_float2(0.0f, 0.0f), acc[PC];
+    if (!CHANNEL) {
+        const float2 step = *reinterpret_cast<const float2*>(st.s + 4 * j);
+        d = make_float2(step.y, step.y);
+#pragma unroll
+        for (uint32_t c = 0; c < PC; c++) v[c] *= step.x;
+    }
+#pragma unroll
+    for (uint32_t c = 0; c < PC; c++) acc[c] = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (uint32_t i = 0; i < NV; i++) {
+        const uint32_t at = j * NP + 4 * lane + 4 * L * i;
+        const float4 q4 = *reinterpret_cast<const float4*>(st.q + at), k4 = *reinterpret_cast<const float4*>(st.k + at);
+        const float2 qa = make_float2(q4.x, q4.y), qb = make_float2(q4.z, q4.w), ka = make_float2(k4.x, k4.y), kb = make_float2(k4.z, k4.w);
+        float2 wa = d, wb = d;
+        if (CHANNEL) {
+            const float4 w4 = *reinterpret_cast<const float4*>(st.w + at);
+            wa = make_float2(w4.x, w4.y);
+            wb = make_float2(w4.z, w4.w);
+        }
+#pragma unroll
+        for (uint32_t c = 0; c < PC; c++) {
+            const float2 vv = make_float2(v[c], v[c]);
+            if (CHANNEL) {
+                acc[c] = __ffma2_rn(qa, S.a[i][c], acc[c]);
+                acc[c] = __ffma2_rn(qb, S.b[i][c], acc[c]);
+            }
+            S.a[i][c] = __ffma2_rn(wa, S.a[i][c], __fmul2_rn(ka, vv));
+            S.b[i][c] = __ffma2_rn(wb, S.b[i][c], __fmul2_rn(kb, vv));
+            if (!CHANNEL) {
+                acc[c] = __ffma2_rn(qa, S.a[i][c], acc[c]);
+                acc[c] = __ffma2_rn(qb, S.b[i][c], acc[c]);
+            }
+        }
+    }
+#pragma unroll
+    for (uint32_t c = 0; c < PC; c++) part[c] = acc[c].x + acc[c].y;
+}
+
+// SUMS sums over L lanes: each exchange halves what a lane still carries; lane l ends with sums l SUMS / L .. in part[0] on.
+template <uint32_t L, uint32_t SUMS>
+__device__ __forceinline__ void spread_sums(float* part, uint32_t lane) {
+    uint32_t half = SUMS / 2;
+#pragma unroll
+    for (uint32_t o = L / 2; o > 0; o /= 2, half /= 2) {
+        const bool up = lane & o;
+#pragma unroll
+        for (uint32_t u = 0; u < SUMS / 2; u++) {
+            if (u >= half) break;
+            const float keep = up ? part[u + half] : part[u], give = up ? part[u] : part[u + half];
+            part[u] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+}
+
+// grid (heads x slices of 16 value channels, runs), 4 L threads: L lanes share PC value channels. tc: tokens a chunk, a multiple of
+// 8; two chunks in shared memory if a run is longer.
+template <uint32_t L, uint32_t NV, bool CHANNEL>
+__global__ void __launch_bounds__(4 * L) scan_kernel(const ScanArgs a, uint32_t tc, bool aligned) {
     pdl_start();
     extern __shared__ __align__(16) float sm[];
-    constexpr uint32_t NP = 32 * NV;
+    constexpr uint32_t NP = 4 * L * NV, THREADS = 4 * L, GROUP = 8;
     const RecurrentCache& c = a.c;
-    const uint32_t slices = (c.P + COLS - 1) / COLS, head = blockIdx.x / slices, p0 = blockIdx.x % slices * COLS, tid = threadIdx.x, lane = tid % LANES, col = tid / LANES;
+    const uint32_t slices = (c.P + COLS - 1) / COLS, head = blockIdx.x / slices, p0 = blockIdx.x % slices * COLS, tid = threadIdx.x, lane = tid % L, col = tid / L * PC;
     const RunIn run = a.runs[blockIdx.y];
-    const uint32_t t0 = run.first, count = run.count, cols = min(COLS, c.P - p0), n0 = 4 * lane;
+    const uint32_t t0 = run.first, count = run.count, cols = min(COLS, c.P - p0), mine = col < cols ? min(PC, cols - col) : 0;
     const bool verify = run.verify && count > 1, two = a.max_run > tc;
     const uint32_t stage_len = stage_floats<CHANNEL>(NP, tc);
     if (c.N != NP || cols != COLS) {  // what no copy writes stays zero
@@ -132,16 +176,16 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(const ScanArgs a, uint32_
             for (uint32_t i = tid; i < 2 * n; i += THREADS) cp_async4(st.s + 4 * (i / 2) + i % 2, D + size_t(i0 + i / 2) * c.heads * 2 + i % 2);
         }
     };
+    float* home = c.state + ((size_t(run.slot) * c.heads + head) * c.P + p0 + (mine ? col : 0)) * NP + 4 * lane;
+    State<NV> S;
+    load_state<L, NV>(S, home, mine);
     fetch(0);
     cp_async_commit();
-    const bool mine = col < cols;
-    float* home = c.state + ((size_t(run.slot) * c.heads + head) * c.P + p0 + (mine ? col : 0)) * NP + n0;
     const bool fresh = a.meta[2 * t0 + 1] == 0;  // a sequence begins: nothing of the slot's last one
-    State<NV> S;
     if (fresh) S.clear();
-    else S.load(home);
     const float skip = CHANNEL ? 0.0f : bf16_to_f32(a.skip[head]);
-    float* Y = a.y + size_t(t0) * c.heads * c.P + size_t(head) * c.P + p0 + col;
+    const size_t ldy = size_t(c.heads) * c.P;
+    float* Y = a.y + size_t(t0) * ldy + size_t(head) * c.P + p0 + col;
     if (verify) {
         // A verified run's rows, at most eight of one tile: each from the state before the run over the rows it descends from. The
         // state itself waits for the accepted path; what it will take is kept.
@@ -151,7 +195,7 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(const ScanArgs a, uint32_
         const size_t kept = size_t(run.slot) * VERIFY_T;
         for (uint32_t i = 0; i < count; i++) {
             const size_t row = kept + i;
-            if (tid < cols) c.keep_v[row * c.heads * c.P + size_t(head) * c.P + p0 + tid] = st.v[i * COLS + tid];
+            for (uint32_t p = tid; p < cols; p += THREADS) c.keep_v[row * ldy + size_t(head) * c.P + p0 + p] = st.v[i * COLS + p];
             if (p0) continue;
             if (head % c.per == 0)
                 for (uint32_t n = tid; n < c.N; n += THREADS) c.keep_k[(row * (c.heads / c.per) + head / c.per) * c.N + n] = st.k[i * NP + n];
@@ -161,15 +205,19 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(const ScanArgs a, uint32_
                 c.keep_d[(row * c.heads + head) * 2 + tid] = st.s[4 * i + tid];
         }
         for (uint32_t i = 0; i < count; i++) {
+            float part[PC];
             if (i) {
                 if (fresh) S.clear();
-                else S.load(home);
-                for (uint32_t before = a.vis[t0 + i] & ((1u << i) - 1); before; before &= before - 1) advance<NV, CHANNEL>(S, st, NP, __ffs(before) - 1, n0, col);
+                else load_state<L, NV>(S, home, mine);
+                for (uint32_t before = a.vis[t0 + i] & ((1u << i) - 1); before; before &= before - 1) advance<L, NV, CHANNEL>(S, st, __ffs(before) - 1, lane, col, part);
             }
-            float y = advance<NV, CHANNEL>(S, st, NP, i, n0, col);
+            advance<L, NV, CHANNEL>(S, st, i, lane, col, part);
 #pragma unroll
-            for (uint32_t o = LANES / 2; o > 0; o /= 2) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (lane == 0 && mine) Y[size_t(i) * c.heads * c.P] = y + (CHANNEL ? st.s[4 * i] : skip) * st.v[i * COLS + col];
+            for (uint32_t p = 0; p < PC; p++) {
+#pragma unroll
+                for (uint32_t o = L / 2; o > 0; o /= 2) part[p] += __shfl_xor_sync(0xffffffffu, part[p], o);
+                if (lane == 0 && p < mine) Y[i * ldy + p] = part[p] + (CHANNEL ? st.s[4 * i] : skip) * st.v[i * COLS + col + p];
+            }
         }
         return;
     }
@@ -180,31 +228,32 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(const ScanArgs a, uint32_
         __syncthreads();
         const Stage st = stage_at<CHANNEL>(sm + (i0 / tc & 1) * stage_len, NP, tc);
         const uint32_t n = min(tc, count - i0);
-        for (uint32_t j0 = 0; j0 < n; j0 += LANES) {
-            float part[LANES];
-            if (j0 + LANES <= n) {
+        for (uint32_t j0 = 0; j0 < n; j0 += GROUP) {
+            float part[GROUP * PC];
+            if (j0 + GROUP <= n) {
 #pragma unroll
-                for (uint32_t u = 0; u < LANES; u++) part[u] = advance<NV, CHANNEL>(S, st, NP, j0 + u, n0, col);
+                for (uint32_t u = 0; u < GROUP; u++) advance<L, NV, CHANNEL>(S, st, j0 + u, lane, col, part + PC * u);
             } else {
 #pragma unroll
-                for (uint32_t u = 0; u < LANES; u++) part[u] = j0 + u < n ? advance<NV, CHANNEL>(S, st, NP, j0 + u, n0, col) : 0.0f;
-            }
-            // Eight sums over eight lanes: each exchange halves what a lane still carries; lane u ends with token u's.
+                for (uint32_t u = 0; u < GROUP; u++) {
+                    if (j0 + u < n) {
+                        advance<L, NV, CHANNEL>(S, st, j0 + u, lane, col, part + PC * u);
+                    } else {
 #pragma unroll
-            for (uint32_t o = LANES / 2; o > 0; o /= 2) {
-                const bool up = lane & o;
-#pragma unroll
-                for (uint32_t u = 0; u < o; u++) {
-                    const float keep = up ? part[u + o] : part[u], give = up ? part[u] : part[u + o];
-                    part[u] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                        for (uint32_t p = 0; p < PC; p++) part[PC * u + p] = 0.0f;
+                    }
                 }
             }
-            const uint32_t j = j0 + lane;
-            if (j < n && mine) Y[size_t(i0 + j) * c.heads * c.P] = part[0] + (CHANNEL ? st.s[4 * j] : skip) * st.v[j * COLS + col];
+            spread_sums<L, GROUP * PC>(part, lane);
+#pragma unroll
+            for (uint32_t r = 0; r < GROUP * PC / L; r++) {
+                const uint32_t sum = lane * (GROUP * PC / L) + r, j = j0 + sum / PC, p = sum % PC;
+                if (j < n && p < mine) Y[(i0 + j) * ldy + p] = part[r] + (CHANNEL ? st.s[4 * j] : skip) * st.v[j * COLS + col + p];
+            }
         }
         __syncthreads();  // the chunk's place is free
     }
-    if (mine && !a.gen[run.slot].done) S.store(home);
+    if (mine && !a.gen[run.slot].done) store_state<L, NV>(S, home, mine);
 }
 
 // grid (heads, caches, runs).
@@ -289,11 +338,12 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs a, const 
     }
 }
 
-// A block per token.
+// grid (tokens, spans of the row).
+template <uint32_t V>
 __global__ void __launch_bounds__(256) token_shift_kernel(const ShiftArgs a, uint32_t n) {
     pdl_start();
     const uint32_t t = blockIdx.x, tid = threadIdx.x, d = a.c.conv_channels;
-    if (t == 0) {
+    if (t == 0 && blockIdx.y == 0) {
         const uint32_t per = (n + a.tile - 1) / a.tile;
         for (uint32_t i = tid; i < 4 * per; i += 256) {
             const uint32_t g = i / per, p = i % per * a.tile;
@@ -303,28 +353,54 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const ShiftArgs a, uin
         }
         if (tid == 0) *a.n_tiles = 4 * per;
     }
+    const uint32_t i = (blockIdx.y * 256 + tid) * V;
+    if (i >= d) return;
     const float *h = row_before(a.c, t, 0), *before = row_before(a.c, t, 1);
-    const uint32_t row = a.c.tin[2 * t + 1], cpos = a.c.meta[2 * (t - row) + 1] + row;
-    float* ring = a.c.ring + (size_t(a.c.meta[2 * t]) * a.c.ring_len + cpos % a.c.ring_len) * d;
-    for (uint32_t i = tid; i < d; i += 256) {
-        const float x = h[i], dx = (before ? before[i] : 0.0f) - x;
+    float x[V], dx[V];
+    load_f32<V>(x, h + i);
 #pragma unroll
-        for (uint32_t m = 0; m < 5; m++) {
-            const float y = fmaf(dx, bf16_to_f32(a.mu[m][i]), x);
-            const size_t o = (size_t((m + 1) % 5) * n + t) * d + i;
-            if (a.out_f32) a.out_f32[o] = y;
-            if (a.out_bf16) a.out_bf16[o] = f32_to_bf16(y);
-        }
-        if (a.c.write_ring) ring[i] = x;
+    for (uint32_t j = 0; j < V; j++) dx[j] = 0.0f;
+    if (before) load_f32<V>(dx, before + i);
+#pragma unroll
+    for (uint32_t j = 0; j < V; j++) dx[j] -= x[j];
+#pragma unroll
+    for (uint32_t m = 0; m < 5; m++) {
+        float y[V];
+        load_bf16<V>(y, a.mu[m] + i);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) y[j] = fmaf(dx[j], y[j], x[j]);
+        const size_t o = (size_t((m + 1) % 5) * n + t) * d + i;
+        if (a.out_f32) store_f32<V>(a.out_f32 + o, y);
+        if (a.out_bf16) store_bf16<V>(a.out_bf16 + o, y);
+    }
+    if (a.c.write_ring) {
+        const uint32_t row = a.c.tin[2 * t + 1], cpos = a.c.meta[2 * (t - row) + 1] + row;
+        store_f32<V>(a.c.ring + (size_t(a.c.meta[2 * t]) * a.c.ring_len + cpos % a.c.ring_len) * d + i, x);
     }
 }
 
-// grid (tokens / 8, heads).
+// grid (tokens / TT, heads): the head's w2 and the tokens' hidden rows in shared memory, a channel and TT / 2 tokens a thread at a time.
+template <uint32_t TT>
 __global__ void __launch_bounds__(128) decay_kernel(const DecayArgs a, uint32_t n) {
     pdl_start();
-    extern __shared__ float th[];  // [8][rank]
-    const uint32_t t0 = blockIdx.x * 8, head = blockIdx.y, tid = threadIdx.x, nt = min(8u, n - t0), warp = tid / 32, lane = tid % 32, K = a.heads * a.dim;
-    for (uint32_t i = tid; i < 8 * a.rank; i += 128) th[i] = i / a.rank < nt ? tanhf(a.hid[size_t(t0 + i / a.rank) * a.ldh + i % a.rank]) : 0.0f;
+    extern __shared__ __align__(16) float sm[];
+    const uint32_t t0 = blockIdx.x * TT, head = blockIdx.y, tid = threadIdx.x, nt = min(TT, n - t0), warp = tid / 32, lane = tid % 32, K = a.heads * a.dim, pitch = a.dim + 1;
+    float *th = sm, *w = sm + TT * a.rank;  // [rank][TT], [rank][pitch]
+    for (uint32_t i = tid; i < TT * a.rank; i += 128) {
+        const uint32_t j = i % a.rank, t = i / a.rank;
+        th[j * TT + t] = t < nt ? tanhf(a.hid[size_t(t0 + t) * a.ldh + j]) : 0.0f;
+    }
+    const uint16_t* w2 = a.w2 + size_t(head) * a.dim * a.rank;
+    if (a.rank % 4 == 0) {
+        for (uint32_t i = 4 * tid; i < a.dim * a.rank; i += 512) {
+            float x[4];
+            load_bf16<4>(x, w2 + i);
+#pragma unroll
+            for (uint32_t u = 0; u < 4; u++) w[(i % a.rank + u) * pitch + i / a.rank] = x[u];
+        }
+    } else {
+        for (uint32_t i = tid; i < a.dim * a.rank; i += 128) w[i % a.rank * pitch + i / a.rank] = bf16_to_f32(w2[i]);
+    }
     for (uint32_t i = warp; i < nt; i += 4) {
         float s = 0.0f;
         for (uint32_t c = lane; c < a.dim; c += 32) {
@@ -335,85 +411,110 @@ __global__ void __launch_bounds__(128) decay_kernel(const DecayArgs a, uint32_t 
         if (lane == 0) a.bonus[size_t(t0 + i) * a.heads + head] = s;
     }
     __syncthreads();
-    for (uint32_t i = tid; i < 2 * a.dim; i += 128) {  // a channel, four tokens
-        const uint32_t c = head * a.dim + i % a.dim, q0 = i / a.dim * 4;
+    constexpr uint32_t PER = TT / 2;
+    for (uint32_t i = tid; i < 2 * a.dim; i += 128) {
+        const uint32_t c = i % a.dim, q0 = i / a.dim * PER;
         if (q0 >= nt) continue;
-        const uint16_t* w = a.w2 + size_t(c) * a.rank;
-        float s[4] = {};
+        float s[PER] = {};
         for (uint32_t j = 0; j < a.rank; j++) {
-            const float wj = bf16_to_f32(w[j]);
+            const float wj = w[j * pitch + c];
 #pragma unroll
-            for (uint32_t u = 0; u < 4; u++) s[u] = fmaf(wj, th[(q0 + u) * a.rank + j], s[u]);
+            for (uint32_t u = 0; u < PER; u += 4) {
+                const float4 h = *reinterpret_cast<const float4*>(th + j * TT + q0 + u);
+                s[u] = fmaf(wj, h.x, s[u]);
+                s[u + 1] = fmaf(wj, h.y, s[u + 1]);
+                s[u + 2] = fmaf(wj, h.z, s[u + 2]);
+                s[u + 3] = fmaf(wj, h.w, s[u + 3]);
+            }
         }
-        const float w0 = bf16_to_f32(a.w0[c]);
+        const float w0 = bf16_to_f32(a.w0[head * a.dim + c]);
 #pragma unroll
-        for (uint32_t u = 0; u < 4; u++)
-            if (q0 + u < nt) a.decay[size_t(t0 + q0 + u) * K + c] = expf(-expf(s[u] + w0));
+        for (uint32_t u = 0; u < PER; u++)
+            if (q0 + u < nt) a.decay[size_t(t0 + q0 + u) * K + head * a.dim + c] = expf(-expf(s[u] + w0));
     }
 }
 
-// A block per token: with eight parts or more a warp takes one at a time, else all threads together.
-__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormArgs a) {
+// A block per token, which keeps the row in shared memory: with eight parts or more a warp takes one at a time, else all threads
+// together.
+template <uint32_t V>
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormArgs a) {
     pdl_start();
-    __shared__ float red[8];
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
     const uint32_t t = blockIdx.x, tid = threadIdx.x, width = a.width / a.groups;
     const bool alone = a.groups >= 8;
-    const uint32_t lanes = alone ? 32 : 256, lane = tid % lanes, first = tid / lanes, step = 256 / lanes;
+    const uint32_t lanes = alone ? 32 : blockDim.x, lane = tid % lanes, first = tid / lanes, step = blockDim.x / lanes;
     const float *y = a.y + size_t(t) * a.width, *gate = a.gate + size_t(t) * a.ldg;
     for (uint32_t g = first; g < a.groups; g += step) {
         const uint32_t c0 = g * width;
         float ss = 0.0f;
-        for (uint32_t c = lane; c < width; c += lanes) {
-            const float v = a.gate_first ? y[c0 + c] * silu(gate[c0 + c]) : y[c0 + c];
-            ss += v * v;
+        for (uint32_t c = lane * V; c < width; c += lanes * V) {
+            float v[V], z[V], w[V];
+            load_f32<V>(v, y + c0 + c);
+            load_f32<V>(z, gate + c0 + c);
+            load_bf16<V>(w, a.w + c0 + c);
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) {
+                const float s = silu(z[j]), gated = v[j] * s;
+                ss += a.gate_first ? gated * gated : v[j] * v[j];
+                v[j] = gated * w[j];
+            }
+            store_f32<V>(row + c0 + c, v);
         }
-        ss = warp_sum(ss);
-        if (!alone) {
-            __syncthreads();  // (the part before this one has been read)
-            if (tid % 32 == 0) red[tid / 32] = ss;
-            __syncthreads();
-            ss = 0.0f;
-            for (uint32_t i = 0; i < 8; i++) ss += red[i];
+        if (alone) {
+            ss = warp_sum(ss);
+        } else {
+            __syncthreads();  // (`red` has been read for the part before this one)
+            ss = block_sum(ss, red);
         }
         const float inv = 1.0f / sqrtf(ss / float(width) + a.eps);
-        for (uint32_t c = lane; c < width; c += lanes) {
-            const float z = silu(gate[c0 + c]), v = y[c0 + c] * inv * bf16_to_f32(a.w[c0 + c]) * z;
-            if (a.out_f32) a.out_f32[size_t(t) * a.width + c0 + c] = v;
-            if (a.out_bf16) a.out_bf16[size_t(t) * a.width + c0 + c] = f32_to_bf16(v);
+        for (uint32_t c = lane * V; c < width; c += lanes * V) {  // (a thread reads back what it wrote)
+            float v[V];
+            load_f32<V>(v, row + c0 + c);
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) v[j] *= inv;
+            const size_t o = size_t(t) * a.width + c0 + c;
+            if (a.out_f32) store_f32<V>(a.out_f32 + o, v);
+            if (a.out_bf16) store_bf16<V>(a.out_bf16 + o, v);
         }
     }
 }
 
-template <uint32_t NV, bool CHANNEL>
+template <uint32_t L, uint32_t NV, bool CHANNEL>
 void scan(const ScanArgs& a, cudaStream_t s) {
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(scan_kernel<NV, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024)); });
+    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(scan_kernel<L, NV, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024)); });
     const uint32_t slices = (a.c.P + COLS - 1) / COLS;
+    constexpr uint32_t NP = 4 * L * NV;
     uint32_t tc = 8;
-    while (tc < 32 && tc < a.max_run && 2 * stage_floats<CHANNEL>(32 * NV, 2 * tc) * 4 <= 72 * 1024) tc *= 2;
-    const size_t smem = size_t(stage_floats<CHANNEL>(32 * NV, tc)) * 4 * (a.max_run > tc ? 2 : 1);
+    while (tc < 32 && tc < a.max_run && 2 * stage_floats<CHANNEL>(NP, 2 * tc) * 4 <= 72 * 1024) tc *= 2;
+    const size_t smem = size_t(stage_floats<CHANNEL>(NP, tc)) * 4 * (a.max_run > tc ? 2 : 1);
     auto whole = [](const void* p, size_t ld) { return reinterpret_cast<uintptr_t>(p) % 16 == 0 && ld % 4 == 0; };
     const bool aligned = a.c.N % 4 == 0 && a.c.P % 4 == 0 && whole(a.q, a.ldq) && whole(a.k, a.ldk) && whole(a.v, a.ldv) && whole(a.decay, 0);
-    launch_pdl(scan_kernel<NV, CHANNEL>, dim3(a.c.heads * slices, a.n_runs), THREADS, smem, s, a, tc, aligned);
+    launch_pdl(scan_kernel<L, NV, CHANNEL>, dim3(a.c.heads * slices, a.n_runs), 4 * L, smem, s, a, tc, aligned);
 }
+struct Kernel {
+    uint32_t pitch;
+    void (*plain)(const ScanArgs&, cudaStream_t);
+    void (*channel)(const ScanArgs&, cudaStream_t);
+};
+template <uint32_t L, uint32_t NV>
+constexpr Kernel kernel() { return {4 * L * NV, scan<L, NV, false>, scan<L, NV, true>}; }
+static const Kernel kernels[] = {kernel<8, 1>(), kernel<16, 1>(), kernel<32, 1>(), kernel<32, 2>(), kernel<32, 3>(), kernel<32, 4>()};
 
 }  // namespace recurrent
 
 void launch_scan(const ScanArgs& a, cudaStream_t s) {
     using namespace recurrent;
     if (!a.n_runs) return;
-    using Fn = void (*)(const ScanArgs&, cudaStream_t);
-    static const struct { uint32_t nv; Fn plain, channel; } kernels[] = {{1, scan<1, false>, scan<1, true>}, {2, scan<2, false>, scan<2, true>},   {3, scan<3, false>, scan<3, true>},
-                                                                         {4, scan<4, false>, scan<4, true>}, {6, scan<6, false>, scan<6, true>},   {8, scan<8, false>, scan<8, true>},
-                                                                         {12, scan<12, false>, scan<12, true>}, {16, scan<16, false>, scan<16, true>}};
-    for (const auto& k : kernels)
-        if (32 * k.nv == a.c.Np) { (a.c.channel_decay ? k.channel : k.plain)(a, s); return; }
+    for (const Kernel& k : kernels)
+        if (k.pitch == a.c.Np) { (a.c.channel_decay ? k.channel : k.plain)(a, s); return; }
     throw Error("internal: a recurrence over " + std::to_string(a.c.N) + " key channels");
 }
 // The key channels a state is laid out for: those of the smallest kernel that takes N.
 uint32_t recurrent_pitch(uint32_t N) {
-    for (uint32_t nv : {1u, 2u, 3u, 4u, 6u, 8u, 12u, 16u})
-        if (N <= 32 * nv) return 32 * nv;
+    for (const recurrent::Kernel& k : recurrent::kernels)
+        if (N <= k.pitch) return k.pitch;
     throw Error("internal: a recurrence over " + std::to_string(N) + " key channels");
 }
 void launch_recurrent_commit(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const RecurrentCache* caches, uint32_t n_runs,
@@ -430,12 +531,29 @@ void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, flo
     if (n >= 64) launch_pdl(recurrent::conv_silu_kernel<4>, dim3((n + 3) / 4, spans), 128, 0, s, a, st, n, y);
     else launch_pdl(recurrent::conv_silu_kernel<1>, dim3(n, spans), 128, 0, s, a, st, n, y);
 }
-void launch_token_shift(const ShiftArgs& a, uint32_t n, cudaStream_t s) { launch_pdl(recurrent::token_shift_kernel, n, 256, 0, s, a, n); }
+void launch_token_shift(const ShiftArgs& a, uint32_t n, cudaStream_t s) {
+    const uint32_t d = a.c.conv_channels;
+    if (d % 4 == 0) launch_pdl(recurrent::token_shift_kernel<4>, dim3(n, (d + 1023) / 1024), 256, 0, s, a, n);
+    else launch_pdl(recurrent::token_shift_kernel<1>, dim3(n, (d + 255) / 256), 256, 0, s, a, n);
+}
 void launch_decay(const DecayArgs& a, uint32_t n, cudaStream_t s) {
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(recurrent::decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); });
-    launch_pdl(recurrent::decay_kernel, dim3((n + 7) / 8, a.heads), 128, size_t(8) * a.rank * 4, s, a, n);
+    configured.once([] {
+        for (auto f : {recurrent::decay_kernel<8>, recurrent::decay_kernel<32>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    });
+    const uint32_t tt = n >= 64 ? 32 : 8;
+    const size_t smem = size_t(a.rank) * (tt + a.dim + 1) * 4;
+    if (tt == 32) launch_pdl(recurrent::decay_kernel<32>, dim3((n + 31) / 32, a.heads), 128, smem, s, a, n);
+    else launch_pdl(recurrent::decay_kernel<8>, dim3((n + 7) / 8, a.heads), 128, smem, s, a, n);
 }
-void launch_gated_norm(const GatedNormArgs& a, uint32_t n, cudaStream_t s) { launch_pdl(recurrent::gated_norm_kernel, n, 256, 0, s, a); }
+void launch_gated_norm(const GatedNormArgs& a, uint32_t n, cudaStream_t s) {
+    static PerDevice configured;
+    configured.once([] {
+        for (auto f : {recurrent::gated_norm_kernel<1>, recurrent::gated_norm_kernel<4>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    const bool four = a.width / a.groups % 4 == 0 && a.ldg % 4 == 0 && reinterpret_cast<uintptr_t>(a.gate) % 16 == 0;
+    if (four) launch_pdl(recurrent::gated_norm_kernel<4>, n, row_threads(a.width, 4), size_t(a.width) * 4, s, a);
+    else launch_pdl(recurrent::gated_norm_kernel<1>, n, row_threads(a.width, 1), size_t(a.width) * 4, s, a);
+}
 
 }  // namespace vlt

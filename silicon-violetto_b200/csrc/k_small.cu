@@ -32,7 +32,16 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
     if (tok >= vocab) tok = 0;
     if (positions) {  // (a draft's rows may reach past the last position: they are not kept then)
         const uint16_t* pv = positions + size_t(min(lens[slot] + depth, n_positions - 1)) * d;
-        for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]) + bf16_to_f32(pv[i]);
+        if (d % 4 == 0) {
+            for (uint32_t i = 4 * tid; i < d; i += 4 * blockDim.x) {
+                float x[4], y[4];
+                load_bf16<4>(x, table + size_t(tok) * d + i);
+                load_bf16<4>(y, pv + i);
+                store_f32<4>(out + size_t(t) * d + i, {x[0] + y[0], x[1] + y[1], x[2] + y[2], x[3] + y[3]});
+            }
+        } else {
+            for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]) + bf16_to_f32(pv[i]);
+        }
     } else if (d % 2 == 0) {
         const uint32_t* row = reinterpret_cast<const uint32_t*>(table + size_t(tok) * d);
         float2* o = reinterpret_cast<float2*>(out + size_t(t) * d);

@@ -31,6 +31,14 @@ struct QkvEpilogue {
 
 __device__ __forceinline__ float weight_of(const RowNorm& n, uint32_t i) { return (n.around_zero ? 1.0f : 0.0f) + bf16_to_f32(n.w[i]); }
 
+template <uint32_t V>
+__device__ __forceinline__ void weights_of(float (&x)[V], const RowNorm& n, uint32_t i) {
+    load_bf16<V>(x, n.w + i);
+    if (n.around_zero)
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) x[j] += 1.0f;
+}
+
 // Y[t][row] = epilogue(W[row] . bf16(X[t])). X fp32 [n][k]; Y fp32 (SWIGLU: [n][m/2]).
 struct MatArgs {
     const uint8_t* W;

@@ -457,10 +457,10 @@ class Engine:
         _check(lib().vlt_debug_profile(self.h, C.c_uint32(int(on))))
 
     def profile_read(self) -> dict:
-        ms = (C.c_double * 5)()
-        n = (C.c_uint32 * 5)()
+        ms = (C.c_double * 6)()
+        n = (C.c_uint32 * 6)()
         _check(lib().vlt_debug_profile_read(self.h, ms, n))
-        names = ("matmul", "attention", "small", "tail", "drafter")
+        names = ("matmul", "attention", "small", "tail", "drafter", "recurrence")
         return {k: dict(ms=ms[i], launches=int(n[i])) for i, k in enumerate(names)}
 
     def step_bytes(self):
