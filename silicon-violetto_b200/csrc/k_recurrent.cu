@@ -2,11 +2,11 @@
 // and its step sizes, time mixing's mixes of neighbouring rows and its decays, and the gated norm of the outputs.
 //
 // The recurrence S = D S + k v^T runs token by token in fp32, the state in registers: a block has 16 value channels of one head of
-// one run; 8, 16 or 32 lanes, by the number of key channels, share four value channels and hold four key channels (or a few
-// times four) of each, in pairs for the packed fp32 instructions: what a lane reads of q, k and decays serves four columns. Rows
-// come in by asynchronous copies, a chunk of tokens ahead; the output's sums over the lanes are taken for eight tokens at a time,
-// by exchanges that halve what a lane carries. A prompt's portion reads and writes the state
-// once, like a decoded token. The result of a row depends on nothing but the rows before it, however they are cut into steps.
+// one run; 8, 16 or 32 lanes share two or four value channels and hold four key channels (or a few times four) of each, in pairs
+// for the packed fp32 instructions: what a lane reads of q, k and decays serves several columns. Rows come in by asynchronous
+// copies, a chunk of tokens ahead; the output's sums over the lanes are taken for eight tokens at a time, by exchanges that halve
+// what a lane carries. A prompt's portion reads and writes the state once, like a decoded token. A row's result depends on nothing
+// but the rows before it, however they are cut into steps.
 #include <algorithm>
 
 #include "kernels.h"
@@ -15,16 +15,27 @@ namespace vlt {
 
 namespace recurrent {
 
-constexpr uint32_t PC = 4, COLS = 4 * PC;  // value channels of a thread, of a block
+constexpr uint32_t COLS = 16;  // value channels of a block; PC: of a thread
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(uint32_t(__cvta_generic_to_shared(dst))), "l"(src) : "memory"); }
-__device__ __forceinline__ void cp_async16(float* dst, const float* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(uint32_t(__cvta_generic_to_shared(dst))), "l"(src) : "memory"); }
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(uint32_t(__cvta_generic_to_shared(dst))), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() {
     asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
+
+// A thread's way through a matrix of `width` columns, `threads` elements at a time: one division where it begins.
+struct Walk {
+    uint32_t r, c, dr, dc, width;
+    __device__ __forceinline__ Walk(uint32_t start, uint32_t threads, uint32_t w) : r(start / w), c(start % w), dr(threads / w), dc(threads % w), width(w) {}
+    __device__ __forceinline__ void next() {
+        r += dr;
+        c += dc;
+        if (c >= width) { c -= width; r++; }
+    }
+};
 
 // A chunk of tokens in shared memory: q and k rows, decays (per channel or two numbers), values, the bonus.
 template <bool CHANNEL>
@@ -44,7 +55,7 @@ __device__ __forceinline__ Stage stage_at(float* base, uint32_t np, uint32_t tok
 }
 
 // The state as a thread holds it: key channels 4 lane + 4 L i .. + 3 of PC neighbouring value channels, in two pairs each.
-template <uint32_t NV>
+template <uint32_t NV, uint32_t PC>
 struct State {
     float2 a[NV][PC], b[NV][PC];
     __device__ __forceinline__ void clear() {
@@ -54,8 +65,8 @@ struct State {
             for (uint32_t c = 0; c < PC; c++) a[i][c] = b[i][c] = make_float2(0.0f, 0.0f);
     }
 };
-template <uint32_t L, uint32_t NV>
-__device__ __forceinline__ void load_state(State<NV>& S, const float* p, uint32_t cols) {  // cols: of the PC, those that exist
+template <uint32_t L, uint32_t NV, uint32_t PC>
+__device__ __forceinline__ void load_state(State<NV, PC>& S, const float* p, uint32_t cols) {  // cols: of the PC, those that exist
 #pragma unroll
     for (uint32_t i = 0; i < NV; i++)
 #pragma unroll
@@ -66,8 +77,8 @@ __device__ __forceinline__ void load_state(State<NV>& S, const float* p, uint32_
             S.b[i][c] = make_float2(x.z, x.w);
         }
 }
-template <uint32_t L, uint32_t NV>
-__device__ __forceinline__ void store_state(const State<NV>& S, float* p, uint32_t cols) {
+template <uint32_t L, uint32_t NV, uint32_t PC>
+__device__ __forceinline__ void store_state(const State<NV, PC>& S, float* p, uint32_t cols) {
 #pragma unroll
     for (uint32_t i = 0; i < NV; i++)
 #pragma unroll
@@ -75,35 +86,53 @@ __device__ __forceinline__ void store_state(const State<NV>& S, float* p, uint32
             if (c < cols) *reinterpret_cast<float4*>(p + (c * NV + i) * 4 * L) = make_float4(S.a[i][c].x, S.a[i][c].y, S.b[i][c].x, S.b[i][c].y);
 }
 
-// One token: the state advances; part[c] is this lane's part of q . S (before the update with channel decays, after it without).
-template <uint32_t L, uint32_t NV, bool CHANNEL>
-__device__ __forceinline__ void advance(State<NV>& S, const Stage& st, uint32_t j, uint32_t lane, uint32_t col, float* part) {
+// What a lane reads of a token.
+template <uint32_t NV, uint32_t PC, bool CHANNEL>
+struct Token {
+    float4 q[NV], k[NV], w[CHANNEL ? NV : 1];
+    float v[PC];
+    float2 step;
+};
+template <uint32_t L, uint32_t NV, uint32_t PC, bool CHANNEL>
+__device__ __forceinline__ void load_token(Token<NV, PC, CHANNEL>& t, const Stage& st, uint32_t j, uint32_t lane, uint32_t col) {
     constexpr uint32_t NP = 4 * L * NV;
-    const float4 v4 = *reinterpret_cast<const float4*>(st.v + j * COLS + col);
-    float v[PC] = {v4.x, v4.y, v4.z, v4.w};
-    float2 d = make_float2(0.0f, 0.0f), acc[PC];
-    if (!CHANNEL) {
-        const float2 step = *reinterpret_cast<const float2*>(st.s + 4 * j);
-        d = make_float2(step.y, step.y);
 #pragma unroll
-        for (uint32_t c = 0; c < PC; c++) v[c] *= step.x;
+    for (uint32_t i = 0; i < NV; i++) {
+        const uint32_t at = j * NP + 4 * lane + 4 * L * i;
+        t.q[i] = *reinterpret_cast<const float4*>(st.q + at);
+        t.k[i] = *reinterpret_cast<const float4*>(st.k + at);
+        if constexpr (CHANNEL) t.w[i] = *reinterpret_cast<const float4*>(st.w + at);
     }
+    if constexpr (PC == 4) {
+        load_f32<4>(t.v, st.v + j * COLS + col);
+    } else {
+        const float2 v2 = *reinterpret_cast<const float2*>(st.v + j * COLS + col);
+        t.v[0] = v2.x;
+        t.v[1] = v2.y;
+    }
+    if constexpr (!CHANNEL) t.step = *reinterpret_cast<const float2*>(st.s + 4 * j);
+}
+
+// One token: the state advances; part[c] is this lane's part of q . S (before the update with channel decays, after it without).
+template <uint32_t NV, uint32_t PC, bool CHANNEL>
+__device__ __forceinline__ void advance(State<NV, PC>& S, const Token<NV, PC, CHANNEL>& t, float* part) {
+    float2 acc[PC];
 #pragma unroll
     for (uint32_t c = 0; c < PC; c++) acc[c] = make_float2(0.0f, 0.0f);
 #pragma unroll
     for (uint32_t i = 0; i < NV; i++) {
-        const uint32_t at = j * NP + 4 * lane + 4 * L * i;
-        const float4 q4 = *reinterpret_cast<const float4*>(st.q + at), k4 = *reinterpret_cast<const float4*>(st.k + at);
-        const float2 qa = make_float2(q4.x, q4.y), qb = make_float2(q4.z, q4.w), ka = make_float2(k4.x, k4.y), kb = make_float2(k4.z, k4.w);
-        float2 wa = d, wb = d;
-        if (CHANNEL) {
-            const float4 w4 = *reinterpret_cast<const float4*>(st.w + at);
-            wa = make_float2(w4.x, w4.y);
-            wb = make_float2(w4.z, w4.w);
+        const float2 qa = make_float2(t.q[i].x, t.q[i].y), qb = make_float2(t.q[i].z, t.q[i].w), ka = make_float2(t.k[i].x, t.k[i].y), kb = make_float2(t.k[i].z, t.k[i].w);
+        float2 wa, wb;
+        if constexpr (CHANNEL) {
+            wa = make_float2(t.w[i].x, t.w[i].y);
+            wb = make_float2(t.w[i].z, t.w[i].w);
+        } else {
+            wa = wb = make_float2(t.step.y, t.step.y);
         }
 #pragma unroll
         for (uint32_t c = 0; c < PC; c++) {
-            const float2 vv = make_float2(v[c], v[c]);
+            const float v = CHANNEL ? t.v[c] : t.v[c] * t.step.x;
+            const float2 vv = make_float2(v, v);
             if (CHANNEL) {
                 acc[c] = __ffma2_rn(qa, S.a[i][c], acc[c]);
                 acc[c] = __ffma2_rn(qb, S.b[i][c], acc[c]);
@@ -119,30 +148,43 @@ __device__ __forceinline__ void advance(State<NV>& S, const Stage& st, uint32_t 
 #pragma unroll
     for (uint32_t c = 0; c < PC; c++) part[c] = acc[c].x + acc[c].y;
 }
+template <uint32_t L, uint32_t NV, uint32_t PC, bool CHANNEL>
+__device__ __forceinline__ void advance(State<NV, PC>& S, const Stage& st, uint32_t j, uint32_t lane, uint32_t col, float* part) {
+    Token<NV, PC, CHANNEL> t;
+    load_token<L, NV, PC, CHANNEL>(t, st, j, lane, col);
+    advance<NV, PC, CHANNEL>(S, t, part);
+}
 
-// SUMS sums over L lanes: each exchange halves what a lane still carries; lane l ends with sums l SUMS / L .. in part[0] on.
+// SUMS sums over L lanes: each exchange halves what a lane still carries, down to one; lane l ends with sums l SUMS / L .. in part[0]
+// on (more lanes than sums: L / SUMS lanes with the same one).
 template <uint32_t L, uint32_t SUMS>
 __device__ __forceinline__ void spread_sums(float* part, uint32_t lane) {
-    uint32_t half = SUMS / 2;
+    uint32_t left = SUMS;
 #pragma unroll
-    for (uint32_t o = L / 2; o > 0; o /= 2, half /= 2) {
+    for (uint32_t o = L / 2; o > 0; o /= 2) {
+        if (left == 1) {
+            part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
+            continue;
+        }
+        left /= 2;
         const bool up = lane & o;
 #pragma unroll
         for (uint32_t u = 0; u < SUMS / 2; u++) {
-            if (u >= half) break;
-            const float keep = up ? part[u + half] : part[u], give = up ? part[u] : part[u + half];
+            if (u >= left) break;
+            const float keep = up ? part[u + left] : part[u], give = up ? part[u] : part[u + left];
             part[u] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
     }
 }
 
-// grid (heads x slices of 16 value channels, runs), 4 L threads: L lanes share PC value channels. tc: tokens a chunk, a multiple of
-// 8; two chunks in shared memory if a run is longer.
-template <uint32_t L, uint32_t NV, bool CHANNEL>
-__global__ void __launch_bounds__(4 * L) scan_kernel(const ScanArgs a, uint32_t tc, bool aligned) {
+// grid (heads x slices of 16 value channels, runs), 16 L / PC threads: L lanes share PC (2 or 4) value channels. tc: tokens a chunk, a multiple of
+// 8; two chunks in shared memory if a run is longer. GROUP: tokens whose sums are taken together (1: steps of short runs, whose
+// kernel holds fewer registers and so has more of the states in flight).
+template <uint32_t L, uint32_t NV, uint32_t PC, bool CHANNEL, uint32_t GROUP>
+__global__ void __launch_bounds__(L * COLS / PC, GROUP == 1 ? 0 : 1) scan_kernel(const ScanArgs a, uint32_t tc, bool aligned) {
     pdl_start();
     extern __shared__ __align__(16) float sm[];
-    constexpr uint32_t NP = 4 * L * NV, THREADS = 4 * L, GROUP = 8;
+    constexpr uint32_t NP = 4 * L * NV, THREADS = L * COLS / PC, SUMS = GROUP * PC, PER = SUMS > L ? SUMS / L : 1;
     const RecurrentCache& c = a.c;
     const uint32_t slices = (c.P + COLS - 1) / COLS, head = blockIdx.x / slices, p0 = blockIdx.x % slices * COLS, tid = threadIdx.x, lane = tid % L, col = tid / L * PC;
     const RunIn run = a.runs[blockIdx.y];
@@ -155,30 +197,29 @@ __global__ void __launch_bounds__(4 * L) scan_kernel(const ScanArgs a, uint32_t 
     }
     const float *Q = a.q + size_t(t0) * a.ldq + size_t(head / c.per) * c.N, *K = a.k + size_t(t0) * a.ldk + size_t(head / c.per) * c.N, *V = a.v + size_t(t0) * a.ldv + size_t(head) * c.P + p0;
     const float* D = CHANNEL ? a.decay + (size_t(t0) * c.heads + head) * c.N : a.decay + (size_t(t0) * c.heads + head) * 2;
-    auto rows = [&](float* dst, uint32_t pitch, const float* src, size_t ld, uint32_t width, uint32_t n) {
-        if (aligned) {
-            const uint32_t w4 = width / 4;
-            for (uint32_t i = tid; i < n * w4; i += THREADS) cp_async16(dst + i / w4 * pitch + i % w4 * 4, src + i / w4 * ld + i % w4 * 4);
-        } else {
-            for (uint32_t i = tid; i < n * width; i += THREADS) cp_async4(dst + i / width * pitch + i % width, src + i / width * ld + i % width);
-        }
+    const Walk key0(tid, THREADS, aligned ? c.N / 4 : c.N), value0(tid, THREADS, aligned ? cols / 4 : cols);
+    auto rows = [&](Walk at, float* dst, uint32_t pitch, const float* src, size_t ld, uint32_t n) {
+        if (aligned)
+            for (; at.r < n; at.next()) cp_async16(dst + at.r * pitch + at.c * 4, src + at.r * ld + at.c * 4);
+        else
+            for (; at.r < n; at.next()) cp_async4(dst + at.r * pitch + at.c, src + at.r * ld + at.c);
     };
     auto fetch = [&](uint32_t i0) {
         const uint32_t n = min(tc, count - i0);
         const Stage st = stage_at<CHANNEL>(sm + (i0 / tc & 1) * stage_len, NP, tc);
-        rows(st.q, NP, Q + size_t(i0) * a.ldq, a.ldq, c.N, n);
-        rows(st.k, NP, K + size_t(i0) * a.ldk, a.ldk, c.N, n);
-        rows(st.v, COLS, V + size_t(i0) * a.ldv, a.ldv, cols, n);
+        rows(key0, st.q, NP, Q + size_t(i0) * a.ldq, a.ldq, n);
+        rows(key0, st.k, NP, K + size_t(i0) * a.ldk, a.ldk, n);
+        rows(value0, st.v, COLS, V + size_t(i0) * a.ldv, a.ldv, n);
         if (CHANNEL) {
-            rows(st.w, NP, D + size_t(i0) * c.heads * c.N, size_t(c.heads) * c.N, c.N, n);
+            rows(key0, st.w, NP, D + size_t(i0) * c.heads * c.N, size_t(c.heads) * c.N, n);
             for (uint32_t i = tid; i < n; i += THREADS) cp_async4(st.s + 4 * i, a.bonus + size_t(t0 + i0 + i) * c.heads + head);
         } else {
             for (uint32_t i = tid; i < 2 * n; i += THREADS) cp_async4(st.s + 4 * (i / 2) + i % 2, D + size_t(i0 + i / 2) * c.heads * 2 + i % 2);
         }
     };
     float* home = c.state + ((size_t(run.slot) * c.heads + head) * c.P + p0 + (mine ? col : 0)) * NP + 4 * lane;
-    State<NV> S;
-    load_state<L, NV>(S, home, mine);
+    State<NV, PC> S;
+    load_state<L, NV, PC>(S, home, mine);
     fetch(0);
     cp_async_commit();
     const bool fresh = a.meta[2 * t0 + 1] == 0;  // a sequence begins: nothing of the slot's last one
@@ -208,10 +249,10 @@ __global__ void __launch_bounds__(4 * L) scan_kernel(const ScanArgs a, uint32_t 
             float part[PC];
             if (i) {
                 if (fresh) S.clear();
-                else load_state<L, NV>(S, home, mine);
-                for (uint32_t before = a.vis[t0 + i] & ((1u << i) - 1); before; before &= before - 1) advance<L, NV, CHANNEL>(S, st, __ffs(before) - 1, lane, col, part);
+                else load_state<L, NV, PC>(S, home, mine);
+                for (uint32_t before = a.vis[t0 + i] & ((1u << i) - 1); before; before &= before - 1) advance<L, NV, PC, CHANNEL>(S, st, __ffs(before) - 1, lane, col, part);
             }
-            advance<L, NV, CHANNEL>(S, st, i, lane, col, part);
+            advance<L, NV, PC, CHANNEL>(S, st, i, lane, col, part);
 #pragma unroll
             for (uint32_t p = 0; p < PC; p++) {
 #pragma unroll
@@ -231,29 +272,35 @@ __global__ void __launch_bounds__(4 * L) scan_kernel(const ScanArgs a, uint32_t 
         for (uint32_t j0 = 0; j0 < n; j0 += GROUP) {
             float part[GROUP * PC];
             if (j0 + GROUP <= n) {
+                Token<NV, PC, CHANNEL> t[2];  // the next token's operands are on their way
+                load_token<L, NV, PC, CHANNEL>(t[0], st, j0, lane, col);
 #pragma unroll
-                for (uint32_t u = 0; u < GROUP; u++) advance<L, NV, CHANNEL>(S, st, j0 + u, lane, col, part + PC * u);
+                for (uint32_t u = 0; u < GROUP; u++) {
+                    if (u + 1 < GROUP) load_token<L, NV, PC, CHANNEL>(t[(u + 1) & 1], st, j0 + u + 1, lane, col);
+                    advance<NV, PC, CHANNEL>(S, t[u & 1], part + PC * u);
+                }
             } else {
 #pragma unroll
                 for (uint32_t u = 0; u < GROUP; u++) {
                     if (j0 + u < n) {
-                        advance<L, NV, CHANNEL>(S, st, j0 + u, lane, col, part + PC * u);
+                        advance<L, NV, PC, CHANNEL>(S, st, j0 + u, lane, col, part + PC * u);
                     } else {
 #pragma unroll
                         for (uint32_t p = 0; p < PC; p++) part[PC * u + p] = 0.0f;
                     }
                 }
             }
-            spread_sums<L, GROUP * PC>(part, lane);
+            spread_sums<L, SUMS>(part, lane);
+            if (SUMS < L && lane % (L / SUMS > 0 ? L / SUMS : 1)) continue;  // (another lane has the same sum)
 #pragma unroll
-            for (uint32_t r = 0; r < GROUP * PC / L; r++) {
-                const uint32_t sum = lane * (GROUP * PC / L) + r, j = j0 + sum / PC, p = sum % PC;
+            for (uint32_t r = 0; r < PER; r++) {
+                const uint32_t sum = SUMS < L ? lane * SUMS / L : lane * PER + r, j = j0 + sum / PC, p = sum % PC;
                 if (j < n && p < mine) Y[(i0 + j) * ldy + p] = part[r] + (CHANNEL ? st.s[4 * j] : skip) * st.v[j * COLS + col + p];
             }
         }
         __syncthreads();  // the chunk's place is free
     }
-    if (mine && !a.gen[run.slot].done) store_state<L, NV>(S, home, mine);
+    if (mine && !a.gen[run.slot].done) store_state<L, NV, PC>(S, home, mine);
 }
 
 // grid (heads, caches, runs).
@@ -379,28 +426,27 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const ShiftArgs a, uin
     }
 }
 
-// grid (tokens / TT, heads): the head's w2 and the tokens' hidden rows in shared memory, a channel and TT / 2 tokens a thread at a time.
+// grid (tokens / TT, heads): the head's rows of w2 and the tokens' hidden rows in shared memory, a channel and TT / 2 tokens a thread
+// at a time.
 template <uint32_t TT>
 __global__ void __launch_bounds__(128) decay_kernel(const DecayArgs a, uint32_t n) {
     pdl_start();
     extern __shared__ __align__(16) float sm[];
-    const uint32_t t0 = blockIdx.x * TT, head = blockIdx.y, tid = threadIdx.x, nt = min(TT, n - t0), warp = tid / 32, lane = tid % 32, K = a.heads * a.dim, pitch = a.dim + 1;
-    float *th = sm, *w = sm + TT * a.rank;  // [rank][TT], [rank][pitch]
-    for (uint32_t i = tid; i < TT * a.rank; i += 128) {
-        const uint32_t j = i % a.rank, t = i / a.rank;
-        th[j * TT + t] = t < nt ? tanhf(a.hid[size_t(t0 + t) * a.ldh + j]) : 0.0f;
-    }
+    const uint32_t rp = (a.rank + 3) / 4 * 4, wp = (a.rank + 7) / 8 * 8 + 8;  // the rows' pitches, in floats and in halves
+    const uint32_t t0 = blockIdx.x * TT, head = blockIdx.y, tid = threadIdx.x, nt = min(TT, n - t0), warp = tid / 32, lane = tid % 32, K = a.heads * a.dim;
+    float* th = sm;                                               // [TT][rp]
+    uint16_t* w = reinterpret_cast<uint16_t*>(sm + TT * rp);      // [dim][wp]
+    const float* hid = a.hid + size_t(t0) * a.ldh;
     const uint16_t* w2 = a.w2 + size_t(head) * a.dim * a.rank;
-    if (a.rank % 4 == 0) {
-        for (uint32_t i = 4 * tid; i < a.dim * a.rank; i += 512) {
-            float x[4];
-            load_bf16<4>(x, w2 + i);
-#pragma unroll
-            for (uint32_t u = 0; u < 4; u++) w[(i % a.rank + u) * pitch + i / a.rank] = x[u];
-        }
+    if (a.rank % 8 == 0 && a.ldh % 4 == 0) {
+        for (Walk at(tid, 128, a.rank / 4); at.r < nt; at.next()) cp_async16(th + at.r * rp + 4 * at.c, hid + size_t(at.r) * a.ldh + 4 * at.c);
+        for (Walk at(tid, 128, a.rank / 8); at.r < a.dim; at.next()) cp_async16(w + at.r * wp + 8 * at.c, w2 + at.r * a.rank + 8 * at.c);
     } else {
-        for (uint32_t i = tid; i < a.dim * a.rank; i += 128) w[i % a.rank * pitch + i / a.rank] = bf16_to_f32(w2[i]);
+        for (Walk at(tid, 128, rp); at.r < nt; at.next()) th[at.r * rp + at.c] = at.c < a.rank ? hid[size_t(at.r) * a.ldh + at.c] : 0.0f;
+        for (Walk at(tid, 128, rp); at.r < a.dim; at.next()) w[at.r * wp + at.c] = at.c < a.rank ? w2[at.r * a.rank + at.c] : uint16_t(0);
     }
+    cp_async_commit();
+#pragma unroll 4
     for (uint32_t i = warp; i < nt; i += 4) {
         float s = 0.0f;
         for (uint32_t c = lane; c < a.dim; c += 32) {
@@ -410,21 +456,22 @@ __global__ void __launch_bounds__(128) decay_kernel(const DecayArgs a, uint32_t 
         s = warp_sum(s);
         if (lane == 0) a.bonus[size_t(t0 + i) * a.heads + head] = s;
     }
+    cp_async_wait<0>();
+    __syncthreads();
+    for (uint32_t i = tid; i < TT * rp; i += 128) th[i] = i < nt * rp ? tanhf(th[i]) : 0.0f;
     __syncthreads();
     constexpr uint32_t PER = TT / 2;
     for (uint32_t i = tid; i < 2 * a.dim; i += 128) {
         const uint32_t c = i % a.dim, q0 = i / a.dim * PER;
         if (q0 >= nt) continue;
         float s[PER] = {};
-        for (uint32_t j = 0; j < a.rank; j++) {
-            const float wj = w[j * pitch + c];
+        for (uint32_t j = 0; j < rp; j += 4) {
+            float wj[4];
+            load_bf16<4>(wj, w + c * wp + j);
 #pragma unroll
-            for (uint32_t u = 0; u < PER; u += 4) {
-                const float4 h = *reinterpret_cast<const float4*>(th + j * TT + q0 + u);
-                s[u] = fmaf(wj, h.x, s[u]);
-                s[u + 1] = fmaf(wj, h.y, s[u + 1]);
-                s[u + 2] = fmaf(wj, h.z, s[u + 2]);
-                s[u + 3] = fmaf(wj, h.w, s[u + 3]);
+            for (uint32_t u = 0; u < PER; u++) {
+                const float4 h = *reinterpret_cast<const float4*>(th + (q0 + u) * rp + j);
+                s[u] = fmaf(wj[3], h.w, fmaf(wj[2], h.z, fmaf(wj[1], h.y, fmaf(wj[0], h.x, s[u]))));
             }
         }
         const float w0 = bf16_to_f32(a.w0[head * a.dim + c]);
@@ -480,27 +527,36 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormArgs a)
     }
 }
 
-template <uint32_t L, uint32_t NV, bool CHANNEL>
+template <uint32_t L, uint32_t NV, uint32_t PC, bool CHANNEL, uint32_t GROUP>
 void scan(const ScanArgs& a, cudaStream_t s) {
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(scan_kernel<L, NV, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024)); });
+    auto* kernel = scan_kernel<L, NV, PC, CHANNEL, GROUP>;
+    configured.once([&] { VLT_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024)); });
     const uint32_t slices = (a.c.P + COLS - 1) / COLS;
     constexpr uint32_t NP = 4 * L * NV;
     uint32_t tc = 8;
     while (tc < 32 && tc < a.max_run && 2 * stage_floats<CHANNEL>(NP, 2 * tc) * 4 <= 72 * 1024) tc *= 2;
+    if (a.max_run < tc) tc = a.max_run;
     const size_t smem = size_t(stage_floats<CHANNEL>(NP, tc)) * 4 * (a.max_run > tc ? 2 : 1);
     auto whole = [](const void* p, size_t ld) { return reinterpret_cast<uintptr_t>(p) % 16 == 0 && ld % 4 == 0; };
     const bool aligned = a.c.N % 4 == 0 && a.c.P % 4 == 0 && whole(a.q, a.ldq) && whole(a.k, a.ldk) && whole(a.v, a.ldv) && whole(a.decay, 0);
-    launch_pdl(scan_kernel<L, NV, CHANNEL>, dim3(a.c.heads * slices, a.n_runs), 4 * L, smem, s, a, tc, aligned);
+    launch_pdl(kernel, dim3(a.c.heads * slices, a.n_runs), L * COLS / PC, smem, s, a, tc, aligned);
 }
+// Per pitch: steps of short runs (bound by the states' traffic) with four columns a lane, longer ones (bound by instructions and
+// their latencies) with two and twice the threads.
 struct Kernel {
     uint32_t pitch;
+    void (*short_plain)(const ScanArgs&, cudaStream_t);
+    void (*short_channel)(const ScanArgs&, cudaStream_t);
     void (*plain)(const ScanArgs&, cudaStream_t);
     void (*channel)(const ScanArgs&, cudaStream_t);
 };
-template <uint32_t L, uint32_t NV>
-constexpr Kernel kernel() { return {4 * L * NV, scan<L, NV, false>, scan<L, NV, true>}; }
-static const Kernel kernels[] = {kernel<8, 1>(), kernel<16, 1>(), kernel<32, 1>(), kernel<32, 2>(), kernel<32, 3>(), kernel<32, 4>()};
+static const Kernel kernels[] = {{32, scan<8, 1, 4, false, 1>, scan<8, 1, 4, true, 1>, scan<8, 1, 2, false, 8>, scan<8, 1, 2, true, 8>},
+                                 {64, scan<16, 1, 4, false, 1>, scan<16, 1, 4, true, 1>, scan<16, 1, 2, false, 8>, scan<16, 1, 2, true, 8>},
+                                 {128, scan<32, 1, 4, false, 1>, scan<32, 1, 4, true, 1>, scan<32, 1, 2, false, 8>, scan<32, 1, 2, true, 8>},
+                                 {256, scan<32, 2, 4, false, 1>, scan<32, 2, 4, true, 1>, scan<32, 2, 2, false, 8>, scan<32, 2, 2, true, 8>},
+                                 {384, scan<32, 3, 4, false, 1>, scan<32, 3, 4, true, 1>, scan<32, 3, 2, false, 8>, scan<32, 3, 2, true, 8>},
+                                 {512, scan<32, 4, 4, false, 1>, scan<32, 4, 4, true, 1>, scan<32, 4, 2, false, 8>, scan<32, 4, 2, true, 8>}};
 
 }  // namespace recurrent
 
@@ -508,7 +564,11 @@ void launch_scan(const ScanArgs& a, cudaStream_t s) {
     using namespace recurrent;
     if (!a.n_runs) return;
     for (const Kernel& k : kernels)
-        if (k.pitch == a.c.Np) { (a.c.channel_decay ? k.channel : k.plain)(a, s); return; }
+        if (k.pitch == a.c.Np) {
+            if (a.max_run <= VERIFY_T) (a.c.channel_decay ? k.short_channel : k.short_plain)(a, s);
+            else (a.c.channel_decay ? k.channel : k.plain)(a, s);
+            return;
+        }
     throw Error("internal: a recurrence over " + std::to_string(a.c.N) + " key channels");
 }
 // The key channels a state is laid out for: those of the smallest kernel that takes N.
@@ -536,13 +596,15 @@ void launch_token_shift(const ShiftArgs& a, uint32_t n, cudaStream_t s) {
     if (d % 4 == 0) launch_pdl(recurrent::token_shift_kernel<4>, dim3(n, (d + 1023) / 1024), 256, 0, s, a, n);
     else launch_pdl(recurrent::token_shift_kernel<1>, dim3(n, (d + 255) / 256), 256, 0, s, a, n);
 }
+static size_t decay_smem(size_t tokens, size_t rank, size_t dim) { return tokens * ((rank + 3) / 4 * 4) * 4 + dim * ((rank + 7) / 8 * 8 + 8) * 2; }
+bool decay_fits(uint32_t rank, uint32_t dim) { return decay_smem(32, rank, dim) <= 220 * 1024; }
 void launch_decay(const DecayArgs& a, uint32_t n, cudaStream_t s) {
     static PerDevice configured;
     configured.once([] {
         for (auto f : {recurrent::decay_kernel<8>, recurrent::decay_kernel<32>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     });
     const uint32_t tt = n >= 64 ? 32 : 8;
-    const size_t smem = size_t(a.rank) * (tt + a.dim + 1) * 4;
+    const size_t smem = decay_smem(tt, a.rank, a.dim);
     if (tt == 32) launch_pdl(recurrent::decay_kernel<32>, dim3((n + 31) / 32, a.heads), 128, smem, s, a, n);
     else launch_pdl(recurrent::decay_kernel<8>, dim3((n + 7) / 8, a.heads), 128, smem, s, a, n);
 }

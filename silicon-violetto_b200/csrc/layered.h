@@ -8,6 +8,8 @@
 
 namespace vlt {
 
+bool decay_fits(uint32_t rank, uint32_t dim);  // of a TimeMix (k_recurrent.cu)
+
 // Of rows: x / sqrt(mean x^2 + eps), times the weight (as stored, or stored around zero: 1 + w).
 struct RowNorm {
     const uint16_t* w = nullptr;

@@ -65,7 +65,7 @@ inline void time_mix(LayeredModel& model, const Json& m, const std::string& pre,
     for (const char* c : {"k", "v", "g"}) w.place(pre + c, {K, d}, false);
     model.matrix(t.rkvg, K, d, at);
     t.rank = w.rows(pre + "w1");  // (no key of config.json has it)
-    if (size_t(t.rank) * (t.dim + 33) * 4 > 220 * 1024) throw Error(pre + ": decays of rank " + std::to_string(t.rank) + " over heads of " + std::to_string(t.dim) + " do not fit shared memory");
+    if (!decay_fits(t.rank, t.dim)) throw Error(pre + ": decays of rank " + std::to_string(t.rank) + " over heads of " + std::to_string(t.dim) + " do not fit shared memory");
     model.padded(t.w1, t.rank, d, w.place(pre + "w1", {t.rank, d}));
     model.point(t.w2, pre + "w2", {K, t.rank});
     model.point(t.w0, pre + "w0", {K});
