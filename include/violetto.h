@@ -47,7 +47,7 @@ typedef struct {
     uint32_t flags;            /* VLT_FLAG_* */
 } VltEngineConfig;
 #define VLT_FLAG_HOST_ONLY 1u /* plan only: no device memory, steps cannot run */
-#define VLT_FLAG_FP32 2u      /* everything in 32-bit (model folders of the Lonasun architecture; others refuse it) */
+#define VLT_FLAG_FP32 2u      /* everything in 32-bit (model folders; the other architectures refuse it) */
 
 /* engine/src/engine.rs:59-95 `Tuning`. The reference's Apple-GPU knobs (gpu_cores,
  * splitk_target, decode_split, verify_ki) are replaced by B200 ones; the rows policy is kept. 0 = default. */
@@ -111,7 +111,7 @@ const char* vlt_last_error(void);
 /* Engine::new, engine/src/engine.rs:221-250. `tuning` may be NULL. The weight file is a plain decoder's (its `meta` tensor
  * describes it: the benchmark's models) or one of the reference's own architecture as tools/convert.py:64-114 writes it (no
  * `meta`; engine/src/model.rs:6-20, with the shapes read off the file). A folder with config.json and model.safetensors is
- * loaded by the architecture config.json names (Lonasun; nothing in the reference corresponds to it). */
+ * loaded by the architecture config.json names (Lonasun, Leduvik; nothing in the reference corresponds to them). */
 int vlt_engine_new(const char* weights_path, const VltEngineConfig* cfg, const VltTuning* tuning, VltEngine** out);
 /* Drop for Engine. */
 void vlt_engine_free(VltEngine* e);
@@ -134,8 +134,8 @@ int vlt_step_rows(VltEngine* e, const VltRun* runs, uint32_t n_runs, const uint3
  * (q | k | v after the folded norm and RoPE, fp32: before the rounding to bf16 and q's softmax scale), sdpa_out
  * [attn_width] (the attention's output), attn_out [d_model] (the o projection's output before the residual add), mlp_in
  * [d_model] (the RMS-normed stream after attention), mlp_out [d_model] (the down projection's output before the residual
- * add); resid_base is the reference's MUDD base (NULL for a plain decoder). A Lonasun model hands out resid_in, sdpa_out (the
- * gated attention, attn_width columns) and resid_out (the stream leaving the layer run); the others are NULL there, and
+ * add); resid_base is the reference's MUDD base (NULL for a plain decoder). A folder's model hands out resid_in, sdpa_out (the
+ * attention with its gate, attn_width columns; NULL in a layer without one) and resid_out (the stream leaving the layer run); the others are NULL there, and
  * resid_out is NULL for a plain decoder. */
 typedef struct {
     uint32_t layer, n, d_model, qkv_width, attn_width;
