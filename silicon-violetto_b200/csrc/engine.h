@@ -252,7 +252,7 @@ class Engine {
         Buffer proj, q_f, q_b, attn_f, attn_b;    // a mixer's projections; finished q; what the output projection reads
         Buffer moe_x, moe_xb, ids, weights, src, place, tiles, n_tiles, hid_f, hid_b, rows, sh_f, sh_b, shared;
         Buffer ff_f, ff_b, branch;                // a dense layer's hidden rows; the outputs of mixers side by side
-        Buffer conv, steps, y, mix_f, mix_b, low, decay;  // a recurrence's inputs and outputs
+        Buffer conv, conv_b, steps, y, mix_f, mix_b, low, decay;  // a recurrence's inputs and outputs
         Buffer rings, states, caches, recurrent_dev;      // caches, recurrent_dev: MixerCache, RecurrentCache on the device
         std::vector<Buffer> rope;                 // per distinct rotation: [position][dims / 2] (cos, sin), fp32
         std::vector<MixerCache> run;              // the host's copy of caches

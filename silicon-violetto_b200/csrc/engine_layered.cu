@@ -86,6 +86,7 @@ void Engine::init_layered() {
     h(z.ff_b, n16 * ff);
     f(z.branch, n * branch);
     f(z.conv, n * channels);
+    h(z.conv_b, n * channels);
     f(z.steps, n * heads);
     f(z.y, n * y);
     if (shift) {
@@ -302,7 +303,10 @@ void Engine::encode_state_space(StepSet& st, const Plan& p, const StateSpace& x,
     c.w = x.conv.w;
     c.bias = x.conv.b;
     sp = span_begin(G_SMALL);
-    launch_conv_silu(c, StepSizeArgs{proj + inner + x.channels(), ld, x.heads, x.dt_bias, x.a_log, z.steps.as<float>()}, n, z.conv.as<float>(), stream);
+    // Long runs on the tensor cores take the convolution's outputs in bf16; the others' recurrence takes them as they are.
+    const bool tensor = !cfg.fp32 && !tuning.plain_attention && ssd_fits(x.state, x.vdim) && p.max_run >= SSD_MIN_RUN;
+    launch_conv_silu(c, StepSizeArgs{proj + inner + x.channels(), ld, x.heads, x.dt_bias, x.a_log, z.steps.as<float>()}, n, tensor && p.n_runs == 1 ? nullptr : z.conv.as<float>(),
+                     tensor ? z.conv_b.as<uint16_t>() : nullptr, stream);
     if (!c.write_ring) launch_conv_state(c, st.in<RunIn>(st.o_runs), p.n_runs, stream);
     span_end(sp);
     ScanArgs a{};
@@ -313,6 +317,12 @@ void Engine::encode_state_space(StepSet& st, const Plan& p, const StateSpace& x,
     a.ldq = a.ldk = a.ldv = x.channels();
     a.decay = z.steps.as<float>();
     a.skip = x.skip;
+    if (tensor) {
+        a.v_b = z.conv_b.as<uint16_t>();
+        a.k_b = a.v_b + inner;
+        a.q_b = a.k_b + x.groups * x.state;
+        a.a_log = x.a_log;
+    }
     GatedNormArgs g{};
     g.gate = proj;
     g.ldg = ld;

@@ -6,7 +6,7 @@
 // for the packed fp32 instructions: what a lane reads of q, k and decays serves several columns. Rows come in by asynchronous
 // copies, a chunk of tokens ahead; the output's sums over the lanes are taken for eight tokens at a time, by exchanges that halve
 // what a lane carries. A prompt's portion reads and writes the state once, like a decoded token. A row's result depends on nothing
-// but the rows before it, however they are cut into steps.
+// but the rows before it, however they are cut into steps. (Longer portions of the state space's go to k_ssd.cu.)
 #include <algorithm>
 
 #include "kernels.h"
@@ -188,6 +188,7 @@ __global__ void __launch_bounds__(L * COLS / PC, GROUP == 1 ? 0 : 1) scan_kernel
     const RecurrentCache& c = a.c;
     const uint32_t slices = (c.P + COLS - 1) / COLS, head = blockIdx.x / slices, p0 = blockIdx.x % slices * COLS, tid = threadIdx.x, lane = tid % L, col = tid / L * PC;
     const RunIn run = a.runs[blockIdx.y];
+    if (a.tensor_min && run.count >= a.tensor_min) return;
     const uint32_t t0 = run.first, count = run.count, cols = min(COLS, c.P - p0), mine = col < cols ? min(PC, cols - col) : 0;
     const bool verify = run.verify && count > 1, two = a.max_run > tc;
     const uint32_t stage_len = stage_floats<CHANNEL>(NP, tc);
@@ -337,7 +338,7 @@ __global__ void __launch_bounds__(256) recurrent_fill_kernel(const RecurrentCach
 
 // grid (tokens / TB, spans of 128 channels, and one more for the step sizes).
 template <uint32_t TB>
-__global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs a, const StepSizeArgs st, uint32_t n, float* __restrict__ y) {
+__global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs a, const StepSizeArgs st, uint32_t n, float* __restrict__ y, uint16_t* __restrict__ y_b) {
     pdl_start();
     __shared__ const float* from[TB][32];
     __shared__ float* into[TB];
@@ -380,7 +381,9 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs a, const 
 #pragma unroll
     for (uint32_t i = 0; i < TB; i++) {
         if (i >= nt) break;
-        y[size_t(t0 + i) * a.conv_channels + c] = silu(s[i]);
+        const float v = silu(s[i]);
+        if (y) y[size_t(t0 + i) * a.conv_channels + c] = v;
+        if (y_b) y_b[size_t(t0 + i) * a.conv_channels + c] = f32_to_bf16(v);
         if (a.write_ring) into[i][c] = last[i];
     }
 }
@@ -560,9 +563,16 @@ static const Kernel kernels[] = {{32, scan<8, 1, 4, false, 1>, scan<8, 1, 4, tru
 
 }  // namespace recurrent
 
-void launch_scan(const ScanArgs& a, cudaStream_t s) {
+void launch_scan(const ScanArgs& all, cudaStream_t s) {
     using namespace recurrent;
+    ScanArgs a = all;
     if (!a.n_runs) return;
+    if (a.q_b && a.max_run >= SSD_MIN_RUN) {
+        a.tensor_min = SSD_MIN_RUN;
+        launch_ssd(a, s);
+        if (a.n_runs == 1) return;
+        a.max_run = SSD_MIN_RUN - 1;  // at most, of the runs that are left
+    }
     for (const Kernel& k : kernels)
         if (k.pitch == a.c.Np) {
             if (a.max_run <= VERIFY_T) (a.c.channel_decay ? k.short_channel : k.short_plain)(a, s);
@@ -586,10 +596,10 @@ void launch_recurrent_fill(const RecurrentCache* caches, uint32_t n_caches, uint
     recurrent::recurrent_fill_kernel<<<n_caches, 256, 0, s>>>(caches, slot, seed);
     launch_counter()++;
 }
-void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, float* y, cudaStream_t s) {
+void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, float* y, uint16_t* y_b, cudaStream_t s) {
     const uint32_t spans = (a.conv_channels + 127) / 128 + 1;
-    if (n >= 64) launch_pdl(recurrent::conv_silu_kernel<4>, dim3((n + 3) / 4, spans), 128, 0, s, a, st, n, y);
-    else launch_pdl(recurrent::conv_silu_kernel<1>, dim3(n, spans), 128, 0, s, a, st, n, y);
+    if (n >= 64) launch_pdl(recurrent::conv_silu_kernel<4>, dim3((n + 3) / 4, spans), 128, 0, s, a, st, n, y, y_b);
+    else launch_pdl(recurrent::conv_silu_kernel<1>, dim3(n, spans), 128, 0, s, a, st, n, y, y_b);
 }
 void launch_token_shift(const ShiftArgs& a, uint32_t n, cudaStream_t s) {
     const uint32_t d = a.c.conv_channels;

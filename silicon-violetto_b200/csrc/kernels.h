@@ -353,21 +353,28 @@ struct ScanArgs {
     const uint32_t *meta, *vis;
     uint32_t n_runs, max_run;
     float* y;                // [n][heads P]
+    // Optional, without channel decays, of shapes that ssd_fits takes: the rows in bf16, as q, k and v are laid out. Runs of
+    // SSD_MIN_RUN tokens or more then go to the tensor cores (k_ssd.cu), and only shorter ones read q, k and v.
+    const uint16_t *q_b, *k_b, *v_b, *a_log;
+    uint32_t tensor_min;     // (launch_scan's: runs from here on are the tensor cores')
 };
+constexpr uint32_t SSD_MIN_RUN = 32;
+bool ssd_fits(uint32_t N, uint32_t P);
+void launch_ssd(const ScanArgs& a, cudaStream_t s);
 uint32_t recurrent_pitch(uint32_t N);  // Np
 void launch_scan(const ScanArgs& a, cudaStream_t s);
 // After acceptance: the states of the verified runs advance over the accepted path's rows.
 void launch_recurrent_commit(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const RecurrentCache* caches, uint32_t n_runs,
                              uint32_t n_caches, uint32_t max_heads, cudaStream_t s);
 void launch_recurrent_fill(const RecurrentCache* caches, uint32_t n_caches, uint32_t slot, uint32_t seed, cudaStream_t s);
-// y[t][c] = silu(bias + convolution) for a.conv_channels channels, and per head softplus(dt + dt_bias) and exp(-exp(a_log) of that).
+// y[t][c] = silu(bias + convolution) for a.conv_channels channels, fp32 and / or bf16, and per head softplus(dt + dt_bias) and exp(-exp(a_log) of that).
 struct StepSizeArgs {
     const float* dt;         // [n][ld]
     uint32_t ld, heads;
     const uint16_t *bias, *a_log;
     float* out;              // [n][heads][2]
 };
-void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, float* y, cudaStream_t s);
+void launch_conv_silu(const ConvArgs& a, const StepSizeArgs& st, uint32_t n, float* y, uint16_t* y_b, cudaStream_t s);
 // Row t's mixes with the row before it, h + (h' - h) mu, five of them: [mix][n][channels], fp32 and / or bf16, the last mu's
 // first. tiles: the grouped projection's table over the four behind it (group, first row, rows), `tile` rows at most.
 struct ShiftArgs {

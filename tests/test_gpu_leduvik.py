@@ -86,6 +86,35 @@ def test_step_sizes_and_decays_at_their_ends(fp32):
         eng.close()
 
 
+@pytest.mark.parametrize("edit", ["", "memory", "ends"])
+def test_state_space_chunks_on_the_tensor_cores(edit):
+    """Portions around the lengths from which the tensor cores take a run, and around their chunks of 64, beside the recurrence
+    token by token (Tuning.plain_attention) and the restatement; short runs of other requests in the same step."""
+    def ends(cfg, bits):
+        for i, lc in enumerate(cfg["layers"]):
+            n = lc["mixer"]["heads"]
+            pick = lambda a, b: lv.to_bf16(np.where(np.arange(n) % 2, a, b).astype(np.float32))
+            bits[f"l{i}.mix.dt_bias"], bits[f"l{i}.mix.A_log"] = pick(0.0, -3.0), pick(4.0, -9.0)  # decays of 1e-12 and of almost 1
+            bits[f"l{i}.mix.D"] = lv.to_bf16(np.full(n, 3.0, np.float32))  # (no output is a small difference, which bf16 would blur)
+    cfg = lv.config(128, 160, [lv.state_space(4, 64, 128, groups=2, norm_groups=2), lv.state_space(6, 32, 64, groups=1, norm_groups=1, conv=2)])
+    bits = lv.random_weights(cfg, 21)
+    {"": lambda c, b: None, "memory": lu.long_memory, "ends": ends}[edit](cfg, bits)
+    folder = lv.write_model(lu._TMP / f"chunks_{edit}", cfg, bits)
+    w = {k: lv.from_bf16(v).astype(np.float64) for k, v in bits.items()}
+    toks, other = prompt(cfg, 300, 6), prompt(cfg, 40, 7)
+    want, want_other = ref.forward(cfg, w, toks)[0], ref.forward(cfg, w, other)[0]
+    fast, plain = lu.engine(folder, False), lu.engine(folder, False, tuning=E.Tuning(plain_attention=True))
+    for sizes in ([300], [31, 32, 33], [64, 1, 63, 65, 2], [1, 127, 129], [200, 100]):
+        got = cut(fast, toks, sizes)
+        close(got, want, False, 0.5)
+        close(got, cut(plain, toks, sizes), False, 0.5)
+    got = lu.replay(fast, {"a": toks, "b": other}, [[("a", 100), ("b", 3)], [("b", 30), ("a", 33)], [("b", 1), ("a", 167)], [("b", 6)]])
+    close(got["a"], want, False, 0.5)
+    close(got["b"], want_other, False, 0.5)
+    fast.close()
+    plain.close()
+
+
 # ---- whole prompts, decoding, portions, batches
 @BOTH
 @pytest.mark.parametrize("name", ["odd", "fast"] + SINGLE)
