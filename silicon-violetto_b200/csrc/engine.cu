@@ -136,7 +136,8 @@ Engine::Engine(const std::string& weights, const EngineConfig& c, const Tuning& 
         std::vector<KvShape> shapes;  // a slice per (layer run, mixer), of no bytes for one without keys
         for (const LayerRun& r : model.layered->runs)
             for (const Mixer& x : model.layered->layers[r.layer].mix)
-                shapes.push_back(x.kind == MixerKind::Attention ? KvShape{x.attn.kv_heads, x.attn.dim, x.attn.vdim} : KvShape{0, 0, 0});
+                shapes.push_back(x.kind == MixerKind::Attention ? KvShape{x.attn.kv_heads, x.attn.dim, x.attn.vdim}
+                                 : x.kind == MixerKind::Latent && x.latent.kv_w() ? KvShape{1, x.latent.key_w(), 0} : KvShape{0, 0, 0});
         kv.init(cfg, md.page, shapes, cfg.fp32 ? 4 : 2, !cfg.host_only);
     } else {
         kv.init(cfg, md.page, std::vector<KvShape>(model.limite ? model.n_global : md.n_layers, {md.n_kv, md.hd, md.hd}), 2, !cfg.host_only);  // (the reference's architecture pages its global layers only)
@@ -465,7 +466,7 @@ void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint3
     a.epi = epi;
     a.vocab_real = vocab_real ? vocab_real : model.md.vocab_real;
     a.eps = model.md.eps;
-    const uint32_t out_w = epi == EPI_SWIGLU ? w.m / 2 : w.m;
+    const uint32_t out_w = epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 8) {
         a.n = std::min(8u, n - t0);
         a.t0 = t0;
@@ -538,7 +539,7 @@ void Engine::matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float*
     // The kernel's N is at most 256 tokens: a longer step (a prompt chunk) goes in blocks of 256, the weights read once per
     // block (the reference's tiled GEMM loops its token tiles the same way, kernels.metal:319-514). Everything indexed by
     // token moves along with the block.
-    const uint32_t out_w = epi == EPI_SWIGLU ? w.m / 2 : w.m;
+    const uint32_t out_w = epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 256) {
         MatArgs b = a;
         b.n = std::min(256u, n - t0);
@@ -939,7 +940,7 @@ void Engine::begin_step(uint32_t set, const Plan& p) {
     const LayeredModel* lm = model.layered.get();
     launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), lm ? lay->x0.as<float>() : s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
                  s.feed.as<uint32_t>(), s.tree.as<uint32_t>(), st.in<uint32_t>(st.o_vis), p.n, model.md.d, model.md.vocab, stream, lm ? lm->positions : nullptr,
-                 lm ? lm->n_positions : 0);
+                 lm ? lm->n_positions : 0, lm && lm->layers[0].post_norm && !cfg.fp32 ? lay->xn_b.as<uint16_t>() : nullptr);
 }
 
 // engine/src/engine/encode.rs:439-451 `encode_replay`.

@@ -248,10 +248,12 @@ class Engine {
     };
     // A model folder's layers (model.layered): caches per (layer run, mixer) beside the paged pool, and scratch.
     struct LayeredState {
-        Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding; a norm's rows; (stream ; embedding)
+        Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding; a norm's rows, or the stream's in bf16; (stream ; embedding)
         Buffer proj, q_f, q_b, attn_f, attn_b;    // a mixer's projections; finished q; what the output projection reads
         Buffer moe_x, moe_xb, ids, weights, src, place, tiles, n_tiles, hid_f, hid_b, rows, sh_f, sh_b, shared;
-        Buffer ff_f, ff_b, branch;                // a dense layer's hidden rows; the outputs of mixers side by side
+        Buffer ff_f, ff_b, branch;                // a dense layer's hidden rows; the outputs of mixers side by side, or of a sublayer with a norm behind it
+        Buffer lat_f, lat_b, uq, part_f, part_b, mid_f, mid_b;  // latent attention: the query row, W_uq's product, its unrotated parts, the sums of c
+        Buffer side, side_f, side_b, row_weight, decays;  // a side input's rows before and behind its gate; experts' sorted scores; fixed decays
         Buffer conv, conv_b, steps, y, mix_f, mix_b, low, decay;  // a recurrence's inputs and outputs
         Buffer rings, states, caches, recurrent_dev;      // caches, recurrent_dev: MixerCache, RecurrentCache on the device
         std::vector<Buffer> rope;                 // per distinct rotation: [position][dims / 2] (cos, sin), fp32
@@ -259,22 +261,27 @@ class Engine {
         std::vector<uint32_t> first;              // a layer run's first entry in it
         std::vector<RecurrentCache> recurrent;
         uint32_t max_heads = 0;                   // of a recurrence
+        const float* in_f = nullptr;              // what the sublayer being queued reads, in fp32 (in bf16: xn_b)
     };
     static constexpr uint32_t EXPERT_TILE_MIN = 16;  // rows of an expert per tile, at least
     static constexpr uint32_t SHIFT_TILE_MIN = 16;   // tokens of a mix per tile, at least
     std::unique_ptr<LayeredState> lay;
     void init_layered();
     void encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm);
+    void encode_side(StepSet& st, const SideInput& x, uint32_t n);
+    void add_norm(const float* x, const RowNorm& norm, uint32_t n);
     ConvArgs conv_args(StepSet& st, const Plan& p, const MixerCache& mc, const float* u, uint32_t ldu, uint32_t taps);
     void mixer_out(const Matrix& o, uint32_t n, const float* cur, float* alone);
     void encode_attention(StepSet& st, const Plan& p, const Attention& a, const MixerCache& mc, const float* cur, float* alone, bool capture);
     void encode_recurrence(StepSet& st, const Plan& p, ScanArgs& a, GatedNormArgs& g);
     void encode_state_space(StepSet& st, const Plan& p, const StateSpace& x, const MixerCache& mc, const float* cur, float* alone);
+    void encode_latent(StepSet& st, const Plan& p, const LatentAttention& a, const MixerCache& mc, float* alone, bool capture);
+    void encode_linear(StepSet& st, const Plan& p, const LinearAttention& x, const MixerCache& mc, float* alone);
     void encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const MixerCache& mc, const float* cur, float* alone);
     void encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
     // Y = epilogue(W x) in the engine's precision: xf in an fp32 engine, else xb through the GEMM, the streamed matmul or,
     // for sizes neither takes, the CUDA cores.
-    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr);
+    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr, uint32_t act_rows = 0);
     std::unique_ptr<LimiteState> lim;
     LimiteKv limite_kv(const LimiteLayer& x) const;
     void encode_forward_limite(uint32_t set, const Plan& p);

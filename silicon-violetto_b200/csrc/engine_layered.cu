@@ -14,9 +14,13 @@ void Engine::init_layered() {
     const bool f32 = cfg.fp32;
     const size_t n = cfg.max_step_tokens, n16 = (n + 15) / 16 * 16, d = md.d;
     size_t proj = 0, q = 0, out = 0, pairs = 0, hid = 0, sff = 0, tiles = 0, top = 0, rows = 0, ff = 0, branch = 0, channels = 0, y = 0, inner = 0, heads = 0, low = 0;
+    size_t halves = 0, lat = 0, uq = 0, part = 0, mid = 0, side = 0, side_wide = 0, fixed = 0;
     bool shift = false;
     for (const FolderLayer& l : m.layers) {
         if (l.mix.size() > 1) branch = 2 * d;
+        else if (l.post_norm) branch = std::max(branch, d);
+        side = std::max<size_t>(side, l.side.gate.m);
+        side_wide = std::max<size_t>(side_wide, l.side.proj.k);
         for (const Mixer& x : l.mix) {
             if (x.kind == MixerKind::Attention) {
                 proj = std::max<size_t>(proj, x.attn.proj.m);
@@ -28,6 +32,22 @@ void Engine::init_layered() {
                 y = std::max<size_t>(y, x.ssm.inner());
                 out = std::max<size_t>(out, x.ssm.inner());
                 heads = std::max<size_t>(heads, 2 * x.ssm.heads);
+            } else if (x.kind == MixerKind::Latent) {
+                const LatentAttention& a = x.latent;
+                proj = std::max<size_t>(proj, a.in.m);
+                q = std::max<size_t>(q, a.heads * a.key_w());
+                out = std::max<size_t>(out, a.out_w());
+                lat = std::max<size_t>(lat, a.q_rank);
+                uq = std::max<size_t>(uq, a.uq.m);
+                part = std::max<size_t>(part, a.heads * a.dim);
+                mid = std::max<size_t>(mid, a.heads * a.kv_rank);
+                tiles = std::max<size_t>(tiles, a.heads * (n / SHIFT_TILE_MIN + 1));
+            } else if (x.kind == MixerKind::Linear) {
+                proj = std::max<size_t>(proj, x.linear.proj.m);
+                halves = std::max<size_t>(halves, x.linear.proj.m);
+                y = std::max<size_t>(y, x.linear.out_w());
+                out = std::max<size_t>(out, x.linear.out_w());
+                fixed += x.linear.heads;
             } else {
                 shift = true;
                 proj = std::max<size_t>(proj, 4 * x.tmix.inner());
@@ -39,7 +59,7 @@ void Engine::init_layered() {
                 tiles = std::max<size_t>(tiles, 4 * (n / SHIFT_TILE_MIN + 1));
             }
         }
-        if (l.mlp == MlpKind::Dense) ff = std::max<size_t>(ff, l.dense.up.m);
+        if (l.mlp == MlpKind::Dense) ff = std::max<size_t>(ff, l.dense.down.k);
         if (l.mlp != MlpKind::Experts) continue;
         const ExpertLayer& e = l.experts;
         const size_t p = n * e.top;
@@ -79,14 +99,25 @@ void Engine::init_layered() {
         w(z.sh_f, n * sff);
         h(z.sh_b, n16 * sff);
         f(z.shared, n * d);
+        f(z.row_weight, pairs);
     }
+    w(z.lat_f, n * lat);
+    h(z.lat_b, n16 * lat);
+    f(z.uq, n * uq);
+    w(z.part_f, n * part);
+    h(z.part_b, n16 * part);
+    w(z.mid_f, n * mid);
+    h(z.mid_b, n16 * mid);
+    f(z.side, n * side);
+    w(z.side_f, n * side_wide);
+    h(z.side_b, n16 * side_wide);
     f(z.tiles, 3 * tiles);
     f(z.n_tiles, 1);
     w(z.ff_f, n * ff);
     h(z.ff_b, n16 * ff);
     f(z.branch, n * branch);
     f(z.conv, n * channels);
-    h(z.conv_b, n * channels);
+    h(z.conv_b, n * std::max(channels, halves));
     f(z.steps, n * heads);
     f(z.y, n * y);
     if (shift) {
@@ -100,7 +131,7 @@ void Engine::init_layered() {
         const uint32_t npos = cfg.max_seq_len + FEED_W, half = r.dims / 2;
         std::vector<float> tab(size_t(npos) * half * 2);
         for (uint32_t i = 0; i < half; i++) {
-            const double freq = std::pow(r.base, -2.0 * i / r.dims);
+            const double freq = std::pow(r.base, -2.0 * i / r.dims) / r.factor;
             for (uint32_t p = 0; p < npos; p++) {
                 tab[(size_t(p) * half + i) * 2] = float(std::cos(p * freq));
                 tab[(size_t(p) * half + i) * 2 + 1] = float(std::sin(p * freq));
@@ -113,8 +144,14 @@ void Engine::init_layered() {
     // Per (layer run, mixer): its pages; a ring per slot of the rows a convolution or shift reaches back over, and room for a
     // verified run past them; a recurrence's state per slot and what a verified run leaves for it.
     uint32_t page_shift = 0;
+    std::vector<bool> shared;  // per cache: its pages are another's, which are compacted and filled there
     while ((1u << page_shift) < md.page) page_shift++;
     const size_t es = f32 ? 4 : 2;
+    std::vector<float> decays;  // of the layers with fixed ones, one after the other
+    for (const FolderLayer& l : m.layers)
+        for (const Mixer& x : l.mix) decays.insert(decays.end(), x.linear.decay.begin(), x.linear.decay.end());
+    f(z.decays, std::max<size_t>(fixed, 1));
+    if (fixed) z.decays.write_vec(0, decays);
     size_t ring = 0, state = 0;
     for (int pass = 0; pass < 2; pass++) {  // sizes, then addresses
         float *rings = z.rings.as<float>(), *states = z.states.as<float>();
@@ -128,25 +165,42 @@ void Engine::init_layered() {
         z.run.clear();
         z.first.clear();
         z.recurrent.clear();
+        std::vector<uint32_t> last(m.layers.size());  // a layer's first cache in its latest run so far
+        shared.clear();
         for (const LayerRun& r : m.runs) {
             z.first.push_back(i);
+            last[r.layer] = i;
             for (const Mixer& x : m.layers[r.layer].mix) {
                 MixerCache c{};
+                shared.push_back(x.kind == MixerKind::Latent && x.latent.kv_from != LatentAttention::OWN);
                 if (x.kind == MixerKind::Attention) {
                     const Attention& a = x.attn;
                     c.kv = PagedKv{kv.k.as<uint8_t>() + kv.k_off[i] * es, kv.v.as<uint8_t>() + kv.v_off[i] * es, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, a.kv_heads, a.dim, a.vdim};
                     if (a.conv.w) { c.channels = a.conv.channels; c.ring_len = a.conv.taps - 1 + VERIFY_T; }
+                } else if (x.kind == MixerKind::Latent) {
+                    const LatentAttention& a = x.latent;
+                    void* keys = kv.k.as<uint8_t>() + kv.k_off[i] * es;
+                    c.kv = PagedKv{keys, keys, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, 1, a.key_w(), a.kv_rank};
+                    if (shared.back()) c.kv = z.run[last[a.kv_from]].kv;
                 } else {
-                    const bool tm = x.kind == MixerKind::TimeMix;
-                    c.channels = tm ? md.d : x.ssm.channels();
-                    c.ring_len = (tm ? 2 : x.ssm.conv.taps) - 1 + VERIFY_T;
+                    const bool tm = x.kind == MixerKind::TimeMix, lin = x.kind == MixerKind::Linear;
+                    if (!lin) {
+                        c.channels = tm ? md.d : x.ssm.channels();
+                        c.ring_len = (tm ? 2 : x.ssm.conv.taps) - 1 + VERIFY_T;
+                    }
                     RecurrentCache rc{};
-                    rc.heads = tm ? x.tmix.heads : x.ssm.heads;
-                    rc.per = tm ? 1 : x.ssm.heads / x.ssm.groups;
-                    rc.N = tm ? x.tmix.dim : x.ssm.state;
+                    rc.heads = lin ? x.linear.heads : tm ? x.tmix.heads : x.ssm.heads;
+                    rc.per = tm || lin ? 1 : x.ssm.heads / x.ssm.groups;
+                    rc.N = lin ? x.linear.dim : tm ? x.tmix.dim : x.ssm.state;
                     rc.Np = recurrent_pitch(rc.N);
-                    rc.P = tm ? x.tmix.dim : x.ssm.vdim;
+                    rc.P = lin ? x.linear.vdim : tm ? x.tmix.dim : x.ssm.vdim;
                     rc.channel_decay = tm;
+                    if (lin) {
+                        size_t before = 0;  // the decays of the layers in front
+                        for (uint32_t j = 0; j < r.layer; j++)
+                            for (const Mixer& y : m.layers[j].mix) before += y.linear.decay.size();
+                        rc.fixed = z.decays.as<float>() + before;
+                    }
                     const size_t kept = size_t(cfg.max_seqs) * VERIFY_T;
                     rc.state = take(size_t(cfg.max_seqs) * rc.heads * rc.P * rc.Np);
                     rc.keep_k = take(kept * (rc.heads / rc.per) * rc.N);
@@ -168,29 +222,33 @@ void Engine::init_layered() {
         }
     }
     z.caches.alloc(z.run.size() * sizeof(MixerCache), false);
-    z.caches.write_vec(0, z.run);
+    std::vector<MixerCache> listed = z.run;
+    for (size_t j = 0; j < listed.size(); j++)
+        if (shared[j]) listed[j].kv.n_kv = 0;
+    z.caches.write_vec(0, listed);
     if (z.recurrent.empty()) return;
     z.recurrent_dev.alloc(z.recurrent.size() * sizeof(RecurrentCache), false);
     z.recurrent_dev.write_vec(0, z.recurrent);
 }
 
-void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base) {
+void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, uint32_t act_rows) {
     const bool gemm = !cfg.fp32 && w.m % 128 == 0 && w.k % 64 == 0, stream_takes = !cfg.fp32 && stream_fits(w, n);
     if (gemm && (gemm_fits(w, n) || !stream_takes)) {  // (few rows that are too long for the streamed kernel's shared memory, too)
-        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr);
+        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr, act_rows);
     } else if (stream_takes) {
-        matmul(w, n, nullptr, y, epi, base, nullptr, 0, nullptr, xb, yb);
+        matmul(w, n, nullptr, y, epi, base, nullptr, act_rows, nullptr, xb, yb);
     } else {
         LinearArgs a{};
         a.W = reinterpret_cast<const uint16_t*>(w.w);
         a.X = cfg.fp32 ? static_cast<const void*>(xf) : xb;
         a.base = base;
         a.Y = y;
-        a.Yb = yb;
+        a.Yb = cfg.fp32 ? nullptr : yb;
         a.n = n;
         a.m = w.m;
         a.k = w.k;
         a.epi = epi;
+        a.act_rows = act_rows;
         launch_linear(a, !cfg.fp32, stream);
     }
 }
@@ -224,7 +282,7 @@ void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, co
     const uint32_t n = p.n;
     const bool f32 = cfg.fp32;
     int sp = span_begin(G_MATMUL);
-    project(a.proj, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), z.proj.as<float>(), nullptr, EPI_RAW);
+    project(a.proj, n, z.in_f, z.xn_b.as<uint16_t>(), z.proj.as<float>(), nullptr, EPI_RAW);
     span_end(sp);
     ConvArgs c = conv_args(st, p, mc, z.proj.as<float>(), a.proj.m, a.conv.w ? a.conv.taps : 1);
     c.w = a.conv.w;
@@ -233,6 +291,9 @@ void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, co
     c.heads = a.heads;
     c.rot_dims = a.rot.dims;
     c.unit_qk = a.unit_qk;
+    c.neighbours = a.rot.neighbours;
+    c.q_norm = a.q_norm;
+    c.k_norm = a.k_norm;
     c.unit_eps = model.md.eps;
     c.temp = a.temp;
     const bool fast_attn = !f32 && !tuning.plain_attention && chunk_attn_fits(a.dim, a.vdim, model.md.page);
@@ -257,6 +318,7 @@ void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, co
     at.chunk = a.chunk;
     at.window = a.window;
     at.scale = a.scale;
+    at.softcap = a.softcap;
     at.out = f32 || capture ? z.attn_f.as<float>() : nullptr;
     at.out_b = z.attn_b.as<uint16_t>();
     uint32_t most = p.max_keys;  // keys a row may see
@@ -297,7 +359,7 @@ void Engine::encode_state_space(StepSet& st, const Plan& p, const StateSpace& x,
     const uint32_t n = p.n, inner = x.inner(), ld = x.in.m;
     float* proj = z.proj.as<float>();
     int sp = span_begin(G_MATMUL);
-    project(x.in, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), proj, nullptr, EPI_RAW);
+    project(x.in, n, z.in_f, z.xn_b.as<uint16_t>(), proj, nullptr, EPI_RAW);
     span_end(sp);
     ConvArgs c = conv_args(st, p, mc, proj + inner, ld, x.conv.taps);
     c.w = x.conv.w;
@@ -340,7 +402,7 @@ void Engine::encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const
     // r, k, v and g are one grouped product over the four mixes they read.
     const bool fast = !f32 && grouped_fits(K, d);
     ShiftArgs sh{};
-    sh.c = conv_args(st, p, mc, z.xn_f.as<float>(), d, 2);
+    sh.c = conv_args(st, p, mc, z.in_f, d, 2);
     for (int i = 0; i < 5; i++) sh.mu[i] = x.mu[i];
     sh.out_f32 = z.mix_f.as<float>();
     sh.out_bf16 = z.mix_b.as<uint16_t>();
@@ -403,6 +465,190 @@ void Engine::encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const
     mixer_out(x.o, n, cur, alone);
 }
 
+// Latent attention: the per-head matrices on the queries' side and on the sums' side, so that all heads read the rows the cache holds.
+void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x, const MixerCache& mc, float* alone, bool capture) {
+    LayeredState& z = *lay;
+    const uint32_t n = p.n;
+    const bool f32 = cfg.fp32;
+    float* proj = z.proj.as<float>();
+    int sp = span_begin(G_MATMUL);
+    project(x.in, n, z.in_f, z.xn_b.as<uint16_t>(), proj, nullptr, EPI_RAW);
+    span_end(sp);
+    LatentRowsArgs r{};
+    r.u = proj;
+    r.ldu = x.in.m;
+    r.q_norm = x.q_norm;
+    r.kv_norm = x.kv_norm;
+    r.rope = z.rope[x.rot.table].as<float>();
+    r.meta = s.meta.as<uint32_t>();
+    r.tin = st.in<uint32_t>(st.o_tin);
+    r.kv = mc.kv;
+    r.q_f = f32 ? z.lat_f.as<float>() : nullptr;
+    r.q_b = f32 ? nullptr : z.lat_b.as<uint16_t>();
+    r.q_rank = x.q_rank;
+    r.kv_rank = x.kv_rank;
+    r.rot_dim = x.rot_dim;
+    r.own = x.kv_from == LatentAttention::OWN;
+    r.neighbours = x.rot.neighbours;
+    r.eps = model.md.eps;
+    sp = span_begin(G_SMALL);
+    launch_latent_rows(r, n, f32, stream);
+    span_end(sp);
+    sp = span_begin(G_MATMUL);
+    project(x.uq, n, z.lat_f.as<float>(), z.lat_b.as<uint16_t>(), z.uq.as<float>(), nullptr, EPI_RAW);
+    span_end(sp);
+    const bool fast_attn = !f32 && !tuning.plain_attention && latent_attn_fits(x.kv_rank, x.rot_dim, model.md.page);
+    const bool fast_q = !f32 && grouped_fits(x.kv_rank, x.dim), fast_v = !f32 && grouped_fits(x.vdim, x.kv_rank);
+    LatentQueryArgs q{};
+    q.u = z.uq.as<float>();
+    q.ldu = x.uq.m;
+    q.rope = r.rope;
+    q.meta = r.meta;
+    q.part_f = f32 ? z.part_f.as<float>() : nullptr;
+    q.part_b = f32 ? nullptr : z.part_b.as<uint16_t>();
+    q.q_f = fast_attn ? nullptr : z.q_f.as<float>();
+    q.q_b = fast_attn ? z.q_b.as<uint16_t>() : nullptr;
+    q.tiles = z.tiles.as<uint32_t>();
+    q.n_tiles = z.n_tiles.as<uint32_t>();
+    q.n = n;
+    q.heads = x.heads;
+    q.dim = x.dim;
+    q.rot_dim = x.rot_dim;
+    q.kv_rank = x.kv_rank;
+    q.tile = 64;
+    if (fast_q && fast_v)
+        for (q.tile = SHIFT_TILE_MIN; q.tile < 128 && q.tile < n;) q.tile *= 2;
+    else if (fast_q || fast_v)
+        for (q.tile = SHIFT_TILE_MIN; q.tile < 64 && q.tile < n;) q.tile *= 2;  // (a tile of the CUDA cores has 64 rows at most)
+    q.neighbours = x.rot.neighbours;
+    q.factor = fast_attn ? x.scale * LOG2E : 1.0f;
+    sp = span_begin(G_SMALL);
+    launch_latent_query(q, stream);
+    span_end(sp);
+    LinearArgs l{};  // W_uk^T on a head's query: in front of the rotated part
+    l.W = reinterpret_cast<const uint16_t*>(x.uk_t.w);
+    l.X = f32 ? static_cast<const void*>(q.part_f) : q.part_b;
+    l.Y = q.q_f;
+    l.Yb = q.q_b;
+    l.m = x.kv_rank;
+    l.k = x.dim;
+    l.epi = EPI_RAW;
+    l.tiles = q.tiles;
+    l.n_tiles = q.n_tiles;
+    l.max_tiles = x.heads * ((n + q.tile - 1) / q.tile);
+    l.by_head = n;
+    l.heads = x.heads;
+    l.ldy = x.key_w();
+    sp = span_begin(G_MATMUL);
+    if (fast_q) launch_grouped(l, x.heads, q.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(l, !f32, stream);
+    span_end(sp);
+    ChunkedAttnArgs at{};
+    at.q_f = q.q_f;
+    at.q_b = q.q_b;
+    at.ctiles = st.in<uint32_t>(st.o_ctiles);
+    at.meta = r.meta;
+    at.tin = r.tin;
+    at.vis = st.in<uint32_t>(st.o_vis);
+    at.kv = mc.kv;
+    at.heads = x.heads;
+    at.scale = x.scale;
+    at.out = f32 ? z.mid_f.as<float>() : nullptr;
+    at.out_b = f32 ? nullptr : z.mid_b.as<uint16_t>();
+    sp = span_begin(G_ATTN);
+    if (fast_attn) launch_attn_latent(at, n, p.chunked ? p.ctiles : 0, p.max_keys, sm_count, tuning.attn_keys_per_cta, stream);
+    else launch_attn_any(at, n, f32, stream);
+    span_end(sp);
+    l.W = reinterpret_cast<const uint16_t*>(x.uv.w);  // W_uv on a head's sum of c, and the gate
+    l.X = f32 ? static_cast<const void*>(at.out) : at.out_b;
+    l.Y = f32 || capture ? z.attn_f.as<float>() : nullptr;
+    l.Yb = f32 ? nullptr : z.attn_b.as<uint16_t>();
+    l.m = x.vdim;
+    l.k = x.kv_rank;
+    l.ldy = x.vdim;
+    l.gate = proj + x.q_rank + x.kv_w();
+    l.ldg = x.in.m;
+    sp = span_begin(G_MATMUL);
+    if (fast_v) launch_grouped(l, x.heads, q.tile, s.err_flag.as<uint32_t>(), stream);
+    else launch_linear(l, !f32, stream);
+    span_end(sp);
+    mixer_out(x.o, n, nullptr, alone);
+}
+
+void Engine::encode_linear(StepSet& st, const Plan& p, const LinearAttention& x, const MixerCache& mc, float* alone) {
+    LayeredState& z = *lay;
+    const uint32_t n = p.n, ld = x.proj.m;
+    float* proj = z.proj.as<float>();
+    // Long runs on the tensor cores take q, k and v in bf16; the others' recurrence takes them as they are.
+    bool tensor = !cfg.fp32 && !tuning.plain_attention && ssd_fits(x.dim, x.vdim) && p.max_run >= SSD_MIN_RUN;
+    for (float d : x.decay) tensor = tensor && d > 0 && d <= 1;  // (products of decays by sums of logarithms that are not positive)
+    int sp = span_begin(G_MATMUL);
+    project(x.proj, n, z.in_f, z.xn_b.as<uint16_t>(), proj, tensor ? z.conv_b.as<uint16_t>() : nullptr, EPI_SILU, nullptr, x.qkv_w());
+    span_end(sp);
+    ScanArgs a{};
+    a.c = z.recurrent[mc.recurrent];
+    a.q = proj;
+    a.k = a.q + x.heads * x.dim;
+    a.v = a.k + x.heads * x.dim;
+    a.ldq = a.ldk = a.ldv = ld;
+    if (tensor) {
+        a.q_b = z.conv_b.as<uint16_t>();
+        a.k_b = a.q_b + x.heads * x.dim;
+        a.v_b = a.k_b + x.heads * x.dim;
+    }
+    GatedNormArgs g{};
+    g.gate = proj + x.qkv_w();
+    g.ldg = ld;
+    g.w = x.norm.w;
+    g.groups = 1;
+    g.sigmoid = true;
+    encode_recurrence(st, p, a, g);
+    mixer_out(x.o, n, nullptr, alone);
+}
+
+// The stream h = x + the norm of what the sublayer has left in `branch`, and its bf16 rows for the next one.
+void Engine::add_norm(const float* x, const RowNorm& norm, uint32_t n) {
+    LayeredState& z = *lay;
+    AddNormArgs a{};
+    a.x = x;
+    a.y = z.branch.as<float>();
+    a.norm = norm;
+    a.out = s.h.as<float>();
+    a.out_b = cfg.fp32 ? nullptr : z.xn_b.as<uint16_t>();
+    a.n = n;
+    a.d = model.md.d;
+    a.eps = model.md.eps;
+    const int sp = span_begin(G_SMALL);
+    launch_add_norm(a, stream);
+    span_end(sp);
+}
+
+void Engine::encode_side(StepSet& st, const SideInput& x, uint32_t n) {
+    LayeredState& z = *lay;
+    int sp = span_begin(G_MATMUL);
+    project(x.gate, n, z.in_f, z.xn_b.as<uint16_t>(), z.side.as<float>(), nullptr, EPI_RAW);
+    span_end(sp);
+    SideGateArgs g{};
+    g.x = z.side.as<float>();
+    g.ldx = x.gate.m;
+    g.table = model.layered->side;
+    g.ld = model.layered->side_w;
+    g.tokens = st.in<uint32_t>(st.o_tokens);
+    g.out_f32 = cfg.fp32 ? z.side_f.as<float>() : nullptr;
+    g.out_bf16 = cfg.fp32 ? nullptr : z.side_b.as<uint16_t>();
+    g.n = n;
+    g.first = x.first;
+    g.dim = x.dim;
+    g.wide = x.proj.k;
+    sp = span_begin(G_SMALL);
+    launch_side_gate(g, stream);
+    span_end(sp);
+    sp = span_begin(G_MATMUL);
+    project(x.proj, n, g.out_f32, g.out_bf16, z.branch.as<float>(), nullptr, EPI_RAW);
+    span_end(sp);
+    add_norm(s.h.as<float>(), x.norm, n);
+}
+
 void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture) {
     const LayeredModel& m = *model.layered;
     const ModelDesc& md = model.md;
@@ -441,7 +687,8 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
         }
         std::vector<float> resid_in, sdpa;
         uint32_t attn_width = 0;
-        if (!normed) {
+        z.in_f = l.post_norm ? cur : z.xn_f.as<float>();
+        if (!normed && !l.post_norm) {
             na.in = cur;
             na.add = m.runs[ri].add_embed ? z.x0.as<float>() : nullptr;
             na.sum = h;
@@ -453,18 +700,20 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
             na.add = nullptr;
         }
         if (capture) resid_in = host(cur, size_t(n) * d);
-        const bool several = l.mix.size() > 1;
+        const bool several = l.mix.size() > 1, own = several || l.post_norm;  // own: a mixer's output goes to a place of its own
         for (uint32_t b = 0; b < l.mix.size(); b++) {
             const Mixer& x = l.mix[b];
             const MixerCache& mc = z.run[z.first[ri] + b];
-            float* alone = several ? z.branch.as<float>() + size_t(b) * n * d : nullptr;
+            float* alone = own ? z.branch.as<float>() + size_t(b) * n * d : nullptr;
             switch (x.kind) {
             case MixerKind::Attention: encode_attention(st, p, x.attn, mc, cur, alone, capture != nullptr); break;
             case MixerKind::StateSpace: encode_state_space(st, p, x.ssm, mc, cur, alone); break;
             case MixerKind::TimeMix: encode_time_mix(st, p, x.tmix, mc, cur, alone); break;
+            case MixerKind::Latent: encode_latent(st, p, x.latent, mc, alone, capture != nullptr); break;
+            case MixerKind::Linear: encode_linear(st, p, x.linear, mc, alone); break;
             }
-            if (capture && x.kind == MixerKind::Attention) {
-                attn_width = x.attn.out_w();
+            if (capture && (x.kind == MixerKind::Attention || x.kind == MixerKind::Latent)) {
+                attn_width = x.kind == MixerKind::Latent ? x.latent.out_w() : x.attn.out_w();
                 sdpa = host(z.attn_f.as<float>(), size_t(n) * attn_width);
             }
         }
@@ -486,14 +735,16 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
             launch_merge_rows(mg, stream);
             span_end(sp);
         }
+        if (l.post_norm) add_norm(cur, l.norm1, n);
         cur = h;
         normed = false;
+        if (l.post_norm) z.in_f = h;
         if (l.mlp == MlpKind::Experts) {
-            const bool next_norm = ri + 1 < m.runs.size() && !m.runs[ri + 1].loop_in && !m.runs[ri + 1].add_embed;
+            const bool next_norm = !l.post_norm && ri + 1 < m.runs.size() && !m.runs[ri + 1].loop_in && !m.runs[ri + 1].add_embed;
             encode_experts(l, n, next_norm ? m.layers[m.runs[ri + 1].layer].norm1 : RowNorm{});
             normed = next_norm;
         } else if (l.mlp == MlpKind::Dense) {
-            if (!several) {
+            if (!several && !l.post_norm) {
                 na.in = h;
                 na.norm = l.norm2;
                 sp = span_begin(G_SMALL);
@@ -501,10 +752,13 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
                 span_end(sp);
             }
             sp = span_begin(G_MATMUL);
-            project(l.dense.up, n, z.xn_f.as<float>(), z.xn_b.as<uint16_t>(), z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), EPI_RELU2);
-            project(l.dense.down, n, z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), h, nullptr, EPI_RESID, h);
+            project(l.dense.up, n, z.in_f, z.xn_b.as<uint16_t>(), f32 ? z.ff_f.as<float>() : nullptr, z.ff_b.as<uint16_t>(), l.dense.hidden == Hidden::SiluGlu ? EPI_GLU : EPI_RELU2);
+            project(l.dense.down, n, z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), l.post_norm ? z.branch.as<float>() : h, nullptr, l.post_norm ? EPI_RAW : EPI_RESID,
+                    l.post_norm ? nullptr : h);
             span_end(sp);
+            if (l.post_norm) add_norm(h, l.norm2, n);
         }
+        if (l.side.dim) encode_side(st, l.side, n);
         if (capture) {
             const std::vector<float> resid_out = host(h, size_t(n) * d);
             LayerCapture lc{ri, n, resid_in.data(), nullptr, nullptr, attn_width ? sdpa.data() : nullptr, nullptr, nullptr, nullptr};
@@ -560,8 +814,10 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     float* h = s.h.as<float>();
     RouterArgs r{};
     r.x = h;
-    r.norm = l.norm2;
+    if (!l.post_norm) r.norm = l.norm2;
     r.router = e.router;
+    r.sigmoid = e.sigmoid;
+    r.renormalized = e.renormalized;
     r.correction = e.correction;
     r.xn = f32 || e.identity ? z.moe_x.as<float>() : nullptr;
     r.xn_b = z.moe_xb.as<uint16_t>();
@@ -579,12 +835,15 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     so.place = z.place.as<uint32_t>();
     so.tiles = z.tiles.as<uint32_t>();
     so.n_tiles = z.n_tiles.as<uint32_t>();
+    so.weights = r.weights;
+    so.row_weight = e.scales_input ? z.row_weight.as<float>() : nullptr;
     so.n = n;
     so.top = e.top;
     so.experts = e.experts;
     // The experts' matrices on the tensor cores where their sizes fit: tiles as long as an expert's rows on average, so that
     // its weights are read once. On the CUDA cores a tile has 64.
-    const bool fast = !f32 && grouped_fits(e.ff, d) && grouped_fits(d, e.ff);
+    const uint32_t hidden = hidden_rows(e.hidden, e.ff);
+    const bool fast = !f32 && grouped_fits(hidden, d) && grouped_fits(d, e.ff);
     so.tile = 64;
     if (fast)
         for (so.tile = EXPERT_TILE_MIN; so.tile < 128 && so.tile < 2 * pairs / (e.experts + e.identity);) so.tile *= 2;
@@ -595,13 +854,17 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     sp = span_begin(G_MATMUL);
     LinearArgs up{};
     up.W = reinterpret_cast<const uint16_t*>(e.up.w);
-    up.X = f32 ? static_cast<const void*>(z.moe_x.as<float>()) : z.moe_xb.as<uint16_t>();
+    const float* in_f = l.post_norm ? z.in_f : z.moe_x.as<float>();  // what the experts read: the stream, or its normed rows
+    const uint16_t* in_b = l.post_norm ? z.xn_b.as<uint16_t>() : z.moe_xb.as<uint16_t>();
+    up.X = f32 ? static_cast<const void*>(in_f) : in_b;
     up.src = so.src;
     up.Y = z.hid_f.as<float>();
     up.Yb = z.hid_b.as<uint16_t>();
-    up.m = e.ff;
+    up.m = hidden;
     up.k = d;
-    up.epi = EPI_RELU2;
+    up.epi = e.hidden == Hidden::ClampedGlu ? EPI_GLU_CLAMP : e.hidden == Hidden::SiluGlu ? EPI_GLU : EPI_RELU2;
+    up.limit = e.limit;
+    up.row_scale = so.row_weight;  // (the first products are linear: onto them instead of onto the rows)
     up.tiles = so.tiles;
     up.n_tiles = so.n_tiles;
     up.max_tiles = pairs / so.tile + std::min(e.experts, pairs);
@@ -611,6 +874,7 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     down.W = reinterpret_cast<const uint16_t*>(e.down.w);
     down.X = f32 ? static_cast<const void*>(z.hid_f.as<float>()) : z.hid_b.as<uint16_t>();
     down.src = nullptr;
+    down.row_scale = nullptr;
     down.Y = z.rows.as<float>();
     down.Yb = nullptr;
     down.m = d;
@@ -619,7 +883,7 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     if (fast) launch_grouped(down, e.experts, so.tile, s.err_flag.as<uint32_t>(), stream);
     else launch_linear(down, !f32, stream);
     if (e.shared_ff) {
-        project(e.shared_up, n, z.moe_x.as<float>(), z.moe_xb.as<uint16_t>(), z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), EPI_RELU2);
+        project(e.shared_up, n, in_f, in_b, z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), EPI_RELU2);
         project(e.shared_down, n, z.sh_f.as<float>(), z.sh_b.as<uint16_t>(), z.shared.as<float>(), nullptr, EPI_RAW);
     }
     span_end(sp);
@@ -630,7 +894,8 @@ void Engine::encode_experts(const FolderLayer& l, uint32_t n, RowNorm norm) {
     c.shared = e.shared_ff ? z.shared.as<float>() : nullptr;
     c.ids = r.ids;
     c.place = so.place;
-    c.weights = r.weights;
+    c.weights = e.scales_input ? nullptr : r.weights;
+    if (l.post_norm) c.post = l.norm2;
     c.out = h;
     c.norm = norm;
     c.next = z.xn_f.as<float>();

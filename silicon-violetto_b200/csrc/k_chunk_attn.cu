@@ -14,53 +14,13 @@
 // the output times sigmoid(gate) where there is a gate, bf16 for the projection after it.
 #include <algorithm>
 
-#include "kernels.h"
-#include "mma.cuh"
+#include "paged_attn.cuh"
 
 namespace vlt {
 
 namespace chunked {
 
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-__device__ __forceinline__ void cluster_sync() { asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ uint32_t cluster_addr(uint32_t addr, uint32_t rank) {
-    uint32_t r;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
-    return r;
-}
-__device__ __forceinline__ float gated(float y, float gate) { return y / (1.0f + __expf(-gate)); }
-
-constexpr uint32_t PAGE_SHIFT = 6, PAGE = 1u << PAGE_SHIFT;
-
-// What token t sees: cached keys [lo, first) and, of its tile of 8 rows that starts at cache position `first`, those `mask`
-// names (its `vis`, less the rows of an earlier chunk or out of the window: the rows of a draft tree may lie on both sides of an edge).
-struct View {
-    uint32_t slot, lo, first, mask;
-};
-__device__ __forceinline__ View view_of(const ChunkedAttnArgs& a, uint32_t t) {
-    const uint32_t pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], i = row % 8;
-    View v;
-    v.slot = a.meta[2 * t];
-    v.first = a.meta[2 * (t - row) + 1] + row - i;
-    v.lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0;
-    v.mask = a.vis[t];
-    if (v.lo) {
-        uint32_t seen = 0;
-        for (uint32_t m = v.mask; m;) {
-            const uint32_t j = __ffs(m) - 1;
-            m &= m - 1;
-            if (a.meta[2 * (t - i + j) + 1] >= v.lo) seen |= 1u << j;
-        }
-        v.mask = seen;
-    }
-    return v;
-}
-__device__ __forceinline__ bool sees(const View& v, uint32_t key) { return key >= v.lo && (key < v.first || (key - v.first < 32 && ((v.mask >> (key - v.first)) & 1u))); }
+using namespace paged;
 
 constexpr uint32_t TILE = 16, WARPS = 4, STAGES = 2, MAX_SPLITS = 16;
 template <uint32_t DK, uint32_t DV>
@@ -78,6 +38,7 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
     const uint32_t t = blockIdx.x, kvh = blockIdx.y % a.kv.n_kv, sp = blockIdx.z, warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane >> 2, tq = lane & 3;
     const uint32_t G = a.heads / a.kv.n_kv, h0 = kvh * G + blockIdx.y / a.kv.n_kv * 8, cols = min(8u, kvh * G + G - h0);
     const View v = view_of(a, t);
+    const float cap = a.softcap * LOG2E, cap_inv = 2.0f / a.softcap;
     // Tiles of 16 positions from the one `lo` lies in up to the last key seen (pages hold whole tiles): an even share.
     const uint32_t tile0 = v.lo / TILE, tiles = (v.first + 32 - __clz(v.mask) + TILE - 1) / TILE - tile0, share = (tiles + gridDim.z - 1) / gridDim.z;
     const uint32_t begin = min(sp * share, tiles), n = min(share, tiles - begin), my = warp < n ? (n - warp + WARPS - 1) / WARPS : 0;
@@ -133,6 +94,10 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
             uint32_t ka[4];
             ldmatrix_x4(ka, kbase + k_row + (((2 * ks + k_c) ^ lr) << 4));
             mma16816(s, ka, q[ks][0], q[ks][1]);
+        }
+        if (a.softcap > 0) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[e] = capped(s[e], cap, cap_inv);
         }
         if (key0 < v.lo || key0 + TILE > v.first) {
             if (!sees(v, key0 + g)) s[0] = s[1] = -INFINITY;
@@ -283,6 +248,7 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
     const uint32_t tile = blockIdx.x, h = blockIdx.y, kvh = h / (a.heads / a.kv.n_kv);
     const uint32_t grp = threadIdx.x / (WARPS * 32), tid = threadIdx.x % (WARPS * 32), warp = tid / 32, lane = tid % 32, g = lane >> 2, tq = lane & 3;
     const uint32_t t0 = a.ctiles[2 * tile], rows = a.ctiles[2 * tile + 1];
+    const float cap = a.softcap * LOG2E, cap_inv = 2.0f / a.softcap;
     uint32_t tok[2], low = 0xffffffffu, end = 0;
     bool live[2];
     View v[2];
@@ -364,6 +330,12 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
                     mma16816(s[j], qa[2 * kp], kb[0], kb[1]);
                     mma16816(s[j], qa[2 * kp + 1], kb[2], kb[3]);
                 }
+            }
+            if (a.softcap > 0) {
+#pragma unroll
+                for (uint32_t j = 0; j < 8; j++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[j][e] = capped(s[j][e], cap, cap_inv);
             }
             if (key0 < lo_max || key0 + CK > first_min || !live[0] || !live[1]) {
 #pragma unroll

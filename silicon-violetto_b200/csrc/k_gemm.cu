@@ -301,6 +301,7 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
     // shared memory.
     auto emit = [&](uint32_t r, bool valid, uint32_t t0, float scale, auto& v) {  // v: 16 or 8 consecutive tokens of row r
         constexpr uint32_t NTOK = sizeof(v) / sizeof(float);
+        constexpr bool PAIRS = EPI == EPI_SWIGLU || EPI == EPI_GLU;  // (rows 2 i and 2 i + 1 make one output)
         const uint32_t row = row0 + r;
         if constexpr (EPI == EPI_QKV) {
             // The row is feature `row` of the qkv projection: dim d of a q, k or v head (whole heads per 64 rows, so
@@ -348,15 +349,16 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
 #pragma unroll
         for (uint32_t j = 0; j < NTOK; j++) {
             const float x = v[j] * scale;
-            if (EPI == EPI_SWIGLU) {
+            if (PAIRS) {
                 const float other = __shfl_xor_sync(0xffffffffu, x, 1);
-                const float gt = x * inv[j], up = other * inv[j];
+                const float gt = EPI == EPI_GLU ? x : x * inv[j], up = EPI == EPI_GLU ? other : other * inv[j];
                 y[j] = gt * __fdividef(1.0f, 1.0f + __expf(-gt)) * up;
             } else if (EPI == EPI_NORM) y[j] = x * inv[j] * m.scale;
             else if (EPI == EPI_RESID) y[j] = m.ra * base[j] + m.rb * (m.scale * x);  // (1, 1, 1 for a plain decoder: the same bits as base + x)
             else if (EPI == EPI_HEAD) y[j] = row < m.vocab_real ? x * inv[j] : -INFINITY;
             else if (EPI == EPI_HEAD_CAP) y[j] = row < m.vocab_real ? 23.0f * (1.0f / (1.0f + __expf(-(x + 5.0f) / 7.5f))) : -INFINITY;  // kernels.metal:196-199
             else if (EPI == EPI_RELU2) y[j] = x > 0.0f ? x * x : 0.0f;
+            else if (EPI == EPI_SILU) y[j] = row < m.vocab_real ? x * __fdividef(1.0f, 1.0f + __expf(-x)) : x;
             else y[j] = x;
         }
         if (EPI == EPI_RESID && m.ssq_out) {
@@ -380,8 +382,8 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
             for (uint32_t bit = 16 / NTOK; bit >= 1; bit /= 2) w[0] += __shfl_xor_sync(0xffffffffu, w[0], bit);
             if ((lane & (32 / NTOK - 1)) == 0) ssq_s[(r / 32) * n_pad + t0 + tk] = w[0];
         }
-        const bool writes = valid && (EPI != EPI_SWIGLU || (lane & 1) == 0);
-        const uint32_t out_w = EPI == EPI_SWIGLU ? m.m / 2 : m.m, out_r = EPI == EPI_SWIGLU ? row / 2 : row;
+        const bool writes = valid && (!PAIRS || (lane & 1) == 0);
+        const uint32_t out_w = PAIRS ? m.m / 2 : m.m, out_r = PAIRS ? row / 2 : row;
         if (writes) {
 #pragma unroll
             for (uint32_t j = 0; j < NTOK; j++)
@@ -533,6 +535,8 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
     case EPI_QKV: return int8 ? gemm::gemm_kernel<true, EPI_QKV> : gemm::gemm_kernel<false, EPI_QKV>;
     case EPI_HEAD_CAP: return int8 ? gemm::gemm_kernel<true, EPI_HEAD_CAP> : gemm::gemm_kernel<false, EPI_HEAD_CAP>;
     case EPI_RELU2: return int8 ? gemm::gemm_kernel<true, EPI_RELU2> : gemm::gemm_kernel<false, EPI_RELU2>;
+    case EPI_SILU: return gemm::gemm_kernel<false, EPI_SILU>;  // (bf16 weights only)
+    case EPI_GLU: return gemm::gemm_kernel<false, EPI_GLU>;
     default: return int8 ? gemm::gemm_kernel<true, EPI_RAW> : gemm::gemm_kernel<false, EPI_RAW>;
     }
 }
@@ -540,7 +544,8 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
 bool gemm_supported(const MatArgs& a) {
     const bool grouped = a.int8 && a.group < a.k;  // scale groups: powers of two from 8
     return a.n >= 1 && a.n <= 256 && a.m % gemm::BM == 0 && a.k % gemm::BK == 0 && (!grouped || (a.group >= 8 && !(a.group & (a.group - 1)))) && a.Xb != nullptr &&
-           (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.epi == EPI_RELU2 || a.inv_in != nullptr || a.ssq_in != nullptr);
+           (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.epi == EPI_RELU2 ||
+            (!a.int8 && (a.epi == EPI_SILU || a.epi == EPI_GLU)) || a.inv_in != nullptr || a.ssq_in != nullptr);
 }
 
 void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaStream_t s, bool allow_paired) {
@@ -583,7 +588,7 @@ void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaSt
     const size_t smem = paired ? need : std::max<size_t>(need, 116 * 1024);
     configured.once([] {
         for (int i8 = 0; i8 < 2; i8++)
-            for (uint32_t epi = EPI_NORM; epi <= EPI_RELU2; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            for (uint32_t epi = EPI_NORM; epi <= EPI_GLU; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
     });

@@ -1,5 +1,5 @@
 // Grouped linear layers on the 5th-generation tensor cores: the experts' matrices of a mixture, each against the tokens that
-// chose it. A block takes one (expert, rows <= N) tile of the sorted pairs (k_moe.cu's table) and 128 of the expert's output
+// chose it, or a matrix per head against that head's part of every token. A block takes one (expert, rows <= N) tile of the sorted pairs (k_moe.cu's table) and 128 of the expert's output
 // rows: the weights are the MMA's M side, so an expert's matrix crosses HBM once for its tile of tokens, from one token on;
 // the tokens are its N side, N rounded to 16 per tile. Weights come by TMA into 128-byte-swizzled stages; four warps fetch
 // the tokens' rows -- gathered through the pair -> token table, or in place -- by 16-byte asynchronous copies into the same
@@ -114,7 +114,8 @@ __global__ void __launch_bounds__(THREADS, 2) grouped_kernel(const __grid_consta
 #pragma unroll
         for (uint32_t j = 0; j < MAX_PER; j++) {
             const uint32_t r = r_first + 16 * j, p = p0 + (r < count ? r : 0);
-            src[j] = X + size_t(j < per ? (a.l.src ? a.l.src[p] : p) : 0) * a.l.k + piece * 8;
+            const size_t from = j >= per ? 0 : a.l.src ? a.l.src[p] : a.l.by_head ? size_t(p - group * a.l.by_head) * a.l.heads + group : p;
+            src[j] = X + from * a.l.k + piece * 8;
         }
         const uint32_t dst0 = base + a_bytes + r_first * 128 + ((piece ^ (r_first & 7)) << 4);
         constexpr uint32_t LAG = 2;  // stages requested ahead of the one reported full
@@ -152,8 +153,19 @@ __global__ void __launch_bounds__(THREADS, 2) grouped_kernel(const __grid_consta
                 for (uint32_t j = 0; j < 16; j++) {
                     if (c0 + j >= count) break;
                     float y = acc[j];
+                    size_t o = size_t(p0 + c0 + j) * a.l.m + row;
                     if (EPI == EPI_RELU2) y = y > 0.0f ? y * y : 0.0f;
-                    const size_t o = size_t(p0 + c0 + j) * a.l.m + row;
+                    if (EPI == EPI_GLU_CLAMP) {
+                        if (a.l.row_scale) y *= a.l.row_scale[p0 + c0 + j];
+                        const float u = __shfl_xor_sync(0xffffffffu, y, 1);
+                        if (lane & 1) continue;  // (a pair's even row has its output)
+                        y = clamped_glu(y, u, a.l.limit);
+                        o = size_t(p0 + c0 + j) * (a.l.m / 2) + row / 2;
+                    } else if (EPI == EPI_RAW && a.l.by_head) {
+                        const size_t t = p0 + c0 + j - group * a.l.by_head;
+                        if (a.l.gate) y *= __fdividef(1.0f, 1.0f + __expf(-a.l.gate[t * a.l.ldg + size_t(group) * a.l.m + row]));
+                        o = (t * a.l.heads + group) * a.l.ldy + row;
+                    }
                     if (a.l.Y) a.l.Y[o] = y;
                     if (a.l.Yb) a.l.Yb[o] = f32_to_bf16(y);
                 }
@@ -181,7 +193,7 @@ void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint3
     static thread_local std::map<std::tuple<const void*, uint32_t, uint32_t, uint32_t>, grouped::Map> maps;
     static PerDevice configured;
     if (!a.max_tiles) return;
-    if (!grouped_fits(a.m, a.k) || tile < 16 || tile > 128 || tile % 16 || (a.epi != EPI_RAW && a.epi != EPI_RELU2)) throw Error("internal: a grouped GEMM of an unsupported shape");
+    if (!grouped_fits(a.m, a.k) || tile < 16 || tile > 128 || tile % 16 || (a.epi != EPI_RAW && a.epi != EPI_RELU2 && a.epi != EPI_GLU_CLAMP) || (a.row_scale && a.epi != EPI_GLU_CLAMP)) throw Error("internal: a grouped GEMM of an unsupported shape");
     auto key = std::make_tuple(static_cast<const void*>(a.W), a.m, a.k, n_groups);
     auto it = maps.find(key);
     if (it == maps.end()) {
@@ -191,7 +203,7 @@ void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint3
     }
     constexpr uint32_t SMEM = 112 * 1024;  // two blocks an SM
     configured.once([] {
-        for (auto f : {grouped::grouped_kernel<EPI_RAW>, grouped::grouped_kernel<EPI_RELU2>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, int(SMEM)));
+        for (auto f : {grouped::grouped_kernel<EPI_RAW>, grouped::grouped_kernel<EPI_RELU2>, grouped::grouped_kernel<EPI_GLU_CLAMP>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, int(SMEM)));
     });
     grouped::Args g;
     g.l = a;
@@ -203,7 +215,8 @@ void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint3
     // (at least 78 KiB, so that no third block, whose tensor memory might not be there, comes onto the SM)
     const size_t smem = std::max<size_t>(size_t(g.stages) * stage + 1024 + (2 * g.stages + 1) * 8 + 16, 78 * 1024);
     const dim3 grid(a.m / grouped::BM, a.max_tiles);
-    if (a.epi == EPI_RELU2) launch_pdl(grouped::grouped_kernel<EPI_RELU2>, grid, grouped::THREADS, smem, s, it->second, g);
+    if (a.epi == EPI_GLU_CLAMP) launch_pdl(grouped::grouped_kernel<EPI_GLU_CLAMP>, grid, grouped::THREADS, smem, s, it->second, g);
+    else if (a.epi == EPI_RELU2) launch_pdl(grouped::grouped_kernel<EPI_RELU2>, grid, grouped::THREADS, smem, s, it->second, g);
     else launch_pdl(grouped::grouped_kernel<EPI_RAW>, grid, grouped::THREADS, smem, s, it->second, g);
 }
 

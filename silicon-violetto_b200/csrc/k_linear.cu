@@ -1,6 +1,7 @@
 // Linear layers on the CUDA cores, for what the tensor-core kernels do not take: activations in fp32 throughout (true fp32
 // products and sums: bf16 weights are exact in fp32), and matrices whose sizes fit neither the streamed kernel nor the GEMM.
-// Also the row passes in front of a projection: RMS norms, two streams side by side, and two mixers' outputs onto the stream.
+// Also the row passes around a projection: RMS norms in front of it or of what it leaves, two streams side by side, two mixers'
+// outputs onto the stream, and a side input's gate.
 #include <algorithm>
 
 #include "kernels.h"
@@ -39,7 +40,8 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
             const uint32_t kk = i % BK, r = i / BK;
             ws[kk][r] = r0 + r < a.m && k0 + kk < a.k ? bf16_to_f32(W[size_t(r0 + r) * a.k + k0 + kk]) : 0.0f;
             const uint32_t p = p0 + r;
-            xs[kk][r] = r < count && k0 + kk < a.k ? load_x(X + size_t(a.src ? a.src[p] : p) * a.k + k0 + kk) : 0.0f;
+            const size_t from = a.src ? a.src[p] : a.by_head ? size_t(p - group * a.by_head) * a.heads + group : p;
+            xs[kk][r] = r < count && k0 + kk < a.k ? load_x(X + from * a.k + k0 + kk) : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -57,15 +59,25 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
 #pragma unroll
     for (int j = 0; j < 4; j++) {
         const uint32_t p = tt + 16 * j;
-        if (p >= count) continue;
+        const float scale = a.row_scale && p < count ? a.row_scale[p0 + p] : 1.0f;
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             const uint32_t r = r0 + tr + 16 * i;
-            if (r >= a.m) continue;
-            const size_t o = size_t(p0 + p) * a.m + r;
-            float y = acc[i][j];
+            float y = acc[i][j] * scale;
+            const bool pairs = a.epi == EPI_GLU || a.epi == EPI_GLU_CLAMP;  // (a pair's rows are neighbouring lanes')
+            const float u = pairs ? __shfl_xor_sync(0xffffffffu, y, 1) : 0.0f;
+            if (p >= count || r >= a.m || (pairs && r % 2)) continue;
+            size_t o = pairs ? size_t(p0 + p) * (a.m / 2) + r / 2 : size_t(p0 + p) * a.m + r;
+            if (a.by_head) {
+                const size_t t = p0 + p - group * a.by_head;
+                if (a.gate) y *= sigmoid_of(a.gate[t * a.ldg + size_t(group) * a.m + r]);
+                o = (t * a.heads + group) * a.ldy + r;
+            }
             if (a.epi == EPI_RESID) y += a.base[o];
             else if (a.epi == EPI_RELU2) y = y > 0.0f ? y * y : 0.0f;
+            else if (a.epi == EPI_SILU) y = r < a.act_rows ? y * sigmoid_of(y) : y;
+            else if (a.epi == EPI_GLU) y = y * sigmoid_of(y) * u;
+            else if (a.epi == EPI_GLU_CLAMP) y = clamped_glu(y, u, a.limit);
             if (a.Y) a.Y[o] = y;
             if (a.Yb) a.Yb[o] = f32_to_bf16(y);
         }
@@ -156,6 +168,51 @@ __global__ void __launch_bounds__(1024) merge_rows_kernel(const MergeArgs a) {
     }
 }
 
+// See AddNormArgs. A block per row.
+template <uint32_t V>
+__global__ void __launch_bounds__(1024) add_norm_kernel(const AddNormArgs a) {
+    pdl_start();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    const uint32_t tid = threadIdx.x * V, step = blockDim.x * V;
+    const size_t from = size_t(blockIdx.x) * a.d;
+    float ss = 0.0f;
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float y[V];
+        load_f32<V>(y, a.y + from + i);
+        store_f32<V>(row + i, y);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) ss += y[j] * y[j];
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / float(a.d) + a.eps);
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float x[V], y[V], w[V];
+        load_f32<V>(x, a.x + from + i);
+        load_f32<V>(y, row + i);
+        weights_of<V>(w, a.norm, i);
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) x[j] += y[j] * inv * w[j];
+        store_f32<V>(a.out + from + i, x);
+        if (a.out_b) store_bf16<V>(a.out_b + from + i, x);
+    }
+}
+
+// See SideGateArgs. grid (tokens, spans of 256 columns).
+__global__ void __launch_bounds__(256) side_gate_kernel(const SideGateArgs a) {
+    pdl_start();
+    const uint32_t t = blockIdx.x, i = blockIdx.y * 256 + threadIdx.x;
+    if (i >= a.wide) return;
+    float y = 0.0f;
+    if (i < a.dim) {
+        const float z = a.x[size_t(t) * a.ldx + i];
+        const float g = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));  // (sqrt(2 / pi))
+        y = g * bf16_to_f32(a.table[size_t(a.tokens[t]) * a.ld + a.first + i]);
+    }
+    const size_t o = size_t(t) * a.wide + i;
+    if (a.out_f32) a.out_f32[o] = y;
+    if (a.out_bf16) a.out_bf16[o] = f32_to_bf16(y);
+}
+
 // out[r] = (a[r] ; b[r]).
 __global__ void __launch_bounds__(256) concat_rows_kernel(const float* __restrict__ a, const float* __restrict__ b, uint32_t d, float* out_f32, uint16_t* out_bf16) {
     pdl_start();
@@ -193,6 +250,18 @@ void launch_merge_rows(const MergeArgs& a, cudaStream_t s) {
     if (!a.n) return;
     if (a.d % 4 == 0) launch_pdl(linear::merge_rows_kernel<4>, a.n, row_threads(a.d, 4), size_t(a.d) * 8, s, a);
     else launch_pdl(linear::merge_rows_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 8, s, a);
+}
+void launch_add_norm(const AddNormArgs& a, cudaStream_t s) {
+    static PerDevice configured;
+    configured.once([] {
+        for (auto f : {linear::add_norm_kernel<1>, linear::add_norm_kernel<4>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    if (!a.n) return;
+    if (a.d % 4 == 0) launch_pdl(linear::add_norm_kernel<4>, a.n, row_threads(a.d, 4), size_t(a.d) * 4, s, a);
+    else launch_pdl(linear::add_norm_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 4, s, a);
+}
+void launch_side_gate(const SideGateArgs& a, cudaStream_t s) {
+    if (a.n) launch_pdl(linear::side_gate_kernel, dim3(a.n, (a.wide + 255) / 256), 256, 0, s, a);
 }
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s) {
     if (n) launch_pdl(linear::concat_rows_kernel, n, 256, 0, s, a, b, d, out_f32, out_bf16);

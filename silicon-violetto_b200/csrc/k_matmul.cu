@@ -24,6 +24,7 @@ __device__ __forceinline__ void store_out(const MatArgs& a, uint32_t t, uint32_t
     case EPI_HEAD: y = row < a.vocab_real ? acc * inv : -INFINITY; break;
     case EPI_HEAD_CAP: y = row < a.vocab_real ? 23.0f * (1.0f / (1.0f + expf(-(acc + 5.0f) / 7.5f))) : -INFINITY; break;
     case EPI_RELU2: y = acc > 0.0f ? acc * acc : 0.0f; break;
+    case EPI_SILU: y = row < a.vocab_real ? acc * sigmoid_of(acc) : acc; break;
     default: y = acc; break;
     }
     if (a.Y) a.Y[o] = y;
@@ -34,7 +35,7 @@ __device__ __forceinline__ void store_swiglu(const MatArgs& a, uint32_t t, uint3
     u *= inv;
     const float y = g * (1.0f / (1.0f + expf(-g))) * u;
     const size_t o = size_t(t) * (a.m / 2) + row / 2;
-    a.Y[o] = y;
+    if (a.Y) a.Y[o] = y;
     if (a.Yb) a.Yb[o] = f32_to_bf16(y);
 }
 
@@ -92,7 +93,7 @@ __global__ void __launch_bounds__(256) matmul_rows_kernel(MatArgs a) {
             const uint32_t t = t0 + b;
             const float inv = a.inv_in ? a.inv_in[t] : rsqrtf(sq / float(a.k) + a.eps);
             if (a.inv_out && row0 == 0) a.inv_out[t] = inv;
-            if (a.epi == EPI_SWIGLU) store_swiglu(a, t, row0, s0, s1, inv);
+            if (a.epi == EPI_SWIGLU || a.epi == EPI_GLU) store_swiglu(a, t, row0, s0, s1, a.epi == EPI_GLU ? 1.0f : inv);
             else { store_out(a, t, row0, s0, inv); store_out(a, t, row0 + 1, s1, inv); }
         }
     }
@@ -466,8 +467,8 @@ __global__ void __launch_bounds__(512, 2) matmul_stream_kernel(MatArgs a, uint32
                 const float partner = __shfl_down_sync(0xffffffffu, sum, 1);  // row r + 1 of the same token (r is even where it is used)
                 if (b < a.n) {
                     const float inv = inv_s[b];
-                    if (a.epi == EPI_SWIGLU) {
-                        if (r % 2 == 0) store_swiglu(a, b, row0 + r, sum, partner, inv);
+                    if (a.epi == EPI_SWIGLU || a.epi == EPI_GLU) {
+                        if (r % 2 == 0) store_swiglu(a, b, row0 + r, sum, partner, a.epi == EPI_GLU ? 1.0f : inv);
                     } else if (a.epi == EPI_QKV) {
                         if (r % 2 == 0) {  // qkv_store_pair with the token's table entries from shared memory
                             const uint32_t hd = a.q.kv.hd, row = row0 + r, head = row / hd, pair = (row % hd) / 2;

@@ -1,5 +1,5 @@
 // The attention mixer's work between its projections and its attention, as parameterised kernels: a short causal
-// convolution over time on q, k and v, rotation of pairs (i, i + dims / 2), q and k heads of unit length, queries that grow with
+// convolution over time on q, k and v, rotation of pairs, q and k heads of unit length, queries that grow with
 // their position (each of them optional), K and V into a paged cache whose heads may have
 // different key and value sizes; the convolution's state -- the projected rows before the step -- in a ring per sequence
 // slot; and a scalar form of the chunked or windowed attention for any head sizes and for fp32 caches.
@@ -15,11 +15,6 @@ __device__ __forceinline__ void store_kv(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_kv(uint16_t* p, float v) { *p = f32_to_bf16(v); }
 __device__ __forceinline__ float load_kv(const float* p) { return *p; }
 __device__ __forceinline__ float load_kv(const uint16_t* p) { return bf16_to_f32(*p); }
-
-__device__ __forceinline__ size_t page_row(const PagedKv& kv, uint32_t slot, uint32_t g, uint32_t pos) {
-    const uint32_t page = kv.page_table[size_t(slot) * kv.max_pages + (pos >> kv.page_shift)], psize = 1u << kv.page_shift;
-    return (size_t(page) * kv.n_kv + g) * psize + (pos & (psize - 1));
-}
 
 // grid (tokens / TB, heads + 2 kv heads): one q, k or v head of TB tokens a block (a step of many tokens: the tokens' chains of
 // dependent loads run side by side).
@@ -86,6 +81,9 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
             for (uint32_t c = back; c < width; c += 32) ss += y[mine * width + c] * y[mine * width + c];
             ss = warp_sum(ss);
             if (back == 0) factor[mine] *= 1.0f / sqrtf(ss / float(width) + a.unit_eps);
+            const RowNorm& weight = kind == 0 ? a.q_norm : a.k_norm;
+            if (weight.w)
+                for (uint32_t c = back; c < width; c += 32) y[mine * width + c] *= weight_of(weight, c);
         }
         __syncthreads();
     }
@@ -96,11 +94,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
             if (i >= nt) break;
             const float* yi = y + i * width;
             float v = yi[c];
-            if (kind < 2 && c < a.rot_dims) {
-                const float2 cs = reinterpret_cast<const float2*>(a.rope)[size_t(pos_s[i]) * half + (c < half ? c : c - half)];
-                v = c < half ? yi[c] * cs.x - yi[c + half] * cs.y : yi[c] * cs.x + yi[c - half] * cs.y;
-            }
-            if (kind < 2) v *= factor[i];
+            if (kind < 2) v = rotated(yi, c, a.rot_dims, a.neighbours, reinterpret_cast<const float2*>(a.rope) + size_t(pos_s[i]) * half) * factor[i];
             if (kind == 0) {
                 const size_t o = (size_t(t0 + i) * a.heads + head) * width + c;
                 if (a.q_f) a.q_f[o] = v;
@@ -145,6 +139,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
     const uint32_t lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0, n_old = p_tile > lo ? p_tile - lo : 0;
     const T* K = static_cast<const T*>(a.kv.k);
     const T* V = static_cast<const T*>(a.kv.v);
+    const uint32_t ldv = a.kv.v == a.kv.k ? a.kv.dk : a.kv.dv;
     for (uint32_t c = tid; c < a.kv.dk; c += 128) q[c] = a.q_f[(size_t(t) * a.heads + h) * a.kv.dk + c];
     for (uint32_t c = tid; c < a.kv.dv; c += 128) o[c] = 0.0f;
     float m = -INFINITY, l = 0.0f;
@@ -166,6 +161,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
             float d = 0.0f;
             for (uint32_t c = 0; c < a.kv.dk; c++) d = fmaf(q[c], load_kv(k + c), d);
             s = d * a.scale;
+            if (a.softcap > 0) s = a.softcap * tanhf(s / a.softcap);
         }
         float mx = warp_max(s);
         if (tid % 32 == 0) red[tid / 32] = mx;
@@ -183,7 +179,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
             for (uint32_t c = tid; c < a.kv.dv; c += 128) {
                 float acc = o[c] * corr;
                 for (uint32_t j = 0; j < n; j++)
-                    if (p[j] != 0.0f) acc = fmaf(p[j], load_kv(V + size_t(rows[j]) * a.kv.dv + c), acc);
+                    if (p[j] != 0.0f) acc = fmaf(p[j], load_kv(V + size_t(rows[j]) * ldv + c), acc);
                 o[c] = acc;
             }
         }
@@ -213,7 +209,8 @@ __global__ void __launch_bounds__(256) mixer_compact_kernel(const RunIn* __restr
         for (uint32_t g = 0; g < mc.kv.n_kv; g++) {
             const size_t src = page_row(mc.kv, slot, g, p0 + from), dst = page_row(mc.kv, slot, g, p0 + j);
             for (uint32_t c = threadIdx.x; c < mc.kv.dk; c += 256) static_cast<T*>(mc.kv.k)[dst * mc.kv.dk + c] = static_cast<const T*>(mc.kv.k)[src * mc.kv.dk + c];
-            for (uint32_t c = threadIdx.x; c < mc.kv.dv; c += 256) static_cast<T*>(mc.kv.v)[dst * mc.kv.dv + c] = static_cast<const T*>(mc.kv.v)[src * mc.kv.dv + c];
+            if (mc.kv.v != mc.kv.k)
+                for (uint32_t c = threadIdx.x; c < mc.kv.dv; c += 256) static_cast<T*>(mc.kv.v)[dst * mc.kv.dv + c] = static_cast<const T*>(mc.kv.v)[src * mc.kv.dv + c];
         }
         float* ring = mc.ring + size_t(slot) * mc.ring_len * mc.channels;
         for (uint32_t c = threadIdx.x; c < mc.channels; c += 256) ring[size_t((p0 + j) % mc.ring_len) * mc.channels + c] = ring[size_t((p0 + from) % mc.ring_len) * mc.channels + c];
@@ -227,7 +224,7 @@ __global__ void __launch_bounds__(256) mixer_fill_kernel(const MixerCache* __res
     const uint32_t pos = from + blockIdx.x;
     for (uint32_t g = 0; g < mc.kv.n_kv; g++) {
         const size_t r = page_row(mc.kv, slot, g, pos);
-        for (uint32_t c = threadIdx.x; c < mc.kv.dk + mc.kv.dv; c += 256) {
+        for (uint32_t c = threadIdx.x; c < mc.kv.dk + (mc.kv.v == mc.kv.k ? 0 : mc.kv.dv); c += 256) {
             const float v = (float(philox(make_uint4(pos, blockIdx.y * 131 + g, c, slot), seed, 0xf111u).x >> 8) * 0x1p-24f - 0.5f) * 0.5f;
             if (c < mc.kv.dk) store_kv(static_cast<T*>(mc.kv.k) + r * mc.kv.dk + c, v);
             else store_kv(static_cast<T*>(mc.kv.v) + r * mc.kv.dv + c - mc.kv.dk, v);
@@ -250,7 +247,7 @@ void launch_conv_state(const ConvArgs& a, const RunIn* runs, uint32_t n_runs, cu
     if (n_runs) launch_pdl(mixer::conv_state_kernel, dim3(n_runs, a.ring_len, (a.conv_channels + 1023) / 1024), 256, 0, s, a, runs);
 }
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
-    const size_t smem = (a.kv.dk + a.kv.dv + 128) * 4;
+    const size_t smem = (a.kv.dk + a.kv.dv + 128) * 4;  // (past 48 KB for rows of some 12 000 entries)
     if (fp32) launch_pdl(mixer::attn_any_kernel<float>, dim3(n, a.heads), 128, smem, s, a);
     else launch_pdl(mixer::attn_any_kernel<uint16_t>, dim3(n, a.heads), 128, smem, s, a);
 }

@@ -1,5 +1,5 @@
-// A mixture of experts: the router (fp32 scores over the experts and the identity experts, a correction that moves the
-// choice but not the weights), the tokens sorted by expert, and the weighted sum of what the experts left. The experts' own
+// A mixture of experts: the router (fp32 scores over the experts and the identity experts, by softmax or sigmoid; a correction that
+// moves the choice but not the weights), the tokens sorted by expert, and the (weighted) sum of what the experts left. The experts' own
 // matrices are grouped linear layers (k_linear.cu, k_grouped.cu).
 #include <algorithm>
 
@@ -9,8 +9,8 @@ namespace vlt {
 
 namespace moe {
 
-// One block per TOK tokens: the RMS norm of their rows (kept for the experts), the scores' logits with a warp per output,
-// softmax and the choice with a warp per token. Ties go to the lower index.
+// One block per TOK tokens: the RMS norm of their rows (kept for the experts; without a weight, the rows as they are), the scores'
+// logits with a warp per output, the scores and the choice with a warp per token. Ties go to the lower index.
 template <uint32_t TOK, uint32_t ROUTER_THREADS>
 __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs a) {
     pdl_start();
@@ -39,6 +39,7 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
         if (j >= nt) break;
         float tot = 0.0f;
         for (uint32_t w = 0; w < NW; w++) tot += red[j][w];
+        if (!a.norm.w) break;
         const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
         for (uint32_t i = tid; i < a.d; i += ROUTER_THREADS) {
             const float v = x[j * a.d + i] * inv * weight_of(a.norm, i);
@@ -99,22 +100,26 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
     for (uint32_t j = warp; j < nt; j += NW) {
         float* zt = z + j * all;
         const uint32_t t = t0 + j;
-        float m = -INFINITY, sum = 0.0f;
-        for (uint32_t e = lane; e < all; e += 32) m = fmaxf(m, zt[e]);
-        m = warp_max(m);
-        for (uint32_t e = lane; e < all; e += 32) {
-            const float p = expf(zt[e] - m);
-            zt[e] = p;
-            sum += p;
+        if (a.sigmoid) {
+            for (uint32_t e = lane; e < all; e += 32) zt[e] = sigmoid_of(zt[e]);
+        } else {
+            float m = -INFINITY, sum = 0.0f;
+            for (uint32_t e = lane; e < all; e += 32) m = fmaxf(m, zt[e]);
+            m = warp_max(m);
+            for (uint32_t e = lane; e < all; e += 32) {
+                const float p = expf(zt[e] - m);
+                zt[e] = p;
+                sum += p;
+            }
+            sum = warp_sum(sum);
+            for (uint32_t e = lane; e < all; e += 32) zt[e] = zt[e] / sum;
         }
-        sum = warp_sum(sum);
-        for (uint32_t e = lane; e < all; e += 32) zt[e] = zt[e] / sum;
         __syncwarp();
         // The choice: the largest score + correction, `top` times, ties to the lower index. Kept as integers that order as
         // the numbers do (0: chosen already), so that a warp's maximum is one instruction.
         uint32_t* ct = reinterpret_cast<uint32_t*>(z + TOK * all) + j * all;
         for (uint32_t e = lane; e < all; e += 32) {
-            const uint32_t u = __float_as_uint(zt[e] + bf16_to_f32(a.correction[e]));
+            const uint32_t u = __float_as_uint(a.correction ? zt[e] + bf16_to_f32(a.correction[e]) : zt[e]);
             ct[e] = max(u & 0x80000000u ? ~u : u | 0x80000000u, 1u);
         }
         __syncwarp();
@@ -137,7 +142,7 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_kernel(const RouterArgs
             if (lane == k) kept = s;
             __syncwarp();
         }
-        const float inv = 1.0f / (total + 1e-20f);
+        const float inv = a.renormalized ? 1.0f / (total + 1e-20f) : 1.0f;
         if (lane < a.top) a.weights[size_t(t) * a.top + lane] = kept * inv;
         for (uint32_t k = 32 + lane; k < a.top; k += 32) a.weights[size_t(t) * a.top + k] *= inv;
     }
@@ -189,13 +194,14 @@ __global__ void __launch_bounds__(1024) sort_kernel(const SortArgs a) {
             const uint32_t p = atomicAdd(cur + e, 1u);
             a.src[p] = i / a.top;
             a.place[i] = p;
+            if (a.row_weight) a.row_weight[p] = a.weights[i];
         }
     }
 }
 
 // out[t] = x[t] + sum_k weight_k (expert k's row, or the token's own normed row for an identity expert) + the shared
-// expert's row, in the order of the choice; and, if asked, the next layer's RMS norm of it. A block per token; V: the
-// columns a thread takes at a time.
+// expert's row, in the order of the choice; and, if asked, the next layer's RMS norm of it. With `post`, what is added to x[t] is
+// the sum's RMS norm. A block per token; V: the columns a thread takes at a time.
 template <typename V>
 __device__ __forceinline__ void fma_v(V& y, float w, const V& v);
 template <>
@@ -221,14 +227,15 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     const float** src = reinterpret_cast<const float**>(wt + (a.top + 1) / 2 * 2);
     for (uint32_t k = tid; k < a.top; k += 256) {
         const size_t i = size_t(t) * a.top + k;
-        wt[k] = a.weights[i];
+        wt[k] = a.weights ? a.weights[i] : 1.0f;
         src[k] = a.ids[i] < a.experts ? a.y + size_t(a.place[i]) * a.d : a.xn + size_t(t) * a.d;
     }
     __syncthreads();
     const V one{};
     float ss = 0.0f;
     for (uint32_t i = tid; i < dv; i += 256) {
-        V y = one, x = reinterpret_cast<const V*>(a.x + size_t(t) * a.d)[i], sh = one;
+        V y = one, x = one, sh = one;
+        if (!a.post.w) x = reinterpret_cast<const V*>(a.x + size_t(t) * a.d)[i];
         if (a.shared) sh = reinterpret_cast<const V*>(a.shared + size_t(t) * a.d)[i];
         for (uint32_t k0 = 0; k0 < a.top; k0 += 8) {
             V v[8];
@@ -240,11 +247,11 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
         }
         fma_v(y, 1.0f, sh);
         fma_v(y, 1.0f, x);
-        reinterpret_cast<V*>(a.out + size_t(t) * a.d)[i] = y;
+        if (!a.post.w) reinterpret_cast<V*>(a.out + size_t(t) * a.d)[i] = y;
         reinterpret_cast<V*>(row)[i] = y;
         ss += square(y);
     }
-    if (!a.norm.w) return;
+    if (!a.norm.w && !a.post.w) return;
     ss = warp_sum(ss);
     if (tid % 32 == 0) red[tid / 32] = ss;
     __syncthreads();
@@ -253,6 +260,12 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
     for (uint32_t i = tid; i < a.d; i += 256) {
         const size_t o = size_t(t) * a.d + i;
+        if (a.post.w) {
+            const float v = a.x[o] + row[i] * inv * weight_of(a.post, i);
+            a.out[o] = v;
+            if (a.next_b) a.next_b[o] = f32_to_bf16(v);
+            continue;
+        }
         const float v = row[i] * inv * weight_of(a.norm, i);
         if (a.next) a.next[o] = v;
         if (a.next_b) a.next_b[o] = f32_to_bf16(v);

@@ -197,7 +197,8 @@ __global__ void __launch_bounds__(L * COLS / PC, GROUP == 1 ? 0 : 1) scan_kernel
         __syncthreads();
     }
     const float *Q = a.q + size_t(t0) * a.ldq + size_t(head / c.per) * c.N, *K = a.k + size_t(t0) * a.ldk + size_t(head / c.per) * c.N, *V = a.v + size_t(t0) * a.ldv + size_t(head) * c.P + p0;
-    const float* D = CHANNEL ? a.decay + (size_t(t0) * c.heads + head) * c.N : a.decay + (size_t(t0) * c.heads + head) * 2;
+    const float* D = a.decay + (size_t(t0) * c.heads + head) * (CHANNEL ? c.N : 2);  // (not read where the decays are fixed)
+    const float fixed = !CHANNEL && c.fixed ? c.fixed[head] : 1.0f;
     const Walk key0(tid, THREADS, aligned ? c.N / 4 : c.N), value0(tid, THREADS, aligned ? cols / 4 : cols);
     auto rows = [&](Walk at, float* dst, uint32_t pitch, const float* src, size_t ld, uint32_t n) {
         if (aligned)
@@ -215,7 +216,10 @@ __global__ void __launch_bounds__(L * COLS / PC, GROUP == 1 ? 0 : 1) scan_kernel
             rows(key0, st.w, NP, D + size_t(i0) * c.heads * c.N, size_t(c.heads) * c.N, n);
             for (uint32_t i = tid; i < n; i += THREADS) cp_async4(st.s + 4 * i, a.bonus + size_t(t0 + i0 + i) * c.heads + head);
         } else {
-            for (uint32_t i = tid; i < 2 * n; i += THREADS) cp_async4(st.s + 4 * (i / 2) + i % 2, D + size_t(i0 + i / 2) * c.heads * 2 + i % 2);
+            if (!c.fixed)
+                for (uint32_t i = tid; i < 2 * n; i += THREADS) cp_async4(st.s + 4 * (i / 2) + i % 2, D + size_t(i0 + i / 2) * c.heads * 2 + i % 2);
+            else
+                for (uint32_t i = tid; i < n; i += THREADS) *reinterpret_cast<float2*>(st.s + 4 * i) = make_float2(1.0f, fixed);
         }
     };
     float* home = c.state + ((size_t(run.slot) * c.heads + head) * c.P + p0 + (mine ? col : 0)) * NP + 4 * lane;
@@ -225,7 +229,7 @@ __global__ void __launch_bounds__(L * COLS / PC, GROUP == 1 ? 0 : 1) scan_kernel
     cp_async_commit();
     const bool fresh = a.meta[2 * t0 + 1] == 0;  // a sequence begins: nothing of the slot's last one
     if (fresh) S.clear();
-    const float skip = CHANNEL ? 0.0f : bf16_to_f32(a.skip[head]);
+    const float skip = CHANNEL || !a.skip ? 0.0f : bf16_to_f32(a.skip[head]);
     const size_t ldy = size_t(c.heads) * c.P;
     float* Y = a.y + size_t(t0) * ldy + size_t(head) * c.P + p0 + col;
     if (verify) {
@@ -321,7 +325,7 @@ __global__ void __launch_bounds__(256) recurrent_commit_kernel(const RunIn* __re
         for (uint32_t j = 0; j < k; j++) {
             const size_t row = size_t(run.slot) * VERIFY_T + path[r * FEED_W + j];
             const float key = c.keep_k[(row * (c.heads / c.per) + head / c.per) * c.N + n], v = c.keep_v[(row * c.heads + head) * c.P + p];
-            const float* d = c.keep_d + (row * c.heads + head) * (c.channel_decay ? c.N : 2);
+            const float* d = c.keep_d + (row * c.heads + head) * (c.channel_decay ? c.N : 2);  // (with fixed decays: 1 and the decay)
             s = c.channel_decay ? fmaf(d[n], s, key * v) : fmaf(d[1], s, key * (v * d[0]));
         }
         S[e] = s;
@@ -505,7 +509,7 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormArgs a)
             load_bf16<V>(w, a.w + c0 + c);
 #pragma unroll
             for (uint32_t j = 0; j < V; j++) {
-                const float s = silu(z[j]), gated = v[j] * s;
+                const float s = a.sigmoid ? sigmoid_of(z[j]) : silu(z[j]), gated = v[j] * s;
                 ss += a.gate_first ? gated * gated : v[j] * v[j];
                 v[j] = gated * w[j];
             }

@@ -14,7 +14,7 @@ namespace vlt {
 // it sees from the node. meta[t] = (slot, lens[slot] + depth). One block per token.
 __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* tokens, float* __restrict__ out, const uint32_t* __restrict__ tin,
                              uint32_t* meta, const uint32_t* __restrict__ lens, const uint32_t* __restrict__ feed, const uint32_t* __restrict__ tree,
-                             uint32_t* vis, uint32_t d, uint32_t vocab, const uint16_t* __restrict__ positions, uint32_t n_positions) {
+                             uint32_t* vis, uint32_t d, uint32_t vocab, const uint16_t* __restrict__ positions, uint32_t n_positions, uint16_t* __restrict__ out_b) {
     pdl_start();
     const uint32_t t = blockIdx.x, tid = threadIdx.x;
     const uint32_t slot = tin[2 * t];
@@ -30,6 +30,8 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
     // An id past the vocabulary can only come from the device (a row of NaN logits has no argmax): read it as 0
     // rather than index out of the table.
     if (tok >= vocab) tok = 0;
+    if (out_b)  // (positions are another design's)
+        for (uint32_t i = tid; i < d; i += blockDim.x) out_b[size_t(t) * d + i] = table[size_t(tok) * d + i];
     if (positions) {  // (a draft's rows may reach past the last position: they are not kept then)
         const uint16_t* pv = positions + size_t(min(lens[slot] + depth, n_positions - 1)) * d;
         if (d % 4 == 0) {
@@ -63,8 +65,8 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
 
 void launch_embed(const uint16_t* table, uint32_t* tokens, float* out, const uint32_t* tin, uint32_t* meta, const uint32_t* lens,
                   const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s, const uint16_t* positions,
-                  uint32_t n_positions) {
-    launch_pdl(embed_kernel, n, 128, 0, s, table, tokens, out, tin, meta, lens, feed, tree, vis, d, vocab, positions, n_positions);
+                  uint32_t n_positions, uint16_t* out_b) {
+    launch_pdl(embed_kernel, n, 128, 0, s, table, tokens, out, tin, meta, lens, feed, tree, vis, d, vocab, positions, n_positions, out_b);
 }
 
 // ------------------------------------------------------- K/V into the cache

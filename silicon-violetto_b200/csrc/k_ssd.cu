@@ -1,5 +1,5 @@
-// The state space's recurrence over a prompt's portion on the tensor cores: S_t = d_t S_(t-1) + e_t k_t v_t^T with a number d_t per
-// head, 64 tokens at a time. With c_t the sum of the logarithms of d up to t within a chunk,
+// Recurrences with a number per head and token as their decay, over a prompt's portion on the tensor cores: S_t = d_t S_(t-1) + e_t k_t v_t^T
+// (the state space's; with e = 1 and a fixed d, linear attention's), 64 tokens at a time. With c_t the sum of the logarithms of d up to t within a chunk,
 //
 //   y_t = sum_(s <= t) (q_t . k_s) 2^(c_t - c_s) e_s v_s + 2^(c_t) q_t S,      S <- 2^(c_end) S + sum_s k_s (2^(c_end - c_s) e_s v_s)^T.
 //
@@ -65,7 +65,7 @@ __global__ void __launch_bounds__(THREADS) ssd_kernel(const ScanArgs a) {
     fetch(0);
     asm volatile("cp.async.commit_group;" ::: "memory");
     const bool fresh = a.meta[2 * t0 + 1] == 0;
-    const float rate = -expf(bf16_to_f32(a.a_log[head])) * LOG2E, skip = bf16_to_f32(a.skip[head]);
+    const float rate = c.fixed ? log2f(c.fixed[head]) : -expf(bf16_to_f32(a.a_log[head])) * LOG2E, skip = a.skip ? bf16_to_f32(a.skip[head]) : 0.0f;
     // The state: rows (key channels) n0 + 16 m + g and + 8, columns (value channels) 8 j + 2 tq and + 1.
     const uint32_t n0 = warp * 16 * MT;
     float* home = c.state + ((size_t(run.slot) * c.heads + head) * c.P + p0) * c.Np;
@@ -100,7 +100,7 @@ __global__ void __launch_bounds__(THREADS) ssd_kernel(const ScanArgs a) {
 #pragma unroll
         for (uint32_t u = 0; u < 2; u++) {
             const uint32_t i = ch * T + 2 * lane + u;
-            ahead[u] = i < count ? a.decay[(size_t(t0 + i) * c.heads + head) * 2] : 0.0f;
+            ahead[u] = i >= count ? 0.0f : c.fixed ? 1.0f : a.decay[(size_t(t0 + i) * c.heads + head) * 2];
         }
     };
     if (warp == 0) steps(0);

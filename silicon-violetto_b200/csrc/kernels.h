@@ -10,7 +10,11 @@
 namespace vlt {
 
 // Epilogues of a matmul, engine/src/engine/kernels.rs:3-9 and kernels.metal:154-209.
-enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI_RAW = 5, EPI_QKV = 6, EPI_HEAD_CAP = 7, EPI_RELU2 = 8 };  // 7: 23 sigmoid((acc + 5) / 7.5), kernels.metal:196-199; 8: max(acc, 0)^2
+enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI_RAW = 5, EPI_QKV = 6, EPI_HEAD_CAP = 7, EPI_RELU2 = 8,  // 7: 23 sigmoid((acc + 5) / 7.5), kernels.metal:196-199; 8: max(acc, 0)^2
+                EPI_SILU = 9,        // silu(acc) for rows below vocab_real, the others as they are
+                EPI_GLU = 10,        // rows in pairs (g, u): silu(g) u, half as many outputs; EPI_SWIGLU's without a norm
+                EPI_GLU_CLAMP = 11   // the same: g sigmoid(1.702 g) (u + 1), g cut off above a limit, u outside of +- the limit
+};
 
 // What the tensor-core GEMM's EPI_QKV epilogue needs to finish the qkv projection the way `qkv_post` does
 // (kernels.metal:749-801): RoPE on q and k, q scaled and rounded to bf16 for the attention, k and v rounded
@@ -31,6 +35,12 @@ struct QkvEpilogue {
 
 __device__ __forceinline__ float weight_of(const RowNorm& n, uint32_t i) { return (n.around_zero ? 1.0f : 0.0f) + bf16_to_f32(n.w[i]); }
 
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_of(1.702f * g) * (u + 1.0f);
+}
 template <uint32_t V>
 __device__ __forceinline__ void weights_of(float (&x)[V], const RowNorm& n, uint32_t i) {
     load_bf16<V>(x, n.w + i);
@@ -51,7 +61,7 @@ struct MatArgs {
     const float* inv_in;  // ... or, if not null, read from here (tensor-core GEMM)
     uint16_t* Yb;       // optional bf16 copy of Y (feeds the next tensor-core GEMM)
     uint32_t n, k, m, group;  // group: 0 for bf16 weights
-    uint32_t epi, vocab_real;
+    uint32_t epi, vocab_real;  // vocab_real: a head's rows from there on are padding; EPI_SILU: rows from there on stay as they are
     float eps;
     // kernels.metal:164-165,188-193: the matrix scale (qkv_scale, o_scale) and EPI_RESID's y = ra base + rb (scale acc). 1 for a
     // plain decoder.
@@ -70,7 +80,8 @@ struct MatArgs {
 
 void launch_embed(const uint16_t* table, uint32_t* tokens, float* out, const uint32_t* tin, uint32_t* meta, const uint32_t* lens,
                   const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s,
-                  const uint16_t* positions = nullptr, uint32_t n_positions = 0);  // positions: [n_positions][d], a vector per position to add
+                  const uint16_t* positions = nullptr, uint32_t n_positions = 0,  // positions: [n_positions][d], a vector per position to add
+                  uint16_t* out_b = nullptr);                                     // out in bf16
 void launch_qkv_post(const float* qkv, const uint32_t* meta, const uint32_t* tin, const float* rope, uint16_t* k_cache, uint16_t* v_cache,
                      const uint32_t* page_table, KvArgs kv, uint32_t layer, uint32_t n, uint32_t n_heads, float scale_log2, uint16_t* q_b, const uint32_t* cpos, cudaStream_t s);
 // q | k | v rows as the attention sees them before rounding (RoPE on q and k, kernels.metal:727-736), for step_capture.
@@ -219,13 +230,21 @@ struct LinearArgs {
     const float* base;       // EPI_RESID
     float* Y;                // optional, as is
     uint16_t* Yb;            // its bf16 copy
-    uint32_t n, m, k, epi;   // EPI_RAW, EPI_RESID or EPI_RELU2
+    uint32_t n, m, k, epi;   // EPI_RAW, EPI_RESID, EPI_RELU2, EPI_SILU, EPI_GLU or EPI_GLU_CLAMP
+    uint32_t act_rows;       // EPI_SILU
+    float limit;             // EPI_GLU_CLAMP
+    const float* row_scale;  // optional, with tiles: what row p's products are multiplied by, before the epilogue
+    // A matrix per head against that head's part of every token (by_head tokens; 0: not so): group g's rows are p = g by_head + t,
+    // read at row t heads + g of X and written at row t heads + g of Y, `ldy` apart. gate (optional): [by_head][ldg], the output is
+    // multiplied by the sigmoid of row t's column g m + r.
+    uint32_t by_head, heads, ldy, ldg;
+    const float* gate;
     const uint32_t* tiles;   // [.][3]: (group, first row, rows)
     const uint32_t* n_tiles;
     uint32_t max_tiles;      // at most so many tiles (the grid)
 };
 void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s);
-bool grouped_fits(uint32_t m, uint32_t k);  // the tensor-core form (k_grouped.cu): bf16 activations, EPI_RAW or EPI_RELU2
+bool grouped_fits(uint32_t m, uint32_t k);  // the tensor-core form (k_grouped.cu): bf16 activations, EPI_RAW, EPI_RELU2 or EPI_GLU_CLAMP
 void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint32_t* err_flag, cudaStream_t s);
 // out[r] = x / sqrt(mean x^2 + eps) times the weight times `scale`, x being row rows[r] (or r) of `in`, plus that of `add`, the
 // sum then left in `sum`.
@@ -254,14 +273,48 @@ struct MergeArgs {
     float eps;
 };
 void launch_merge_rows(const MergeArgs& a, cudaStream_t s);
+// out[r] = x[r] + y[r] / sqrt(mean y^2 + eps) times the weight, and its bf16 copy.
+struct AddNormArgs {
+    const float *x, *y;
+    RowNorm norm;
+    float* out;              // may be x
+    uint16_t* out_b;         // optional
+    uint32_t n, d;
+    float eps;
+};
+void launch_add_norm(const AddNormArgs& a, cudaStream_t s);
+// out[t][i] = gelu(x[t][i]) times entry first + i of token t's row in a bf16 table, i < dim; zeros from there to `wide`.
+struct SideGateArgs {
+    const float* x;          // [n][ldx]
+    const uint16_t* table;   // [vocab][ld]
+    const uint32_t* tokens;
+    float* out_f32;          // optional
+    uint16_t* out_bf16;      // optional
+    uint32_t n, ldx, ld, first, dim, wide;
+};
+void launch_side_gate(const SideGateArgs& a, cudaStream_t s);
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
 
-// One layer run's pages: [page][kv head][position in page][dk or dv] for K and for V, bf16 or fp32.
+// One layer run's pages: [page][kv head][position in page][dk or dv] for K and for V, bf16 or fp32. v == k: a value is its key's
+// first dv entries, and there is no V pool.
 struct PagedKv {
     void *k, *v;
     const uint32_t* page_table;
     uint32_t max_pages, page_shift, n_kv, dk, dv;
 };
+__device__ __forceinline__ size_t page_row(const PagedKv& kv, uint32_t slot, uint32_t g, uint32_t pos) {
+    const uint32_t page = kv.page_table[size_t(slot) * kv.max_pages + (pos >> kv.page_shift)], psize = 1u << kv.page_shift;
+    return (size_t(page) * kv.n_kv + g) * psize + (pos & (psize - 1));
+}
+// Entry c of a vector whose first `dims` entries turn (see Rotation); cs: the position's (cos, sin) per pair.
+__device__ __forceinline__ float rotated(const float* y, uint32_t c, uint32_t dims, bool neighbours, const float2* cs) {
+    const uint32_t half = dims / 2;
+    if (c >= dims) return y[c];
+    const float2 t = cs[neighbours ? c / 2 : c < half ? c : c - half];
+    const bool first = neighbours ? c % 2 == 0 : c < half;
+    const float other = y[neighbours ? c ^ 1u : first ? c + half : c - half];
+    return first ? y[c] * t.x - other * t.y : y[c] * t.x + other * t.y;
+}
 // A mixer's cache as the path compaction and the benchmark's fill see it (kv.n_kv 0: no pages; channels 0: no ring).
 struct MixerCache {
     PagedKv kv;
@@ -283,8 +336,9 @@ struct ConvArgs {
     float q_scale;
     uint32_t ldu, taps, ring_len, conv_channels, heads, rot_dims;
     bool write_ring;                      // false: launch_conv_state does it afterwards
-    float unit_eps;                       // with unit_qk: q's and k's heads over sqrt(mean square + unit_eps)
-    bool unit_qk;
+    float unit_eps;                       // with unit_qk: q's and k's heads over sqrt(mean square + unit_eps), times a weight (optional)
+    bool unit_qk, neighbours;             // neighbours: see Rotation
+    RowNorm q_norm, k_norm;
     QueryTemperature temp;
 };
 // Where the row `back` positions before token t lies: among the rows of its own tile of 8 that it descends from (its `vis` mask
@@ -319,13 +373,44 @@ struct ChunkedAttnArgs {
     PagedKv kv;
     const float* gate;                    // optional [n][ldg]: the output is multiplied by sigmoid(gate)
     uint32_t ldg, heads, chunk, window;   // what a position sees (see Attention); both 0: every position before
-    float scale;
+    float scale, softcap;                 // softcap: see Attention
     float* out;                           // optional [n][heads][dv]
     uint16_t* out_b;                      // optional
 };
 bool chunk_attn_fits(uint32_t dk, uint32_t dv, uint32_t page);  // k_chunk_attn.cu's kernels, bf16 caches; else launch_attn_any
 void launch_attn_chunked(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s);
+// What stands between a latent attention's projections (k_latent.cu). From the rows q | c | r of the first one: n(q) for the query
+// projection, and n(c) and r rotated into the cache (kv.dk entries a row).
+struct LatentRowsArgs {
+    const float* u;                       // [n][ldu]
+    RowNorm q_norm, kv_norm;
+    const float* rope;
+    const uint32_t *meta, *tin;
+    PagedKv kv;
+    float* q_f;                           // optional: [n][q_rank]
+    uint16_t* q_b;                        // optional
+    uint32_t ldu, q_rank, kv_rank, rot_dim;
+    bool own, neighbours;                 // own: (c ; r) is this layer's to write
+    float eps;
+};
+void launch_latent_rows(const LatentRowsArgs& a, uint32_t n, bool fp32, cudaStream_t s);
+// From the query projection's rows, per head dim | rot_dim: the first parts gathered [n][heads][dim], the rotated ones into their
+// place behind kv_rank entries of q [n][heads][kv_rank + rot_dim], all times `factor`; and the per-head products' table of tiles.
+struct LatentQueryArgs {
+    const float* u;                       // [n][ldu]
+    const float* rope;
+    const uint32_t* meta;
+    float *part_f, *q_f;                  // fp32 ...
+    uint16_t *part_b, *q_b;               // ... or bf16, each pair optional
+    uint32_t *tiles, *n_tiles;
+    uint32_t n, ldu, heads, dim, rot_dim, kv_rank, tile;
+    bool neighbours;
+    float factor;
+};
+void launch_latent_query(const LatentQueryArgs& a, cudaStream_t s);
+bool latent_attn_fits(uint32_t kv_rank, uint32_t rot_dim, uint32_t page);  // k_latent_attn.cu's kernels, bf16 caches; else launch_attn_any
+void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
 void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_caches,
                           bool fp32, cudaStream_t s);
 void launch_mixer_fill(const MixerCache* caches, uint32_t n_caches, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s);
@@ -335,6 +420,7 @@ void launch_mixer_fill(const MixerCache* caches, uint32_t n_caches, uint32_t slo
 // Np being N rounded up to a multiple of 32 (recurrent_pitch) with zeros behind.
 struct RecurrentCache {
     float* state;
+    const float* fixed;  // optional, without channel decays: [heads], every token's decay (its key's factor is 1)
     // The rows of a verified run, kept until it is known which of them stand: keys [slot][8][heads / per][N], decays
     // [slot][8][heads][N] or (key scale, decay) [slot][8][heads][2], values [slot][8][heads][P].
     float *keep_k, *keep_d, *keep_v;
@@ -344,9 +430,9 @@ struct RecurrentCache {
 struct ScanArgs {
     const float *q, *k, *v;  // row t's of head h at q + t ldq + (h / per) N, k likewise, v + t ldv + h P
     uint32_t ldq, ldk, ldv;
-    const float* decay;      // per channel: [n][heads][N]; else [n][heads][2] (the key's factor, the decay)
+    const float* decay;      // per channel: [n][heads][N]; else [n][heads][2] (the key's factor, the decay), unless c.fixed has them
     const float* bonus;      // per channel: [n][heads], what of v is added to the output, which is read before the update; ...
-    const uint16_t* skip;    // ... else per head bf16, the output being read after it
+    const uint16_t* skip;    // ... else per head bf16 (optional), the output being read after it
     RecurrentCache c;
     const RunIn* runs;
     const GenState* gen;     // a sequence that has ended keeps its state
@@ -395,12 +481,13 @@ struct DecayArgs {
     float *decay, *bonus;    // [n][heads][dim], [n][heads]
 };
 void launch_decay(const DecayArgs& a, uint32_t n, cudaStream_t s);
-// Rows of `groups` equal parts, each over its own root mean square, times w; silu(gate) goes on before the norm or at the end.
+// Rows of `groups` equal parts, each over its own root mean square, times w; silu(gate), or sigmoid(gate), goes on before the norm
+// or at the end.
 struct GatedNormArgs {
     const float *y, *gate;   // [n][width], [n][ldg]
     const uint16_t* w;
     uint32_t width, ldg, groups;
-    bool gate_first;
+    bool gate_first, sigmoid;
     float eps;
     float* out_f32;          // optional
     uint16_t* out_bf16;      // optional
@@ -410,8 +497,9 @@ void launch_gated_norm(const GatedNormArgs& a, uint32_t n, cudaStream_t s);
 // A mixture of experts (k_moe.cu).
 struct RouterArgs {
     const float* x;                       // the stream [n][d]
-    RowNorm norm;
-    const uint16_t *router, *correction;
+    RowNorm norm;                         // optional
+    const uint16_t *router, *correction;  // correction: optional
+    bool sigmoid, renormalized;           // see ExpertLayer
     float* xn;                            // optional: its normed rows
     uint16_t* xn_b;                       // optional, bf16
     uint32_t* ids;                        // [n][top]; experts and beyond: an identity expert
@@ -423,6 +511,8 @@ void launch_router(const RouterArgs& a, cudaStream_t s);
 struct SortArgs {
     const uint32_t* ids;
     uint32_t *src, *place;                // row -> token, (token, choice) -> row
+    const float* weights;                 // with row_weight: [n][top], sorted into it
+    float* row_weight;                    // optional
     uint32_t *tiles, *n_tiles;
     uint32_t n, top, experts, tile;
 };
@@ -430,8 +520,9 @@ void launch_expert_sort(const SortArgs& a, cudaStream_t s);
 struct CombineArgs {
     const float *x, *y, *xn, *shared;     // the stream, the experts' rows, the normed stream, the shared expert's rows (optional)
     const uint32_t *ids, *place;
-    const float* weights;
+    const float* weights;                 // optional (1)
     float* out;                           // may be x
+    RowNorm post;                         // optional: of the sum, before it goes onto x; next_b is then the new row itself
     RowNorm norm;                         // optional: the next layer's norm, into next / next_b
     float* next;
     uint16_t* next_b;

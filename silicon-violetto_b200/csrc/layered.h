@@ -1,5 +1,5 @@
 // Model folders: decoders whose config.json lists their layers one by one. This file has the mechanisms a layer can hold, each a
-// parameter struct of its own, the list of layer runs, and what the readers of the designs (lonasun.h, leduvik.h) share: the
+// parameter struct of its own, the list of layer runs, and what the readers of the designs (lonasun.h, leduvik.h, pasovik.h) share: the
 // tensors' places and the loop over a span of layers. A design's reader fills it; engine_layered.cu runs it.
 #pragma once
 #include <memory>
@@ -20,10 +20,12 @@ struct ShortConv {
     const uint16_t *w = nullptr, *b = nullptr;  // [channels][taps] bf16, no weights: none; [channels], optional
     uint32_t channels = 0, taps = 1;
 };
-// Dimensions i and i + dims / 2 of a head's first `dims` turn by position * base^(-2 i / dims).
+// Pairs of a head's first `dims` dimensions -- i and i + dims / 2, or the neighbours 2 i and 2 i + 1 -- turn by
+// position * base^(-2 i / dims) / factor.
 struct Rotation {
     uint32_t dims = 0;
-    double base = 1;
+    double base = 1, factor = 1;
+    bool neighbours = false;
     uint32_t table = 0;  // index among the model's rotations
 };
 // Queries are multiplied by 1 + coef ln(floor((position + 1) / every) + 1). every 0: not at all.
@@ -36,8 +38,10 @@ struct QueryTemperature {
 struct Attention {
     uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, chunk = 0, window = 0;
     float scale = 1;
-    bool unit_qk = false;  // q's and k's heads are divided by their root mean square
-    bool gated = false;    // the output times sigmoid(gate)
+    float softcap = 0;       // scores become softcap tanh(score / softcap); 0: they stay
+    bool unit_qk = false;    // q's and k's heads are divided by their root mean square, ...
+    RowNorm q_norm, k_norm;  // ... and multiplied by a weight of one head's size (optional)
+    bool gated = false;      // the output times sigmoid(gate)
     Rotation rot;
     QueryTemperature temp;
     ShortConv conv;  // over q | k | v
@@ -65,24 +69,67 @@ struct TimeMix {
     const uint16_t *w2 = nullptr, *w0 = nullptr, *bonus = nullptr, *norm = nullptr;  // w2 [heads dim][rank], bonus [heads][dim]
     uint32_t inner() const { return heads * dim; }
 };
-enum class MixerKind { Attention, StateSpace, TimeMix };
+// Attention whose keys and values are linear in a short normed row c of every position: per head, the key is (W_uk c ; r) with a
+// rotated part r that all heads share, the value W_uv c. Only (c ; r) is kept. W_uk goes onto the queries and W_uv onto the sums of
+// c: the heads are query heads of one kv head whose key is (c ; r) and whose value is c. Queries come from a normed row of their own.
+struct LatentAttention {
+    static constexpr uint32_t OWN = 0xffffffffu;
+    uint32_t heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0, q_rank = 0;
+    float scale = 1;
+    Rotation rot;             // of the rotated parts
+    uint32_t kv_from = OWN;   // the layer whose (c ; r) this one reads
+    Matrix in;                // W_dq | W_dkv (unless kv_from) | W_g stacked
+    Matrix uq, uk_t, uv, o;   // uk_t, uv: per head [kv_rank][dim] and [vdim][kv_rank], stacked
+    RowNorm q_norm, kv_norm;
+    uint32_t key_w() const { return kv_rank + rot_dim; }
+    uint32_t out_w() const { return heads * vdim; }
+    uint32_t kv_w() const { return kv_from == OWN ? key_w() : 0; }  // rows of W_dkv in `in`
+};
+// Linear attention with a fixed decay per head: S = d_h S + k v^T, o = S^T q; q, k and v through silu; o normed as one row, times
+// sigmoid(gate).
+struct LinearAttention {
+    uint32_t heads = 0, dim = 0, vdim = 0;
+    std::vector<float> decay;
+    Matrix proj, o;  // proj: q | k | v | gate
+    RowNorm norm;
+    uint32_t qkv_w() const { return heads * (2 * dim + vdim); }
+    uint32_t out_w() const { return heads * vdim; }
+};
+enum class MixerKind { Attention, StateSpace, TimeMix, Latent, Linear };
 struct Mixer {
     MixerKind kind = MixerKind::Attention;
     Attention attn;
     StateSpace ssm;
     TimeMix tmix;
+    LatentAttention latent;
+    LinearAttention linear;
     RowNorm out;  // on the output, in layers of several mixers
 };
-// relu(W_up h)^2 through W_down, `top` of `experts` + `identity` per token, softmax scores, a shared expert (ff 0: none).
+// A feed-forward's hidden rows: relu(W_up h)^2; silu(g) u with (g, u) = (W_gate, W_up) h; or g sigmoid(1.702 g) (u + 1) with g cut
+// off above `limit` and u outside of +- limit.
+enum class Hidden { Relu2, SiluGlu, ClampedGlu };
+inline uint32_t hidden_rows(Hidden h, uint32_t ff) { return h == Hidden::Relu2 ? ff : 2 * ff; }  // of `up`: with a gate, its rows and W_up's in turn
+// `top` of `experts` + `identity` per token, scores by softmax or sigmoid, the chosen ones' summing to 1 or as they are; a shared
+// expert (ff 0: none).
 struct ExpertLayer {
     uint32_t experts = 0, identity = 0, top = 0, ff = 0, shared_ff = 0;
-    const uint16_t *router = nullptr, *correction = nullptr;  // [experts + identity][d], [experts + identity]
-    Matrix up, down;                                          // all experts': [experts * ff][d], [experts * d][ff]
+    Hidden hidden = Hidden::Relu2;
+    float limit = 0;
+    bool sigmoid = false, renormalized = true;
+    bool scales_input = false;                                // a score multiplies its expert's input, not its output
+    const uint16_t *router = nullptr, *correction = nullptr;  // [experts + identity][d], [experts + identity] (optional)
+    Matrix up, down;                                          // all experts': [experts * rows][d], [experts * d][ff]
     Matrix shared_up, shared_down;
 };
-// W_down relu(W_up h)^2.
 struct DenseLayer {
+    Hidden hidden = Hidden::Relu2;
     Matrix up, down;
+};
+// n(W_proj (gelu(W_gate x) * e)) onto the stream, e a span of the token's row in the model's side table; gelu by tanh.
+struct SideInput {
+    uint32_t dim = 0, first = 0;  // the span; dim 0: none
+    Matrix gate, proj;            // gate's rows and proj's columns padded with zeros
+    RowNorm norm;
 };
 enum class MlpKind { None, Experts, Dense };
 struct FolderLayer {
@@ -91,6 +138,8 @@ struct FolderLayer {
     MlpKind mlp = MlpKind::None;
     ExpertLayer experts;
     DenseLayer dense;
+    bool post_norm = false;  // norm1 and norm2 go onto what the mixer and the feed-forward leave; both read the stream itself
+    SideInput side;          // (layers with post_norm)
 };
 // A layer run: with a loop a layer runs several times, each with a cache of its own.
 struct LayerRun {
@@ -121,6 +170,8 @@ struct LayeredModel {
     Matrix loop_in, head;
     const uint16_t *embed = nullptr, *positions = nullptr;  // positions: a learned vector per position (optional)
     uint32_t n_positions = 0;                               // rows of it; sequences are no longer than that
+    const uint16_t* side = nullptr;                         // the layers' side inputs: a row of side_w per token id (optional)
+    uint32_t side_w = 0;
     RowNorm final_norm;
     float logit_scale = 1;
 
@@ -179,6 +230,11 @@ struct LayeredModel {
         a.vdim = m.at("vdim").count("vdim");
         a.scale = float(m.at("scale").number("scale"));
     }
+    // The rotation's table is the model's: one for all layers that turn alike.
+    void share(Rotation& rot) {
+        rot.table = uint32_t(std::find_if(rotations.begin(), rotations.end(), [&](const Rotation& r) { return r.dims == rot.dims && r.base == rot.base && r.factor == rot.factor; }) - rotations.begin());
+        if (rot.table == rotations.size()) rotations.push_back(rot);
+    }
     void check_taps(const ShortConv& c, const std::string& pre) const {
         if (c.taps == 0 || c.taps > MAX_TAPS) throw Error(pre + ": a convolution takes 1 to " + std::to_string(MAX_TAPS) + " taps");
     }
@@ -210,13 +266,19 @@ struct LayeredModel {
         md.n_layers = uint32_t(runs.size());
         for (const FolderLayer& l : layers) {
             for (const Mixer& x : l.mix) {
+                if (x.kind == MixerKind::Latent) {
+                    md.n_heads = std::max(md.n_heads, x.latent.heads);
+                    md.n_kv = std::max(md.n_kv, 1u);
+                    md.hd = std::max(md.hd, x.latent.dim + x.latent.rot_dim);
+                    if (md.attn_scale == 0) md.attn_scale = x.latent.scale;
+                }
                 if (x.kind != MixerKind::Attention) continue;
                 md.n_heads = std::max(md.n_heads, x.attn.heads);
                 md.n_kv = std::max(md.n_kv, x.attn.kv_heads);
                 md.hd = std::max(md.hd, x.attn.dim);
                 if (md.attn_scale == 0) md.attn_scale = x.attn.scale;
             }
-            md.ffn = std::max(md.ffn, std::max(l.experts.ff, l.dense.up.m));
+            md.ffn = std::max(md.ffn, std::max(l.experts.ff, l.dense.down.k));
         }
     }
 };

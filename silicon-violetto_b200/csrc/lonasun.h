@@ -26,9 +26,7 @@ inline void read_layer(LayeredModel& model, const Json& c, const std::string& pr
     a.rot.base = m.at("rot").at("base").number("rot.base");
     if (a.rot.dims % 2 || a.rot.dims > a.dim) throw Error(pre + ": rot.dims does not fit the heads");
     model.check_taps(a.conv, pre);
-    auto& rotations = model.rotations;
-    a.rot.table = uint32_t(std::find_if(rotations.begin(), rotations.end(), [&](const Rotation& r) { return r.dims == a.rot.dims && r.base == a.rot.base; }) - rotations.begin());
-    if (a.rot.table == rotations.size()) rotations.push_back(a.rot);
+    model.share(a.rot);
     const std::string mx = pre + "mix.";
     model.attention_matrices(a, mx, d);
     const uint32_t qw = a.heads * a.dim, kw = a.kv_heads * a.dim, vw = a.kv_heads * a.vdim;

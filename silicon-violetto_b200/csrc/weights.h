@@ -142,7 +142,7 @@ struct SafeTensors {
         std::memcpy(&n, base, 8);
         if (n > map_bytes - 8) throw Error(p + ": the header is longer than the file");
         const Json head = Json::parse(reinterpret_cast<const char*>(base + 8), n, p);
-        const size_t room = map_bytes - 8 - n;
+        const size_t left = map_bytes - 8 - n;
         size_t total = 0;
         for (const auto& [name, t] : head.fields) {
             if (name == "__metadata__") continue;
@@ -156,13 +156,13 @@ struct SafeTensors {
             const std::vector<Json>& off = t.at("data_offsets").items;
             if (off.size() != 2) throw Error(name + ": bad data_offsets");
             const double a = off[0].number("data_offsets"), b = off[1].number("data_offsets");
-            if (!(a >= 0 && b >= a && b <= double(room))) throw Error(name + ": its data lies outside the file");
+            if (!(a >= 0 && b >= a && b <= double(left))) throw Error(name + ": its data lies outside the file");
             e.data = base + 8 + n + size_t(a);
             e.nbytes = size_t(b - a);
             const size_t size = e.dtype == "BF16" || e.dtype == "F16" ? 2 : e.dtype == "F32" || e.dtype == "I32" ? 4 : 0;
             if (size && e.nbytes != count * size) throw Error(name + ": its data does not fit its shape");
             total += e.nbytes + 256;
-            if (e.shape.size() == 2) total += size_t(128) * e.shape[1] * 2;  // (room for `zeros`; untouched pages of it cost nothing)
+            if (e.shape.size() == 2) total += size_t(128) * e.shape[1] * 2 + size_t(126) * e.shape[0];  // (room for `zeros` and `place_wide`; untouched pages of it cost nothing)
             entries[name] = e;
         }
         buffer.alloc(total + 256, true);  // (filled on the host, then moved to the device in one copy: see to_device)
@@ -182,11 +182,36 @@ struct SafeTensors {
     // placed before it without a gap (a stack of rows).
     size_t place(const std::string& name, const std::vector<uint32_t>& shape, bool fresh = true) {
         const Entry& e = get(name, shape);
-        if (fresh) used = (used + 255) / 256 * 256;
-        const size_t at = used;
-        if (at + e.nbytes > buffer.bytes) throw Error(path + ": a tensor is placed twice");
+        const size_t at = room(e.nbytes, fresh);
         std::memcpy(buffer.as<uint8_t>() + at, e.data, e.nbytes);
-        used += e.nbytes;
+        return at;
+    }
+    // Two matrices of one shape with their rows in turn: a, b, a, b, ...
+    size_t place_pairs(const std::string& a, const std::string& b, const std::vector<uint32_t>& shape, bool fresh = true) {
+        const Entry &ea = get(a, shape), &eb = get(b, shape);
+        const size_t row = size_t(shape[1]) * 2, at = room(2 * ea.nbytes, fresh);
+        uint8_t* dst = buffer.as<uint8_t>() + at;
+        for (size_t r = 0; r < shape[0]; r++) {
+            std::memcpy(dst + 2 * r * row, ea.data + r * row, row);
+            std::memcpy(dst + (2 * r + 1) * row, eb.data + r * row, row);
+        }
+        return at;
+    }
+    // A stack of `blocks` matrices [rows][k], each as its transpose [k][rows].
+    size_t place_transposed(const std::string& name, uint32_t blocks, uint32_t rows, uint32_t k) {
+        const Entry& e = get(name, {blocks * rows, k});
+        const size_t at = room(e.nbytes, true);
+        uint16_t* dst = reinterpret_cast<uint16_t*>(buffer.as<uint8_t>() + at);
+        for (size_t b = 0; b < blocks; b++)
+            for (size_t r = 0; r < rows; r++)
+                for (size_t c = 0; c < k; c++) std::memcpy(dst + (b * k + c) * rows + r, e.data + ((b * rows + r) * k + c) * 2, 2);
+        return at;
+    }
+    // A matrix [rows][k] with columns of zeros up to `wide`, fewer than 64 of them.
+    size_t place_wide(const std::string& name, uint32_t rows, uint32_t k, uint32_t wide) {
+        const Entry& e = get(name, {rows, k});
+        const size_t at = room(size_t(rows) * wide * 2, true);
+        for (size_t r = 0; r < rows; r++) std::memcpy(buffer.as<uint8_t>() + at + r * wide * 2, e.data + r * k * 2, size_t(k) * 2);
         return at;
     }
     // Zero bytes after the tensor placed last.
@@ -212,6 +237,13 @@ struct SafeTensors {
     }
 
   private:
+    size_t room(size_t nbytes, bool fresh) {
+        if (fresh) used = (used + 255) / 256 * 256;
+        const size_t at = used;
+        if (at + nbytes > buffer.bytes) throw Error(path + ": a tensor is placed twice");
+        used += nbytes;
+        return at;
+    }
     void* map = nullptr;
     size_t map_bytes = 0;
 };
