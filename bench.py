@@ -402,6 +402,53 @@ def leduvik_work(size):
     return c, {"leduvik": at(seen + ctx, ctx * ctx / 2 + seen * (ctx - seen / 2), ours, state), "plain": at(3 * ctx, 3 * ctx * ctx / 2, plain, 0)}
 
 
+# Layers of real models' sizes, in blocks of the design's three kinds, as many and as wide as Leduvik's above, which is the
+# framework's closest other model; a later block's latent layer reads the first one's rows.
+PASOVIK_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536), linear=16, ff=5376,
+                 moe=dict(experts=64, top=8, ff=640), side=256, vocab=32768, blocks=2, ctx=8000),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536), linear=32, ff=9472,
+                 moe=dict(experts=32, top=4, ff=2304), side=256, vocab=32768, blocks=1, ctx=1900),
+}
+
+
+def pasovik_files(size):
+    """A Pasovik model (PASOVIK_SIZES) beside leduvik_files's two, random-init, bf16, written once per box."""
+    from silicon_violetto_b200 import pasovik
+    CACHE.mkdir(parents=True, exist_ok=True)
+    c = PASOVIK_SIZES[size]
+    layers = []
+    for b in range(c["blocks"]):
+        layers += [pasovik.lightning(128, 128, [1 - 2.0 ** -(2 + 8 * h / c["linear"]) for h in range(c["linear"])], mlp=pasovik.dense(c["ff"])),
+                   pasovik.attention(c["heads"], c["kv_heads"], c["dim"], c["dim"], softcap=50.0, rot_dims=64, base=500000.0, factor=8.0, mlp=pasovik.moe(**c["moe"])),
+                   pasovik.latent(**c["latent"], base=500000.0, kv_from=2 if b else None, mlp=pasovik.dense(c["ff"]))]
+    folder = CACHE / f"pasovik_{size}"
+    if not (folder / "ok").exists():
+        cfg = pasovik.config(c["width"], c["vocab"], layers, side=c["side"])
+        pasovik.write_model(folder, cfg, pasovik.random_weights(cfg))
+        (folder / "ok").write_text("ok")
+    return (folder, *leduvik_files(size))
+
+
+def pasovik_work(size):
+    """What a Pasovik model of PASOVIK_SIZES reads and computes, beside leduvik_work's."""
+    c = PASOVIK_SIZES[size]
+    d, ctx, B, l, m = c["width"], c["ctx"], c["blocks"], c["latent"], c["moe"]
+    attn_p = ((2 * c["heads"] + 2 * c["kv_heads"]) * c["dim"]) * d
+    lin_p = 5 * c["linear"] * 128 * d
+    lat_p = (l["q_rank"] + 2 * l["heads"] * l["vdim"]) * d + l["heads"] * (l["q_rank"] * (l["dim"] + l["rot_dim"]) + l["kv_rank"] * (l["dim"] + l["vdim"]))
+    own_p = (l["kv_rank"] + l["rot_dim"]) * d  # the first latent layer's alone
+    common = B * (attn_p + lin_p + lat_p + 2 * 3 * c["ff"] * d + 3 * 2 * c["side"] * d) + own_p
+    experts = lambda touched: B * touched * 3 * m["ff"] * d
+    touched = lambda n: m["experts"] * (1 - (1 - m["top"] / m["experts"]) ** n)
+    row = l["kv_rank"] + l["rot_dim"]
+    kv = B * 2 * (2 * c["kv_heads"] * c["dim"] + row) * ctx
+    flops = B * 2.0 * (2 * c["heads"] * c["dim"] + l["heads"] * (row + l["kv_rank"])) * ctx * ctx / 2  # (as the kernel does them: all heads on the rows)
+    ours = {"decode_weights": lambda n: common + experts(touched(n)), "prompt_weights": common + experts(m["top"]), "kv": kv, "state": B * 2 * 4 * c["linear"] * 128 * 128,
+            "attention_flops": flops}
+    return c, {"pasovik": ours, **leduvik_work(size)[1]}
+
+
 def folder_figure(E, local, c, files, work, steps, stream_counts, hbm_peak, tc_peak):
     """Decoding over a filled context and a prompt of the same length in portions of 512, the folder's model and the plain
     decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their own) the
@@ -512,11 +559,11 @@ def main():
     ap.add_argument("--attn-keys", type=int, default=0, help="keys per attention block (0: the engine's own choice)")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers: a profiler-size case, not a bench value")
     ap.add_argument("--no-limite", action="store_true", help="skip the reference-architecture pass of the extras (it writes a 2 GB file first)")
-    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite, lonasun and leduvik")
+    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite, lonasun, leduvik and pasovik")
     ap.add_argument("--limite-drafter", action="store_true", help="--only limite: with the reference's block drafter loaded (tree drafts of up to 8 rows)")
     ap.add_argument("--limite-int8", action="store_true", help="--only limite: int8 weights in the reference converter's default groups (64; the head 8)")
     ap.add_argument("--limite-keys", type=int, default=0, help="--only limite: keys per attention block (VltTuning.attn_keys_per_cta); 0 = the library's choice")
-    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) 'lonasun' or 'leduvik' (models of those designs beside plain decoders of equal size): run that one pass alone and print its figure (not the bench line)")
+    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) 'lonasun', 'leduvik' or 'pasovik' (models of those designs beside others of equal size): run that one pass alone and print its figure (not the bench line)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank, world, local = int(os.environ.get("RANK", 0)), int(os.environ.get("WORLD_SIZE", 1)), int(os.environ.get("LOCAL_RANK", 0))
@@ -562,9 +609,10 @@ def main():
     solo = lambda: torch.cuda.synchronize(local)
     _package()
     from silicon_violetto_b200 import engine as E
-    if args.only in ("lonasun", "leduvik"):
+    if args.only in ("lonasun", "leduvik", "pasovik"):
         peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
-        sizes, files, work = {"lonasun": (LONASUN_SIZES, lonasun_files, lonasun_work), "leduvik": (LEDUVIK_SIZES, leduvik_files, leduvik_work)}[args.only]
+        sizes, files, work = {"lonasun": (LONASUN_SIZES, lonasun_files, lonasun_work), "leduvik": (LEDUVIK_SIZES, leduvik_files, leduvik_work),
+                              "pasovik": (PASOVIK_SIZES, pasovik_files, pasovik_work)}[args.only]
         figures = {}
         for n in sizes:
             c, w = work(n)
@@ -581,7 +629,7 @@ def main():
         elif args.only == "limite":
             print(json.dumps(limite_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], args.limite_keys, args.limite_drafter, args.limite_int8)))
         else:
-            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite', 'lonasun' or 'leduvik'")
+            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite', 'lonasun', 'leduvik' or 'pasovik'")
         return
     total = args.warmup + args.steps + 6
     # The headline pass, on every rank: the int8 target with the chain drafter loaded (1 layer + fc + a head over 16 384 draft

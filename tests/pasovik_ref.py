@@ -44,21 +44,18 @@ def soften(score, cap):
     return cap * np.tanh(score / cap)
 
 
-def softmax_sum(score, v):
-    """score [keys], v [keys, size]."""
-    p = np.exp(score - score.max())
-    return (p / p.sum()) @ v
-
-
 def causal(q, k, v, scale, cap=None):
     """q [time, H, dim], k [time, G, dim], v [time, G, vdim] -> [time, H, vdim]: every position over itself and all before it."""
     time, heads, _ = q.shape
     per = heads // k.shape[1]
     out = np.zeros((time, heads, v.shape[2]))
-    for t in range(time):
-        for h in range(heads):
-            s = (k[:t + 1, h // per] @ q[t, h]) * scale
-            out[t, h] = softmax_sum(soften(s, cap) if cap else s, v[:t + 1, h // per])
+    for h in range(heads):
+        s = q[:, h] @ k[:, h // per].T * scale
+        if cap:
+            s = soften(s, cap)
+        s = np.where(np.tri(time, dtype=bool), s, -np.inf)
+        p = np.exp(s - s.max(axis=1, keepdims=True))
+        out[:, h] = p / p.sum(axis=1, keepdims=True) @ v[:, h // per]
     return out
 
 
@@ -96,13 +93,10 @@ def latent_attention(x, w, pre, m, eps, kept):
 
 def lightning_core(q, k, v, decay):
     """q, k [time, H, dim], v [time, H, vdim]: the state fades, takes the token in, and is read."""
-    time, heads, dim = q.shape
-    out = np.zeros((time, heads, v.shape[2]))
-    for h in range(heads):
-        S = np.zeros((dim, v.shape[2]))
-        for t in range(time):
-            S = decay[h] * S + np.outer(k[t, h], v[t, h])
-            out[t, h] = S.T @ q[t, h]
+    S, out = np.zeros((q.shape[1], q.shape[2], v.shape[2])), np.zeros_like(v)
+    for t in range(len(q)):
+        S = np.asarray(decay)[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out[t] = np.einsum("hkv,hk->hv", S, q[t])
     return out
 
 
