@@ -175,12 +175,12 @@ void Engine::init_layered() {
                 shared.push_back(x.kind == MixerKind::Latent && x.latent.kv_from != LatentAttention::OWN);
                 if (x.kind == MixerKind::Attention) {
                     const Attention& a = x.attn;
-                    c.kv = PagedKv{kv.k.as<uint8_t>() + kv.k_off[i] * es, kv.v.as<uint8_t>() + kv.v_off[i] * es, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, a.kv_heads, a.dim, a.vdim};
+                    c.kv = PagedKv{kv.k.as<uint8_t>() + kv.k_off[i] * es, kv.v.as<uint8_t>() + kv.v_off[i] * es, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, a.kv_heads, a.dim, a.vdim, kv.n_pages};
                     if (a.conv.w) { c.channels = a.conv.channels; c.ring_len = a.conv.taps - 1 + VERIFY_T; }
                 } else if (x.kind == MixerKind::Latent) {
                     const LatentAttention& a = x.latent;
                     void* keys = kv.k.as<uint8_t>() + kv.k_off[i] * es;
-                    c.kv = PagedKv{keys, keys, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, 1, a.key_w(), a.kv_rank};
+                    c.kv = PagedKv{keys, keys, kv.page_table.as<uint32_t>(), kv.max_pages, page_shift, 1, a.key_w(), a.kv_rank, kv.n_pages};
                     if (shared.back()) c.kv = z.run[last[a.kv_from]].kv;
                 } else {
                     const bool tm = x.kind == MixerKind::TimeMix, lin = x.kind == MixerKind::Linear;
@@ -556,7 +556,7 @@ void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x,
     at.out = f32 ? z.mid_f.as<float>() : nullptr;
     at.out_b = f32 ? nullptr : z.mid_b.as<uint16_t>();
     sp = span_begin(G_ATTN);
-    if (fast_attn) launch_attn_latent(at, n, p.chunked ? p.ctiles : 0, p.max_keys, sm_count, tuning.attn_keys_per_cta, stream);
+    if (fast_attn) launch_attn_latent(at, n, p.chunked ? p.ctiles : 0, p.max_keys, sm_count, tuning.attn_keys_per_cta, s.err_flag.as<uint32_t>(), stream);
     else launch_attn_any(at, n, f32, stream);
     span_end(sp);
     l.W = reinterpret_cast<const uint16_t*>(x.uv.w);  // W_uv on a head's sum of c, and the gate

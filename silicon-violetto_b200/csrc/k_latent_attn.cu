@@ -1,297 +1,434 @@
-// Latent attention over paged rows (c ; r) on the tensor cores (sizes it does not take and fp32 caches: k_mixer.cu's scalar kernel).
-// All query heads read one row per position, whose first part is the value as well: what a row costs to fetch is shared by as
-// many (token, head) rows as a block holds.
+// Latent attention over paged rows (c ; r) on the 5th-generation tensor cores (sizes it does not take and fp32 caches: k_mixer.cu's
+// scalar kernel). All query heads read one row per position, whose first part is the value as well, so a block's (token, head) rows
+// share the rows it fetches:
 //
-//   A block has 16, 32 or 64 (token, head) rows of one run -- decoding, a token's heads; a prompt's portion, the heads of several
-//   neighbouring tokens -- and goes through its share of the run's pages 32 positions at a time, which asynchronous copies bring
-//   into a ring. Eight warps split the scores by rows and positions (16 rows: also by the columns they sum over), meet in shared
-//   memory for the softmax in fp32, and split the sums of c by rows and columns. A row's positions may be split over a cluster of
-//   blocks, each of which finishes a span of the columns from what the others store into its shared memory.
+//   S[row][position] = Q (c ; r)^T          the rows are the MMA's M side (64, as many of them as a block has meaning something)
+//   O^T[column][row] += c^T P^T             128 columns of c a time are its M side, the rows its N side
+//
+// so that O takes rows x columns / 128 of tensor memory's columns, and c is read as it lies: its positions are the second product's
+// k side, 64 neighbouring columns a swizzled line. A block has 16, 32 or 64 (token, head) rows of one run -- decoding, a token's
+// heads; a prompt's portion, the heads of several neighbouring tokens -- and goes through its share of the run's positions a tile
+// at a time:
+//
+//   warp 0       a tile of rows by TMA, 64 columns a box, into a ring of stages
+//   warp 1       the MMAs: the scores of the tile to come in front of this tile's sums
+//   warps 2..5   softmax in fp32 (a warp has 16 rows: 64 MMA rows lie on the first 16 lanes of each quarter of tensor memory), P in bf16
+//                through shared memory; the running maximum moves when a score exceeds it by more than 8, and only then does O come
+//                through registers; in the end O
+//
+// A row's positions may be split over a cluster of blocks, each of which finishes a span of the columns from what the others store
+// into its shared memory. Every wait is bounded: when one runs out, the kernel sets the error word, waits for nothing more, and
+// leaves by the way it always does.
 //
 // It takes q with scale * log2(e) folded in, rounded to bf16, and leaves the sums in bf16 for the per-head product after it.
 #include <algorithm>
+#include <map>
+#include <tuple>
 
 #include "paged_attn.cuh"
+#include "tcgen05.cuh"
 
 namespace vlt {
 
 namespace latent {
 
+using gemm::elect_one;
+using gemm::instr_desc;
+using gemm::mbar_arrive;
+using gemm::mbar_expect_tx;
+using gemm::mbar_init;
+using gemm::mma_commit;
+using gemm::mma_f16;
+using gemm::tma_load_2d;
+using gemm::tmem_ld16;
+using gemm::wait_or_abort;
 using namespace paged;
 
-constexpr uint32_t WARPS = 8, THREADS = WARPS * 32, KT = 32, EXTRA = 64, MAX_SPLITS = 16;  // EXTRA: room for the rotated part behind R columns
+constexpr uint32_t THREADS = 192, SOFTMAX = 128, MAX_SPLITS = 16, MAX_STAGES = 6, MISC = 2048;
+constexpr uint32_t SMEM = 227 * 1024, SMEM_MIN = 116 * 1024;  // (at least half an SM's: one block an SM, which never waits for another's tensor memory)
+template <uint32_t ROWS>
+constexpr uint32_t tile_keys() { return ROWS == 64 ? 64 : 32; }
 
-// R: columns of c a block is laid out for; ROWS: its (token, head) rows.
-template <uint32_t R, uint32_t ROWS>
-struct Shape {
-    static constexpr uint32_t WIDTH = R + EXTRA, PITCH = WIDTH * 2 + 16, STAGE = KT * PITCH;           // a staged row; bytes that keep ldmatrix free of conflicts
-    static constexpr uint32_t RG = ROWS / 16, KG = RG == 4 ? 2 : 4, KH = WARPS / (RG * KG);             // row groups, key groups, parts of the columns
-    static constexpr uint32_t NT = KT / KG / 8;                                                         // scores: tiles of 8 keys of a warp
-    static constexpr uint32_t CG = WARPS / RG, CW = R / CG < 16 ? 16 : R / CG;                          // sums: column groups, columns of a warp
-    static constexpr uint32_t STAGES = ROWS == 16 ? 5 : ROWS == 32 ? 4 : 3;
-    static constexpr uint32_t TPR = THREADS / ROWS, KPT = KT / TPR, SP = KT + 4, PP = KT + 8;           // softmax: threads of a row, keys of a thread; pitches
-    static constexpr uint32_t O_Q = STAGES * STAGE, O_S = O_Q + ROWS * PITCH, O_P = O_S + KH * ROWS * SP * 4, O_STAT = O_P + ROWS * PP * 2;
-    static constexpr uint32_t BYTES = O_STAT + ROWS * 12 + MAX_SPLITS * ROWS * 8;
-    static_assert(ROWS * R * 4 <= O_STAT, "the cluster's sums must fit in front of the statistics");
-    static_assert(BYTES <= 227 * 1024, "shared memory");
+struct Map {
+    alignas(64) uint8_t a[128];
 };
+struct Args {
+    ChunkedAttnArgs c;
+    uint32_t groups, sub, toks;                      // see latent_kernel
+    uint32_t blocks, ksteps, mtiles, stages, tmem_cols;  // of a row: boxes of 64 columns, steps of 16 that hold something; 128-column tiles of c
+    uint32_t* err_flag;
+};
+
+// 8 KT / 32 columns of 8 of this warp's first 16 lanes: thread (g, tq) has row g's columns 8 j + 2 tq, + 1 and row g + 8's, for each j.
+__device__ __forceinline__ void ld_scores(uint32_t taddr, float (&s)[4][4]) {
+    uint32_t r[16];
+    asm volatile("tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
+                   "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+                 : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 16; i++) s[i / 4][i % 4] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const float (&v)[16]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]),
+                 "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]), "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15])
+                 : "memory");
+}
+__device__ __forceinline__ bool softmax_any(bool mine) {
+    uint32_t any;
+    asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 p, %1, 0;\nbar.red.or.pred q, 1, %2, p;\nselp.u32 %0, 1, 0, q;\n}" : "=r"(any) : "r"(uint32_t(mine)), "n"(SOFTMAX) : "memory");
+    return any != 0;
+}
+__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, %0;" ::"n"(SOFTMAX) : "memory"); }
+// As gemm::smem_desc, of an operand whose lines are its k: 64 entries of the M side a line, the next 64 `next` bytes on.
+__device__ __forceinline__ uint64_t mn_major_desc(uint32_t addr, uint32_t next) {
+    return uint64_t((addr & 0x3FFFFu) >> 4) | (uint64_t(next >> 4) << 16) | (uint64_t(1024 >> 4) << 32) | (uint64_t(1) << 46) | (uint64_t(2) << 61);
+}
 
 // grid (tiles, 1, key splits). Prompts (sub > 0): tile = (chunk tile, one of its `sub` spans of `toks` tokens, group of ROWS heads); else
 // (token, group).
-template <uint32_t R, uint32_t ROWS>
-__global__ void __launch_bounds__(THREADS, 1) latent_kernel(const ChunkedAttnArgs a, uint32_t groups, uint32_t sub, uint32_t toks) {
+template <uint32_t ROWS>
+__global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constant__ Map map, const Args p) {
     pdl_start();
-    using S = Shape<R, ROWS>;
-    extern __shared__ __align__(1024) uint8_t smem[];
-    __shared__ uint32_t end_s;
-    const uint32_t tid = threadIdx.x, warp = tid / 32, lane = tid % 32, g = lane >> 2, tq = lane & 3, lm = lane >> 3, lr = lane & 7;
-    const uint32_t grp = blockIdx.x % groups, unit = blockIdx.x / groups, sp = blockIdx.z, splits = gridDim.z;
+    constexpr uint32_t KT = tile_keys<ROWS>(), BOX = KT * 128, QB = ROWS * 128, ACTIVE = ROWS / 16;
+    extern __shared__ uint8_t smem_raw[];
+    const ChunkedAttnArgs& a = p.c;
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    const uint32_t tid = threadIdx.x, warp = tid / 32, lane = tid % 32, grp = blockIdx.x % p.groups, unit = blockIdx.x / p.groups, sp = blockIdx.z, splits = gridDim.z;
     uint32_t t0 = unit, n_tok = 1;
-    if (sub) {
-        const uint32_t tile = unit / sub, at = unit % sub * toks, rows = a.ctiles[2 * tile + 1];
+    if (p.sub) {
+        const uint32_t tile = unit / p.sub, at = unit % p.sub * p.toks, rows = a.ctiles[2 * tile + 1];
         if (at >= rows) return;  // (all of a cluster's blocks together)
         t0 = a.ctiles[2 * tile] + at;
-        n_tok = min(toks, rows - at);
+        n_tok = min(p.toks, rows - at);
     }
-    const uint32_t hpt = min(a.heads, ROWS), dk = a.kv.dk, rank = a.kv.dv;
-    auto row_at = [&](uint32_t r, uint32_t& tok, uint32_t& head) {  // whether row r of the tile exists
+    const uint32_t S = p.stages, stage = p.blocks * BOX, dk = a.kv.dk, rank = a.kv.dv;
+    const uint32_t base = smem_u32(smem), ring = base + p.blocks * QB, probs = ring + S * stage;  // Q | the ring | P | what follows
+    uint8_t* misc = smem + p.blocks * QB + S * stage + QB;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(misc);  // full[S], empty[S], scores[2], P, sums
+    const uint32_t bar_full = smem_u32(bars), bar_empty = bar_full + 8 * S, bar_scores = bar_empty + 8 * S, bar_p = bar_scores + 16, bar_sums = bar_p + 8;
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_STAGES + 4));
+    volatile uint32_t* abort_flag = tmem_slot + 1;
+    uint32_t* end_s = const_cast<uint32_t*>(tmem_slot) + 2;
+    int* from = reinterpret_cast<int*>(misc + 256);  // a row's place among the queries and the outputs, -1: none
+    float *corr_s = reinterpret_cast<float*>(from + ROWS), *m_s = corr_s + ROWS, *l_s = m_s + ROWS;
+    if (tid == 0) {
+        for (uint32_t i = 0; i < S; i++) {
+            mbar_init(bar_full + 8 * i, 1);
+            mbar_init(bar_empty + 8 * i, 1);
+        }
+        mbar_init(bar_scores, 1);
+        mbar_init(bar_scores + 8, 1);
+        mbar_init(bar_p, ACTIVE);
+        mbar_init(bar_sums, 1);
+        *abort_flag = 0;
+        *end_s = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(tmem_slot))), "r"(p.tmem_cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    const uint32_t hpt = min(a.heads, ROWS);
+    auto row_at = [&](uint32_t r, uint32_t& tok) {
         tok = t0 + r / hpt;
-        head = grp * ROWS + r % hpt;
-        return r / hpt < n_tok && head < a.heads;
+        const uint32_t head = grp * ROWS + r % hpt;
+        return r / hpt < n_tok && head < a.heads ? int(tok * a.heads + head) : -1;
     };
-    // The softmax's row of this thread.
-    const uint32_t my_row = tid / S::TPR, my_key = tid % S::TPR * S::KPT;
-    uint32_t my_tok, my_head;
-    const bool live = row_at(my_row, my_tok, my_head);
-    const View v = view_of(a, live ? my_tok : t0);
-    if (tid == 0) end_s = 0;
     __syncthreads();
-    if (live && tid % S::TPR == 0) atomicMax(&end_s, v.first + 32 - __clz(v.mask));
-    // The query rows, zeros where there are none, and zeros behind the staged rows' ends (no copy writes there).
-    const uint32_t pieces = dk / 8, whole = S::WIDTH / 8;
-    for (uint32_t i = tid; i < ROWS * whole; i += THREADS) {
-        const uint32_t r = i / whole, c = i % whole;
-        uint32_t tok, head;
+    const uint32_t slot = a.meta[2 * t0];
+    if (tid < ROWS) {
+        uint32_t tok;
+        from[tid] = row_at(tid, tok);
+        if (from[tid] >= 0) {
+            const View v = view_of(a, tok);
+            atomicMax(end_s, v.first + 32 - __clz(v.mask));
+        }
+    }
+    for (uint32_t i = tid; i < ROWS * p.blocks * 8; i += THREADS) {  // Q in the MMA's swizzle: zeros where there are no rows or columns
+        const uint32_t r = i / (p.blocks * 8), c = i % (p.blocks * 8);
+        uint32_t tok;
+        const int at = row_at(r, tok);
         uint4 x = make_uint4(0, 0, 0, 0);
-        if (row_at(r, tok, head) && c < pieces) x = reinterpret_cast<const uint4*>(a.q_b + (size_t(tok) * a.heads + head) * dk)[c];
-        *reinterpret_cast<uint4*>(smem + S::O_Q + r * S::PITCH + c * 16) = x;
+        if (at >= 0 && c * 8 < dk) x = *reinterpret_cast<const uint4*>(a.q_b + size_t(at) * dk + c * 8);
+        *reinterpret_cast<uint4*>(smem + c / 8 * QB + r * 128 + ((c % 8 ^ (r & 7)) << 4)) = x;
     }
-    for (uint32_t i = tid; i < S::STAGES * KT * (whole - pieces); i += THREADS)
-        *reinterpret_cast<uint4*>(smem + i / (whole - pieces) * S::PITCH + (pieces + i % (whole - pieces)) * 16) = make_uint4(0, 0, 0, 0);
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
-    const uint32_t tiles = (end_s + KT - 1) / KT, share = (tiles + splits - 1) / splits, begin = min(sp * share, tiles), n = min(share, tiles - begin);
-
-    const uint32_t* pages = a.kv.page_table + size_t(v.slot) * a.kv.max_pages;
-    const uint16_t* K = static_cast<const uint16_t*>(a.kv.k);
-    const uint32_t base = smem_u32(smem);
-    auto issue = [&](uint32_t i) {
-        const uint32_t key0 = (begin + i) * KT;
-        const uint16_t* src = K + ((size_t(pages[key0 >> PAGE_SHIFT]) << PAGE_SHIFT) + (key0 & (PAGE - 1))) * dk;
-        const uint32_t dst = base + i % S::STAGES * S::STAGE;
-        uint32_t key = tid / pieces, c = tid % pieces;
-        const uint32_t dkey = THREADS / pieces, dc = THREADS % pieces;
-        while (key < KT) {
-            cp_async16(dst + key * S::PITCH + c * 16, src + size_t(key) * dk + c * 8);
-            key += dkey;
-            c += dc;
-            if (c >= pieces) { c -= pieces; key++; }
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem = *tmem_slot, tmem_o = tmem + 2 * KT;
+    const uint32_t tiles = (*end_s + KT - 1) / KT, share = (tiles + splits - 1) / splits, begin = min(sp * share, tiles), n = min(share, tiles - begin);
+    bool ok = true;
+    if (warp == 0) {
+        if (lane == 0) {
+            const uint32_t* pages = a.kv.page_table + size_t(slot) * a.kv.max_pages;
+            uint32_t st = 0, ph = 1, page = n ? pages[begin * KT >> PAGE_SHIFT] : 0;
+            for (uint32_t i = 0; i < n; i++) {
+                const uint32_t key0 = (begin + i) * KT, row = (page << PAGE_SHIFT) + (key0 & (PAGE - 1));
+                if (i + 1 < n) page = pages[(key0 + KT) >> PAGE_SHIFT];
+                ok = wait_or_abort(bar_empty + 8 * st, ph, abort_flag);
+                if (!ok) break;
+                mbar_expect_tx(bar_full + 8 * st, stage);
+                for (uint32_t b = 0; b < p.blocks; b++) tma_load_2d(ring + st * stage + b * BOX, &map, int(b * 64), int(row), bar_full + 8 * st);
+                if (++st == S) { st = 0; ph ^= 1; }
+            }
         }
-    };
+        __syncwarp();
+    } else if (warp == 1) {
+        const uint32_t leader = elect_one(), idesc_s = instr_desc(64, KT), idesc_o = instr_desc(128, ROWS) | (1u << 15);  // (bit 15: A's lines are its k)
+        const uint64_t q0 = gemm::smem_desc(base), p0 = gemm::smem_desc(probs);
+        uint32_t st_s = 0, ph_s = 0, st_o = 0;  // the stage the next scores read, the one the next sums read
+        auto scores = [&](uint32_t i) {
+            ok = ok && wait_or_abort(bar_full + 8 * st_s, ph_s, abort_flag);
+            ok = __all_sync(0xffffffffu, ok);
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (leader && ok) {
+                const uint64_t k0 = gemm::smem_desc(ring + st_s * stage);
+                for (uint32_t x = 0; x < p.ksteps; x++)
+                    mma_f16(tmem + (i & 1) * KT, q0 + (x / 4 * (QB >> 4) + x % 4 * 2), k0 + (x / 4 * (BOX >> 4) + x % 4 * 2), idesc_s, x != 0 ? 1u : 0u);
+                mma_commit(bar_scores + 8 * (i & 1));
+            }
+            __syncwarp();
+            if (++st_s == S) { st_s = 0; ph_s ^= 1; }
+        };
+        if (n) scores(0);
+        for (uint32_t i = 0; i < n && ok; i++) {
+            if (i + 1 < n) scores(i + 1);
+            ok = ok && wait_or_abort(bar_p, i & 1, abort_flag);
+            ok = __all_sync(0xffffffffu, ok);
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (leader && ok) {
+                for (uint32_t m = 0; m < p.mtiles; m++) {
+                    const uint64_t v0 = mn_major_desc(ring + st_o * stage + 2 * m * BOX, BOX);
 #pragma unroll
-    for (uint32_t i = 0; i < S::STAGES - 1; i++) {
-        if (i < n) issue(i);
-        cp_async_commit();
-    }
-    float *scores = reinterpret_cast<float*>(smem + S::O_S), *corr_s = reinterpret_cast<float*>(smem + S::O_STAT), *m_s = corr_s + ROWS, *l_s = m_s + ROWS;
-    uint16_t* probs = reinterpret_cast<uint16_t*>(smem + S::O_P);
-    const uint32_t rg = warp % S::RG, kg = warp / S::RG % S::KG, kh = warp / (S::RG * S::KG), cg = warp / S::RG, col0 = cg * S::CW;
-    const bool sums = col0 < R;
-    float o[S::CW / 8][4], m_run = -INFINITY, l_run = 0.0f;
-#pragma unroll
-    for (uint32_t j = 0; j < S::CW / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
-    const uint32_t q_addr = base + S::O_Q + (rg * 16 + lane % 16) * S::PITCH + lane / 16 * 16, p_addr = base + S::O_P + ((rg * 16 + lane % 16) * S::PP + lane / 16 * 8) * 2;
-    const float cap = a.softcap * LOG2E, cap_inv = 2.0f / a.softcap;
-    for (uint32_t i = 0; i < n; i++) {
-        cp_async_wait<S::STAGES - 2>();
-        __syncthreads();  // everybody's copies of the tile are in, and everybody is done with the tile before
-        if (i + S::STAGES - 1 < n) issue(i + S::STAGES - 1);
-        cp_async_commit();
-        const uint32_t stage = base + i % S::STAGES * S::STAGE, key0 = (begin + i) * KT;
-        {
-            float s[S::NT][2][4];
-#pragma unroll
-            for (uint32_t j = 0; j < S::NT; j++)
-#pragma unroll
-                for (uint32_t e = 0; e < 4; e++) s[j][0][e] = s[j][1][e] = 0.0f;
-            constexpr uint32_t PAIRS = S::WIDTH / 32 / S::KH;  // pairs of 16 columns
-            const uint32_t k_addr = stage + (kg * S::NT * 8 + lr) * S::PITCH + lm * 16 + kh * PAIRS * 64, qa = q_addr + kh * PAIRS * 64;
-#pragma unroll 6
-            for (uint32_t kp = 0; kp < PAIRS; kp++) {
-                uint32_t a0[4], a1[4];
-                ldmatrix_x4(a0, qa + kp * 64);
-                ldmatrix_x4(a1, qa + kp * 64 + 32);
-#pragma unroll
-                for (uint32_t j = 0; j < S::NT; j++) {
-                    uint32_t kb[4];
-                    ldmatrix_x4(kb, k_addr + j * 8 * S::PITCH + kp * 64);
-                    mma16816(s[j][0], a0, kb[0], kb[1]);
-                    mma16816(s[j][1], a1, kb[2], kb[3]);
+                    for (uint32_t kk = 0; kk < KT / 16; kk++) mma_f16(tmem_o + m * ROWS, v0 + kk * (2048 >> 4), p0 + kk * 2, idesc_o, (i | kk) != 0 ? 1u : 0u);
                 }
+                mma_commit(bar_empty + 8 * st_o);
+                mma_commit(bar_sums);
             }
-            float* dst = scores + (kh * ROWS + rg * 16 + g) * S::SP + kg * S::NT * 8 + 2 * tq;
-#pragma unroll
-            for (uint32_t j = 0; j < S::NT; j++) {
-                *reinterpret_cast<float2*>(dst + 8 * j) = make_float2(s[j][0][0] + s[j][1][0], s[j][0][1] + s[j][1][1]);
-                *reinterpret_cast<float2*>(dst + 8 * S::SP + 8 * j) = make_float2(s[j][0][2] + s[j][1][2], s[j][0][3] + s[j][1][3]);
-            }
+            __syncwarp();
+            if (++st_o == S) st_o = 0;
         }
-        __syncthreads();
-        {
-            float s[S::KPT], mx = -INFINITY;
-#pragma unroll
-            for (uint32_t e = 0; e < S::KPT; e++) {
-                s[e] = scores[my_row * S::SP + my_key + e];
-                if (S::KH == 2) s[e] += scores[(ROWS + my_row) * S::SP + my_key + e];
-                if (a.softcap > 0) s[e] = capped(s[e], cap, cap_inv);
-                const uint32_t key = key0 + my_key + e;
-                if (!live || (key >= v.first && !sees(v, key))) s[e] = -INFINITY;
-                mx = fmaxf(mx, s[e]);
-            }
-#pragma unroll
-            for (uint32_t x = 1; x < S::TPR; x *= 2) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-            // The running maximum only has to keep 2^(s - m) in range: it moves when a score exceeds it by more than 8.
-            float corr = 1.0f;
-            if (mx > m_run + 8.0f) {
-                corr = fast_exp2(m_run - mx);  // (0 from -infinity)
-                m_run = mx;
-            }
-            const float m = m_run == -INFINITY ? 0.0f : m_run;
-            float sum = 0.0f;
-            uint32_t packed[S::KPT / 2];
-#pragma unroll
-            for (uint32_t e = 0; e < S::KPT; e += 2) {
-                const float p0 = fast_exp2(s[e] - m), p1 = fast_exp2(s[e + 1] - m);
-                sum += p0 + p1;
-                packed[e / 2] = pack_bf16(p0, p1);
-                *reinterpret_cast<uint32_t*>(probs + my_row * S::PP + my_key + e) = packed[e / 2];
-            }
-            l_run = l_run * corr + sum;
-            if (tid % S::TPR == 0) corr_s[my_row] = corr;
-        }
-        __syncthreads();
-        const float c0 = corr_s[rg * 16 + g], c1 = corr_s[rg * 16 + g + 8];
-        if (__any_sync(0xffffffffu, c0 != 1.0f || c1 != 1.0f)) {
-#pragma unroll
-            for (uint32_t j = 0; j < S::CW / 8; j++) {
-                o[j][0] *= c0;
-                o[j][1] *= c0;
-                o[j][2] *= c1;
-                o[j][3] *= c1;
-            }
-        }
-        if (sums) {
-            uint32_t pa[KT / 16][4];
-#pragma unroll
-            for (uint32_t kk = 0; kk < KT / 16; kk++) ldmatrix_x4(pa[kk], p_addr + kk * 32);
-            const uint32_t v_addr = stage + (8 * (lm & 1) + lr) * S::PITCH + (col0 + 8 * (lm >> 1)) * 2;
-#pragma unroll
-            for (uint32_t dp = 0; dp < S::CW / 16; dp++)
-#pragma unroll
-                for (uint32_t kk = 0; kk < KT / 16; kk++) {
-                    uint32_t vb[4];
-                    ldmatrix_x4_trans(vb, v_addr + kk * 16 * S::PITCH + dp * 32);
-                    mma16816(o[2 * dp], pa[kk], vb[0], vb[1]);
-                    mma16816(o[2 * dp + 1], pa[kk], vb[2], vb[3]);
-                }
-        }
-    }
-    cp_async_wait<0>();
-#pragma unroll
-    for (uint32_t x = 1; x < S::TPR; x *= 2) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
-    if (splits == 1) {
-        if (tid % S::TPR == 0) l_s[my_row] = l_run;
-        __syncthreads();
-        if (!sums) return;
+    } else {
+        const uint32_t quarter = warp & 3, g = lane >> 2, tq = lane & 3, o_addr = tmem_o + ((quarter * 32) << 16);
+        const bool active = quarter < ACTIVE;
+        const float cap = a.softcap * LOG2E, cap_inv = 2.0f / a.softcap;
+        View v[2];
+        bool live[2];
+        float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 #pragma unroll
         for (uint32_t r = 0; r < 2; r++) {
-            const uint32_t row = rg * 16 + g + 8 * r;
-            uint32_t tok, head;
-            if (!row_at(row, tok, head)) continue;
-            const float inv = 1.0f / l_s[row];
-            const size_t at = (size_t(tok) * a.heads + head) * rank;
+            uint32_t tok;
+            live[r] = active && row_at(quarter * 16 + g + 8 * r, tok) >= 0;
+            v[r] = view_of(a, live[r] ? tok : t0);
+        }
+        const uint32_t first = min(v[0].first, v[1].first);
+        for (uint32_t i = 0; i < n; i++) {
+            float s[KT / 8][4], m_new[2] = {m_run[0], m_run[1]};
+            bool need = false;
+            if (active) {
+                ok = ok && wait_or_abort(bar_scores + 8 * (i & 1), (i >> 1) & 1, abort_flag);
+                ok = __all_sync(0xffffffffu, ok);
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-            for (uint32_t j = 0; j < S::CW / 8; j++) {
-                const uint32_t c = col0 + 8 * j + 2 * tq;
-                if (c < rank) *reinterpret_cast<uint32_t*>(a.out_b + at + c) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+                for (uint32_t x = 0; x < KT / 32; x++) ld_scores(tmem + (i & 1) * KT + 32 * x + ((quarter * 32) << 16), *reinterpret_cast<float(*)[4][4]>(&s[4 * x]));
+                asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                if (a.softcap > 0) {
+#pragma unroll
+                    for (uint32_t j = 0; j < KT / 8; j++)
+#pragma unroll
+                        for (uint32_t e = 0; e < 4; e++) s[j][e] = capped(s[j][e], cap, cap_inv);
+                }
+                const uint32_t key0 = (begin + i) * KT;
+                if (key0 + KT > first || !live[0] || !live[1]) {
+#pragma unroll
+                    for (uint32_t j = 0; j < KT / 8; j++)
+#pragma unroll
+                        for (uint32_t e = 0; e < 4; e++)
+                            if (!live[e >> 1] || !sees(v[e >> 1], key0 + 8 * j + 2 * tq + (e & 1))) s[j][e] = -INFINITY;
+                }
+#pragma unroll
+                for (uint32_t r = 0; r < 2; r++) {
+                    float mx = -INFINITY;
+#pragma unroll
+                    for (uint32_t j = 0; j < KT / 8; j++) mx = fmaxf(mx, fmaxf(s[j][2 * r], s[j][2 * r + 1]));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                    if (mx > m_run[r] + 8.0f) {
+                        need = true;
+                        m_new[r] = mx;
+                    }
+                }
             }
-        }
-        return;
-    }
-    // The cluster: block b finishes columns b R / splits on. [source][row][column of the span] in front of the statistics, (m, l) per
-    // (source, row) behind them. The first barrier: every block is done with its ring; the second: every partial has arrived.
-    cluster_sync();
-    const uint32_t span = R / splits, ml = S::O_STAT + ROWS * 12;
-    if (tid % S::TPR == 0)
-        for (uint32_t b = 0; b < splits; b++) {
-            const uint32_t dst = cluster_addr(base + ml + (sp * ROWS + my_row) * 8, b);
-            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(m_run) : "memory");
-            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + 4), "f"(l_run) : "memory");
-        }
-    if (sums) {
+            if (softmax_any(need)) {  // some row's maximum moves (the first tile's do)
+                if (active) {
 #pragma unroll
-        for (uint32_t j = 0; j < S::CW / 8; j++) {
-            const uint32_t c = col0 + 8 * j + 2 * tq, owner = c / span;
-            const uint32_t dst = cluster_addr(base + ((sp * ROWS + rg * 16 + g) * span + c % span) * 4, owner);
+                    for (uint32_t r = 0; r < 2; r++) {
+                        const float corr = m_new[r] == m_run[r] ? 1.0f : fast_exp2(m_run[r] - m_new[r]);  // (0 from -infinity)
+                        m_run[r] = m_new[r];
+                        l_run[r] *= corr;
+                        if (tq == 0) corr_s[quarter * 16 + g + 8 * r] = corr;
+                    }
+                }
+                softmax_sync();
+                if (i) {
+                    ok = ok && wait_or_abort(bar_sums, (i - 1) & 1, abort_flag);
+                    ok = __all_sync(0xffffffffu, ok);
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
+                        float o[16];
+                        tmem_ld16(o_addr + c, o);
+#pragma unroll
+                        for (uint32_t j = 0; j < 16; j++) o[j] *= corr_s[c % ROWS + j];
+                        tmem_st16(o_addr + c, o);
+                    }
+                    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+                    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                }
+                softmax_sync();
+            }
+            if (!active) continue;
+            if (i) ok = ok && wait_or_abort(bar_sums, (i - 1) & 1, abort_flag);  // P has been read
+            ok = __all_sync(0xffffffffu, ok);
 #pragma unroll
             for (uint32_t r = 0; r < 2; r++) {
-                asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + r * 8 * span * 4), "f"(o[j][2 * r]) : "memory");
-                asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + r * 8 * span * 4 + 4), "f"(o[j][2 * r + 1]) : "memory");
+                const float m = m_run[r] == -INFINITY ? 0.0f : m_run[r];
+                const uint32_t row = quarter * 16 + g + 8 * r;
+                uint8_t* dst = smem + (probs - base) + row * 128 + tq * 4;
+#pragma unroll
+                for (uint32_t j = 0; j < KT / 8; j++) {
+                    const float e0 = fast_exp2(s[j][2 * r] - m), e1 = fast_exp2(s[j][2 * r + 1] - m);
+                    l_run[r] += e0 + e1;
+                    *reinterpret_cast<uint32_t*>(dst + ((j ^ (row & 7)) << 4)) = pack_bf16(e0, e1);
+                }
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_p);
+        }
+        if (active) {
+#pragma unroll
+            for (uint32_t r = 0; r < 2; r++) {
+                l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+                l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+                if (tq == 0) {
+                    m_s[quarter * 16 + g + 8 * r] = m_run[r];
+                    l_s[quarter * 16 + g + 8 * r] = l_run[r];
+                }
+            }
+        }
+        if (n) ok = ok && wait_or_abort(bar_sums, (n - 1) & 1, abort_flag);
+        ok = __all_sync(0xffffffffu, ok);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        softmax_sync();
+        if (splits == 1) {
+            for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
+                float o[16];
+                tmem_ld16(o_addr + c, o);
+                const uint32_t x = c / ROWS * 128 + quarter * 32 + lane, r0 = c % ROWS;
+#pragma unroll
+                for (uint32_t j = 0; j < 16; j++)
+                    if (from[r0 + j] >= 0 && x < rank) a.out_b[size_t(from[r0 + j]) * rank + x] = f32_to_bf16(__fdividef(o[j], l_s[r0 + j]));
             }
         }
     }
-    cluster_sync();
-    const float *recv = reinterpret_cast<const float*>(smem), *stat = reinterpret_cast<const float*>(smem + ml);
-    for (uint32_t i = tid; i < ROWS * span / 2; i += THREADS) {
-        const uint32_t row = i / (span / 2), x = i % (span / 2) * 2, c = sp * span + x;
-        uint32_t tok, head;
-        if (!row_at(row, tok, head) || c >= rank) continue;
-        float m = -INFINITY, l = 0.0f, y0 = 0.0f, y1 = 0.0f;
-        for (uint32_t k = 0; k < splits; k++) m = fmaxf(m, stat[(k * ROWS + row) * 2]);
-        for (uint32_t k = 0; k < splits; k++) {
-            const float mk = stat[(k * ROWS + row) * 2], w = mk == -INFINITY ? 0.0f : fast_exp2(mk - m);
-            const float2 y = *reinterpret_cast<const float2*>(recv + (k * ROWS + row) * span + x);
-            l += stat[(k * ROWS + row) * 2 + 1] * w;
-            y0 += y.x * w;
-            y1 += y.y * w;
+    if (!ok) {
+        *abort_flag = 1;
+        atomicExch(p.err_flag, 6u);
+    }
+    __syncwarp();
+    if (splits > 1) {
+        // The cluster: block b finishes columns b span on. [source][row][column of the span] and behind them (m, l) per (source, row), in the
+        // room of Q and the ring. The first barrier: every block is done with them; the second: every partial has arrived.
+        cluster_sync();
+        const uint32_t span = p.mtiles * 128 / splits, stats = splits * ROWS * span * 4;
+        if (warp >= 2) {
+            const uint32_t quarter = warp & 3, me = tid - 64;
+            if (me < ROWS)
+                for (uint32_t b = 0; b < splits; b++) {
+                    const uint32_t dst = cluster_addr(base + stats + (sp * ROWS + me) * 8, b);
+                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(m_s[me]) : "memory");
+                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + 4), "f"(l_s[me]) : "memory");
+                }
+            for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
+                float o[16];
+                tmem_ld16(tmem_o + ((quarter * 32) << 16) + c, o);
+                const uint32_t x = c / ROWS * 128 + quarter * 32 + lane;
+                const uint32_t dst = cluster_addr(base + ((sp * ROWS + c % ROWS) * span + x % span) * 4, x / span);
+#pragma unroll
+                for (uint32_t j = 0; j < 16; j++) asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + j * span * 4), "f"(n ? o[j] : 0.0f) : "memory");
+            }
         }
-        *reinterpret_cast<uint32_t*>(a.out_b + (size_t(tok) * a.heads + head) * rank + c) = pack_bf16(y0 / l, y1 / l);
+        __syncwarp();
+        cluster_sync();
+        const float *recv = reinterpret_cast<const float*>(smem), *stat = reinterpret_cast<const float*>(smem + stats);
+        for (uint32_t i = tid; i < ROWS * span; i += THREADS) {
+            const uint32_t row = i / span, x = sp * span + i % span;
+            if (from[row] < 0 || x >= rank) continue;
+            float m = -INFINITY, l = 0.0f, y = 0.0f;
+            for (uint32_t k = 0; k < splits; k++) m = fmaxf(m, stat[(k * ROWS + row) * 2]);
+            for (uint32_t k = 0; k < splits; k++) {
+                const float mk = stat[(k * ROWS + row) * 2], w = mk == -INFINITY ? 0.0f : fast_exp2(mk - m);
+                l += stat[(k * ROWS + row) * 2 + 1] * w;
+                y += recv[(k * ROWS + row) * span + i % span] * w;
+            }
+            a.out_b[size_t(from[row]) * rank + x] = f32_to_bf16(y / l);
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(p.tmem_cols) : "memory");
     }
 }
 
-template <uint32_t R, uint32_t ROWS>
-void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s) {
-    using S = Shape<R, ROWS>;
+template <uint32_t ROWS>
+void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s) {
+    constexpr uint32_t KT = tile_keys<ROWS>();
     static PerDevice configured;
     configured.once([] {
-        VLT_CUDA(cudaFuncSetAttribute(latent_kernel<R, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(S::BYTES)));
-        VLT_CUDA(cudaFuncSetAttribute(latent_kernel<R, ROWS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+        VLT_CUDA(cudaFuncSetAttribute(latent_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(SMEM)));
+        VLT_CUDA(cudaFuncSetAttribute(latent_kernel<ROWS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
     });
-    const uint32_t groups = (a.heads + ROWS - 1) / ROWS, toks = n_ctiles ? std::max(1u, ROWS / a.heads) : 1, sub = n_ctiles ? (64 + toks - 1) / toks : 0;
-    // A tile's positions over 1, 2, 4 or 8 blocks, or 16 where 8 leave most SMs idle: the count that makes waves of blocks (one an SM where
-    // the ring is large) times a block's positions, plus a fixed part, least.
-    const uint32_t units = std::max(1u, (n + toks - 1) / toks * groups), most = units * 16 <= sm_count ? MAX_SPLITS : 8;
+    static thread_local std::map<std::tuple<const void*, uint32_t, uint32_t>, Map> maps;
+    auto key = std::make_tuple(static_cast<const void*>(a.kv.k), a.kv.dk, a.kv.n_pages);
+    auto it = maps.find(key);
+    if (it == maps.end()) {
+        Map m;
+        make_tensor_map_2d(m.a, a.kv.k, a.kv.dk, uint64_t(a.kv.n_pages) * PAGE, 64, KT, 2, true);
+        it = maps.emplace(key, m).first;
+    }
+    Args p;
+    p.c = a;
+    p.err_flag = err_flag;
+    p.groups = (a.heads + ROWS - 1) / ROWS;
+    p.toks = n_ctiles ? std::max(1u, ROWS / a.heads) : 1;
+    p.sub = n_ctiles ? (64 + p.toks - 1) / p.toks : 0;
+    p.mtiles = (a.kv.dv + 127) / 128;
+    p.blocks = std::max((a.kv.dk + 63) / 64, 2 * p.mtiles);
+    p.ksteps = (a.kv.dk + 15) / 16;
+    const uint32_t fixed = 1024 + (p.blocks + 1) * ROWS * 128 + MISC, stage = p.blocks * KT * 128;
+    p.stages = std::min(MAX_STAGES, (SMEM - fixed) / stage);
+    p.tmem_cols = 32;
+    while (p.tmem_cols < 2 * KT + p.mtiles * ROWS) p.tmem_cols *= 2;
+    // A tile's positions over 1, 2, 4 or 8 blocks, or 16 where 8 leave most SMs idle: the count that makes waves of blocks (one an SM) times
+    // a block's positions, plus a fixed part, least.
+    const uint32_t units = std::max(1u, (n + p.toks - 1) / p.toks * p.groups), most = units * 16 <= sm_count ? MAX_SPLITS : 8;
     uint32_t splits = 1;
     uint64_t best = ~0ull;
     for (uint32_t c = 1; c <= most && (c == 1 || max_keys / c >= 64); c *= 2) {
-        const uint64_t cost = uint64_t((units * c + sm_count - 1) / sm_count) * ((max_keys + c - 1) / c + 128);
+        const uint64_t cost = uint64_t((units * c + sm_count - 1) / sm_count) * ((max_keys + c - 1) / c + 256);
         if (cost < best) { best = cost; splits = c; }
     }
     if (keys_per_block)
         for (splits = 1; splits < MAX_SPLITS && splits * keys_per_block < max_keys;) splits *= 2;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((sub ? n_ctiles * sub : n) * groups, 1, splits);
+    cfg.gridDim = dim3((p.sub ? n_ctiles * p.sub : n) * p.groups, 1, splits);
     cfg.blockDim = dim3(THREADS);
-    cfg.dynamicSmemBytes = S::BYTES;
+    cfg.dynamicSmemBytes = std::max(SMEM_MIN, fixed + p.stages * stage);
     cfg.stream = s;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -301,29 +438,19 @@ void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t ma
     attr[1].val.clusterDim.z = splits;
     cfg.attrs = attr;
     cfg.numAttrs = splits > 1 ? 2 : 1;
-    VLT_CUDA(cudaLaunchKernelEx(&cfg, latent_kernel<R, ROWS>, a, groups, sub, toks));
+    VLT_CUDA(cudaLaunchKernelEx(&cfg, latent_kernel<ROWS>, it->second, p));
     launch_counter()++;
 }
-template <uint32_t R>
-void by_rows(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s) {
-    if (n_ctiles || a.heads > 32) launch<R, 64>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s);
-    else if (a.heads > 16) launch<R, 32>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s);
-    else launch<R, 16>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s);
-}
-static uint32_t columns(uint32_t rank) { return rank <= 64 ? 64 : rank <= 128 ? 128 : rank <= 256 ? 256 : 512; }
 
 }  // namespace latent
 
 bool latent_attn_fits(uint32_t kv_rank, uint32_t rot_dim, uint32_t page) {
-    return page == paged::PAGE && kv_rank <= 512 && kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank + rot_dim <= latent::columns(kv_rank) + latent::EXTRA;
+    return page == paged::PAGE && kv_rank <= 512 && kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank + rot_dim <= 576;
 }
-void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s) {
-    switch (latent::columns(a.kv.dv)) {
-    case 64: latent::by_rows<64>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s); break;
-    case 128: latent::by_rows<128>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s); break;
-    case 256: latent::by_rows<256>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s); break;
-    default: latent::by_rows<512>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, s);
-    }
+void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s) {
+    if (n_ctiles || a.heads > 32) latent::launch<64>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);
+    else if (a.heads > 16) latent::launch<32>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);
+    else latent::launch<16>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);
 }
 
 }  // namespace vlt

@@ -301,6 +301,7 @@ struct PagedKv {
     void *k, *v;
     const uint32_t* page_table;
     uint32_t max_pages, page_shift, n_kv, dk, dv;
+    uint32_t n_pages;  // of the pool
 };
 __device__ __forceinline__ size_t page_row(const PagedKv& kv, uint32_t slot, uint32_t g, uint32_t pos) {
     const uint32_t page = kv.page_table[size_t(slot) * kv.max_pages + (pos >> kv.page_shift)], psize = 1u << kv.page_shift;
@@ -410,7 +411,7 @@ struct LatentQueryArgs {
 };
 void launch_latent_query(const LatentQueryArgs& a, cudaStream_t s);
 bool latent_attn_fits(uint32_t kv_rank, uint32_t rot_dim, uint32_t page);  // k_latent_attn.cu's kernels, bf16 caches; else launch_attn_any
-void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
+void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s);
 void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_caches,
                           bool fp32, cudaStream_t s);
 void launch_mixer_fill(const MixerCache* caches, uint32_t n_caches, uint32_t slot, uint32_t from, uint32_t to, uint32_t seed, bool fp32, cudaStream_t s);
