@@ -10,8 +10,9 @@
 // heads; a prompt's portion, the heads of several neighbouring tokens -- and goes through its share of the run's positions a tile
 // at a time:
 //
-//   warp 0       a tile of rows by TMA, 64 columns a box, into a ring of stages
-//   warp 1       the MMAs: the scores of the tile to come in front of this tile's sums
+//   warp 0       tiles of 64 positions by TMA, 64 columns a box: the columns of c in pairs of boxes, each pair a slot of a ring, the boxes
+//                behind them (of r) in a ring of their own
+//   warp 1       the MMAs: a tile's sums as soon as its P is there, else the next tile's scores, pair by pair as they come
 //   warps 2..5   softmax in fp32 (a warp has 16 rows: 64 MMA rows lie on the first 16 lanes of each quarter of tensor memory), P in bf16
 //                through shared memory; the running maximum moves when a score exceeds it by more than 8, and only then does O come
 //                through registers; in the end O
@@ -44,10 +45,9 @@ using gemm::tmem_ld16;
 using gemm::wait_or_abort;
 using namespace paged;
 
-constexpr uint32_t THREADS = 192, SOFTMAX = 128, MAX_SPLITS = 16, MAX_STAGES = 6, MISC = 2048;
+constexpr uint32_t THREADS = 192, SOFTMAX = 128, MAX_SPLITS = 16, KT = 64, BOX = KT * 128;  // KT: positions of a tile (a page)
+constexpr uint32_t MAX_SLOTS = 16, REST_SLOTS = 3, MISC = 2048;
 constexpr uint32_t SMEM = 227 * 1024, SMEM_MIN = 116 * 1024;  // (at least half an SM's: one block an SM, which never waits for another's tensor memory)
-template <uint32_t ROWS>
-constexpr uint32_t tile_keys() { return ROWS == 64 ? 64 : 32; }
 
 struct Map {
     alignas(64) uint8_t a[128];
@@ -55,11 +55,12 @@ struct Map {
 struct Args {
     ChunkedAttnArgs c;
     uint32_t groups, sub, toks;                      // see latent_kernel
-    uint32_t blocks, ksteps, mtiles, stages, tmem_cols;  // of a row: boxes of 64 columns, steps of 16 that hold something; 128-column tiles of c
+    uint32_t boxes, mtiles, rest;                    // of a row: boxes of 64 columns; pairs of them that hold c; those behind the pairs
+    uint32_t slots, rest_slots, tmem_cols;
     uint32_t* err_flag;
 };
 
-// 8 KT / 32 columns of 8 of this warp's first 16 lanes: thread (g, tq) has row g's columns 8 j + 2 tq, + 1 and row g + 8's, for each j.
+// Four times 8 columns of this warp's first 16 lanes: thread (g, tq) has row g's columns 8 j + 2 tq, + 1 and row g + 8's, for each j.
 __device__ __forceinline__ void ld_scores(uint32_t taddr, float (&s)[4][4]) {
     uint32_t r[16];
     asm volatile("tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
@@ -74,6 +75,11 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const float (&v)[16]) 
     asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]),
                  "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]), "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15])
                  : "memory");
+}
+__device__ __forceinline__ bool arrived(uint32_t bar, uint32_t parity) {  // (without waiting for it)
+    uint32_t ok;
+    asm volatile("{\n.reg .pred p;\nmbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
+    return ok != 0;
 }
 __device__ __forceinline__ bool softmax_any(bool mine) {
     uint32_t any;
@@ -91,7 +97,7 @@ __device__ __forceinline__ uint64_t mn_major_desc(uint32_t addr, uint32_t next) 
 template <uint32_t ROWS>
 __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constant__ Map map, const Args p) {
     pdl_start();
-    constexpr uint32_t KT = tile_keys<ROWS>(), BOX = KT * 128, QB = ROWS * 128, ACTIVE = ROWS / 16;
+    constexpr uint32_t QB = ROWS * 128, ACTIVE = ROWS / 16;
     extern __shared__ uint8_t smem_raw[];
     const ChunkedAttnArgs& a = p.c;
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -103,21 +109,19 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         t0 = a.ctiles[2 * tile] + at;
         n_tok = min(p.toks, rows - at);
     }
-    const uint32_t S = p.stages, stage = p.blocks * BOX, dk = a.kv.dk, rank = a.kv.dv;
-    const uint32_t base = smem_u32(smem), ring = base + p.blocks * QB, probs = ring + S * stage;  // Q | the ring | P | what follows
-    uint8_t* misc = smem + p.blocks * QB + S * stage + QB;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(misc);  // full[S], empty[S], scores[2], P, sums
-    const uint32_t bar_full = smem_u32(bars), bar_empty = bar_full + 8 * S, bar_scores = bar_empty + 8 * S, bar_p = bar_scores + 16, bar_sums = bar_p + 8;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_STAGES + 4));
+    const uint32_t dk = a.kv.dk, rank = a.kv.dv, NP = p.slots, NR = p.rest_slots;
+    // Q | the pairs' ring | the ring behind them | P | what follows
+    const uint32_t base = smem_u32(smem), ring = base + p.boxes * QB, rest = ring + NP * 2 * BOX, probs = rest + NR * p.rest * BOX;
+    uint8_t* misc = smem + (probs - base) + QB;
+    const uint32_t bar_full = smem_u32(misc), bar_empty = bar_full + 8 * MAX_SLOTS, bar_rest = bar_empty + 8 * MAX_SLOTS, bar_free = bar_rest + 8 * REST_SLOTS, bar_scores = bar_free + 8 * REST_SLOTS,
+                   bar_p = bar_scores + 16, bar_sums = bar_p + 8;
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_SLOTS + 2 * REST_SLOTS + 4));
     volatile uint32_t* abort_flag = tmem_slot + 1;
     uint32_t* end_s = const_cast<uint32_t*>(tmem_slot) + 2;
-    int* from = reinterpret_cast<int*>(misc + 256);  // a row's place among the queries and the outputs, -1: none
+    int* from = reinterpret_cast<int*>(misc + 512);  // a row's place among the queries and the outputs, -1: none
     float *corr_s = reinterpret_cast<float*>(from + ROWS), *m_s = corr_s + ROWS, *l_s = m_s + ROWS;
     if (tid == 0) {
-        for (uint32_t i = 0; i < S; i++) {
-            mbar_init(bar_full + 8 * i, 1);
-            mbar_init(bar_empty + 8 * i, 1);
-        }
+        for (uint32_t i = 0; i < 2 * MAX_SLOTS + 2 * REST_SLOTS; i++) mbar_init(bar_full + 8 * i, 1);
         mbar_init(bar_scores, 1);
         mbar_init(bar_scores + 8, 1);
         mbar_init(bar_p, ACTIVE);
@@ -146,8 +150,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             atomicMax(end_s, v.first + 32 - __clz(v.mask));
         }
     }
-    for (uint32_t i = tid; i < ROWS * p.blocks * 8; i += THREADS) {  // Q in the MMA's swizzle: zeros where there are no rows or columns
-        const uint32_t r = i / (p.blocks * 8), c = i % (p.blocks * 8);
+    for (uint32_t i = tid; i < ROWS * p.boxes * 8; i += THREADS) {  // Q in the MMA's swizzle: zeros where there are no rows or columns
+        const uint32_t r = i / (p.boxes * 8), c = i % (p.boxes * 8);
         uint32_t tok;
         const int at = row_at(r, tok);
         uint4 x = make_uint4(0, 0, 0, 0);
@@ -164,53 +168,79 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     if (warp == 0) {
         if (lane == 0) {
             const uint32_t* pages = a.kv.page_table + size_t(slot) * a.kv.max_pages;
-            uint32_t st = 0, ph = 1, page = n ? pages[begin * KT >> PAGE_SHIFT] : 0;
-            for (uint32_t i = 0; i < n; i++) {
-                const uint32_t key0 = (begin + i) * KT, row = (page << PAGE_SHIFT) + (key0 & (PAGE - 1));
-                if (i + 1 < n) page = pages[(key0 + KT) >> PAGE_SHIFT];
-                ok = wait_or_abort(bar_empty + 8 * st, ph, abort_flag);
+            uint32_t st = 0, ph = 1, rs = 0, rph = 1, page = n ? pages[begin] : 0;
+            for (uint32_t i = 0; i < n && ok; i++) {
+                const int row = int(page << PAGE_SHIFT);
+                if (i + 1 < n) page = pages[begin + i + 1];
+                for (uint32_t m = 0; m < p.mtiles && ok; m++) {
+                    const bool two = 2 * m + 1 < p.boxes;
+                    ok = wait_or_abort(bar_empty + 8 * st, ph, abort_flag);
+                    if (!ok) break;
+                    mbar_expect_tx(bar_full + 8 * st, two ? 2 * BOX : BOX);
+                    tma_load_2d(ring + st * 2 * BOX, &map, int(m * 128), row, bar_full + 8 * st);
+                    if (two) tma_load_2d(ring + st * 2 * BOX + BOX, &map, int(m * 128 + 64), row, bar_full + 8 * st);
+                    if (++st == NP) { st = 0; ph ^= 1; }
+                }
+                if (!p.rest || !ok) continue;
+                ok = wait_or_abort(bar_free + 8 * rs, rph, abort_flag);
                 if (!ok) break;
-                mbar_expect_tx(bar_full + 8 * st, stage);
-                for (uint32_t b = 0; b < p.blocks; b++) tma_load_2d(ring + st * stage + b * BOX, &map, int(b * 64), int(row), bar_full + 8 * st);
-                if (++st == S) { st = 0; ph ^= 1; }
+                mbar_expect_tx(bar_rest + 8 * rs, p.rest * BOX);
+                for (uint32_t b = 0; b < p.rest; b++) tma_load_2d(rest + (rs * p.rest + b) * BOX, &map, int((2 * p.mtiles + b) * 64), row, bar_rest + 8 * rs);
+                if (++rs == NR) { rs = 0; rph ^= 1; }
             }
         }
         __syncwarp();
     } else if (warp == 1) {
-        const uint32_t leader = elect_one(), idesc_s = instr_desc(64, KT), idesc_o = instr_desc(128, ROWS) | (1u << 15);  // (bit 15: A's lines are its k)
-        const uint64_t q0 = gemm::smem_desc(base), p0 = gemm::smem_desc(probs);
-        uint32_t st_s = 0, ph_s = 0, st_o = 0;  // the stage the next scores read, the one the next sums read
-        auto scores = [&](uint32_t i) {
-            ok = ok && wait_or_abort(bar_full + 8 * st_s, ph_s, abort_flag);
-            ok = __all_sync(0xffffffffu, ok);
-            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            if (leader && ok) {
-                const uint64_t k0 = gemm::smem_desc(ring + st_s * stage);
-                for (uint32_t x = 0; x < p.ksteps; x++)
-                    mma_f16(tmem + (i & 1) * KT, q0 + (x / 4 * (QB >> 4) + x % 4 * 2), k0 + (x / 4 * (BOX >> 4) + x % 4 * 2), idesc_s, x != 0 ? 1u : 0u);
-                mma_commit(bar_scores + 8 * (i & 1));
-            }
-            __syncwarp();
-            if (++st_s == S) { st_s = 0; ph_s ^= 1; }
-        };
-        if (n) scores(0);
-        for (uint32_t i = 0; i < n && ok; i++) {
-            if (i + 1 < n) scores(i + 1);
-            ok = ok && wait_or_abort(bar_p, i & 1, abort_flag);
-            ok = __all_sync(0xffffffffu, ok);
-            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            if (leader && ok) {
-                for (uint32_t m = 0; m < p.mtiles; m++) {
-                    const uint64_t v0 = mn_major_desc(ring + st_o * stage + 2 * m * BOX, BOX);
+        if (elect_one()) {
+            constexpr uint32_t idesc_s = instr_desc(64, KT), idesc_o = instr_desc(128, ROWS) | (1u << 15);  // (bit 15: A's lines are its k)
+            const uint64_t k_major = gemm::smem_desc(0), mn_major = mn_major_desc(0, BOX);
+            auto lo = [](uint32_t addr) { return (addr & 0x3FFFFu) >> 4; };  // (an address in a cluster has the block's rank above these bits)
+            const uint32_t q0 = lo(base), ring0 = lo(ring), rest0 = lo(rest), p0 = lo(probs);
+            uint32_t st_s = 0, ph_s = 0, rs = 0, rph = 0, st_o = 0, next_s = 0, next_o = 0, idle = 0;
+            auto box = [&](uint32_t b, uint32_t at, uint32_t d) {  // box b of a tile, which lies at `at`: four steps of 16 columns
 #pragma unroll
-                    for (uint32_t kk = 0; kk < KT / 16; kk++) mma_f16(tmem_o + m * ROWS, v0 + kk * (2048 >> 4), p0 + kk * 2, idesc_o, (i | kk) != 0 ? 1u : 0u);
+                for (uint32_t x = 0; x < 4; x++) mma_f16(d, k_major + (q0 + b * (QB >> 4) + 2 * x), k_major + (at + 2 * x), idesc_s, (b | x) != 0 ? 1u : 0u);
+            };
+            while (next_o < n && ok) {
+                if (next_o < next_s && arrived(bar_p, next_o & 1)) {
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    for (uint32_t m = 0; m < p.mtiles; m++) {
+#pragma unroll
+                        for (uint32_t kk = 0; kk < KT / 16; kk++)
+                            mma_f16(tmem_o + m * ROWS, mn_major + (ring0 + st_o * (2 * BOX >> 4) + kk * (2048 >> 4)), k_major + (p0 + kk * 2), idesc_o, (next_o | kk) != 0 ? 1u : 0u);
+                        mma_commit(bar_empty + 8 * st_o);
+                        if (++st_o == NP) st_o = 0;
+                    }
+                    mma_commit(bar_sums);
+                    next_o++;
+                    idle = 0;
+                } else if (next_s < n && next_s <= next_o + 1 && arrived(bar_full + 8 * st_s, ph_s)) {
+                    // (scores two tiles ahead of the sums would go where the softmax may still read)
+                    const uint32_t d = tmem + (next_s & 1) * KT;
+                    for (uint32_t m = 0; m < p.mtiles && ok; m++) {
+                        ok = wait_or_abort(bar_full + 8 * st_s, ph_s, abort_flag);
+                        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                        if (!ok) break;
+                        box(2 * m, ring0 + st_s * (2 * BOX >> 4), d);
+                        if (2 * m + 1 < p.boxes) box(2 * m + 1, ring0 + st_s * (2 * BOX >> 4) + (BOX >> 4), d);
+                        if (++st_s == NP) { st_s = 0; ph_s ^= 1; }
+                    }
+                    if (p.rest && ok) {
+                        ok = wait_or_abort(bar_rest + 8 * rs, rph, abort_flag);
+                        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                        for (uint32_t b = 0; b < p.rest && ok; b++) box(2 * p.mtiles + b, rest0 + (rs * p.rest + b) * (BOX >> 4), d);
+                        if (ok) mma_commit(bar_free + 8 * rs);
+                        if (++rs == NR) { rs = 0; rph ^= 1; }
+                    }
+                    if (ok) mma_commit(bar_scores + 8 * (next_s & 1));
+                    next_s++;
+                    idle = 0;
+                } else if (++idle == gemm::SPIN || ((idle & 1023u) == 1023u && *abort_flag)) {
+                    ok = false;
                 }
-                mma_commit(bar_empty + 8 * st_o);
-                mma_commit(bar_sums);
             }
-            __syncwarp();
-            if (++st_o == S) st_o = 0;
         }
+        __syncwarp();
     } else {
         const uint32_t quarter = warp & 3, g = lane >> 2, tq = lane & 3, o_addr = tmem_o + ((quarter * 32) << 16);
         const bool active = quarter < ACTIVE;
@@ -363,18 +393,39 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         }
         __syncwarp();
         cluster_sync();
-        const float *recv = reinterpret_cast<const float*>(smem), *stat = reinterpret_cast<const float*>(smem + stats);
-        for (uint32_t i = tid; i < ROWS * span; i += THREADS) {
-            const uint32_t row = i / span, x = sp * span + i % span;
-            if (from[row] < 0 || x >= rank) continue;
-            float m = -INFINITY, l = 0.0f, y = 0.0f;
-            for (uint32_t k = 0; k < splits; k++) m = fmaxf(m, stat[(k * ROWS + row) * 2]);
-            for (uint32_t k = 0; k < splits; k++) {
-                const float mk = stat[(k * ROWS + row) * 2], w = mk == -INFINITY ? 0.0f : fast_exp2(mk - m);
-                l += stat[(k * ROWS + row) * 2 + 1] * w;
-                y += recv[(k * ROWS + row) * span + i % span] * w;
+        const float* recv = reinterpret_cast<const float*>(smem);
+        float* stat = reinterpret_cast<float*>(smem + stats);
+        if (tid < ROWS) {  // what each source's sums of the row are worth
+            float m = -INFINITY, l = 0.0f, w[MAX_SPLITS];
+#pragma unroll
+            for (uint32_t k = 0; k < MAX_SPLITS; k++) {
+                w[k] = k < splits ? stat[(k * ROWS + tid) * 2] : -INFINITY;
+                m = fmaxf(m, w[k]);
             }
-            a.out_b[size_t(from[row]) * rank + x] = f32_to_bf16(y / l);
+#pragma unroll
+            for (uint32_t k = 0; k < MAX_SPLITS; k++) {
+                w[k] = w[k] == -INFINITY ? 0.0f : fast_exp2(w[k] - m);
+                if (k < splits) l += stat[(k * ROWS + tid) * 2 + 1] * w[k];
+            }
+#pragma unroll
+            for (uint32_t k = 0; k < MAX_SPLITS; k++)
+                if (k < splits) stat[(k * ROWS + tid) * 2] = w[k] / l;
+        }
+        __syncthreads();
+        for (uint32_t i = tid; i < ROWS * span / 4; i += THREADS) {
+            const uint32_t row = i / (span / 4), c = i % (span / 4) * 4, x = sp * span + c;
+            if (from[row] < 0 || x >= rank) continue;
+            float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 4
+            for (uint32_t k = 0; k < splits; k++) {
+                const float w = stat[(k * ROWS + row) * 2];
+                const float4 v = *reinterpret_cast<const float4*>(recv + (k * ROWS + row) * span + c);
+                y.x = fmaf(w, v.x, y.x);
+                y.y = fmaf(w, v.y, y.y);
+                y.z = fmaf(w, v.z, y.z);
+                y.w = fmaf(w, v.w, y.w);
+            }
+            *reinterpret_cast<uint2*>(a.out_b + size_t(from[row]) * rank + x) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -387,7 +438,6 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
 
 template <uint32_t ROWS>
 void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s) {
-    constexpr uint32_t KT = tile_keys<ROWS>();
     static PerDevice configured;
     configured.once([] {
         VLT_CUDA(cudaFuncSetAttribute(latent_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(SMEM)));
@@ -408,10 +458,13 @@ void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t ma
     p.toks = n_ctiles ? std::max(1u, ROWS / a.heads) : 1;
     p.sub = n_ctiles ? (64 + p.toks - 1) / p.toks : 0;
     p.mtiles = (a.kv.dv + 127) / 128;
-    p.blocks = std::max((a.kv.dk + 63) / 64, 2 * p.mtiles);
-    p.ksteps = (a.kv.dk + 15) / 16;
-    const uint32_t fixed = 1024 + (p.blocks + 1) * ROWS * 128 + MISC, stage = p.blocks * KT * 128;
-    p.stages = std::min(MAX_STAGES, (SMEM - fixed) / stage);
+    p.boxes = (a.kv.dk + 63) / 64;
+    p.rest = p.boxes > 2 * p.mtiles ? p.boxes - 2 * p.mtiles : 0;
+    // Room for two tiles at least (the sums of one wait for their P while the scores of the next come in).
+    const uint32_t fixed = 1024 + (p.boxes + 1) * ROWS * 128 + MISC;
+    p.rest_slots = fixed + (p.rest * REST_SLOTS + 4 * p.mtiles) * BOX <= SMEM ? REST_SLOTS : 2;
+    p.slots = std::min(MAX_SLOTS, (SMEM - fixed - p.rest * p.rest_slots * BOX) / (2 * BOX));
+    if (p.slots < 2 * p.mtiles) throw Error("internal: latent attention over " + std::to_string(a.kv.dk) + " columns");
     p.tmem_cols = 32;
     while (p.tmem_cols < 2 * KT + p.mtiles * ROWS) p.tmem_cols *= 2;
     // A tile's positions over 1, 2, 4 or 8 blocks, or 16 where 8 leave most SMs idle: the count that makes waves of blocks (one an SM) times
@@ -428,7 +481,7 @@ void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t ma
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((p.sub ? n_ctiles * p.sub : n) * p.groups, 1, splits);
     cfg.blockDim = dim3(THREADS);
-    cfg.dynamicSmemBytes = std::max(SMEM_MIN, fixed + p.stages * stage);
+    cfg.dynamicSmemBytes = std::max(SMEM_MIN, fixed + (p.rest * p.rest_slots + 2 * p.slots) * BOX);
     cfg.stream = s;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
