@@ -12,8 +12,9 @@
 //
 //   warp 0       tiles of 64 positions by TMA, 64 columns a box: the columns of c in pairs of boxes, each pair a slot of a ring, the boxes
 //                behind them (of r) in a ring of their own
-//   warp 1       the MMAs: a tile's sums as soon as its P is there, else the next tile's scores, pair by pair as they come
-//   warps 2..5   softmax in fp32 (a warp has 16 rows: 64 MMA rows lie on the first 16 lanes of each quarter of tensor memory), P in bf16
+//   warp 1       the scores' MMAs, a pair of boxes at a time as they come
+//   warp 2       the sums' MMAs (a warp of their own: neither kind waits in front of the other's barriers)
+//   warps 3..6   softmax in fp32 (a warp has 16 rows: 64 MMA rows lie on the first 16 lanes of each quarter of tensor memory), P in bf16
 //                through shared memory; the running maximum moves when a score exceeds it by more than 8, and only then does O come
 //                through registers; in the end O
 //
@@ -45,7 +46,7 @@ using gemm::tmem_ld16;
 using gemm::wait_or_abort;
 using namespace paged;
 
-constexpr uint32_t THREADS = 192, SOFTMAX = 128, MAX_SPLITS = 16, KT = 64, BOX = KT * 128;  // KT: positions of a tile (a page)
+constexpr uint32_t THREADS = 224, SOFTMAX = 128, MAX_SPLITS = 16, KT = 64, BOX = KT * 128;  // KT: positions of a tile (a page)
 constexpr uint32_t MAX_SLOTS = 16, REST_SLOTS = 3, MISC = 2048;
 constexpr uint32_t SMEM = 227 * 1024, SMEM_MIN = 116 * 1024;  // (at least half an SM's: one block an SM, which never waits for another's tensor memory)
 
@@ -76,11 +77,6 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const float (&v)[16]) 
                  "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]), "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15])
                  : "memory");
 }
-__device__ __forceinline__ bool arrived(uint32_t bar, uint32_t parity) {  // (without waiting for it)
-    uint32_t ok;
-    asm volatile("{\n.reg .pred p;\nmbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    return ok != 0;
-}
 __device__ __forceinline__ bool softmax_any(bool mine) {
     uint32_t any;
     asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 p, %1, 0;\nbar.red.or.pred q, 1, %2, p;\nselp.u32 %0, 1, 0, q;\n}" : "=r"(any) : "r"(uint32_t(mine)), "n"(SOFTMAX) : "memory");
@@ -96,14 +92,14 @@ __device__ __forceinline__ uint64_t mn_major_desc(uint32_t addr, uint32_t next) 
 // (token, group).
 template <uint32_t ROWS>
 __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constant__ Map map, const Args p) {
-    pdl_start();
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     constexpr uint32_t QB = ROWS * 128, ACTIVE = ROWS / 16;
     extern __shared__ uint8_t smem_raw[];
     const ChunkedAttnArgs& a = p.c;
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     const uint32_t tid = threadIdx.x, warp = tid / 32, lane = tid % 32, grp = blockIdx.x % p.groups, unit = blockIdx.x / p.groups, sp = blockIdx.z, splits = gridDim.z;
     uint32_t t0 = unit, n_tok = 1;
-    if (p.sub) {
+    if (p.sub) {  // (the step's inputs: uploaded before its first kernel)
         const uint32_t tile = unit / p.sub, at = unit % p.sub * p.toks, rows = a.ctiles[2 * tile + 1];
         if (at >= rows) return;  // (all of a cluster's blocks together)
         t0 = a.ctiles[2 * tile] + at;
@@ -114,10 +110,10 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     const uint32_t base = smem_u32(smem), ring = base + p.boxes * QB, rest = ring + NP * 2 * BOX, probs = rest + NR * p.rest * BOX;
     uint8_t* misc = smem + (probs - base) + QB;
     const uint32_t bar_full = smem_u32(misc), bar_empty = bar_full + 8 * MAX_SLOTS, bar_rest = bar_empty + 8 * MAX_SLOTS, bar_free = bar_rest + 8 * REST_SLOTS, bar_scores = bar_free + 8 * REST_SLOTS,
-                   bar_p = bar_scores + 16, bar_sums = bar_p + 8;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_SLOTS + 2 * REST_SLOTS + 4));
+                   bar_p = bar_scores + 16, bar_sums = bar_p + 16;
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_SLOTS + 2 * REST_SLOTS + 6));
     volatile uint32_t* abort_flag = tmem_slot + 1;
-    uint32_t* end_s = const_cast<uint32_t*>(tmem_slot) + 2;
+    volatile uint32_t* end_s = tmem_slot + 2;
     int* from = reinterpret_cast<int*>(misc + 512);  // a row's place among the queries and the outputs, -1: none
     float *corr_s = reinterpret_cast<float*>(from + ROWS), *m_s = corr_s + ROWS, *l_s = m_s + ROWS;
     if (tid == 0) {
@@ -125,10 +121,12 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         mbar_init(bar_scores, 1);
         mbar_init(bar_scores + 8, 1);
         mbar_init(bar_p, ACTIVE);
+        mbar_init(bar_p + 8, ACTIVE);
         mbar_init(bar_sums, 1);
         *abort_flag = 0;
-        *end_s = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&map) : "memory");
     }
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(tmem_slot))), "r"(p.tmem_cols) : "memory");
@@ -140,104 +138,137 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         const uint32_t head = grp * ROWS + r % hpt;
         return r / hpt < n_tok && head < a.heads ? int(tok * a.heads + head) : -1;
     };
-    __syncthreads();
-    const uint32_t slot = a.meta[2 * t0];
-    if (tid < ROWS) {
-        uint32_t tok;
-        from[tid] = row_at(tid, tok);
-        if (from[tid] >= 0) {
-            const View v = view_of(a, tok);
-            atomicMax(end_s, v.first + 32 - __clz(v.mask));
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    // Tile i's boxes, into slots that are free; false: they did not become so.
+    const uint32_t* pages = a.kv.page_table + size_t(a.meta[2 * t0]) * a.kv.max_pages;
+    uint32_t begin = 0, n = 0, st = 0, ph = 1, rs = 0, rph = 1;
+    auto load = [&](uint32_t page) {
+        const int row = int(page << PAGE_SHIFT);
+        for (uint32_t m = 0; m < p.mtiles; m++) {
+            const bool two = 2 * m + 1 < p.boxes;
+            if (!wait_or_abort(bar_empty + 8 * st, ph, abort_flag)) return false;
+            mbar_expect_tx(bar_full + 8 * st, two ? 2 * BOX : BOX);
+            tma_load_2d(ring + st * 2 * BOX, &map, int(m * 128), row, bar_full + 8 * st);
+            if (two) tma_load_2d(ring + st * 2 * BOX + BOX, &map, int(m * 128 + 64), row, bar_full + 8 * st);
+            if (++st == NP) { st = 0; ph ^= 1; }
+        }
+        if (!p.rest) return true;
+        if (!wait_or_abort(bar_free + 8 * rs, rph, abort_flag)) return false;
+        mbar_expect_tx(bar_rest + 8 * rs, p.rest * BOX);
+        for (uint32_t b = 0; b < p.rest; b++) tma_load_2d(rest + (rs * p.rest + b) * BOX, &map, int((2 * p.mtiles + b) * 64), row, bar_rest + 8 * rs);
+        if (++rs == NR) { rs = 0; rph ^= 1; }
+        return true;
+    };
+    auto share_of = [&](uint32_t end) {
+        const uint32_t tiles = (end + KT - 1) / KT, share = (tiles + splits - 1) / splits;
+        begin = min(sp * share, tiles);
+        n = min(share, tiles - begin);
+    };
+    bool ok = true;
+    if (warp == 0) {  // how far the rows see, and the first two tiles on their way while the others fetch the queries
+        uint32_t end = 0;
+        for (uint32_t i = lane; i < n_tok; i += 32) {
+            const View v = view_of(a, t0 + i);
+            end = max(end, v.first + 32 - __clz(v.mask));
+        }
+        end = __reduce_max_sync(0xffffffffu, end);
+        share_of(end);
+        if (lane == 0) {
+            *end_s = end;
+            for (uint32_t i = 0; i < min(n, 2u) && ok; i++) ok = load(pages[begin + i]);
+        }
+    } else {
+        if (tid - 32 < ROWS) {
+            uint32_t tok;
+            from[tid - 32] = row_at(tid - 32, tok);
+        }
+        // Q in the MMA's swizzle: zeros where there are no rows or columns. Six loads at a time.
+        const uint32_t all = ROWS * p.boxes * 8;
+        for (uint32_t i0 = tid - 32; i0 < all; i0 += 6 * (THREADS - 32)) {
+            uint4 x[6];
+#pragma unroll
+            for (uint32_t u = 0; u < 6; u++) {
+                const uint32_t i = i0 + u * (THREADS - 32), r = i / (p.boxes * 8), c = i % (p.boxes * 8);
+                uint32_t tok;
+                const int at = i < all ? row_at(r, tok) : -1;
+                x[u] = at >= 0 && c * 8 < dk ? *reinterpret_cast<const uint4*>(a.q_b + size_t(at) * dk + c * 8) : make_uint4(0, 0, 0, 0);
+            }
+#pragma unroll
+            for (uint32_t u = 0; u < 6; u++) {
+                const uint32_t i = i0 + u * (THREADS - 32), r = i / (p.boxes * 8), c = i % (p.boxes * 8);
+                if (i < all) *reinterpret_cast<uint4*>(smem + c / 8 * QB + r * 128 + ((c % 8 ^ (r & 7)) << 4)) = x[u];
+            }
         }
     }
-    for (uint32_t i = tid; i < ROWS * p.boxes * 8; i += THREADS) {  // Q in the MMA's swizzle: zeros where there are no rows or columns
-        const uint32_t r = i / (p.boxes * 8), c = i % (p.boxes * 8);
-        uint32_t tok;
-        const int at = row_at(r, tok);
-        uint4 x = make_uint4(0, 0, 0, 0);
-        if (at >= 0 && c * 8 < dk) x = *reinterpret_cast<const uint4*>(a.q_b + size_t(at) * dk + c * 8);
-        *reinterpret_cast<uint4*>(smem + c / 8 * QB + r * 128 + ((c % 8 ^ (r & 7)) << 4)) = x;
-    }
+    __syncwarp();
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = *tmem_slot, tmem_o = tmem + 2 * KT;
-    const uint32_t tiles = (*end_s + KT - 1) / KT, share = (tiles + splits - 1) / splits, begin = min(sp * share, tiles), n = min(share, tiles - begin);
-    bool ok = true;
+    share_of(*end_s);
+    auto lo = [](uint32_t addr) { return (addr & 0x3FFFFu) >> 4; };  // (an address in a cluster has the block's rank above these bits)
+    const uint64_t k_major = gemm::smem_desc(0);
     if (warp == 0) {
         if (lane == 0) {
-            const uint32_t* pages = a.kv.page_table + size_t(slot) * a.kv.max_pages;
-            uint32_t st = 0, ph = 1, rs = 0, rph = 1, page = n ? pages[begin] : 0;
-            for (uint32_t i = 0; i < n && ok; i++) {
-                const int row = int(page << PAGE_SHIFT);
+            uint32_t page = n > 2 ? pages[begin + 2] : 0;
+            for (uint32_t i = 2; i < n && ok; i++) {
+                const uint32_t now = page;
                 if (i + 1 < n) page = pages[begin + i + 1];
-                for (uint32_t m = 0; m < p.mtiles && ok; m++) {
-                    const bool two = 2 * m + 1 < p.boxes;
-                    ok = wait_or_abort(bar_empty + 8 * st, ph, abort_flag);
-                    if (!ok) break;
-                    mbar_expect_tx(bar_full + 8 * st, two ? 2 * BOX : BOX);
-                    tma_load_2d(ring + st * 2 * BOX, &map, int(m * 128), row, bar_full + 8 * st);
-                    if (two) tma_load_2d(ring + st * 2 * BOX + BOX, &map, int(m * 128 + 64), row, bar_full + 8 * st);
-                    if (++st == NP) { st = 0; ph ^= 1; }
-                }
-                if (!p.rest || !ok) continue;
-                ok = wait_or_abort(bar_free + 8 * rs, rph, abort_flag);
-                if (!ok) break;
-                mbar_expect_tx(bar_rest + 8 * rs, p.rest * BOX);
-                for (uint32_t b = 0; b < p.rest; b++) tma_load_2d(rest + (rs * p.rest + b) * BOX, &map, int((2 * p.mtiles + b) * 64), row, bar_rest + 8 * rs);
-                if (++rs == NR) { rs = 0; rph ^= 1; }
+                ok = load(now);
             }
         }
         __syncwarp();
     } else if (warp == 1) {
         if (elect_one()) {
-            constexpr uint32_t idesc_s = instr_desc(64, KT), idesc_o = instr_desc(128, ROWS) | (1u << 15);  // (bit 15: A's lines are its k)
-            const uint64_t k_major = gemm::smem_desc(0), mn_major = mn_major_desc(0, BOX);
-            auto lo = [](uint32_t addr) { return (addr & 0x3FFFFu) >> 4; };  // (an address in a cluster has the block's rank above these bits)
-            const uint32_t q0 = lo(base), ring0 = lo(ring), rest0 = lo(rest), p0 = lo(probs);
-            uint32_t st_s = 0, ph_s = 0, rs = 0, rph = 0, st_o = 0, next_s = 0, next_o = 0, idle = 0;
-            auto box = [&](uint32_t b, uint32_t at, uint32_t d) {  // box b of a tile, which lies at `at`: four steps of 16 columns
+            constexpr uint32_t idesc = instr_desc(64, KT);
+            const uint32_t q0 = lo(base), ring0 = lo(ring), rest0 = lo(rest);
+            uint32_t fs = 0, fph = 0, frs = 0, frph = 0;
+            for (uint32_t i = 0; i < n && ok; i++) {
+                const uint32_t d = tmem + (i & 1) * KT;
+                auto box = [&](uint32_t b, uint32_t at) {  // box b of the tile, which lies at `at`: four steps of 16 columns
 #pragma unroll
-                for (uint32_t x = 0; x < 4; x++) mma_f16(d, k_major + (q0 + b * (QB >> 4) + 2 * x), k_major + (at + 2 * x), idesc_s, (b | x) != 0 ? 1u : 0u);
-            };
-            while (next_o < n && ok) {
-                if (next_o < next_s && arrived(bar_p, next_o & 1)) {
+                    for (uint32_t x = 0; x < 4; x++) mma_f16(d, k_major + (q0 + b * (QB >> 4) + 2 * x), k_major + (at + 2 * x), idesc, (b | x) != 0 ? 1u : 0u);
+                };
+                if (i >= 2) {  // the softmax has read the scores that lie there
+                    ok = wait_or_abort(bar_p + 8 * (i & 1), (i / 2 - 1) & 1, abort_flag);
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                    for (uint32_t m = 0; m < p.mtiles; m++) {
-#pragma unroll
-                        for (uint32_t kk = 0; kk < KT / 16; kk++)
-                            mma_f16(tmem_o + m * ROWS, mn_major + (ring0 + st_o * (2 * BOX >> 4) + kk * (2048 >> 4)), k_major + (p0 + kk * 2), idesc_o, (next_o | kk) != 0 ? 1u : 0u);
-                        mma_commit(bar_empty + 8 * st_o);
-                        if (++st_o == NP) st_o = 0;
-                    }
-                    mma_commit(bar_sums);
-                    next_o++;
-                    idle = 0;
-                } else if (next_s < n && next_s <= next_o + 1 && arrived(bar_full + 8 * st_s, ph_s)) {
-                    // (scores two tiles ahead of the sums would go where the softmax may still read)
-                    const uint32_t d = tmem + (next_s & 1) * KT;
-                    for (uint32_t m = 0; m < p.mtiles && ok; m++) {
-                        ok = wait_or_abort(bar_full + 8 * st_s, ph_s, abort_flag);
-                        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                        if (!ok) break;
-                        box(2 * m, ring0 + st_s * (2 * BOX >> 4), d);
-                        if (2 * m + 1 < p.boxes) box(2 * m + 1, ring0 + st_s * (2 * BOX >> 4) + (BOX >> 4), d);
-                        if (++st_s == NP) { st_s = 0; ph_s ^= 1; }
-                    }
-                    if (p.rest && ok) {
-                        ok = wait_or_abort(bar_rest + 8 * rs, rph, abort_flag);
-                        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                        for (uint32_t b = 0; b < p.rest && ok; b++) box(2 * p.mtiles + b, rest0 + (rs * p.rest + b) * (BOX >> 4), d);
-                        if (ok) mma_commit(bar_free + 8 * rs);
-                        if (++rs == NR) { rs = 0; rph ^= 1; }
-                    }
-                    if (ok) mma_commit(bar_scores + 8 * (next_s & 1));
-                    next_s++;
-                    idle = 0;
-                } else if (++idle == gemm::SPIN || ((idle & 1023u) == 1023u && *abort_flag)) {
-                    ok = false;
                 }
+                for (uint32_t m = 0; m < p.mtiles && ok; m++) {
+                    ok = wait_or_abort(bar_full + 8 * fs, fph, abort_flag);
+                    if (!ok) break;
+                    box(2 * m, ring0 + fs * (2 * BOX >> 4));
+                    if (2 * m + 1 < p.boxes) box(2 * m + 1, ring0 + fs * (2 * BOX >> 4) + (BOX >> 4));
+                    if (++fs == NP) { fs = 0; fph ^= 1; }
+                }
+                if (p.rest && ok) {
+                    ok = wait_or_abort(bar_rest + 8 * frs, frph, abort_flag);
+                    for (uint32_t b = 0; b < p.rest && ok; b++) box(2 * p.mtiles + b, rest0 + (frs * p.rest + b) * (BOX >> 4));
+                    if (ok) mma_commit(bar_free + 8 * frs);
+                    if (++frs == NR) { frs = 0; frph ^= 1; }
+                }
+                if (ok) mma_commit(bar_scores + 8 * (i & 1));
+            }
+        }
+        __syncwarp();
+    } else if (warp == 2) {
+        if (elect_one()) {
+            constexpr uint32_t idesc = instr_desc(128, ROWS) | (1u << 15);  // (bit 15: A's lines are its k)
+            const uint64_t mn_major = mn_major_desc(0, BOX);
+            const uint32_t ring0 = lo(ring), p0 = lo(probs);
+            uint32_t fs = 0;
+            for (uint32_t i = 0; i < n && ok; i++) {
+                ok = wait_or_abort(bar_p + 8 * (i & 1), (i >> 1) & 1, abort_flag);  // (P comes of the scores, and they of the whole tile)
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                for (uint32_t m = 0; m < p.mtiles; m++) {
+#pragma unroll
+                    for (uint32_t kk = 0; kk < KT / 16; kk++)
+                        mma_f16(tmem_o + m * ROWS, mn_major + (ring0 + fs * (2 * BOX >> 4) + kk * (2048 >> 4)), k_major + (p0 + kk * 2), idesc, (i | kk) != 0 ? 1u : 0u);
+                    mma_commit(bar_empty + 8 * fs);
+                    if (++fs == NP) fs = 0;
+                }
+                mma_commit(bar_sums);
             }
         }
         __syncwarp();
@@ -336,7 +367,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             }
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             __syncwarp();
-            if (lane == 0) mbar_arrive(bar_p);
+            if (lane == 0) mbar_arrive(bar_p + 8 * (i & 1));
         }
         if (active) {
 #pragma unroll
@@ -370,26 +401,27 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     }
     __syncwarp();
     if (splits > 1) {
-        // The cluster: block b finishes columns b span on. [source][row][column of the span] and behind them (m, l) per (source, row), in the
-        // room of Q and the ring. The first barrier: every block is done with them; the second: every partial has arrived.
+        // The cluster: block b finishes columns b span on. [source][column of the span][row] and behind them (m, l) per (source, row), in the
+        // room of Q and the rings. The first barrier: every block is done with them; the second: every partial has arrived.
         cluster_sync();
-        const uint32_t span = p.mtiles * 128 / splits, stats = splits * ROWS * span * 4;
-        if (warp >= 2) {
-            const uint32_t quarter = warp & 3, me = tid - 64;
-            if (me < ROWS)
-                for (uint32_t b = 0; b < splits; b++) {
-                    const uint32_t dst = cluster_addr(base + stats + (sp * ROWS + me) * 8, b);
-                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(m_s[me]) : "memory");
-                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + 4), "f"(l_s[me]) : "memory");
-                }
+        constexpr uint32_t RP = ROWS + 4;  // a column's pitch
+        const uint32_t span = p.mtiles * 128 / splits, stats = splits * span * RP * 4;
+        if (warp >= 3) {
+            const uint32_t quarter = warp & 3, me = tid - 96;
             for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
                 float o[16];
                 tmem_ld16(tmem_o + ((quarter * 32) << 16) + c, o);
                 const uint32_t x = c / ROWS * 128 + quarter * 32 + lane;
-                const uint32_t dst = cluster_addr(base + ((sp * ROWS + c % ROWS) * span + x % span) * 4, x / span);
+                const uint32_t dst = cluster_addr(base + ((sp * span + x % span) * RP + c % ROWS) * 4, x / span);
 #pragma unroll
-                for (uint32_t j = 0; j < 16; j++) asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst + j * span * 4), "f"(n ? o[j] : 0.0f) : "memory");
+                for (uint32_t j = 0; j < 16; j += 4) {
+                    if (!n) o[j] = o[j + 1] = o[j + 2] = o[j + 3] = 0.0f;
+                    asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst + j * 4), "f"(o[j]), "f"(o[j + 1]), "f"(o[j + 2]), "f"(o[j + 3]) : "memory");
+                }
             }
+            if (me < ROWS)
+                for (uint32_t b = 0; b < splits; b++)
+                    asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(cluster_addr(base + stats + (sp * ROWS + me) * 8, b)), "f"(m_s[me]), "f"(l_s[me]) : "memory");
         }
         __syncwarp();
         cluster_sync();
@@ -412,20 +444,23 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
                 if (k < splits) stat[(k * ROWS + tid) * 2] = w[k] / l;
         }
         __syncthreads();
-        for (uint32_t i = tid; i < ROWS * span / 4; i += THREADS) {
-            const uint32_t row = i / (span / 4), c = i % (span / 4) * 4, x = sp * span + c;
-            if (from[row] < 0 || x >= rank) continue;
+        for (uint32_t i = tid; i < ROWS * span / 4; i += THREADS) {  // a column of four rows
+            const uint32_t r0 = i / span * 4, c = i % span, x = sp * span + c;
+            if (x >= rank) continue;
             float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll 4
             for (uint32_t k = 0; k < splits; k++) {
-                const float w = stat[(k * ROWS + row) * 2];
-                const float4 v = *reinterpret_cast<const float4*>(recv + (k * ROWS + row) * span + c);
-                y.x = fmaf(w, v.x, y.x);
-                y.y = fmaf(w, v.y, y.y);
-                y.z = fmaf(w, v.z, y.z);
-                y.w = fmaf(w, v.w, y.w);
+                const float4 v = *reinterpret_cast<const float4*>(recv + (k * span + c) * RP + r0);
+                const float* w = stat + (k * ROWS + r0) * 2;
+                y.x = fmaf(w[0], v.x, y.x);
+                y.y = fmaf(w[2], v.y, y.y);
+                y.z = fmaf(w[4], v.z, y.z);
+                y.w = fmaf(w[6], v.w, y.w);
             }
-            *reinterpret_cast<uint2*>(a.out_b + size_t(from[row]) * rank + x) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
+            const float ys[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+            for (uint32_t j = 0; j < 4; j++)
+                if (from[r0 + j] >= 0) a.out_b[size_t(from[r0 + j]) * rank + x] = f32_to_bf16(ys[j]);
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
