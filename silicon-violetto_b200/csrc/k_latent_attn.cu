@@ -182,21 +182,27 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             uint32_t tok;
             from[tid - 32] = row_at(tid - 32, tok);
         }
-        // Q in the MMA's swizzle: zeros where there are no rows or columns. Six loads at a time.
-        const uint32_t all = ROWS * p.boxes * 8;
-        for (uint32_t i0 = tid - 32; i0 < all; i0 += 6 * (THREADS - 32)) {
-            uint4 x[6];
+        // Q in the MMA's swizzle, zeros where there are no rows or columns: a row a warp, three of them at a time, 16 bytes a lane and load.
+        constexpr uint32_t WARPS = THREADS / 32 - 1, AT_ONCE = 3;
+        for (uint32_t r0 = warp - 1; r0 < ROWS; r0 += AT_ONCE * WARPS) {
+            uint4 x[AT_ONCE][3];
 #pragma unroll
-            for (uint32_t u = 0; u < 6; u++) {
-                const uint32_t i = i0 + u * (THREADS - 32), r = i / (p.boxes * 8), c = i % (p.boxes * 8);
+            for (uint32_t u = 0; u < AT_ONCE; u++) {
                 uint32_t tok;
-                const int at = i < all ? row_at(r, tok) : -1;
-                x[u] = at >= 0 && c * 8 < dk ? *reinterpret_cast<const uint4*>(a.q_b + size_t(at) * dk + c * 8) : make_uint4(0, 0, 0, 0);
+                const uint32_t r = r0 + u * WARPS;
+                const int at = r < ROWS ? row_at(r, tok) : -1;
+                const uint4* src = reinterpret_cast<const uint4*>(a.q_b + size_t(max(at, 0)) * dk);
+#pragma unroll
+                for (uint32_t y = 0; y < 3; y++) x[u][y] = at >= 0 && (lane + 32 * y) * 8 < dk ? src[lane + 32 * y] : make_uint4(0, 0, 0, 0);
             }
 #pragma unroll
-            for (uint32_t u = 0; u < 6; u++) {
-                const uint32_t i = i0 + u * (THREADS - 32), r = i / (p.boxes * 8), c = i % (p.boxes * 8);
-                if (i < all) *reinterpret_cast<uint4*>(smem + c / 8 * QB + r * 128 + ((c % 8 ^ (r & 7)) << 4)) = x[u];
+            for (uint32_t u = 0; u < AT_ONCE; u++) {
+                const uint32_t r = r0 + u * WARPS;
+#pragma unroll
+                for (uint32_t y = 0; y < 3; y++) {
+                    const uint32_t c = lane + 32 * y;
+                    if (r < ROWS && c < p.boxes * 8) *reinterpret_cast<uint4*>(smem + c / 8 * QB + r * 128 + ((c % 8 ^ (r & 7)) << 4)) = x[u][y];
+                }
             }
         }
     }
@@ -427,28 +433,29 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         cluster_sync();
         const float* recv = reinterpret_cast<const float*>(smem);
         float* stat = reinterpret_cast<float*>(smem + stats);
+        // (Code that runs once a block: rolled loops, as its instructions have to be fetched.)
         if (tid < ROWS) {  // what each source's sums of the row are worth
-            float m = -INFINITY, l = 0.0f, w[MAX_SPLITS];
-#pragma unroll
-            for (uint32_t k = 0; k < MAX_SPLITS; k++) {
-                w[k] = k < splits ? stat[(k * ROWS + tid) * 2] : -INFINITY;
-                m = fmaxf(m, w[k]);
+            float m = -INFINITY, l = 0.0f;
+#pragma unroll 1
+            for (uint32_t k = 0; k < splits; k++) {
+                const float2 ml = *reinterpret_cast<const float2*>(stat + (k * ROWS + tid) * 2);
+                const float top = fmaxf(m, ml.x);
+                if (top != -INFINITY) l = l * fast_exp2(m - top) + ml.y * fast_exp2(ml.x - top);
+                m = top;
             }
-#pragma unroll
-            for (uint32_t k = 0; k < MAX_SPLITS; k++) {
-                w[k] = w[k] == -INFINITY ? 0.0f : fast_exp2(w[k] - m);
-                if (k < splits) l += stat[(k * ROWS + tid) * 2 + 1] * w[k];
+#pragma unroll 1
+            for (uint32_t k = 0; k < splits; k++) {
+                float* w = stat + (k * ROWS + tid) * 2;
+                *w = *w == -INFINITY ? 0.0f : __fdividef(fast_exp2(*w - m), l);
             }
-#pragma unroll
-            for (uint32_t k = 0; k < MAX_SPLITS; k++)
-                if (k < splits) stat[(k * ROWS + tid) * 2] = w[k] / l;
         }
         __syncthreads();
-        for (uint32_t i = tid; i < ROWS * span / 4; i += THREADS) {  // a column of four rows
-            const uint32_t r0 = i / span * 4, c = i % span, x = sp * span + c;
-            if (x >= rank) continue;
+#pragma unroll 1
+        for (uint32_t u = warp, per = (span + 31) / 32; u < ROWS / 4 * per; u += THREADS / 32) {  // 32 neighbouring columns of four rows
+            const uint32_t r0 = u / per * 4, c = u % per * 32 + lane, x = sp * span + c;
+            if (c >= span || x >= rank) continue;
             float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 4
+#pragma unroll 2
             for (uint32_t k = 0; k < splits; k++) {
                 const float4 v = *reinterpret_cast<const float4*>(recv + (k * span + c) * RP + r0);
                 const float* w = stat + (k * ROWS + r0) * 2;
