@@ -110,12 +110,13 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     const uint32_t base = smem_u32(smem), ring = base + p.boxes * QB, rest = ring + NP * 2 * BOX, probs = rest + NR * p.rest * BOX;
     uint8_t* misc = smem + (probs - base) + QB;
     const uint32_t bar_full = smem_u32(misc), bar_empty = bar_full + 8 * MAX_SLOTS, bar_rest = bar_empty + 8 * MAX_SLOTS, bar_free = bar_rest + 8 * REST_SLOTS, bar_scores = bar_free + 8 * REST_SLOTS,
-                   bar_p = bar_scores + 16, bar_sums = bar_p + 16;
+                   bar_p = bar_scores + 16, bar_sums = bar_p + 16, bar_merge = bar_sums + 8;
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_SLOTS + 2 * REST_SLOTS + 6));
     volatile uint32_t* abort_flag = tmem_slot + 1;
     volatile uint32_t* end_s = tmem_slot + 2;
     int* from = reinterpret_cast<int*>(misc + 512);  // a row's place among the queries and the outputs, -1: none
-    float *corr_s = reinterpret_cast<float*>(from + ROWS), *m_s = corr_s + ROWS, *l_s = m_s + ROWS;
+    float* corr_s = reinterpret_cast<float*>(from + ROWS);
+    float2* ml_s = reinterpret_cast<float2*>(corr_s + ROWS);  // a row's maximum and the sum under it
     if (tid == 0) {
         for (uint32_t i = 0; i < 2 * MAX_SLOTS + 2 * REST_SLOTS; i++) mbar_init(bar_full + 8 * i, 1);
         mbar_init(bar_scores, 1);
@@ -123,6 +124,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         mbar_init(bar_p, ACTIVE);
         mbar_init(bar_p + 8, ACTIVE);
         mbar_init(bar_sums, 1);
+        mbar_init(bar_merge, 1);
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -164,6 +166,11 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         begin = min(sp * share, tiles);
         n = min(share, tiles - begin);
     };
+    // Splits: what the cluster's blocks send of their sums arrives as [source][column of this block's span][row], (m, l) per (source, row)
+    // behind it, in the room of Q and the rings; there, too, this block's own, to be copied from.
+    constexpr uint32_t RP = ROWS + 4;     // a column's pitch
+    constexpr bool BULK = ROWS < 64;      // (64 rows: no room for both; stored one by one)
+    const uint32_t span = p.mtiles * 128 / splits, stats = splits * span * RP * 4, own = stats + splits * ROWS * 8;
     bool ok = true;
     if (warp == 0) {  // how far the rows see, and the first two tiles on their way while the others fetch the queries
         uint32_t end = 0;
@@ -380,24 +387,29 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             for (uint32_t r = 0; r < 2; r++) {
                 l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
                 l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
-                if (tq == 0) {
-                    m_s[quarter * 16 + g + 8 * r] = m_run[r];
-                    l_s[quarter * 16 + g + 8 * r] = l_run[r];
-                }
+                if (tq == 0) ml_s[quarter * 16 + g + 8 * r] = make_float2(m_run[r], l_run[r]);
             }
         }
         if (n) ok = ok && wait_or_abort(bar_sums, (n - 1) & 1, abort_flag);
         ok = __all_sync(0xffffffffu, ok);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         softmax_sync();
-        if (splits == 1) {
+        if (splits > 1 && BULK) {  // O as the cluster's blocks will take it, a column's rows together
+            for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
+                float o[16];
+                tmem_ld16(o_addr + c, o);
+                float4* dst = reinterpret_cast<float4*>(smem + own + ((c / ROWS * 128 + quarter * 32 + lane) * RP + c % ROWS) * 4);
+#pragma unroll
+                for (uint32_t j = 0; j < 4; j++) dst[j] = n ? make_float4(o[4 * j], o[4 * j + 1], o[4 * j + 2], o[4 * j + 3]) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+        } else if (splits == 1) {
             for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
                 float o[16];
                 tmem_ld16(o_addr + c, o);
                 const uint32_t x = c / ROWS * 128 + quarter * 32 + lane, r0 = c % ROWS;
 #pragma unroll
                 for (uint32_t j = 0; j < 16; j++)
-                    if (from[r0 + j] >= 0 && x < rank) a.out_b[size_t(from[r0 + j]) * rank + x] = f32_to_bf16(__fdividef(o[j], l_s[r0 + j]));
+                    if (from[r0 + j] >= 0 && x < rank) a.out_b[size_t(from[r0 + j]) * rank + x] = f32_to_bf16(__fdividef(o[j], ml_s[r0 + j].y));
             }
         }
     }
@@ -407,30 +419,49 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     }
     __syncwarp();
     if (splits > 1) {
-        // The cluster: block b finishes columns b span on. [source][column of the span][row] and behind them (m, l) per (source, row), in the
-        // room of Q and the rings. The first barrier: every block is done with them; the second: every partial has arrived.
-        cluster_sync();
-        constexpr uint32_t RP = ROWS + 4;  // a column's pitch
-        const uint32_t span = p.mtiles * 128 / splits, stats = splits * span * RP * 4;
-        if (warp >= 3) {
-            const uint32_t quarter = warp & 3, me = tid - 96;
-            for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
-                float o[16];
-                tmem_ld16(tmem_o + ((quarter * 32) << 16) + c, o);
-                const uint32_t x = c / ROWS * 128 + quarter * 32 + lane;
-                const uint32_t dst = cluster_addr(base + ((sp * span + x % span) * RP + c % ROWS) * 4, x / span);
-#pragma unroll
-                for (uint32_t j = 0; j < 16; j += 4) {
-                    if (!n) o[j] = o[j + 1] = o[j + 2] = o[j + 3] = 0.0f;
-                    asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst + j * 4), "f"(o[j]), "f"(o[j + 1]), "f"(o[j + 2]), "f"(o[j + 3]) : "memory");
-                }
+        // The cluster: block b finishes columns b span on.
+        if (BULK) {
+            if (tid == 0) mbar_expect_tx(bar_merge, splits * (span * RP * 4 + ROWS * 8));
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            __syncwarp();
+            cluster_sync();  // every block is done with its ring, has laid out its sums and expects the others'
+            if (tid < splits) {
+                auto copy = [&](uint32_t to, uint32_t src, uint32_t bytes) {
+                    asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(cluster_addr(base + to, tid)), "r"(src), "r"(bytes),
+                                 "r"(cluster_addr(bar_merge, tid))
+                                 : "memory");
+                };
+                copy(sp * span * RP * 4, base + own + tid * span * RP * 4, span * RP * 4);
+                copy(stats + sp * ROWS * 8, smem_u32(ml_s), ROWS * 8);
             }
-            if (me < ROWS)
-                for (uint32_t b = 0; b < splits; b++)
-                    asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(cluster_addr(base + stats + (sp * ROWS + me) * 8, b)), "f"(m_s[me]), "f"(l_s[me]) : "memory");
+            ok = gemm::mbar_wait(bar_merge, 0);  // (they come whatever went wrong before)
+            if (!ok) atomicExch(p.err_flag, 6u);
+            __syncwarp();
+            // (No block leaves before every copy, its own among them, has arrived.)
+            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+        } else {
+            cluster_sync();  // every block is done with its ring
+            if (warp >= 3) {
+                const uint32_t quarter = warp & 3, me = tid - 96;
+                for (uint32_t c = 0; c < p.mtiles * ROWS; c += 16) {
+                    float o[16];
+                    tmem_ld16(tmem_o + ((quarter * 32) << 16) + c, o);
+                    const uint32_t x = c / ROWS * 128 + quarter * 32 + lane;
+                    const uint32_t dst = cluster_addr(base + ((sp * span + x % span) * RP + c % ROWS) * 4, x / span);
+#pragma unroll
+                    for (uint32_t j = 0; j < 16; j += 4) {
+                        if (!n) o[j] = o[j + 1] = o[j + 2] = o[j + 3] = 0.0f;
+                        asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst + j * 4), "f"(o[j]), "f"(o[j + 1]), "f"(o[j + 2]), "f"(o[j + 3]) : "memory");
+                    }
+                }
+                if (me < ROWS)
+                    for (uint32_t b = 0; b < splits; b++)
+                        asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(cluster_addr(base + stats + (sp * ROWS + me) * 8, b)), "f"(ml_s[me].x), "f"(ml_s[me].y) : "memory");
+            }
+            __syncwarp();
+            cluster_sync();  // every partial has arrived
+            asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
         }
-        __syncwarp();
-        cluster_sync();
         const float* recv = reinterpret_cast<const float*>(smem);
         float* stat = reinterpret_cast<float*>(smem + stats);
         // (Code that runs once a block: rolled loops, as its instructions have to be fetched.)
@@ -469,6 +500,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             for (uint32_t j = 0; j < 4; j++)
                 if (from[r0 + j] >= 0) a.out_b[size_t(from[r0 + j]) * rank + x] = f32_to_bf16(ys[j]);
         }
+        __syncwarp();
+        asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
@@ -509,21 +542,42 @@ void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t ma
     if (p.slots < 2 * p.mtiles) throw Error("internal: latent attention over " + std::to_string(a.kv.dk) + " columns");
     p.tmem_cols = 32;
     while (p.tmem_cols < 2 * KT + p.mtiles * ROWS) p.tmem_cols *= 2;
-    // A tile's positions over 1, 2, 4 or 8 blocks, or 16 where 8 leave most SMs idle: the count that makes waves of blocks (one an SM) times
-    // a block's positions, plus a fixed part, least.
-    const uint32_t units = std::max(1u, (n + p.toks - 1) / p.toks * p.groups), most = units * 16 <= sm_count ? MAX_SPLITS : 8;
+    // A tile's positions over 1, 2, 4, 8 or 16 blocks: the count that makes waves of clusters times a block's positions, plus what a block and
+    // a cluster's exchange cost besides (as much as some hundred positions), least.
+    const uint32_t units = std::max(1u, (n + p.toks - 1) / p.toks * p.groups), smem = std::max(SMEM_MIN, fixed + (p.rest * p.rest_slots + 2 * p.slots) * BOX);
+    static thread_local std::map<std::pair<uint32_t, uint32_t>, uint32_t> wave;  // (shared memory, cluster size) -> clusters that run at once
+    auto at_once = [&](uint32_t c) {
+        if (c == 1) return sm_count;
+        auto w = wave.find({smem, c});
+        if (w != wave.end()) return w->second;
+        cudaLaunchConfig_t q = {};
+        q.gridDim = dim3(sm_count, 1, c);
+        q.blockDim = dim3(THREADS);
+        q.dynamicSmemBytes = smem;
+        cudaLaunchAttribute qa[1];
+        qa[0].id = cudaLaunchAttributeClusterDimension;
+        qa[0].val.clusterDim.x = qa[0].val.clusterDim.y = 1;
+        qa[0].val.clusterDim.z = c;
+        q.attrs = qa;
+        q.numAttrs = 1;
+        int clusters = 0;
+        const cudaError_t e = cudaOccupancyMaxActiveClusters(&clusters, latent_kernel<ROWS>, &q);
+        return wave.emplace(std::make_pair(smem, c), e == cudaSuccess ? uint32_t(clusters) : 0u).first->second;
+    };
     uint32_t splits = 1;
     uint64_t best = ~0ull;
-    for (uint32_t c = 1; c <= most && (c == 1 || max_keys / c >= 64); c *= 2) {
-        const uint64_t cost = uint64_t((units * c + sm_count - 1) / sm_count) * ((max_keys + c - 1) / c + 256);
+    for (uint32_t c = 1; c <= MAX_SPLITS && (c == 1 || max_keys / c >= KT); c *= 2) {
+        const uint32_t w = at_once(c);
+        if (!w) continue;
+        const uint64_t cost = uint64_t((units + w - 1) / w) * ((max_keys + c - 1) / c + (c > 1 ? 550 : 300));
         if (cost < best) { best = cost; splits = c; }
     }
     if (keys_per_block)
-        for (splits = 1; splits < MAX_SPLITS && splits * keys_per_block < max_keys;) splits *= 2;
+        for (splits = 1; splits < MAX_SPLITS && splits * keys_per_block < max_keys && at_once(2 * splits);) splits *= 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((p.sub ? n_ctiles * p.sub : n) * p.groups, 1, splits);
     cfg.blockDim = dim3(THREADS);
-    cfg.dynamicSmemBytes = std::max(SMEM_MIN, fixed + (p.rest * p.rest_slots + 2 * p.slots) * BOX);
+    cfg.dynamicSmemBytes = smem;
     cfg.stream = s;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;

@@ -46,7 +46,7 @@ CONFIGS = {
     "dense": pv.config(128, 200, [pv.lightning(64, 64, [0.9, 0.8], mlp=pv.dense(192))]),
 }
 # Latents up to the largest kernel's, in every number of rows a block may have, and in ranks between those a kernel is laid out for.
-for rank, rot, heads in ((512, 64, 16), (512, 64, 24), (512, 64, 40), (384, 32, 70), (256, 64, 8), (256, 128, 4), (136, 8, 5), (40, 88, 33), (512, 128, 2)):
+for rank, rot, heads in ((512, 64, 16), (512, 64, 24), (512, 64, 40), (384, 32, 70), (256, 64, 8), (256, 128, 4), (136, 8, 5), (40, 88, 33), (24, 8, 3), (512, 128, 2)):
     CONFIGS[f"rank{rank}_{rot}_{heads}"] = pv.config(128, 96, [pv.latent(heads, 64, rot, 16, rank, 64, scale=0.12)], side=64)
 # Key channels up to the largest kernel's.
 for n, N in enumerate((5, 40, 70, 100, 170, 230, 300, 512)):
