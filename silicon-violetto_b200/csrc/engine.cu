@@ -450,7 +450,7 @@ Plan Engine::plan(uint32_t set, const std::vector<PlanRun>& runs, Rows hidden) {
 // tensor cores from registers; larger ones go in token blocks of 8 (the weights of one matrix
 // stay in L2 between blocks).
 void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint32_t epi, const float* base, float* inv_out, uint32_t vocab_real,
-                    const QkvEpilogue* q, const uint16_t* xb, uint16_t* yb, float scale, float ra, float rb) {
+                    const QkvEpilogue* q, const uint16_t* xb, uint16_t* yb, float scale, float ra, float rb, const SideTable* side) {
     MatArgs a{};
     a.scale = scale;
     a.ra = ra;
@@ -466,10 +466,12 @@ void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint3
     a.epi = epi;
     a.vocab_real = vocab_real ? vocab_real : model.md.vocab_real;
     a.eps = model.md.eps;
-    const uint32_t out_w = epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
+    if (side) a.side = *side;
+    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 8) {
         a.n = std::min(8u, n - t0);
         a.t0 = t0;
+        if (side) a.side.tokens = side->tokens + t0;
         a.X = x + size_t(t0) * w.k;
         a.Xb = xb ? xb + size_t(t0) * w.k : nullptr;
         a.Y = y ? y + size_t(t0) * out_w : nullptr;
@@ -511,7 +513,7 @@ bool Engine::layer_carries(const Layer& l, uint32_t n) const {
 }
 
 void Engine::matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, const float* inv,
-                         uint32_t vocab_real, const QkvEpilogue* q, float* ssq_out, const float* ssq_in, float scale, float ra, float rb) {
+                         uint32_t vocab_real, const QkvEpilogue* q, float* ssq_out, const float* ssq_in, float scale, float ra, float rb, const SideTable* side) {
     MatArgs a{};
     a.scale = scale;
     a.ra = ra;
@@ -539,10 +541,12 @@ void Engine::matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float*
     // The kernel's N is at most 256 tokens: a longer step (a prompt chunk) goes in blocks of 256, the weights read once per
     // block (the reference's tiled GEMM loops its token tiles the same way, kernels.metal:319-514). Everything indexed by
     // token moves along with the block.
-    const uint32_t out_w = epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
+    if (side) a.side = *side;
+    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 256) {
         MatArgs b = a;
         b.n = std::min(256u, n - t0);
+        if (side) b.side.tokens = side->tokens + t0;
         b.Xb = xb + size_t(t0) * w.k;
         b.Y = y ? y + size_t(t0) * out_w : nullptr;
         b.Yb = yb ? yb + size_t(t0) * out_w : nullptr;

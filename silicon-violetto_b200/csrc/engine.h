@@ -281,7 +281,7 @@ class Engine {
     void encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
     // Y = epilogue(W x) in the engine's precision: xf in an fp32 engine, else xb through the GEMM, the streamed matmul or,
     // for sizes neither takes, the CUDA cores.
-    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr, uint32_t act_rows = 0);
+    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr, uint32_t act_rows = 0, const SideTable* side = nullptr);
     std::unique_ptr<LimiteState> lim;
     LimiteKv limite_kv(const LimiteLayer& x) const;
     void encode_forward_limite(uint32_t set, const Plan& p);
@@ -326,12 +326,12 @@ class Engine {
   private:
     KvArgs kv_args() const;
     void matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint32_t epi, const float* base, float* inv_out, uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr,
-                const uint16_t* xb = nullptr, uint16_t* yb = nullptr, float scale = 1.0f, float ra = 1.0f, float rb = 1.0f);
+                const uint16_t* xb = nullptr, uint16_t* yb = nullptr, float scale = 1.0f, float ra = 1.0f, float rb = 1.0f, const SideTable* side = nullptr);
     bool stream_fits(const Matrix& w, uint32_t n = 1) const;
     // The tensor-core GEMM: xb is x in bf16, inv the rows' 1/rms (normed epilogues), yb an optional bf16 copy of y.
     void matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, const float* inv,
                      uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr, float* ssq_out = nullptr, const float* ssq_in = nullptr, float scale = 1.0f, float ra = 1.0f,
-                     float rb = 1.0f);
+                     float rb = 1.0f, const SideTable* side = nullptr);
     bool use_gemm(const Matrix& w, uint32_t n) const;
     bool gemm_fits(const Matrix& w, uint32_t n) const;
     // A layer of n tokens runs on the tensor-core GEMM and its last projection leaves bf16(h) in h_b and h's sums of squares in ssq.

@@ -231,12 +231,12 @@ void Engine::init_layered() {
     z.recurrent_dev.write_vec(0, z.recurrent);
 }
 
-void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, uint32_t act_rows) {
+void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, uint32_t act_rows, const SideTable* side) {
     const bool gemm = !cfg.fp32 && w.m % 128 == 0 && w.k % 64 == 0, stream_takes = !cfg.fp32 && stream_fits(w, n);
     if (gemm && (gemm_fits(w, n) || !stream_takes)) {  // (few rows that are too long for the streamed kernel's shared memory, too)
-        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr, act_rows);
+        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr, act_rows, nullptr, nullptr, nullptr, 1.0f, 1.0f, 1.0f, side);
     } else if (stream_takes) {
-        matmul(w, n, nullptr, y, epi, base, nullptr, act_rows, nullptr, xb, yb);
+        matmul(w, n, nullptr, y, epi, base, nullptr, act_rows, nullptr, xb, yb, 1.0f, 1.0f, 1.0f, side);
     } else {
         LinearArgs a{};
         a.W = reinterpret_cast<const uint16_t*>(w.w);
@@ -625,24 +625,23 @@ void Engine::add_norm(const float* x, const RowNorm& norm, uint32_t n) {
 
 void Engine::encode_side(StepSet& st, const SideInput& x, uint32_t n) {
     LayeredState& z = *lay;
-    int sp = span_begin(G_MATMUL);
-    project(x.gate, n, z.in_f, z.xn_b.as<uint16_t>(), z.side.as<float>(), nullptr, EPI_RAW);
-    span_end(sp);
     SideGateArgs g{};
-    g.x = z.side.as<float>();
-    g.ldx = x.gate.m;
-    g.table = model.layered->side;
-    g.ld = model.layered->side_w;
-    g.tokens = st.in<uint32_t>(st.o_tokens);
+    g.side = SideTable{model.layered->side, st.in<uint32_t>(st.o_tokens), model.layered->side_w, x.first, x.dim, x.proj.k};
     g.out_f32 = cfg.fp32 ? z.side_f.as<float>() : nullptr;
     g.out_bf16 = cfg.fp32 ? nullptr : z.side_b.as<uint16_t>();
-    g.n = n;
-    g.first = x.first;
-    g.dim = x.dim;
-    g.wide = x.proj.k;
-    sp = span_begin(G_SMALL);
-    launch_side_gate(g, stream);
+    const bool fused = !cfg.fp32 && x.gate.m >= x.proj.k && ((x.gate.m % 128 == 0 && x.gate.k % 64 == 0) || stream_fits(x.gate, n));  // (the kernels that have the gate as an epilogue)
+    int sp = span_begin(G_MATMUL);
+    if (fused) project(x.gate, n, nullptr, z.xn_b.as<uint16_t>(), nullptr, g.out_bf16, EPI_SIDE, nullptr, 0, &g.side);
+    else project(x.gate, n, z.in_f, z.xn_b.as<uint16_t>(), z.side.as<float>(), nullptr, EPI_RAW);
     span_end(sp);
+    if (!fused) {
+        g.x = z.side.as<float>();
+        g.ldx = x.gate.m;
+        g.n = n;
+        sp = span_begin(G_SMALL);
+        launch_side_gate(g, stream);
+        span_end(sp);
+    }
     sp = span_begin(G_MATMUL);
     project(x.proj, n, g.out_f32, g.out_bf16, z.branch.as<float>(), nullptr, EPI_RAW);
     span_end(sp);

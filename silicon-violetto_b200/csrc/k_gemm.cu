@@ -358,6 +358,7 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
             else if (EPI == EPI_HEAD) y[j] = row < m.vocab_real ? x * inv[j] : -INFINITY;
             else if (EPI == EPI_HEAD_CAP) y[j] = row < m.vocab_real ? 23.0f * (1.0f / (1.0f + __expf(-(x + 5.0f) / 7.5f))) : -INFINITY;  // kernels.metal:196-199
             else if (EPI == EPI_RELU2) y[j] = x > 0.0f ? x * x : 0.0f;
+            else if (EPI == EPI_SIDE) y[j] = t0 + j < m.n ? side_of(m.side, t0 + j, row, x) : 0.0f;
             else if (EPI == EPI_SILU) y[j] = row < m.vocab_real ? x * __fdividef(1.0f, 1.0f + __expf(-x)) : x;
             else y[j] = x;
         }
@@ -382,8 +383,8 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
             for (uint32_t bit = 16 / NTOK; bit >= 1; bit /= 2) w[0] += __shfl_xor_sync(0xffffffffu, w[0], bit);
             if ((lane & (32 / NTOK - 1)) == 0) ssq_s[(r / 32) * n_pad + t0 + tk] = w[0];
         }
-        const bool writes = valid && (!PAIRS || (lane & 1) == 0);
-        const uint32_t out_w = PAIRS ? m.m / 2 : m.m, out_r = PAIRS ? row / 2 : row;
+        const bool writes = valid && (!PAIRS || (lane & 1) == 0) && (EPI != EPI_SIDE || row < m.side.wide);
+        const uint32_t out_w = EPI == EPI_SIDE ? m.side.wide : PAIRS ? m.m / 2 : m.m, out_r = PAIRS ? row / 2 : row;
         if (writes) {
 #pragma unroll
             for (uint32_t j = 0; j < NTOK; j++)
@@ -416,6 +417,11 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
                 }
             }
             inv_s[t] = inv;
+            if (EPI == EPI_SIDE && t < a.m.n && row0 < a.m.side.dim) {  // the table's entries for this tile on their way while the products run
+                const uint16_t* e = a.m.side.table + size_t(a.m.side.tokens[t]) * a.m.side.ld + a.m.side.first + row0;
+                for (uint32_t i = 0; i < min(BM, a.m.side.dim - row0); i += 64) asm volatile("prefetch.global.L1 [%0];" ::"l"(e + i));
+                asm volatile("prefetch.global.L1 [%0];" ::"l"(e + min(BM, a.m.side.dim - row0) - 1));
+            }
             if (EPI == EPI_QKV) {
                 const QkvEpilogue& qe = a.m.q;
                 uint32_t pos = 0, kvrow = NO_TOK;
@@ -537,6 +543,7 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
     case EPI_RELU2: return int8 ? gemm::gemm_kernel<true, EPI_RELU2> : gemm::gemm_kernel<false, EPI_RELU2>;
     case EPI_SILU: return gemm::gemm_kernel<false, EPI_SILU>;  // (bf16 weights only)
     case EPI_GLU: return gemm::gemm_kernel<false, EPI_GLU>;
+    case EPI_SIDE: return gemm::gemm_kernel<false, EPI_SIDE>;
     default: return int8 ? gemm::gemm_kernel<true, EPI_RAW> : gemm::gemm_kernel<false, EPI_RAW>;
     }
 }
@@ -545,7 +552,7 @@ bool gemm_supported(const MatArgs& a) {
     const bool grouped = a.int8 && a.group < a.k;  // scale groups: powers of two from 8
     return a.n >= 1 && a.n <= 256 && a.m % gemm::BM == 0 && a.k % gemm::BK == 0 && (!grouped || (a.group >= 8 && !(a.group & (a.group - 1)))) && a.Xb != nullptr &&
            (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.epi == EPI_RELU2 ||
-            (!a.int8 && (a.epi == EPI_SILU || a.epi == EPI_GLU)) || a.inv_in != nullptr || a.ssq_in != nullptr);
+            (!a.int8 && (a.epi == EPI_SILU || a.epi == EPI_GLU || a.epi == EPI_SIDE)) || a.inv_in != nullptr || a.ssq_in != nullptr);
 }
 
 void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaStream_t s, bool allow_paired) {
@@ -588,7 +595,7 @@ void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaSt
     const size_t smem = paired ? need : std::max<size_t>(need, 116 * 1024);
     configured.once([] {
         for (int i8 = 0; i8 < 2; i8++)
-            for (uint32_t epi = EPI_NORM; epi <= EPI_GLU; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+            for (uint32_t epi = EPI_NORM; epi <= EPI_SIDE; epi++) VLT_CUDA(cudaFuncSetAttribute(gemm_entry(i8 != 0, epi), cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024));
         VLT_CUDA(cudaFuncSetAttribute(gemm_entry(true, EPI_HEAD, true), cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
     });

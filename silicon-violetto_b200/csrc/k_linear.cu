@@ -201,14 +201,9 @@ __global__ void __launch_bounds__(1024) add_norm_kernel(const AddNormArgs a) {
 __global__ void __launch_bounds__(256) side_gate_kernel(const SideGateArgs a) {
     pdl_start();
     const uint32_t t = blockIdx.x, i = blockIdx.y * 256 + threadIdx.x;
-    if (i >= a.wide) return;
-    float y = 0.0f;
-    if (i < a.dim) {
-        const float z = a.x[size_t(t) * a.ldx + i];
-        const float g = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));  // (sqrt(2 / pi))
-        y = g * bf16_to_f32(a.table[size_t(a.tokens[t]) * a.ld + a.first + i]);
-    }
-    const size_t o = size_t(t) * a.wide + i;
+    if (i >= a.side.wide) return;
+    const float y = side_of(a.side, t, i, i < a.side.dim ? a.x[size_t(t) * a.ldx + i] : 0.0f);
+    const size_t o = size_t(t) * a.side.wide + i;
     if (a.out_f32) a.out_f32[o] = y;
     if (a.out_bf16) a.out_bf16[o] = f32_to_bf16(y);
 }
@@ -261,7 +256,7 @@ void launch_add_norm(const AddNormArgs& a, cudaStream_t s) {
     else launch_pdl(linear::add_norm_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 4, s, a);
 }
 void launch_side_gate(const SideGateArgs& a, cudaStream_t s) {
-    if (a.n) launch_pdl(linear::side_gate_kernel, dim3(a.n, (a.wide + 255) / 256), 256, 0, s, a);
+    if (a.n) launch_pdl(linear::side_gate_kernel, dim3(a.n, (a.side.wide + 255) / 256), 256, 0, s, a);
 }
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s) {
     if (n) launch_pdl(linear::concat_rows_kernel, n, 256, 0, s, a, b, d, out_f32, out_bf16);

@@ -16,9 +16,14 @@ namespace vlt {
 // kernels.metal:184-209 `epilogue`, `epilogue_swiglu`. A plain decoder's scales and residual lambdas are 1 and its head has
 // no cap; the reference's own architecture sets them and takes EPI_HEAD_CAP.
 __device__ __forceinline__ void store_out(const MatArgs& a, uint32_t t, uint32_t row, float acc, float inv) {
-    const size_t o = size_t(t) * a.m + row;
+    size_t o = size_t(t) * a.m + row;
     float y;
     switch (a.epi) {
+    case EPI_SIDE:
+        if (row >= a.side.wide) return;
+        y = side_of(a.side, t, row, acc);
+        o = size_t(t) * a.side.wide + row;
+        break;
     case EPI_NORM: y = acc * inv * a.scale; break;
     case EPI_RESID: y = a.ra * a.base[o] + a.rb * (a.scale * acc); break;
     case EPI_HEAD: y = row < a.vocab_real ? acc * inv : -INFINITY; break;

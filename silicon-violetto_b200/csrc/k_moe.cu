@@ -258,14 +258,22 @@ __global__ void __launch_bounds__(256) combine_kernel(const CombineArgs a) {
     float tot = 0.0f;
     for (uint32_t w = 0; w < 8; w++) tot += red[w];
     const float inv = 1.0f / sqrtf(tot / float(a.d) + a.eps);
+    if (a.post.w) {
+        for (uint32_t i = tid * W; i < a.d; i += 256 * W) {
+            const size_t o = size_t(t) * a.d + i;
+            float x[W], y[W], w[W];
+            load_f32<W>(x, a.x + o);
+            load_f32<W>(y, row + i);
+            weights_of<W>(w, a.post, i);
+#pragma unroll
+            for (uint32_t j = 0; j < W; j++) x[j] += y[j] * inv * w[j];
+            store_f32<W>(a.out + o, x);
+            if (a.next_b) store_bf16<W>(a.next_b + o, x);
+        }
+        return;
+    }
     for (uint32_t i = tid; i < a.d; i += 256) {
         const size_t o = size_t(t) * a.d + i;
-        if (a.post.w) {
-            const float v = a.x[o] + row[i] * inv * weight_of(a.post, i);
-            a.out[o] = v;
-            if (a.next_b) a.next_b[o] = f32_to_bf16(v);
-            continue;
-        }
         const float v = row[i] * inv * weight_of(a.norm, i);
         if (a.next) a.next[o] = v;
         if (a.next_b) a.next_b[o] = f32_to_bf16(v);

@@ -13,7 +13,8 @@ namespace vlt {
 enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI_RAW = 5, EPI_QKV = 6, EPI_HEAD_CAP = 7, EPI_RELU2 = 8,  // 7: 23 sigmoid((acc + 5) / 7.5), kernels.metal:196-199; 8: max(acc, 0)^2
                 EPI_SILU = 9,        // silu(acc) for rows below vocab_real, the others as they are
                 EPI_GLU = 10,        // rows in pairs (g, u): silu(g) u, half as many outputs; EPI_SWIGLU's without a norm
-                EPI_GLU_CLAMP = 11   // the same: g sigmoid(1.702 g) (u + 1), g cut off above a limit, u outside of +- the limit
+                EPI_SIDE = 12,       // gelu(acc) times an entry of the token's row in a table (MatArgs::side)
+                EPI_GLU_CLAMP = 11   // EPI_GLU's pairs: g sigmoid(1.702 g) (u + 1), g cut off above a limit, u outside of +- the limit
 };
 
 // What the tensor-core GEMM's EPI_QKV epilogue needs to finish the qkv projection the way `qkv_post` does
@@ -49,6 +50,19 @@ __device__ __forceinline__ void weights_of(float (&x)[V], const RowNorm& n, uint
         for (uint32_t j = 0; j < V; j++) x[j] += 1.0f;
 }
 
+// A row's gate (launch_side_gate, EPI_SIDE): entry i < dim is gelu(z_i) times entry first + i of the token's row in a bf16 table; zeros
+// from there to `wide`.
+struct SideTable {
+    const uint16_t* table;   // [vocab][ld]
+    const uint32_t* tokens;
+    uint32_t ld, first, dim, wide;
+};
+__device__ __forceinline__ float side_of(const SideTable& s, uint32_t t, uint32_t i, float z) {
+    if (i >= s.dim) return 0.0f;
+    const float g = z * sigmoid_of(1.5957691216057308f * (z + 0.044715f * z * z * z));  // (1 + tanh u) / 2 is sigmoid(2 u), u = sqrt(2 / pi) (z + ...)
+    return g * bf16_to_f32(s.table[size_t(s.tokens[t]) * s.ld + s.first + i]);
+}
+
 // Y[t][row] = epilogue(W[row] . bf16(X[t])). X fp32 [n][k]; Y fp32 (SWIGLU: [n][m/2]).
 struct MatArgs {
     const uint8_t* W;
@@ -67,7 +81,8 @@ struct MatArgs {
     // plain decoder.
     float scale = 1.0f, ra = 1.0f, rb = 1.0f;
     bool int8;
-    QkvEpilogue q;  // EPI_QKV only
+    QkvEpilogue q;   // EPI_QKV only
+    SideTable side;  // EPI_SIDE only, whose outputs are `side.wide` to a token
     uint32_t t0;    // EPI_QKV in the streamed matmul: the step's token that this launch's token 0 is
     uint32_t* err_flag;  // streamed matmul: device word set if a bounded wait ran out (optional)
     // The residual stream's sum of squares per token, kept by the tensor-core GEMMs themselves so that no row pass is
@@ -283,14 +298,12 @@ struct AddNormArgs {
     float eps;
 };
 void launch_add_norm(const AddNormArgs& a, cudaStream_t s);
-// out[t][i] = gelu(x[t][i]) times entry first + i of token t's row in a bf16 table, i < dim; zeros from there to `wide`.
 struct SideGateArgs {
     const float* x;          // [n][ldx]
-    const uint16_t* table;   // [vocab][ld]
-    const uint32_t* tokens;
-    float* out_f32;          // optional
+    SideTable side;
+    float* out_f32;          // optional, [n][wide]
     uint16_t* out_bf16;      // optional
-    uint32_t n, ldx, ld, first, dim, wide;
+    uint32_t n, ldx;
 };
 void launch_side_gate(const SideGateArgs& a, cudaStream_t s);
 void launch_concat_rows(const float* a, const float* b, uint32_t n, uint32_t d, float* out_f32, uint16_t* out_bf16, cudaStream_t s);
