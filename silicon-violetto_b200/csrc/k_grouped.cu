@@ -148,6 +148,12 @@ __global__ void __launch_bounds__(THREADS, 2) grouped_kernel(const __grid_consta
             const uint32_t quarter = warp & 3, row = row0 + quarter * 32 + lane;
             for (uint32_t c0 = 0; c0 < n; c0 += 16) {
                 float acc[16];
+                float gate[16];
+                if (EPI == EPI_RAW && a.l.by_head && a.l.gate) {  // (their loads go out together)
+                    const float* from = a.l.gate + size_t(p0 + c0 - group * a.l.by_head) * a.l.ldg + size_t(group) * a.l.m + row;
+#pragma unroll
+                    for (uint32_t j = 0; j < 16; j++) gate[j] = c0 + j < count ? from[size_t(j) * a.l.ldg] : 0.0f;
+                }
                 tmem_ld16(tmem + ((quarter * 32) << 16) + c0, acc);
 #pragma unroll
                 for (uint32_t j = 0; j < 16; j++) {
@@ -163,7 +169,7 @@ __global__ void __launch_bounds__(THREADS, 2) grouped_kernel(const __grid_consta
                         o = size_t(p0 + c0 + j) * (a.l.m / 2) + row / 2;
                     } else if (EPI == EPI_RAW && a.l.by_head) {
                         const size_t t = p0 + c0 + j - group * a.l.by_head;
-                        if (a.l.gate) y *= __fdividef(1.0f, 1.0f + __expf(-a.l.gate[t * a.l.ldg + size_t(group) * a.l.m + row]));
+                        if (a.l.gate) y *= __fdividef(1.0f, 1.0f + __expf(-gate[j]));
                         o = (t * a.l.heads + group) * a.l.ldy + row;
                     }
                     if (a.l.Y) a.l.Y[o] = y;
