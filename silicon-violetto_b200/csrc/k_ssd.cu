@@ -3,7 +3,7 @@
 //
 //   y_t = sum_(s <= t) (q_t . k_s) 2^(c_t - c_s) e_s v_s + 2^(c_t) q_t S,      S <- 2^(c_end) S + sum_s k_s (2^(c_end - c_s) e_s v_s)^T.
 //
-// A block has 32 value channels of one head of one run and goes through the run's chunks in order: four warps, q, k and v rows in
+// A block has 32 (or 16, where there are few blocks) value channels of one head of one run and goes through the run's chunks in order: four warps, q, k and v rows in
 // bf16 (a convolution's outputs), the state in the fp32 accumulators of the last product. What is computed in 32-bit and enters a
 // product -- the weights of the first sum, the state as it is read, the scaled values -- does so as two bf16 parts, whose sum
 // has 16 bits. No exponent is positive: every term weighs at most its step size.
@@ -16,7 +16,7 @@ namespace vlt {
 
 namespace ssd {
 
-constexpr uint32_t T = 64, PS = 32, PP = PS + 8, THREADS = 128;  // tokens of a chunk, value channels of a block and their pitch
+constexpr uint32_t T = 64, THREADS = 128;  // tokens of a chunk
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
 // v0 and v1 as bf16 pairs: the rounded values and what the rounding left.
@@ -25,21 +25,23 @@ __device__ __forceinline__ void split(float v0, float v1, uint32_t& hi, uint32_t
     lo = pack_bf16(v0 - bf16lo(hi), v1 - bf16hi(hi));
 }
 
-template <uint32_t N>
+// PS: value channels of a block.
+template <uint32_t N, uint32_t PS>
 struct Shared {
-    static constexpr uint32_t NP = N + 8;  // pitches that keep ldmatrix free of conflicts
+    static constexpr uint32_t NP = N + 8, PP = PS + 8;  // pitches that keep ldmatrix free of conflicts
     uint16_t q[2][T * NP], k[2][T * NP], v[2][T * PP];
     uint16_t vh[T * PP], vl[T * PP], sh[N * PP], sl[N * PP];  // the scaled values and the state in two parts
     float cum[T], step[T], weight[T];
 };
 
-// grid (heads x spans of 32 value channels, runs).
-template <uint32_t N>
+// grid (heads x spans of PS value channels, runs).
+template <uint32_t N, uint32_t PS>
 __global__ void __launch_bounds__(THREADS) ssd_kernel(const ScanArgs a) {
     pdl_start();
     extern __shared__ __align__(16) uint8_t raw[];
-    Shared<N>& sm = *reinterpret_cast<Shared<N>*>(raw);
-    constexpr uint32_t NP = Shared<N>::NP, MT = N / 64, KS = N / 16, PT = PS / 8;
+    using Sh = Shared<N, PS>;
+    Sh& sm = *reinterpret_cast<Sh*>(raw);
+    constexpr uint32_t NP = Sh::NP, PP = Sh::PP, MT = N / 64, KS = N / 16, PT = PS / 8;
     const RunIn run = a.runs[blockIdx.y];
     if (run.count < a.tensor_min) return;
     const RecurrentCache& c = a.c;
@@ -47,7 +49,7 @@ __global__ void __launch_bounds__(THREADS) ssd_kernel(const ScanArgs a) {
     const uint32_t t0 = run.first, count = run.count, chunks = (count + T - 1) / T;
     const uint16_t *Q = a.q_b + size_t(t0) * a.ldq + head / c.per * N, *K = a.k_b + size_t(t0) * a.ldk + head / c.per * N, *V = a.v_b + size_t(t0) * a.ldv + head * c.P + p0;
     if (count % T) {  // (rows past the last token: finite, and weighed by zero)
-        for (uint32_t i = tid; i < sizeof(Shared<N>) / 16; i += THREADS) reinterpret_cast<uint4*>(raw)[i] = make_uint4(0, 0, 0, 0);
+        for (uint32_t i = tid; i < sizeof(Sh) / 16; i += THREADS) reinterpret_cast<uint4*>(raw)[i] = make_uint4(0, 0, 0, 0);
         __syncthreads();
     }
     auto fetch = [&](uint32_t ch) {
@@ -247,20 +249,22 @@ __global__ void __launch_bounds__(THREADS) ssd_kernel(const ScanArgs a) {
             for (uint32_t e = 0; e < 4; e++) home[(8 * j + 2 * tq + (e & 1)) * c.Np + n0 + 16 * m + g + 8 * (e >> 1)] = S[m][j][e];
 }
 
-template <uint32_t N>
+template <uint32_t N, uint32_t PS>
 void launch(const ScanArgs& a, cudaStream_t s) {
+    using Sh = Shared<N, PS>;
     static PerDevice configured;
-    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(ssd_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(sizeof(Shared<N>)))); });
-    static_assert(sizeof(Shared<N>) % 16 == 0, "cleared by 16 bytes");
-    launch_pdl(ssd_kernel<N>, dim3(a.c.heads * (a.c.P / PS), a.n_runs), THREADS, sizeof(Shared<N>), s, a);
+    configured.once([] { VLT_CUDA(cudaFuncSetAttribute(ssd_kernel<N, PS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(sizeof(Sh)))); });
+    static_assert(sizeof(Sh) % 16 == 0, "cleared by 16 bytes");
+    launch_pdl(ssd_kernel<N, PS>, dim3(a.c.heads * (a.c.P / PS), a.n_runs), THREADS, sizeof(Sh), s, a);
 }
 
 }  // namespace ssd
 
-bool ssd_fits(uint32_t N, uint32_t P) { return (N == 64 || N == 128) && P % ssd::PS == 0; }
+bool ssd_fits(uint32_t N, uint32_t P) { return (N == 64 || N == 128) && P % 32 == 0; }
 void launch_ssd(const ScanArgs& a, cudaStream_t s) {
-    if (a.c.N == 64) ssd::launch<64>(a, s);
-    else ssd::launch<128>(a, s);
+    const bool few = a.c.heads * (a.c.P / 32) * a.n_runs <= 74;  // (half the SMs)
+    if (a.c.N == 64) few ? ssd::launch<64, 16>(a, s) : ssd::launch<64, 32>(a, s);
+    else few ? ssd::launch<128, 16>(a, s) : ssd::launch<128, 32>(a, s);
 }
 
 }  // namespace vlt

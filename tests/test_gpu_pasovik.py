@@ -107,6 +107,21 @@ def test_decays_at_their_ends(decays):
         e.close()
 
 
+@pytest.mark.parametrize("dim,vdim", [(64, 32), (128, 64)])
+def test_chunks_of_many_heads(dim, vdim):
+    """Enough heads, or runs, that a block of the tensor cores' recurrence has 32 value channels; fewer give it 16."""
+    cfg = pv.config(64, 96, [pv.lightning(dim, vdim, list(np.linspace(0.4, 0.999, 80)))], side=9)
+    bits = pv.random_weights(cfg, 22)
+    folder = pv.write_model(pu._TMP / f"many_{dim}", cfg, bits)
+    w = {k: pv.from_bf16(v).astype(np.float64) for k, v in bits.items()}
+    prompts = {n: prompt(cfg, k, 8 + k) for n, k in (("a", 150), ("b", 97), ("c", 40))}
+    eng = pu.engine(folder, False)
+    got = pu.replay(eng, prompts, [[("a", 70), ("b", 64), ("c", 33)], [("c", 1), ("a", 33), ("b", 1)], [("b", 32), ("a", 47), ("c", 6)]])
+    eng.close()
+    for n, toks in prompts.items():
+        close(got[n], ref.forward(cfg, w, toks)[0], False)
+
+
 @BOTH
 @pytest.mark.parametrize("top,experts", [(1, 1), (4, 4), (2, 40)])
 def test_choices_of_experts(top, experts, fp32):
