@@ -19,8 +19,8 @@
 //                through registers; in the end O
 //
 // A row's positions may be split over a cluster of blocks, each of which finishes a span of the columns from what the others store
-// into its shared memory. Every wait is bounded: when one runs out, the kernel sets the error word, waits for nothing more, and
-// leaves by the way it always does.
+// into its shared memory. Every wait is bounded: when one runs out, the kernel sets the error word, goes on without waiting for more of
+// the kind, and leaves by the way it always does.
 //
 // It takes q with scale * log2(e) folded in, rounded to bf16, and leaves the sums in bf16 for the per-head product after it.
 #include <algorithm>
@@ -141,10 +141,9 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         return r / hpt < n_tok && head < a.heads ? int(tok * a.heads + head) : -1;
     };
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    // Tile i's boxes, into slots that are free; false: they did not become so.
     const uint32_t* pages = a.kv.page_table + size_t(a.meta[2 * t0]) * a.kv.max_pages;
     uint32_t begin = 0, n = 0, st = 0, ph = 1, rs = 0, rph = 1;
-    auto load = [&](uint32_t page) {
+    auto load = [&](uint32_t page) {  // a tile's boxes, into slots that are free; false: they did not become so
         const int row = int(page << PAGE_SHIFT);
         for (uint32_t m = 0; m < p.mtiles; m++) {
             const bool two = 2 * m + 1 < p.boxes;
