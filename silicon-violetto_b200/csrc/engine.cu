@@ -450,8 +450,10 @@ Plan Engine::plan(uint32_t set, const std::vector<PlanRun>& runs, Rows hidden) {
 // tensor cores from registers; larger ones go in token blocks of 8 (the weights of one matrix
 // stay in L2 between blocks).
 void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint32_t epi, const float* base, float* inv_out, uint32_t vocab_real,
-                    const QkvEpilogue* q, const uint16_t* xb, uint16_t* yb, float scale, float ra, float rb, const SideTable* side) {
+                    const QkvEpilogue* q, const uint16_t* xb, uint16_t* yb, float scale, float ra, float rb, const SideTable* side, float limit) {
     MatArgs a{};
+    a.bias = w.bias;
+    a.limit = limit;
     a.scale = scale;
     a.ra = ra;
     a.rb = rb;
@@ -467,7 +469,7 @@ void Engine::matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint3
     a.vocab_real = vocab_real ? vocab_real : model.md.vocab_real;
     a.eps = model.md.eps;
     if (side) a.side = *side;
-    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
+    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi_pairs(epi) ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 8) {
         a.n = std::min(8u, n - t0);
         a.t0 = t0;
@@ -513,8 +515,10 @@ bool Engine::layer_carries(const Layer& l, uint32_t n) const {
 }
 
 void Engine::matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, const float* inv,
-                         uint32_t vocab_real, const QkvEpilogue* q, float* ssq_out, const float* ssq_in, float scale, float ra, float rb, const SideTable* side) {
+                         uint32_t vocab_real, const QkvEpilogue* q, float* ssq_out, const float* ssq_in, float scale, float ra, float rb, const SideTable* side, float limit) {
     MatArgs a{};
+    a.bias = w.bias;
+    a.limit = limit;
     a.scale = scale;
     a.ra = ra;
     a.rb = rb;
@@ -542,7 +546,7 @@ void Engine::matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float*
     // block (the reference's tiled GEMM loops its token tiles the same way, kernels.metal:319-514). Everything indexed by
     // token moves along with the block.
     if (side) a.side = *side;
-    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi == EPI_SWIGLU || epi == EPI_GLU ? w.m / 2 : w.m;
+    const uint32_t out_w = epi == EPI_SIDE ? side->wide : epi_pairs(epi) ? w.m / 2 : w.m;
     for (uint32_t t0 = 0; t0 < n; t0 += 256) {
         MatArgs b = a;
         b.n = std::min(256u, n - t0);
@@ -944,7 +948,7 @@ void Engine::begin_step(uint32_t set, const Plan& p) {
     const LayeredModel* lm = model.layered.get();
     launch_embed(model.embed, st.in<uint32_t>(st.o_tokens), lm ? lay->x0.as<float>() : s.h.as<float>(), st.in<uint32_t>(st.o_tin), s.meta.as<uint32_t>(), s.lens.as<uint32_t>(),
                  s.feed.as<uint32_t>(), s.tree.as<uint32_t>(), st.in<uint32_t>(st.o_vis), p.n, model.md.d, model.md.vocab, stream, lm ? lm->positions : nullptr,
-                 lm ? lm->n_positions : 0, lm && lm->layers[0].post_norm && !cfg.fp32 ? lay->xn_b.as<uint16_t>() : nullptr);
+                 lm ? lm->n_positions : 0, lm && lm->layers[0].post_norm && !cfg.fp32 ? lay->xn_b.as<uint16_t>() : nullptr, lm ? lm->embed_scale : 1.0f);
 }
 
 // engine/src/engine/encode.rs:439-451 `encode_replay`.

@@ -248,12 +248,13 @@ class Engine {
     };
     // A model folder's layers (model.layered): caches per (layer run, mixer) beside the paged pool, and scratch.
     struct LayeredState {
-        Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding; a norm's rows, or the stream's in bf16; (stream ; embedding)
+        Buffer x0, xn_f, xn_b, cat_f, cat_b;      // the embedding (and behind it, for averages over them, every run's result); a norm's rows, or the stream's in bf16; (stream ; embedding)
         Buffer proj, q_f, q_b, attn_f, attn_b;    // a mixer's projections; finished q; what the output projection reads
         Buffer moe_x, moe_xb, ids, weights, src, place, tiles, n_tiles, hid_f, hid_b, rows, sh_f, sh_b, shared;
         Buffer ff_f, ff_b, branch;                // a dense layer's hidden rows; the outputs of mixers side by side, or of a sublayer with a norm behind it
         Buffer lat_f, lat_b, uq, part_f, part_b, mid_f, mid_b;  // latent attention: the query row, W_uq's product, its unrotated parts, the sums of c
-        Buffer side, side_f, side_b, row_weight, decays;  // a side input's rows before and behind its gate; experts' sorted scores; fixed decays
+        Buffer side, side_f, side_b, row_weight, per_head;  // a side input's rows before and behind its gate; experts' sorted scores; fixed decays and slopes
+        Buffer v_first;                           // the values other layers mix in
         Buffer conv, conv_b, steps, y, mix_f, mix_b, low, decay;  // a recurrence's inputs and outputs
         Buffer rings, states, caches, recurrent_dev;      // caches, recurrent_dev: MixerCache, RecurrentCache on the device
         std::vector<Buffer> rope;                 // per distinct rotation: [position][dims / 2] (cos, sin), fp32
@@ -262,6 +263,7 @@ class Engine {
         std::vector<RecurrentCache> recurrent;
         uint32_t max_heads = 0;                   // of a recurrence
         const float* in_f = nullptr;              // what the sublayer being queued reads, in fp32 (in bf16: xn_b)
+        float* result = nullptr;                  // where the stream goes on from the sublayer being queued
     };
     static constexpr uint32_t EXPERT_TILE_MIN = 16;  // rows of an expert per tile, at least
     static constexpr uint32_t SHIFT_TILE_MIN = 16;   // tokens of a mix per tile, at least
@@ -275,13 +277,13 @@ class Engine {
     void encode_attention(StepSet& st, const Plan& p, const Attention& a, const MixerCache& mc, const float* cur, float* alone, bool capture);
     void encode_recurrence(StepSet& st, const Plan& p, ScanArgs& a, GatedNormArgs& g);
     void encode_state_space(StepSet& st, const Plan& p, const StateSpace& x, const MixerCache& mc, const float* cur, float* alone);
-    void encode_latent(StepSet& st, const Plan& p, const LatentAttention& a, const MixerCache& mc, float* alone, bool capture);
+    void encode_latent(StepSet& st, const Plan& p, const LatentAttention& a, const MixerCache& mc, const float* cur, float* alone, bool capture);
     void encode_linear(StepSet& st, const Plan& p, const LinearAttention& x, const MixerCache& mc, float* alone);
     void encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const MixerCache& mc, const float* cur, float* alone);
     void encode_forward_layered(uint32_t set, const Plan& p, const std::function<void(const LayerCapture&)>* capture = nullptr);
     // Y = epilogue(W x) in the engine's precision: xf in an fp32 engine, else xb through the GEMM, the streamed matmul or,
     // for sizes neither takes, the CUDA cores.
-    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr, uint32_t act_rows = 0, const SideTable* side = nullptr);
+    void project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base = nullptr, uint32_t act_rows = 0, const SideTable* side = nullptr, float limit = 0.0f);
     std::unique_ptr<LimiteState> lim;
     LimiteKv limite_kv(const LimiteLayer& x) const;
     void encode_forward_limite(uint32_t set, const Plan& p);
@@ -326,12 +328,12 @@ class Engine {
   private:
     KvArgs kv_args() const;
     void matmul(const Matrix& w, uint32_t n, const float* x, float* y, uint32_t epi, const float* base, float* inv_out, uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr,
-                const uint16_t* xb = nullptr, uint16_t* yb = nullptr, float scale = 1.0f, float ra = 1.0f, float rb = 1.0f, const SideTable* side = nullptr);
+                const uint16_t* xb = nullptr, uint16_t* yb = nullptr, float scale = 1.0f, float ra = 1.0f, float rb = 1.0f, const SideTable* side = nullptr, float limit = 0.0f);
     bool stream_fits(const Matrix& w, uint32_t n = 1) const;
     // The tensor-core GEMM: xb is x in bf16, inv the rows' 1/rms (normed epilogues), yb an optional bf16 copy of y.
     void matmul_gemm(const Matrix& w, uint32_t n, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, const float* inv,
                      uint32_t vocab_real = 0, const QkvEpilogue* q = nullptr, float* ssq_out = nullptr, const float* ssq_in = nullptr, float scale = 1.0f, float ra = 1.0f,
-                     float rb = 1.0f, const SideTable* side = nullptr);
+                     float rb = 1.0f, const SideTable* side = nullptr, float limit = 0.0f);
     bool use_gemm(const Matrix& w, uint32_t n) const;
     bool gemm_fits(const Matrix& w, uint32_t n) const;
     // A layer of n tokens runs on the tensor-core GEMM and its last projection leaves bf16(h) in h_b and h's sums of squares in ssq.

@@ -14,11 +14,12 @@ void Engine::init_layered() {
     const bool f32 = cfg.fp32;
     const size_t n = cfg.max_step_tokens, n16 = (n + 15) / 16 * 16, d = md.d;
     size_t proj = 0, q = 0, out = 0, pairs = 0, hid = 0, sff = 0, tiles = 0, top = 0, rows = 0, ff = 0, branch = 0, channels = 0, y = 0, inner = 0, heads = 0, low = 0;
-    size_t halves = 0, lat = 0, uq = 0, part = 0, mid = 0, side = 0, side_wide = 0, fixed = 0;
-    bool shift = false;
+    size_t halves = 0, lat = 0, uq = 0, part = 0, mid = 0, side = 0, side_wide = 0, v_first = 0;
+    bool shift = false, depth = false;
     for (const FolderLayer& l : m.layers) {
         if (l.mix.size() > 1) branch = 2 * d;
         else if (l.post_norm) branch = std::max(branch, d);
+        depth = depth || l.depth;
         side = std::max<size_t>(side, l.side.gate.m);
         side_wide = std::max<size_t>(side_wide, l.side.proj.k);
         for (const Mixer& x : l.mix) {
@@ -26,6 +27,7 @@ void Engine::init_layered() {
                 proj = std::max<size_t>(proj, x.attn.proj.m);
                 q = std::max<size_t>(q, x.attn.heads * x.attn.dim);
                 out = std::max<size_t>(out, x.attn.out_w());
+                if (x.attn.mix.share) v_first = std::max<size_t>(v_first, x.attn.v_w());
             } else if (x.kind == MixerKind::StateSpace) {
                 proj = std::max<size_t>(proj, x.ssm.in.m);
                 channels = std::max<size_t>(channels, x.ssm.channels());
@@ -47,7 +49,6 @@ void Engine::init_layered() {
                 halves = std::max<size_t>(halves, x.linear.proj.m);
                 y = std::max<size_t>(y, x.linear.out_w());
                 out = std::max<size_t>(out, x.linear.out_w());
-                fixed += x.linear.heads;
             } else {
                 shift = true;
                 proj = std::max<size_t>(proj, 4 * x.tmix.inner());
@@ -73,7 +74,8 @@ void Engine::init_layered() {
     auto f = [](Buffer& b, size_t floats) { b.alloc(floats * 4, false); };
     auto h = [&](Buffer& b, size_t halves) { if (!f32) b.alloc(halves * 2, false); };  // the 16-bit copies
     auto w = [&](Buffer& b, size_t floats) { if (f32) b.alloc(floats * 4, false); };   // their 32-bit counterparts
-    f(z.x0, n * d);
+    f(z.x0, (depth ? m.runs.size() + 1 : 1) * n * d);
+    f(z.v_first, n * v_first);
     if (shift) f(z.xn_f, n * d);  // (rows are mixed in 32-bit)
     else w(z.xn_f, n * d);
     h(z.xn_b, n16 * d);
@@ -147,11 +149,15 @@ void Engine::init_layered() {
     std::vector<bool> shared;  // per cache: its pages are another's, which are compacted and filled there
     while ((1u << page_shift) < md.page) page_shift++;
     const size_t es = f32 ? 4 : 2;
-    std::vector<float> decays;  // of the layers with fixed ones, one after the other
-    for (const FolderLayer& l : m.layers)
-        for (const Mixer& x : l.mix) decays.insert(decays.end(), x.linear.decay.begin(), x.linear.decay.end());
-    f(z.decays, std::max<size_t>(fixed, 1));
-    if (fixed) z.decays.write_vec(0, decays);
+    std::vector<float> per_head;  // the layers' fixed decays and slopes, one after the other
+    std::vector<size_t> from;     // where a layer's begin
+    for (const FolderLayer& l : m.layers) {
+        from.push_back(per_head.size());
+        for (const Mixer& x : l.mix)
+            for (const std::vector<float>* v : {&x.linear.decay, &x.attn.slopes}) per_head.insert(per_head.end(), v->begin(), v->end());
+    }
+    f(z.per_head, std::max<size_t>(per_head.size(), 1));
+    if (!per_head.empty()) z.per_head.write_vec(0, per_head);
     size_t ring = 0, state = 0;
     for (int pass = 0; pass < 2; pass++) {  // sizes, then addresses
         float *rings = z.rings.as<float>(), *states = z.states.as<float>();
@@ -170,8 +176,11 @@ void Engine::init_layered() {
         for (const LayerRun& r : m.runs) {
             z.first.push_back(i);
             last[r.layer] = i;
+            const float* mine = z.per_head.as<float>() + from[r.layer];
             for (const Mixer& x : m.layers[r.layer].mix) {
                 MixerCache c{};
+                c.per_head = mine;
+                mine += x.linear.decay.size() + x.attn.slopes.size();
                 shared.push_back(x.kind == MixerKind::Latent && x.latent.kv_from != LatentAttention::OWN);
                 if (x.kind == MixerKind::Attention) {
                     const Attention& a = x.attn;
@@ -195,12 +204,7 @@ void Engine::init_layered() {
                     rc.Np = recurrent_pitch(rc.N);
                     rc.P = lin ? x.linear.vdim : tm ? x.tmix.dim : x.ssm.vdim;
                     rc.channel_decay = tm;
-                    if (lin) {
-                        size_t before = 0;  // the decays of the layers in front
-                        for (uint32_t j = 0; j < r.layer; j++)
-                            for (const Mixer& y : m.layers[j].mix) before += y.linear.decay.size();
-                        rc.fixed = z.decays.as<float>() + before;
-                    }
+                    if (lin) rc.fixed = c.per_head;
                     const size_t kept = size_t(cfg.max_seqs) * VERIFY_T;
                     rc.state = take(size_t(cfg.max_seqs) * rc.heads * rc.P * rc.Np);
                     rc.keep_k = take(kept * (rc.heads / rc.per) * rc.N);
@@ -231,12 +235,12 @@ void Engine::init_layered() {
     z.recurrent_dev.write_vec(0, z.recurrent);
 }
 
-void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, uint32_t act_rows, const SideTable* side) {
+void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_t* xb, float* y, uint16_t* yb, uint32_t epi, const float* base, uint32_t act_rows, const SideTable* side, float limit) {
     const bool gemm = !cfg.fp32 && w.m % 128 == 0 && w.k % 64 == 0, stream_takes = !cfg.fp32 && stream_fits(w, n);
     if (gemm && (gemm_fits(w, n) || !stream_takes)) {  // (few rows that are too long for the streamed kernel's shared memory, too)
-        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr, act_rows, nullptr, nullptr, nullptr, 1.0f, 1.0f, 1.0f, side);
+        matmul_gemm(w, n, xb, y, yb, epi, base, nullptr, act_rows, nullptr, nullptr, nullptr, 1.0f, 1.0f, 1.0f, side, limit);
     } else if (stream_takes) {
-        matmul(w, n, nullptr, y, epi, base, nullptr, act_rows, nullptr, xb, yb, 1.0f, 1.0f, 1.0f, side);
+        matmul(w, n, nullptr, y, epi, base, nullptr, act_rows, nullptr, xb, yb, 1.0f, 1.0f, 1.0f, side, limit);
     } else {
         LinearArgs a{};
         a.W = reinterpret_cast<const uint16_t*>(w.w);
@@ -249,6 +253,8 @@ void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_
         a.k = w.k;
         a.epi = epi;
         a.act_rows = act_rows;
+        a.bias = w.bias;
+        a.limit = limit;
         launch_linear(a, !cfg.fp32, stream);
     }
 }
@@ -257,7 +263,7 @@ void Engine::project(const Matrix& w, uint32_t n, const float* xf, const uint16_
 void Engine::mixer_out(const Matrix& o, uint32_t n, const float* cur, float* alone) {
     LayeredState& z = *lay;
     const int sp = span_begin(G_MATMUL);
-    project(o, n, z.attn_f.as<float>(), z.attn_b.as<uint16_t>(), alone ? alone : s.h.as<float>(), nullptr, alone ? EPI_RAW : EPI_RESID, alone ? nullptr : cur);
+    project(o, n, z.attn_f.as<float>(), z.attn_b.as<uint16_t>(), alone ? alone : z.result, nullptr, alone ? EPI_RAW : EPI_RESID, alone ? nullptr : cur);
     span_end(sp);
 }
 
@@ -291,6 +297,9 @@ void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, co
     c.heads = a.heads;
     c.rot_dims = a.rot.dims;
     c.unit_qk = a.unit_qk;
+    c.unit_v = a.unit_v;
+    c.mix = a.mix;
+    c.v_first = z.v_first.as<float>();
     c.neighbours = a.rot.neighbours;
     c.q_norm = a.q_norm;
     c.k_norm = a.k_norm;
@@ -317,13 +326,15 @@ void Engine::encode_attention(StepSet& st, const Plan& p, const Attention& a, co
     at.heads = a.heads;
     at.chunk = a.chunk;
     at.window = a.window;
+    at.keep = a.keep;
     at.scale = a.scale;
     at.softcap = a.softcap;
+    at.slopes = a.slopes.empty() ? nullptr : mc.per_head;
     at.out = f32 || capture ? z.attn_f.as<float>() : nullptr;
     at.out_b = z.attn_b.as<uint16_t>();
     uint32_t most = p.max_keys;  // keys a row may see
     for (uint32_t bound : {a.chunk, a.window})
-        if (bound) most = std::min(most, bound);
+        if (bound) most = std::min(most, bound + a.keep);
     sp = span_begin(G_ATTN);
     if (fast_attn) launch_attn_chunked(at, n, p.chunked ? p.ctiles : 0, most, sm_count, tuning.attn_keys_per_cta, stream);
     else launch_attn_any(at, n, f32, stream);
@@ -466,10 +477,10 @@ void Engine::encode_time_mix(StepSet& st, const Plan& p, const TimeMix& x, const
 }
 
 // Latent attention: the per-head matrices on the queries' side and on the sums' side, so that all heads read the rows the cache holds.
-void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x, const MixerCache& mc, float* alone, bool capture) {
+void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x, const MixerCache& mc, const float* cur, float* alone, bool capture) {
     LayeredState& z = *lay;
     const uint32_t n = p.n;
-    const bool f32 = cfg.fp32;
+    const bool f32 = cfg.fp32, direct = x.q_rank == 0;  // direct: the queries are in the first projection
     float* proj = z.proj.as<float>();
     int sp = span_begin(G_MATMUL);
     project(x.in, n, z.in_f, z.xn_b.as<uint16_t>(), proj, nullptr, EPI_RAW);
@@ -486,22 +497,25 @@ void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x,
     r.q_f = f32 ? z.lat_f.as<float>() : nullptr;
     r.q_b = f32 ? nullptr : z.lat_b.as<uint16_t>();
     r.q_rank = x.q_rank;
+    r.key_at = x.first_w();
     r.kv_rank = x.kv_rank;
     r.rot_dim = x.rot_dim;
     r.own = x.kv_from == LatentAttention::OWN;
     r.neighbours = x.rot.neighbours;
     r.eps = model.md.eps;
-    sp = span_begin(G_SMALL);
-    launch_latent_rows(r, n, f32, stream);
-    span_end(sp);
-    sp = span_begin(G_MATMUL);
-    project(x.uq, n, z.lat_f.as<float>(), z.lat_b.as<uint16_t>(), z.uq.as<float>(), nullptr, EPI_RAW);
-    span_end(sp);
+    if (!direct) {
+        sp = span_begin(G_SMALL);
+        launch_latent_rows(r, n, f32, stream);
+        span_end(sp);
+        sp = span_begin(G_MATMUL);
+        project(x.uq, n, z.lat_f.as<float>(), z.lat_b.as<uint16_t>(), z.uq.as<float>(), nullptr, EPI_RAW);
+        span_end(sp);
+    }
     const bool fast_attn = !f32 && !tuning.plain_attention && latent_attn_fits(x.kv_rank, x.rot_dim, model.md.page);
     const bool fast_q = !f32 && grouped_fits(x.kv_rank, x.dim), fast_v = !f32 && grouped_fits(x.vdim, x.kv_rank);
     LatentQueryArgs q{};
-    q.u = z.uq.as<float>();
-    q.ldu = x.uq.m;
+    q.u = direct ? proj : z.uq.as<float>();
+    q.ldu = direct ? x.in.m : x.uq.m;
     q.rope = r.rope;
     q.meta = r.meta;
     q.part_f = f32 ? z.part_f.as<float>() : nullptr;
@@ -523,7 +537,8 @@ void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x,
     q.neighbours = x.rot.neighbours;
     q.factor = fast_attn ? x.scale * LOG2E : 1.0f;
     sp = span_begin(G_SMALL);
-    launch_latent_query(q, stream);
+    if (direct) launch_latent_split(r, q, f32, stream);
+    else launch_latent_query(q, stream);
     span_end(sp);
     LinearArgs l{};  // W_uk^T on a head's query: in front of the rotated part
     l.W = reinterpret_cast<const uint16_t*>(x.uk_t.w);
@@ -552,11 +567,14 @@ void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x,
     at.vis = st.in<uint32_t>(st.o_vis);
     at.kv = mc.kv;
     at.heads = x.heads;
+    at.window = x.window;
+    at.sink = x.sink;
     at.scale = x.scale;
     at.out = f32 ? z.mid_f.as<float>() : nullptr;
     at.out_b = f32 ? nullptr : z.mid_b.as<uint16_t>();
     sp = span_begin(G_ATTN);
-    if (fast_attn) launch_attn_latent(at, n, p.chunked ? p.ctiles : 0, p.max_keys, sm_count, tuning.attn_keys_per_cta, s.err_flag.as<uint32_t>(), stream);
+    const uint32_t most = x.window ? std::min(p.max_keys, x.window) : p.max_keys;  // keys a row may see
+    if (fast_attn) launch_attn_latent(at, n, p.chunked ? p.ctiles : 0, most, sm_count, tuning.attn_keys_per_cta, s.err_flag.as<uint32_t>(), stream);
     else launch_attn_any(at, n, f32, stream);
     span_end(sp);
     l.W = reinterpret_cast<const uint16_t*>(x.uv.w);  // W_uv on a head's sum of c, and the gate
@@ -566,13 +584,14 @@ void Engine::encode_latent(StepSet& st, const Plan& p, const LatentAttention& x,
     l.m = x.vdim;
     l.k = x.kv_rank;
     l.ldy = x.vdim;
-    l.gate = proj + x.q_rank + x.kv_w();
+    l.gate = proj + x.first_w() + x.kv_w();
     l.ldg = x.in.m;
+    l.gate_w = x.gate_by_head ? 1 : x.vdim;
     sp = span_begin(G_MATMUL);
     if (fast_v) launch_grouped(l, x.heads, q.tile, s.err_flag.as<uint32_t>(), stream);
     else launch_linear(l, !f32, stream);
     span_end(sp);
-    mixer_out(x.o, n, nullptr, alone);
+    mixer_out(x.o, n, cur, alone);
 }
 
 void Engine::encode_linear(StepSet& st, const Plan& p, const LinearAttention& x, const MixerCache& mc, float* alone) {
@@ -658,6 +677,7 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
     const uint32_t n = p.n, d = md.d;
     float* h = s.h.as<float>();
     const float* cur = z.x0.as<float>();  // the stream; h from the first layer on
+    const size_t apart = size_t(cfg.max_step_tokens) * d;  // from one of the results an average takes to the next
     bool normed = false;  // the layer before has left norm1's rows
     auto host = [&](const float* dev, size_t count) {
         std::vector<float> v(count);
@@ -687,6 +707,7 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
         std::vector<float> resid_in, sdpa;
         uint32_t attn_width = 0;
         z.in_f = l.post_norm ? cur : z.xn_f.as<float>();
+        z.result = l.depth ? z.x0.as<float>() + (ri + 1) * apart : h;
         if (!normed && !l.post_norm) {
             na.in = cur;
             na.add = m.runs[ri].add_embed ? z.x0.as<float>() : nullptr;
@@ -708,7 +729,7 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
             case MixerKind::Attention: encode_attention(st, p, x.attn, mc, cur, alone, capture != nullptr); break;
             case MixerKind::StateSpace: encode_state_space(st, p, x.ssm, mc, cur, alone); break;
             case MixerKind::TimeMix: encode_time_mix(st, p, x.tmix, mc, cur, alone); break;
-            case MixerKind::Latent: encode_latent(st, p, x.latent, mc, alone, capture != nullptr); break;
+            case MixerKind::Latent: encode_latent(st, p, x.latent, mc, cur, alone, capture != nullptr); break;
             case MixerKind::Linear: encode_linear(st, p, x.linear, mc, alone); break;
             }
             if (capture && (x.kind == MixerKind::Attention || x.kind == MixerKind::Latent)) {
@@ -735,6 +756,7 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
             span_end(sp);
         }
         if (l.post_norm) add_norm(cur, l.norm1, n);
+        float* res = z.result;
         cur = h;
         normed = false;
         if (l.post_norm) z.in_f = h;
@@ -743,21 +765,40 @@ void Engine::encode_forward_layered(uint32_t set, const Plan& p, const std::func
             encode_experts(l, n, next_norm ? m.layers[m.runs[ri + 1].layer].norm1 : RowNorm{});
             normed = next_norm;
         } else if (l.mlp == MlpKind::Dense) {
-            if (!several && !l.post_norm) {
-                na.in = h;
+            if (!several && !l.post_norm && !l.parallel) {
+                na.in = res;
                 na.norm = l.norm2;
                 sp = span_begin(G_SMALL);
                 launch_norm_rows(na, stream);
                 span_end(sp);
             }
             sp = span_begin(G_MATMUL);
-            project(l.dense.up, n, z.in_f, z.xn_b.as<uint16_t>(), f32 ? z.ff_f.as<float>() : nullptr, z.ff_b.as<uint16_t>(), l.dense.hidden == Hidden::SiluGlu ? EPI_GLU : EPI_RELU2);
-            project(l.dense.down, n, z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), l.post_norm ? z.branch.as<float>() : h, nullptr, l.post_norm ? EPI_RAW : EPI_RESID,
-                    l.post_norm ? nullptr : h);
+            project(l.dense.up, n, z.in_f, z.xn_b.as<uint16_t>(), f32 ? z.ff_f.as<float>() : nullptr, z.ff_b.as<uint16_t>(),
+                    l.dense.hidden == Hidden::SiluGlu ? EPI_GLU : l.dense.hidden == Hidden::ClampedGlu ? EPI_GLU_CLAMP : EPI_RELU2, nullptr, 0, nullptr, l.dense.limit);
+            project(l.dense.down, n, z.ff_f.as<float>(), z.ff_b.as<uint16_t>(), l.post_norm ? z.branch.as<float>() : res, nullptr, l.post_norm ? EPI_RAW : EPI_RESID,
+                    l.post_norm ? nullptr : res);
             span_end(sp);
             if (l.post_norm) add_norm(h, l.norm2, n);
         }
         if (l.side.dim) encode_side(st, l.side, n);
+        if (l.depth) {
+            DepthArgs a{};
+            a.x = z.x0.as<float>();
+            a.stride = apart;
+            a.share = l.depth;
+            a.count = ri + 2;
+            a.out = h;
+            normed = ri + 1 < m.runs.size();
+            if (normed) a.norm = m.layers[m.runs[ri + 1].layer].norm1;
+            a.next = f32 ? na.out_f32 : nullptr;
+            a.next_b = f32 ? nullptr : na.out_bf16;
+            a.n = n;
+            a.d = d;
+            a.eps = md.eps;
+            sp = span_begin(G_SMALL);
+            launch_depth_average(a, stream);
+            span_end(sp);
+        }
         if (capture) {
             const std::vector<float> resid_out = host(h, size_t(n) * d);
             LayerCapture lc{ri, n, resid_in.data(), nullptr, nullptr, attn_width ? sdpa.data() : nullptr, nullptr, nullptr, nullptr};

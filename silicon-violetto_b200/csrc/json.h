@@ -40,6 +40,10 @@ struct Json {
         if (!(v >= 0 && v <= 4294967295.0) || v != std::floor(v)) throw Error("config: `" + what + "` is not a size");
         return uint32_t(v);
     }
+    bool flag(const std::string& what) const {  // (absent or null: no)
+        if (kind != Kind::Bool && kind != Kind::Null) throw Error("config: `" + what + "` is neither true nor false");
+        return kind == Kind::Bool && b;
+    }
     const std::string& text(const std::string& what) const {
         if (kind != Kind::String) throw Error("config: `" + what + "` is not a string");
         return str;

@@ -1,6 +1,7 @@
 // Attention over paged keys on the tensor cores, chunked, windowed or over everything before, for head sizes that are instantiated
 // below (other sizes and fp32 caches: k_mixer.cu's scalar kernel). What a row walks begins wherever its chunk or window does, in
-// the middle of a page or not, and is bounded by it.
+// the middle of a page or not, and is bounded by it; in front of a window come the tiles of the first positions, if some are kept.
+// Scores may be capped, and lowered by a head's slope times the distance.
 //
 //   chunk_decode_kernel   a row (token) and up to 8 query heads of one kv head per block: the keys are the MMAs' M side, the
 //                         heads its columns; four warps take tiles of 16 keys in turn, each with its own ring of asynchronous
@@ -39,8 +40,13 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
     const uint32_t G = a.heads / a.kv.n_kv, h0 = kvh * G + blockIdx.y / a.kv.n_kv * 8, cols = min(8u, kvh * G + G - h0);
     const View v = view_of(a, t);
     const float cap = a.softcap * LOG2E, cap_inv = 2.0f / a.softcap;
-    // Tiles of 16 positions from the one `lo` lies in up to the last key seen (pages hold whole tiles): an even share.
-    const uint32_t tile0 = v.lo / TILE, tiles = (v.first + 32 - __clz(v.mask) + TILE - 1) / TILE - tile0, share = (tiles + gridDim.z - 1) / gridDim.z;
+    float slope[2] = {0.0f, 0.0f};
+    if (a.slopes)
+#pragma unroll
+        for (uint32_t e = 0; e < 2; e++) slope[e] = a.slopes[h0 + min(2 * tq + e, cols - 1)] * LOG2E;
+    // Tiles of 16 positions up to the last key seen (pages hold whole tiles): an even share.
+    const Tiles<TILE> walk(v.lo, v.keep);
+    const uint32_t tiles = walk.count(v.first + 32 - __clz(v.mask)), share = (tiles + gridDim.z - 1) / gridDim.z;
     const uint32_t begin = min(sp * share, tiles), n = min(share, tiles - begin), my = warp < n ? (n - warp + WARPS - 1) / WARPS : 0;
 
     uint32_t q[KS][2];
@@ -61,7 +67,7 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
     const uint16_t* V = static_cast<const uint16_t*>(a.kv.v);
     const uint32_t wbuf = smem_u32(smem) + warp * STAGES * (KB + VB);
     auto issue = [&](uint32_t i) {  // this warp's tile i: 16 neighbouring rows of K and of V
-        const uint32_t key0 = (tile0 + begin + warp + i * WARPS) * TILE;
+        const uint32_t key0 = walk.at(begin + warp + i * WARPS) * TILE;
         const size_t r0 = ((size_t(pages[key0 >> PAGE_SHIFT]) * a.kv.n_kv + kvh) << PAGE_SHIFT) + (key0 & (PAGE - 1));
         const uint32_t dst = wbuf + (i % STAGES) * (KB + VB);
 #pragma unroll
@@ -87,7 +93,7 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
     for (uint32_t i = 0; i < my; i++) {
         cp_async_wait<STAGES - 1>();
         __syncwarp();
-        const uint32_t kbase = wbuf + (i % STAGES) * (KB + VB), vbase = kbase + KB, key0 = (tile0 + begin + warp + i * WARPS) * TILE;
+        const uint32_t kbase = wbuf + (i % STAGES) * (KB + VB), vbase = kbase + KB, key0 = walk.at(begin + warp + i * WARPS) * TILE;
         float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};  // [0, 1] key g, columns 2 tq, 2 tq + 1; [2, 3] key g + 8
 #pragma unroll
         for (uint32_t ks = 0; ks < KS; ks++) {
@@ -98,6 +104,16 @@ __global__ void __launch_bounds__(WARPS * 32, 3) chunk_decode_kernel(const Chunk
         if (a.softcap > 0) {
 #pragma unroll
             for (int e = 0; e < 4; e++) s[e] = capped(s[e], cap, cap_inv);
+        }
+        if (a.slopes) {
+            const bool tree = key0 + TILE > v.first;
+#pragma unroll
+            for (uint32_t r = 0; r < 2; r++) {
+                const uint32_t key = key0 + g + 8 * r;
+                const float back = tree && sees(v, key) ? distance(a, v, key) : float(int(v.pos) - int(key));
+#pragma unroll
+                for (uint32_t e = 0; e < 2; e++) s[2 * r + e] = fmaf(-slope[e], back, s[2 * r + e]);
+            }
         }
         if (key0 < v.lo || key0 + TILE > v.first) {
             if (!sees(v, key0 + g)) s[0] = s[1] = -INFINITY;
@@ -270,7 +286,9 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
     }
     if (lane == 0 && grp == 0) { lows[warp] = low; ends[warp] = end; }
     __syncthreads();
-    const uint32_t b0 = min(min(lows[0], lows[1]), min(lows[2], lows[3])) / CK + grp, b1 = (max(max(ends[0], ends[1]), max(ends[2], ends[3])) + CK - 1) / CK;
+    const Tiles<CK> walk(min(min(lows[0], lows[1]), min(lows[2], lows[3])), a.keep);
+    const uint32_t b0 = grp, b1 = walk.count(max(max(ends[0], ends[1]), max(ends[2], ends[3])));
+    const float slope = a.slopes ? a.slopes[h] * LOG2E : 0.0f;
 
     const uint32_t* pages = a.kv.page_table + size_t(v[0].slot) * a.kv.max_pages;
     const uint16_t* K = static_cast<const uint16_t*>(a.kv.k);
@@ -278,7 +296,7 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
     const uint32_t ring = smem_u32(smem) + grp * ST * (KB + VB);
     auto group_sync = [&] { asm volatile("bar.sync %0, %1;" ::"r"(1 + grp), "n"(WARPS * 32) : "memory"); };
     auto issue = [&](uint32_t b) {  // a page of keys
-        const size_t r0 = (size_t(pages[b]) * a.kv.n_kv + kvh) << PAGE_SHIFT;
+        const size_t r0 = (size_t(pages[walk.at(b)]) * a.kv.n_kv + kvh) << PAGE_SHIFT;
         const uint32_t dst = ring + (b - b0) / GROUPS % ST * (KB + VB);
 #pragma unroll
         for (uint32_t c = tid; c < CK * KC; c += WARPS * 32) {
@@ -316,8 +334,8 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
     for (uint32_t b = b0; b < b1; b += GROUPS) {
         cp_async_wait<ST - 1>();
         group_sync();  // everybody's copies of the page are in
-        const uint32_t kbase = ring + (b - b0) / GROUPS % ST * (KB + VB), vbase = kbase + KB, key0 = b * CK;
-        if (key0 < ends[warp] && key0 + CK > lows[warp]) {  // (a warp whose rows see nothing of the page skips the arithmetic, not the barriers)
+        const uint32_t kbase = ring + (b - b0) / GROUPS % ST * (KB + VB), vbase = kbase + KB, key0 = walk.at(b) * CK;
+        if (key0 < ends[warp] && (key0 + CK > lows[warp] || key0 < a.keep)) {  // (a warp whose rows see nothing of the page skips the arithmetic, not the barriers)
             float s[8][4];
 #pragma unroll
             for (uint32_t j = 0; j < 8; j++) {
@@ -336,6 +354,18 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
                 for (uint32_t j = 0; j < 8; j++)
 #pragma unroll
                     for (int e = 0; e < 4; e++) s[j][e] = capped(s[j][e], cap, cap_inv);
+            }
+            if (a.slopes) {
+                const bool tree = key0 + CK > first_min;
+#pragma unroll
+                for (uint32_t j = 0; j < 8; j++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const View& w = v[e >> 1];
+                        const uint32_t key = key0 + 8 * j + 2 * tq + (e & 1);
+                        const float back = tree && key >= w.first && live[e >> 1] && sees(w, key) ? distance(a, w, key) : float(int(w.pos) - int(key));
+                        s[j][e] = fmaf(-slope, back, s[j][e]);
+                    }
             }
             if (key0 < lo_max || key0 + CK > first_min || !live[0] || !live[1]) {
 #pragma unroll
@@ -476,6 +506,7 @@ bool chunk_attn_fits(uint32_t dk, uint32_t dv, uint32_t page) { return (dk == 64
 // n_ctiles: tiles of at most 64 rows, if the step holds a run longer than a verified one (then every row goes by tile);
 // max_keys: the most keys a row may see; keys_per_block overrides the split.
 void launch_attn_chunked(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s) {
+    if (a.sink) throw Error("internal: attention over chunks has no sinks");
     // A row's keys over at most 8 blocks, or 16 where 8 leave most SMs idle: the count that makes waves of blocks (three an SM) times a block's keys, plus a
     // fixed part of about 128 keys' worth, least.
     const uint32_t units = std::max(n * a.kv.n_kv * ((a.heads / a.kv.n_kv + 7) / 8), 1u), slots = 3 * sm_count;

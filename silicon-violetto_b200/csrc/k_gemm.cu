@@ -301,8 +301,9 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
     // shared memory.
     auto emit = [&](uint32_t r, bool valid, uint32_t t0, float scale, auto& v) {  // v: 16 or 8 consecutive tokens of row r
         constexpr uint32_t NTOK = sizeof(v) / sizeof(float);
-        constexpr bool PAIRS = EPI == EPI_SWIGLU || EPI == EPI_GLU;  // (rows 2 i and 2 i + 1 make one output)
+        constexpr bool PAIRS = epi_pairs(EPI);
         const uint32_t row = row0 + r;
+        const float bias = !INT8 && m.bias ? bf16_to_f32(__ldg(m.bias + row)) : 0.0f;
         if constexpr (EPI == EPI_QKV) {
             // The row is feature `row` of the qkv projection: dim d of a q, k or v head (whole heads per 64 rows, so
             // a warp's 32 rows are of one kind). RoPE pairs are neighbouring rows, i.e. neighbouring lanes.
@@ -348,8 +349,10 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
         }
 #pragma unroll
         for (uint32_t j = 0; j < NTOK; j++) {
-            const float x = v[j] * scale;
-            if (PAIRS) {
+            const float x = INT8 ? v[j] * scale : v[j] + bias;
+            if (EPI == EPI_GLU_CLAMP) {
+                y[j] = clamped_glu(x, __shfl_xor_sync(0xffffffffu, x, 1), m.limit);
+            } else if (PAIRS) {
                 const float other = __shfl_xor_sync(0xffffffffu, x, 1);
                 const float gt = EPI == EPI_GLU ? x : x * inv[j], up = EPI == EPI_GLU ? other : other * inv[j];
                 y[j] = gt * __fdividef(1.0f, 1.0f + __expf(-gt)) * up;
@@ -543,6 +546,7 @@ static GemmEntry gemm_entry(bool int8, uint32_t epi, bool paired = false) {
     case EPI_RELU2: return int8 ? gemm::gemm_kernel<true, EPI_RELU2> : gemm::gemm_kernel<false, EPI_RELU2>;
     case EPI_SILU: return gemm::gemm_kernel<false, EPI_SILU>;  // (bf16 weights only)
     case EPI_GLU: return gemm::gemm_kernel<false, EPI_GLU>;
+    case EPI_GLU_CLAMP: return gemm::gemm_kernel<false, EPI_GLU_CLAMP>;
     case EPI_SIDE: return gemm::gemm_kernel<false, EPI_SIDE>;
     default: return int8 ? gemm::gemm_kernel<true, EPI_RAW> : gemm::gemm_kernel<false, EPI_RAW>;
     }
@@ -552,7 +556,7 @@ bool gemm_supported(const MatArgs& a) {
     const bool grouped = a.int8 && a.group < a.k;  // scale groups: powers of two from 8
     return a.n >= 1 && a.n <= 256 && a.m % gemm::BM == 0 && a.k % gemm::BK == 0 && (!grouped || (a.group >= 8 && !(a.group & (a.group - 1)))) && a.Xb != nullptr &&
            (a.epi == EPI_RESID || a.epi == EPI_RAW || a.epi == EPI_HEAD_CAP || a.epi == EPI_RELU2 ||
-            (!a.int8 && (a.epi == EPI_SILU || a.epi == EPI_GLU || a.epi == EPI_SIDE)) || a.inv_in != nullptr || a.ssq_in != nullptr);
+            (!a.int8 && (a.epi == EPI_SILU || a.epi == EPI_GLU || a.epi == EPI_GLU_CLAMP || a.epi == EPI_SIDE)) || a.inv_in != nullptr || a.ssq_in != nullptr);
 }
 
 void launch_gemm(const MatArgs& a, uint32_t sm_count, uint32_t* err_flag, cudaStream_t s, bool allow_paired) {

@@ -150,7 +150,7 @@ __global__ void __launch_bounds__(THREADS, 2) grouped_kernel(const __grid_consta
                 float acc[16];
                 float gate[16];
                 if (EPI == EPI_RAW && a.l.by_head && a.l.gate) {  // (their loads go out together)
-                    const float* from = a.l.gate + size_t(p0 + c0 - group * a.l.by_head) * a.l.ldg + size_t(group) * a.l.m + row;
+                    const float* from = a.l.gate + size_t(p0 + c0 - group * a.l.by_head) * a.l.ldg + (a.l.gate_w == 1 ? group : size_t(group) * a.l.m + row);
 #pragma unroll
                     for (uint32_t j = 0; j < 16; j++) gate[j] = c0 + j < count ? from[size_t(j) * a.l.ldg] : 0.0f;
                 }
@@ -199,7 +199,7 @@ void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint3
     static thread_local std::map<std::tuple<const void*, uint32_t, uint32_t, uint32_t>, grouped::Map> maps;
     static PerDevice configured;
     if (!a.max_tiles) return;
-    if (!grouped_fits(a.m, a.k) || tile < 16 || tile > 128 || tile % 16 || (a.epi != EPI_RAW && a.epi != EPI_RELU2 && a.epi != EPI_GLU_CLAMP) || (a.row_scale && a.epi != EPI_GLU_CLAMP)) throw Error("internal: a grouped GEMM of an unsupported shape");
+    if (!grouped_fits(a.m, a.k) || tile < 16 || tile > 128 || tile % 16 || (a.epi != EPI_RAW && a.epi != EPI_RELU2 && a.epi != EPI_GLU_CLAMP) || (a.row_scale && a.epi != EPI_GLU_CLAMP) || a.bias) throw Error("internal: a grouped GEMM of an unsupported shape");
     auto key = std::make_tuple(static_cast<const void*>(a.W), a.m, a.k, n_groups);
     auto it = maps.find(key);
     if (it == maps.end()) {

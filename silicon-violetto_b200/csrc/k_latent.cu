@@ -11,15 +11,11 @@ namespace latent {
 __device__ __forceinline__ void store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store(uint16_t* p, float v) { *p = f32_to_bf16(v); }
 
-// grid (tokens, 1 or 2): the query row; (c ; r) if it is this layer's own. T: the cache's element.
+// Token t's query row, or its (c ; r). T: the cache's element.
 template <typename T>
-__global__ void __launch_bounds__(256) rows_kernel(const LatentRowsArgs a) {
-    pdl_start();
-    __shared__ float red[32];
-    const uint32_t t = blockIdx.x, tid = threadIdx.x;
-    const bool key = blockIdx.y == 1;
-    const uint32_t width = key ? a.kv_rank : a.q_rank;
-    const float* u = a.u + size_t(t) * a.ldu + (key ? a.q_rank : 0);
+__device__ __forceinline__ void normed_row(const LatentRowsArgs& a, uint32_t t, bool key, float* red) {
+    const uint32_t tid = threadIdx.x, width = key ? a.kv_rank : a.q_rank;
+    const float* u = a.u + size_t(t) * a.ldu + (key ? a.key_at : 0);
     const RowNorm& norm = key ? a.kv_norm : a.q_norm;
     float ss = 0.0f;
     for (uint32_t i = tid; i < width; i += 256) ss += u[i] * u[i];
@@ -39,11 +35,10 @@ __global__ void __launch_bounds__(256) rows_kernel(const LatentRowsArgs a) {
     for (uint32_t i = tid; i < a.rot_dim; i += 256) store(dst + width + i, rotated(u + width, i, a.rot_dim, a.neighbours, cs));
 }
 
-// grid (tokens, spans of 1024 entries of a row).
-__global__ void __launch_bounds__(256) query_kernel(const LatentQueryArgs a) {
-    pdl_start();
-    const uint32_t t = blockIdx.x, tid = threadIdx.x, head_w = a.dim + a.rot_dim, all = a.heads * head_w;
-    if (t == 0 && blockIdx.y == 0) {
+// Token t's queries, a span of 1024 of their entries.
+__device__ __forceinline__ void query_span(const LatentQueryArgs& a, uint32_t t, uint32_t span) {
+    const uint32_t tid = threadIdx.x, head_w = a.dim + a.rot_dim, all = a.heads * head_w;
+    if (t == 0 && span == 0) {
         const uint32_t per = (a.n + a.tile - 1) / a.tile;
         for (uint32_t i = tid; i < a.heads * per; i += 256) {
             const uint32_t h = i / per, p = i % per * a.tile;
@@ -55,8 +50,8 @@ __global__ void __launch_bounds__(256) query_kernel(const LatentQueryArgs a) {
     }
     const float* u = a.u + size_t(t) * a.ldu;
     const float2* cs = reinterpret_cast<const float2*>(a.rope) + size_t(a.meta[2 * t + 1]) * (a.rot_dim / 2);
-    const uint32_t end = min(all, (blockIdx.y + 1) * 1024);
-    for (uint32_t i = blockIdx.y * 1024 + tid; i < end; i += 256) {
+    const uint32_t end = min(all, (span + 1) * 1024);
+    for (uint32_t i = span * 1024 + tid; i < end; i += 256) {
         const uint32_t h = i / head_w, c = i % head_w;
         if (c < a.dim) {
             const size_t o = (size_t(t) * a.heads + h) * a.dim + c;
@@ -72,6 +67,29 @@ __global__ void __launch_bounds__(256) query_kernel(const LatentQueryArgs a) {
     }
 }
 
+// grid (tokens, 1 or 2): the query row; (c ; r) if it is this layer's own.
+template <typename T>
+__global__ void __launch_bounds__(256) rows_kernel(const LatentRowsArgs a) {
+    pdl_start();
+    __shared__ float red[32];
+    normed_row<T>(a, blockIdx.x, blockIdx.y == 1, red);
+}
+
+// grid (tokens, spans).
+__global__ void __launch_bounds__(256) query_kernel(const LatentQueryArgs a) {
+    pdl_start();
+    query_span(a, blockIdx.x, blockIdx.y);
+}
+
+// grid (tokens, 1 + spans).
+template <typename T>
+__global__ void __launch_bounds__(256) split_kernel(const LatentRowsArgs r, const LatentQueryArgs q) {
+    pdl_start();
+    __shared__ float red[32];
+    if (blockIdx.y == 0) normed_row<T>(r, blockIdx.x, true, red);
+    else query_span(q, blockIdx.x, blockIdx.y - 1);
+}
+
 }  // namespace latent
 
 void launch_latent_rows(const LatentRowsArgs& a, uint32_t n, bool fp32, cudaStream_t s) {
@@ -81,6 +99,11 @@ void launch_latent_rows(const LatentRowsArgs& a, uint32_t n, bool fp32, cudaStre
 }
 void launch_latent_query(const LatentQueryArgs& a, cudaStream_t s) {
     launch_pdl(latent::query_kernel, dim3(a.n, (a.heads * (a.dim + a.rot_dim) + 1023) / 1024), 256, 0, s, a);
+}
+void launch_latent_split(const LatentRowsArgs& r, const LatentQueryArgs& q, bool fp32, cudaStream_t s) {
+    const dim3 grid(q.n, 1 + (q.heads * (q.dim + q.rot_dim) + 1023) / 1024);
+    if (fp32) launch_pdl(latent::split_kernel<float>, grid, 256, 0, s, r, q);
+    else launch_pdl(latent::split_kernel<uint16_t>, grid, 256, 0, s, r, q);
 }
 
 }  // namespace vlt

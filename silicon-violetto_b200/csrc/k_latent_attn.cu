@@ -114,6 +114,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(misc + 8 * (2 * MAX_SLOTS + 2 * REST_SLOTS + 6));
     volatile uint32_t* abort_flag = tmem_slot + 1;
     volatile uint32_t* end_s = tmem_slot + 2;
+    volatile uint32_t* low_s = tmem_slot + 3;
     int* from = reinterpret_cast<int*>(misc + 512);  // a row's place among the queries and the outputs, -1: none
     float* corr_s = reinterpret_cast<float*>(from + ROWS);
     float2* ml_s = reinterpret_cast<float2*>(corr_s + ROWS);  // a row's maximum and the sum under it
@@ -142,7 +143,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     };
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const uint32_t* pages = a.kv.page_table + size_t(a.meta[2 * t0]) * a.kv.max_pages;
-    uint32_t begin = 0, n = 0, st = 0, ph = 1, rs = 0, rph = 1;
+    uint32_t begin = 0, n = 0, head = 0, skip = 0, st = 0, ph = 1, rs = 0, rph = 1;
     auto load = [&](uint32_t page) {  // a tile's boxes, into slots that are free; false: they did not become so
         const int row = int(page << PAGE_SHIFT);
         for (uint32_t m = 0; m < p.mtiles; m++) {
@@ -160,11 +161,15 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
         if (++rs == NR) { rs = 0; rph ^= 1; }
         return true;
     };
-    auto share_of = [&](uint32_t end) {
-        const uint32_t tiles = (end + KT - 1) / KT, share = (tiles + splits - 1) / splits;
+    auto share_of = [&](uint32_t low, uint32_t end) {  // this block's tiles: `n` from number `begin` on (see Tiles)
+        const Tiles<KT> walk(low, a.keep);
+        const uint32_t tiles = walk.count(end), share = (tiles + splits - 1) / splits;
         begin = min(sp * share, tiles);
         n = min(share, tiles - begin);
+        head = walk.head;
+        skip = walk.skip;
     };
+    auto tile_at = [&](uint32_t i) { return begin + i < head ? begin + i : begin + i + skip; };
     // Splits: what the cluster's blocks send of their sums arrives as [source][column of this block's span][row], (m, l) per (source, row)
     // behind it, in the room of Q and the rings; there, too, this block's own, to be copied from.
     constexpr uint32_t RP = ROWS + 4;     // a column's pitch
@@ -172,16 +177,19 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     const uint32_t span = p.mtiles * 128 / splits, stats = splits * span * RP * 4, own = stats + splits * ROWS * 8;
     bool ok = true;
     if (warp == 0) {  // how far the rows see, and the first two tiles on their way while the others fetch the queries
-        uint32_t end = 0;
+        uint32_t end = 0, low = 0xffffffffu;
         for (uint32_t i = lane; i < n_tok; i += 32) {
             const View v = view_of(a, t0 + i);
             end = max(end, v.first + 32 - __clz(v.mask));
+            low = min(low, v.lo);
         }
         end = __reduce_max_sync(0xffffffffu, end);
-        share_of(end);
+        low = __reduce_min_sync(0xffffffffu, low);
+        share_of(low, end);
         if (lane == 0) {
             *end_s = end;
-            for (uint32_t i = 0; i < min(n, 2u) && ok; i++) ok = load(pages[begin + i]);
+            *low_s = low;
+            for (uint32_t i = 0; i < min(n, 2u) && ok; i++) ok = load(pages[tile_at(i)]);
         }
     } else {
         if (tid - 32 < ROWS) {
@@ -218,15 +226,15 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = *tmem_slot, tmem_o = tmem + 2 * KT;
-    share_of(*end_s);
+    share_of(*low_s, *end_s);
     auto lo = [](uint32_t addr) { return (addr & 0x3FFFFu) >> 4; };  // (an address in a cluster has the block's rank above these bits)
     const uint64_t k_major = gemm::smem_desc(0);
     if (warp == 0) {
         if (lane == 0) {
-            uint32_t page = n > 2 ? pages[begin + 2] : 0;
+            uint32_t page = n > 2 ? pages[tile_at(2)] : 0;
             for (uint32_t i = 2; i < n && ok; i++) {
                 const uint32_t now = page;
-                if (i + 1 < n) page = pages[begin + i + 1];
+                if (i + 1 < n) page = pages[tile_at(i + 1)];
                 ok = load(now);
             }
         }
@@ -297,7 +305,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             live[r] = active && row_at(quarter * 16 + g + 8 * r, tok) >= 0;
             v[r] = view_of(a, live[r] ? tok : t0);
         }
-        const uint32_t first = min(v[0].first, v[1].first);
+        const uint32_t first = min(v[0].first, v[1].first), lo_max = max(v[0].lo, v[1].lo);
         for (uint32_t i = 0; i < n; i++) {
             float s[KT / 8][4], m_new[2] = {m_run[0], m_run[1]};
             bool need = false;
@@ -314,8 +322,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
 #pragma unroll
                         for (uint32_t e = 0; e < 4; e++) s[j][e] = capped(s[j][e], cap, cap_inv);
                 }
-                const uint32_t key0 = (begin + i) * KT;
-                if (key0 + KT > first || !live[0] || !live[1]) {
+                const uint32_t key0 = tile_at(i) * KT;
+                if (key0 < lo_max || key0 + KT > first || !live[0] || !live[1]) {
 #pragma unroll
                     for (uint32_t j = 0; j < KT / 8; j++)
 #pragma unroll
@@ -386,6 +394,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
             for (uint32_t r = 0; r < 2; r++) {
                 l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
                 l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+                if (splits == 1 && a.sink && live[r]) l_run[r] += fast_exp2(bf16_to_f32(a.sink[grp * ROWS + (quarter * 16 + g + 8 * r) % hpt]) * LOG2E - m_run[r]);
                 if (tq == 0) ml_s[quarter * 16 + g + 8 * r] = make_float2(m_run[r], l_run[r]);
             }
         }
@@ -473,6 +482,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_kernel(const __grid_constan
                 if (top != -INFINITY) l = l * fast_exp2(m - top) + ml.y * fast_exp2(ml.x - top);
                 m = top;
             }
+            if (a.sink && from[tid] >= 0) l += fast_exp2(bf16_to_f32(a.sink[from[tid] % a.heads]) * LOG2E - m);
 #pragma unroll 1
             for (uint32_t k = 0; k < splits; k++) {
                 float* w = stat + (k * ROWS + tid) * 2;
@@ -596,6 +606,7 @@ bool latent_attn_fits(uint32_t kv_rank, uint32_t rot_dim, uint32_t page) {
     return page == paged::PAGE && kv_rank <= 512 && kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank + rot_dim <= 576;
 }
 void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s) {
+    if (a.slopes) throw Error("internal: latent attention has no slopes");
     if (n_ctiles || a.heads > 32) latent::launch<64>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);
     else if (a.heads > 16) latent::launch<32>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);
     else latent::launch<16>(a, n, n_ctiles, max_keys, sm_count, keys_per_block, err_flag, s);

@@ -1,7 +1,7 @@
 // Linear layers on the CUDA cores, for what the tensor-core kernels do not take: activations in fp32 throughout (true fp32
 // products and sums: bf16 weights are exact in fp32), and matrices whose sizes fit neither the streamed kernel nor the GEMM.
-// Also the row passes around a projection: RMS norms in front of it or of what it leaves, two streams side by side, two mixers'
-// outputs onto the stream, and a side input's gate.
+// Also the row passes around a projection: norms in front of it or of what it leaves, two streams side by side, two mixers'
+// outputs onto the stream, the average over the layers' results, and a side input's gate.
 #include <algorithm>
 
 #include "kernels.h"
@@ -64,13 +64,14 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
         for (int i = 0; i < 4; i++) {
             const uint32_t r = r0 + tr + 16 * i;
             float y = acc[i][j] * scale;
-            const bool pairs = a.epi == EPI_GLU || a.epi == EPI_GLU_CLAMP;  // (a pair's rows are neighbouring lanes')
+            if (a.bias && r < a.m) y += bf16_to_f32(a.bias[r]);
+            const bool pairs = epi_pairs(a.epi);  // (a pair's rows are neighbouring lanes')
             const float u = pairs ? __shfl_xor_sync(0xffffffffu, y, 1) : 0.0f;
             if (p >= count || r >= a.m || (pairs && r % 2)) continue;
             size_t o = pairs ? size_t(p0 + p) * (a.m / 2) + r / 2 : size_t(p0 + p) * a.m + r;
             if (a.by_head) {
                 const size_t t = p0 + p - group * a.by_head;
-                if (a.gate) y *= sigmoid_of(a.gate[t * a.ldg + size_t(group) * a.m + r]);
+                if (a.gate) y *= sigmoid_of(a.gate[t * a.ldg + (a.gate_w == 1 ? group : size_t(group) * a.m + r)]);
                 o = (t * a.heads + group) * a.ldy + r;
             }
             if (a.epi == EPI_RESID) y += a.base[o];
@@ -84,12 +85,49 @@ __global__ void __launch_bounds__(256) linear_kernel(const LinearArgs a) {
     }
 }
 
-// See NormArgs. A block per row, which it keeps in shared memory.
+// What a norm makes of the row a block keeps in shared memory, each thread its own entries; ss: their squares' sum if it is not centered.
+template <uint32_t V>
+__device__ __forceinline__ void norm_row(float* row, uint32_t width, const RowNorm& norm, float ss, float eps, float scale, float* red, float* out, uint16_t* out_b) {
+    const uint32_t tid = threadIdx.x * V, step = blockDim.x * V;
+    float mean = 0.0f;
+    if (norm.centered) {  // (the squares in a pass of their own: of what is left of the row)
+        float sum = 0.0f;
+        for (uint32_t i = tid; i < width; i += step)
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) sum += row[i + j];
+        mean = block_sum(sum, red) / float(width);
+        red += 32;
+        ss = 0.0f;
+        for (uint32_t i = tid; i < width; i += step)
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) ss += (row[i + j] - mean) * (row[i + j] - mean);
+    }
+    const float inv = scale / sqrtf(block_sum(ss, red) / float(width) + eps);
+    for (uint32_t i = tid; i < width; i += step) {
+        float x[V], w[V];
+        load_f32<V>(x, row + i);
+        weights_of<V>(w, norm, i);
+        if (norm.centered)
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) x[j] -= mean;
+#pragma unroll
+        for (uint32_t j = 0; j < V; j++) x[j] *= inv * w[j];
+        if (norm.b) {
+            load_bf16<V>(w, norm.b + i);
+#pragma unroll
+            for (uint32_t j = 0; j < V; j++) x[j] += scale * w[j];
+        }
+        if (out) store_f32<V>(out + i, x);
+        if (out_b) store_bf16<V>(out_b + i, x);
+    }
+}
+
+// See NormArgs. A block per row.
 template <uint32_t V>
 __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormArgs a) {
     pdl_start();
     extern __shared__ __align__(16) float row[];
-    __shared__ float red[32];
+    __shared__ float red[64];
     const uint32_t r = blockIdx.x, tid = threadIdx.x * V, step = blockDim.x * V;
     const size_t from = size_t(a.rows ? a.rows[r] : r) * a.k;
     float ss = 0.0f;
@@ -107,16 +145,42 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(const NormArgs a) {
 #pragma unroll
         for (uint32_t j = 0; j < V; j++) ss += x[j] * x[j];
     }
-    const float inv = a.scale / sqrtf(block_sum(ss, red) / float(a.k) + a.eps);
-    for (uint32_t i = tid; i < a.k; i += step) {
-        float x[V], w[V];
-        load_f32<V>(x, row + i);
-        weights_of<V>(w, a.norm, i);
+    const size_t to = size_t(r) * a.k;
+    norm_row<V>(row, a.k, a.norm, ss, a.eps, a.scale, red, a.out_f32 ? a.out_f32 + to : nullptr, a.out_bf16 ? a.out_bf16 + to : nullptr);
+}
+
+// See DepthArgs. A block per row.
+template <uint32_t V>
+__global__ void __launch_bounds__(1024) depth_average_kernel(const DepthArgs a) {
+    pdl_start();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[64];
+    const uint32_t tid = threadIdx.x * V, step = blockDim.x * V;
+    const size_t from = size_t(blockIdx.x) * a.d;
+    constexpr uint32_t AT_ONCE = 4;  // results whose loads go out together
+    float ss = 0.0f;
+    for (uint32_t i = tid; i < a.d; i += step) {
+        float sum[V] = {};
+        for (uint32_t j0 = 0; j0 < a.count; j0 += AT_ONCE) {
+            float x[AT_ONCE][V], share[AT_ONCE];
 #pragma unroll
-        for (uint32_t j = 0; j < V; j++) x[j] *= inv * w[j];
-        if (a.out_f32) store_f32<V>(a.out_f32 + size_t(r) * a.k + i, x);
-        if (a.out_bf16) store_bf16<V>(a.out_bf16 + size_t(r) * a.k + i, x);
+            for (uint32_t k = 0; k < AT_ONCE; k++) {
+                const uint32_t j = min(j0 + k, a.count - 1);
+                share[k] = j0 + k < a.count ? bf16_to_f32(a.share[j]) : 0.0f;
+                load_f32<V>(x[k], a.x + j * a.stride + from + i);
+            }
+#pragma unroll
+            for (uint32_t k = 0; k < AT_ONCE; k++)
+                if (j0 + k < a.count)
+#pragma unroll
+                    for (uint32_t v = 0; v < V; v++) sum[v] = fmaf(share[k], x[k][v], sum[v]);
+        }
+        store_f32<V>(a.out + from + i, sum);
+        store_f32<V>(row + i, sum);
+#pragma unroll
+        for (uint32_t v = 0; v < V; v++) ss += sum[v] * sum[v];
     }
+    if (a.norm.w) norm_row<V>(row, a.d, a.norm, ss, a.eps, 1.0f, red, a.next ? a.next + from : nullptr, a.next_b ? a.next_b + from : nullptr);
 }
 
 // See MergeArgs. A block per row.
@@ -254,6 +318,15 @@ void launch_add_norm(const AddNormArgs& a, cudaStream_t s) {
     if (!a.n) return;
     if (a.d % 4 == 0) launch_pdl(linear::add_norm_kernel<4>, a.n, row_threads(a.d, 4), size_t(a.d) * 4, s, a);
     else launch_pdl(linear::add_norm_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 4, s, a);
+}
+void launch_depth_average(const DepthArgs& a, cudaStream_t s) {
+    static PerDevice configured;
+    configured.once([] {
+        for (auto f : {linear::depth_average_kernel<1>, linear::depth_average_kernel<4>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    });
+    if (!a.n) return;
+    if (a.d % 4 == 0) launch_pdl(linear::depth_average_kernel<4>, a.n, row_threads(a.d, 4), size_t(a.d) * 4, s, a);
+    else launch_pdl(linear::depth_average_kernel<1>, a.n, row_threads(a.d, 1), size_t(a.d) * 4, s, a);
 }
 void launch_side_gate(const SideGateArgs& a, cudaStream_t s) {
     if (a.n) launch_pdl(linear::side_gate_kernel, dim3(a.n, (a.side.wide + 255) / 256), 256, 0, s, a);

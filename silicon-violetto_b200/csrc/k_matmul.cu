@@ -35,10 +35,12 @@ __device__ __forceinline__ void store_out(const MatArgs& a, uint32_t t, uint32_t
     if (a.Y) a.Y[o] = y;
     if (a.Yb) a.Yb[o] = f32_to_bf16(y);
 }
-__device__ __forceinline__ void store_swiglu(const MatArgs& a, uint32_t t, uint32_t row, float g, float u, float inv) {
-    g *= inv;
-    u *= inv;
-    const float y = g * (1.0f / (1.0f + expf(-g))) * u;
+__device__ __forceinline__ void store_pair(const MatArgs& a, uint32_t t, uint32_t row, float g, float u, float inv) {
+    if (a.epi == EPI_SWIGLU) {
+        g *= inv;
+        u *= inv;
+    }
+    const float y = a.epi == EPI_GLU_CLAMP ? clamped_glu(g, u, a.limit) : g * (1.0f / (1.0f + expf(-g))) * u;
     const size_t o = size_t(t) * (a.m / 2) + row / 2;
     if (a.Y) a.Y[o] = y;
     if (a.Yb) a.Yb[o] = f32_to_bf16(y);
@@ -93,12 +95,17 @@ __global__ void __launch_bounds__(256) matmul_rows_kernel(MatArgs a) {
 #pragma unroll
         for (int b = 0; b < 8; b++) {
             if (t0 + b >= a.n) break;
-            const float s0 = warp_sum(acc[0][b]), s1 = warp_sum(acc[1][b]), sq = warp_sum(ss[b]);
+            float s0 = warp_sum(acc[0][b]), s1 = warp_sum(acc[1][b]);
+            const float sq = warp_sum(ss[b]);
             if (lane != 0) continue;
+            if (a.bias) {
+                s0 += bf16_to_f32(a.bias[row0]);
+                s1 += bf16_to_f32(a.bias[row0 + 1]);
+            }
             const uint32_t t = t0 + b;
             const float inv = a.inv_in ? a.inv_in[t] : rsqrtf(sq / float(a.k) + a.eps);
             if (a.inv_out && row0 == 0) a.inv_out[t] = inv;
-            if (a.epi == EPI_SWIGLU || a.epi == EPI_GLU) store_swiglu(a, t, row0, s0, s1, a.epi == EPI_GLU ? 1.0f : inv);
+            if (epi_pairs(a.epi)) store_pair(a, t, row0, s0, s1, inv);
             else { store_out(a, t, row0, s0, inv); store_out(a, t, row0 + 1, s1, inv); }
         }
     }
@@ -396,7 +403,8 @@ __global__ void __launch_bounds__(512, 2) matmul_stream_kernel(MatArgs a, uint32
             row_sh = bf16_to_f32(a.scales[row0 + g + 8]);
         }
         // The residual this thread will add to (warps 0..3, see below): asked for now, there when the sums are.
-        float resid = 0.0f;
+        float resid = 0.0f, bias = 0.0f;
+        if (!INT8 && a.bias && sl + 1 == slices && tid < 128) bias = bf16_to_f32(a.bias[row0 + tid % 16]);
         if (a.epi == EPI_RESID && sl + 1 == slices && tid < 128 && tid / 16 < a.n) resid = a.base[size_t(tid / 16) * a.m + row0 + tid % 16];
         if (!st_mbar_wait(st_smem_u32(&bars[st]), (item / n_stages) & 1) && lane == 0 && a.err_flag) atomicExch(a.err_flag, 2u);
         const uint8_t* sw = stages + size_t(st) * STREAM_STAGE;
@@ -469,11 +477,12 @@ __global__ void __launch_bounds__(512, 2) matmul_stream_kernel(MatArgs a, uint32
 #pragma unroll
                 for (int w = 0; w < NW; w++) sum += rp[w * 128];
                 if (INT8) sum *= x_up[b];  // exact: a power of two
+                else sum += bias;
                 const float partner = __shfl_down_sync(0xffffffffu, sum, 1);  // row r + 1 of the same token (r is even where it is used)
                 if (b < a.n) {
                     const float inv = inv_s[b];
-                    if (a.epi == EPI_SWIGLU || a.epi == EPI_GLU) {
-                        if (r % 2 == 0) store_swiglu(a, b, row0 + r, sum, partner, a.epi == EPI_GLU ? 1.0f : inv);
+                    if (epi_pairs(a.epi)) {
+                        if (r % 2 == 0) store_pair(a, b, row0 + r, sum, partner, inv);
                     } else if (a.epi == EPI_QKV) {
                         if (r % 2 == 0) {  // qkv_store_pair with the token's table entries from shared memory
                             const uint32_t hd = a.q.kv.hd, row = row0 + r, head = row / hd, pair = (row % hd) / 2;

@@ -1,11 +1,12 @@
 // The attention mixer's work between its projections and its attention, as parameterised kernels: a short causal
-// convolution over time on q, k and v, rotation of pairs, q and k heads of unit length, queries that grow with
-// their position (each of them optional), K and V into a paged cache whose heads may have
+// convolution over time on q, k and v, rotation of pairs, q, k and v heads of unit length, queries that grow with
+// their position, values mixed with an earlier layer's (each of them optional), K and V into a paged cache whose heads may have
 // different key and value sizes; the convolution's state -- the projected rows before the step -- in a ring per sequence
 // slot; and a scalar form of the chunked or windowed attention for any head sizes and for fp32 caches.
 #include <algorithm>
 
 #include "kernels.h"
+#include "paged_attn.cuh"
 
 namespace vlt {
 
@@ -25,7 +26,7 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
     __shared__ const float* from[TB][32];
     __shared__ uint32_t pos_s[TB], cpos_s[TB], slot_s[TB];
     __shared__ size_t row_s[TB];  // where the head's key or value goes in the cache
-    __shared__ float factor[TB];  // what multiplies the head of a query or key
+    __shared__ float factor[TB];  // what multiplies the head
     const uint32_t t0 = blockIdx.x * TB, unit = blockIdx.y, tid = threadIdx.x, nt = min(TB, n - t0);
     const uint32_t kind = unit < a.heads ? 0u : unit < a.heads + a.kv.n_kv ? 1u : 2u;
     const uint32_t head = kind == 0 ? unit : kind == 1 ? unit - a.heads : unit - a.heads - a.kv.n_kv, width = kind == 2 ? a.kv.dv : a.kv.dk;
@@ -75,26 +76,33 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvArgs a, uint32_
         }
     }
     __syncthreads();
-    if (a.unit_qk && kind < 2) {  // a warp per token
+    if (kind < 2 ? a.unit_qk : a.unit_v) {  // a warp per token
         if (mine < TB) {
             float ss = 0.0f;
             for (uint32_t c = back; c < width; c += 32) ss += y[mine * width + c] * y[mine * width + c];
             ss = warp_sum(ss);
             if (back == 0) factor[mine] *= 1.0f / sqrtf(ss / float(width) + a.unit_eps);
             const RowNorm& weight = kind == 0 ? a.q_norm : a.k_norm;
-            if (weight.w)
+            if (kind < 2 && weight.w)
                 for (uint32_t c = back; c < width; c += 32) y[mine * width + c] *= weight_of(weight, c);
         }
         __syncthreads();
     }
     const uint32_t half = a.rot_dims / 2;
+    const float share = kind == 2 && a.mix.share && !a.mix.first ? bf16_to_f32(*a.mix.share) : 0.0f;
     for (uint32_t c = tid; c < width; c += 128) {
 #pragma unroll
         for (uint32_t i = 0; i < TB; i++) {
             if (i >= nt) break;
             const float* yi = y + i * width;
             float v = yi[c];
-            if (kind < 2) v = rotated(yi, c, a.rot_dims, a.neighbours, reinterpret_cast<const float2*>(a.rope) + size_t(pos_s[i]) * half) * factor[i];
+            if (kind < 2) v = rotated(yi, c, a.rot_dims, a.neighbours, reinterpret_cast<const float2*>(a.rope) + size_t(pos_s[i]) * half);
+            v *= factor[i];
+            if (kind == 2 && a.mix.share) {
+                float* first = a.v_first + (size_t(t0 + i) * a.kv.n_kv + head) * width + c;
+                if (a.mix.first) *first = v;
+                else v = (1.0f - share) * v + share * *first;
+            }
             if (kind == 0) {
                 const size_t o = (size_t(t0 + i) * a.heads + head) * width + c;
                 if (a.q_f) a.q_f[o] = v;
@@ -123,9 +131,9 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const ConvArgs a, const
     }
 }
 
-// Attention of one token and query head per block: the cached keys from the chunk's or window's first position (or the
-// sequence's) up to the token's tile of 8, then the tile's rows its `vis` names that lie no further back than that; softmax in fp32 with a running
-// maximum over blocks of 128 keys; the gate, if there is one, on the result.
+// Attention of one token and query head per block: the cached keys that are kept and those from the chunk's or window's first position
+// (or the sequence's) up to the token's tile of 8, then the tile's rows its `vis` names that it sees; softmax in fp32 with a running
+// maximum over blocks of 128 keys; a sink's share and the gate, if there are such, on the result.
 template <typename T>
 __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) {
     pdl_start();
@@ -134,34 +142,29 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
     __shared__ uint32_t rows[128];  // (a key's row in the pool; pools of more than 2^32 rows do not exist)
     __shared__ float red[8];
     const uint32_t t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, g = h / (a.heads / a.kv.n_kv);
-    const uint32_t slot = a.meta[2 * t], pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], mask = a.vis[t];
-    const uint32_t tile0 = t - row % 8, p_tile = a.meta[2 * (t - row) + 1] + row - row % 8;  // the tile's first token and cache position
-    const uint32_t lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0, n_old = p_tile > lo ? p_tile - lo : 0;
+    const paged::View view = paged::view_of(a, t);
+    const uint32_t kept = min(view.keep, min(view.lo, view.first)), n_old = kept + (view.first > view.lo ? view.first - view.lo : 0);  // keys in front of the tile
     const T* K = static_cast<const T*>(a.kv.k);
     const T* V = static_cast<const T*>(a.kv.v);
     const uint32_t ldv = a.kv.v == a.kv.k ? a.kv.dk : a.kv.dv;
     for (uint32_t c = tid; c < a.kv.dk; c += 128) q[c] = a.q_f[(size_t(t) * a.heads + h) * a.kv.dk + c];
     for (uint32_t c = tid; c < a.kv.dv; c += 128) o[c] = 0.0f;
     float m = -INFINITY, l = 0.0f;
+    const float slope = a.slopes ? a.slopes[h] : 0.0f;
     __syncthreads();
     for (uint32_t i0 = 0; i0 < n_old + 8; i0 += 128) {
         const uint32_t i = i0 + tid;
         float s = -INFINITY;
-        bool seen = i < n_old;
-        uint32_t kp = lo + i;
-        if (!seen && i < n_old + 8) {
-            const uint32_t j = i - n_old;
-            kp = p_tile + j;
-            seen = ((mask >> j) & 1u) && a.meta[2 * (tile0 + j) + 1] >= lo;
-        }
-        if (seen) {
-            const size_t r = page_row(a.kv, slot, g, kp);
+        const uint32_t kp = i < kept ? i : i < n_old ? view.lo + i - kept : view.first + i - n_old;
+        if (i < n_old + 8 && paged::sees(view, kp)) {
+            const size_t r = page_row(a.kv, view.slot, g, kp);
             rows[tid] = uint32_t(r);
             const T* k = K + r * a.kv.dk;
             float d = 0.0f;
             for (uint32_t c = 0; c < a.kv.dk; c++) d = fmaf(q[c], load_kv(k + c), d);
             s = d * a.scale;
             if (a.softcap > 0) s = a.softcap * tanhf(s / a.softcap);
+            if (a.slopes) s -= slope * paged::distance(a, view, kp);
         }
         float mx = warp_max(s);
         if (tid % 32 == 0) red[tid / 32] = mx;
@@ -185,6 +188,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const ChunkedAttnArgs a) 
         }
         __syncthreads();
     }
+    if (a.sink) l += expf(bf16_to_f32(a.sink[h]) - m);
     for (uint32_t c = tid; c < a.kv.dv; c += 128) {
         const float gt = a.gate ? 1.0f / (1.0f + expf(-a.gate[size_t(t) * a.ldg + h * a.kv.dv + c])) : 1.0f, y = o[c] / l * gt;
         const size_t at = (size_t(t) * a.heads + h) * a.kv.dv + c;

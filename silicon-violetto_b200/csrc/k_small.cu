@@ -14,7 +14,7 @@ namespace vlt {
 // it sees from the node. meta[t] = (slot, lens[slot] + depth). One block per token.
 __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* tokens, float* __restrict__ out, const uint32_t* __restrict__ tin,
                              uint32_t* meta, const uint32_t* __restrict__ lens, const uint32_t* __restrict__ feed, const uint32_t* __restrict__ tree,
-                             uint32_t* vis, uint32_t d, uint32_t vocab, const uint16_t* __restrict__ positions, uint32_t n_positions, uint16_t* __restrict__ out_b) {
+                             uint32_t* vis, uint32_t d, uint32_t vocab, const uint16_t* __restrict__ positions, uint32_t n_positions, uint16_t* __restrict__ out_b, float scale) {
     pdl_start();
     const uint32_t t = blockIdx.x, tid = threadIdx.x;
     const uint32_t slot = tin[2 * t];
@@ -31,7 +31,7 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
     // rather than index out of the table.
     if (tok >= vocab) tok = 0;
     if (out_b)  // (positions are another design's)
-        for (uint32_t i = tid; i < d; i += blockDim.x) out_b[size_t(t) * d + i] = table[size_t(tok) * d + i];
+        for (uint32_t i = tid; i < d; i += blockDim.x) out_b[size_t(t) * d + i] = f32_to_bf16(bf16_to_f32(table[size_t(tok) * d + i]) * scale);
     if (positions) {  // (a draft's rows may reach past the last position: they are not kept then)
         const uint16_t* pv = positions + size_t(min(lens[slot] + depth, n_positions - 1)) * d;
         if (d % 4 == 0) {
@@ -39,20 +39,20 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
                 float x[4], y[4];
                 load_bf16<4>(x, table + size_t(tok) * d + i);
                 load_bf16<4>(y, pv + i);
-                store_f32<4>(out + size_t(t) * d + i, {x[0] + y[0], x[1] + y[1], x[2] + y[2], x[3] + y[3]});
+                store_f32<4>(out + size_t(t) * d + i, {x[0] * scale + y[0], x[1] * scale + y[1], x[2] * scale + y[2], x[3] * scale + y[3]});
             }
         } else {
-            for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]) + bf16_to_f32(pv[i]);
+            for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]) * scale + bf16_to_f32(pv[i]);
         }
     } else if (d % 2 == 0) {
         const uint32_t* row = reinterpret_cast<const uint32_t*>(table + size_t(tok) * d);
         float2* o = reinterpret_cast<float2*>(out + size_t(t) * d);
         for (uint32_t i = tid; i < d / 2; i += blockDim.x) {
             const uint32_t w = row[i];
-            o[i] = make_float2(bf16lo(w), bf16hi(w));
+            o[i] = make_float2(bf16lo(w) * scale, bf16hi(w) * scale);
         }
     } else {
-        for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]);
+        for (uint32_t i = tid; i < d; i += blockDim.x) out[size_t(t) * d + i] = bf16_to_f32(table[size_t(tok) * d + i]) * scale;
     }
     __syncthreads();  // every thread has read tokens[t]
     if (tid == 0) {
@@ -65,8 +65,8 @@ __global__ void embed_kernel(const uint16_t* __restrict__ table, uint32_t* token
 
 void launch_embed(const uint16_t* table, uint32_t* tokens, float* out, const uint32_t* tin, uint32_t* meta, const uint32_t* lens,
                   const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s, const uint16_t* positions,
-                  uint32_t n_positions, uint16_t* out_b) {
-    launch_pdl(embed_kernel, n, 128, 0, s, table, tokens, out, tin, meta, lens, feed, tree, vis, d, vocab, positions, n_positions, out_b);
+                  uint32_t n_positions, uint16_t* out_b, float scale) {
+    launch_pdl(embed_kernel, n, 128, 0, s, table, tokens, out, tin, meta, lens, feed, tree, vis, d, vocab, positions, n_positions, out_b, scale);
 }
 
 // ------------------------------------------------------- K/V into the cache

@@ -16,6 +16,8 @@ enum : uint32_t { EPI_NORM = 1, EPI_RESID = 2, EPI_SWIGLU = 3, EPI_HEAD = 4, EPI
                 EPI_SIDE = 12,       // gelu(acc) times an entry of the token's row in a table (MatArgs::side)
                 EPI_GLU_CLAMP = 11   // EPI_GLU's pairs: g sigmoid(1.702 g) (u + 1), g cut off above a limit, u outside of +- the limit
 };
+// Rows 2 i and 2 i + 1 make output i.
+__host__ __device__ constexpr bool epi_pairs(uint32_t epi) { return epi == EPI_SWIGLU || epi == EPI_GLU || epi == EPI_GLU_CLAMP; }
 
 // What the tensor-core GEMM's EPI_QKV epilogue needs to finish the qkv projection the way `qkv_post` does
 // (kernels.metal:749-801): RoPE on q and k, q scaled and rounded to bf16 for the attention, k and v rounded
@@ -77,6 +79,8 @@ struct MatArgs {
     uint32_t n, k, m, group;  // group: 0 for bf16 weights
     uint32_t epi, vocab_real;  // vocab_real: a head's rows from there on are padding; EPI_SILU: rows from there on stay as they are
     float eps;
+    const uint16_t* bias;  // optional, bf16 [m] (bf16 weights): onto the sums in front of everything else
+    float limit;           // EPI_GLU_CLAMP
     // kernels.metal:164-165,188-193: the matrix scale (qkv_scale, o_scale) and EPI_RESID's y = ra base + rb (scale acc). 1 for a
     // plain decoder.
     float scale = 1.0f, ra = 1.0f, rb = 1.0f;
@@ -96,7 +100,8 @@ struct MatArgs {
 void launch_embed(const uint16_t* table, uint32_t* tokens, float* out, const uint32_t* tin, uint32_t* meta, const uint32_t* lens,
                   const uint32_t* feed, const uint32_t* tree, uint32_t* vis, uint32_t n, uint32_t d, uint32_t vocab, cudaStream_t s,
                   const uint16_t* positions = nullptr, uint32_t n_positions = 0,  // positions: [n_positions][d], a vector per position to add
-                  uint16_t* out_b = nullptr);                                     // out in bf16
+                  uint16_t* out_b = nullptr,                                      // out in bf16
+                  float scale = 1.0f);                                            // of the table's rows
 void launch_qkv_post(const float* qkv, const uint32_t* meta, const uint32_t* tin, const float* rope, uint16_t* k_cache, uint16_t* v_cache,
                      const uint32_t* page_table, KvArgs kv, uint32_t layer, uint32_t n, uint32_t n_heads, float scale_log2, uint16_t* q_b, const uint32_t* cpos, cudaStream_t s);
 // q | k | v rows as the attention sees them before rounding (RoPE on q and k, kernels.metal:727-736), for step_capture.
@@ -248,11 +253,12 @@ struct LinearArgs {
     uint32_t n, m, k, epi;   // EPI_RAW, EPI_RESID, EPI_RELU2, EPI_SILU, EPI_GLU or EPI_GLU_CLAMP
     uint32_t act_rows;       // EPI_SILU
     float limit;             // EPI_GLU_CLAMP
+    const uint16_t* bias;    // optional, without tiles: [m], onto the sums
     const float* row_scale;  // optional, with tiles: what row p's products are multiplied by, before the epilogue
     // A matrix per head against that head's part of every token (by_head tokens; 0: not so): group g's rows are p = g by_head + t,
     // read at row t heads + g of X and written at row t heads + g of Y, `ldy` apart. gate (optional): [by_head][ldg], the output is
-    // multiplied by the sigmoid of row t's column g m + r.
-    uint32_t by_head, heads, ldy, ldg;
+    // multiplied by the sigmoid of row t's column g m + r, or (gate_w 1) g.
+    uint32_t by_head, heads, ldy, ldg, gate_w;
     const float* gate;
     const uint32_t* tiles;   // [.][3]: (group, first row, rows)
     const uint32_t* n_tiles;
@@ -262,7 +268,7 @@ void launch_linear(const LinearArgs& a, bool x_bf16, cudaStream_t s);
 bool grouped_fits(uint32_t m, uint32_t k);  // the tensor-core form (k_grouped.cu): bf16 activations, EPI_RAW, EPI_RELU2 or EPI_GLU_CLAMP
 void launch_grouped(const LinearArgs& a, uint32_t n_groups, uint32_t tile, uint32_t* err_flag, cudaStream_t s);
 // out[r] = x / sqrt(mean x^2 + eps) times the weight times `scale`, x being row rows[r] (or r) of `in`, plus that of `add`, the
-// sum then left in `sum`.
+// sum then left in `sum`. (A centered norm: of x less its mean, plus its b times `scale`.)
 struct NormArgs {
     const float* in;
     const uint32_t* rows;    // optional
@@ -298,6 +304,19 @@ struct AddNormArgs {
     float eps;
 };
 void launch_add_norm(const AddNormArgs& a, cudaStream_t s);
+// out[r] = the sum over j < count of share[j] X_j[r], X_j at x + j stride; norm.w (optional): its normed rows as well.
+struct DepthArgs {
+    const float* x;
+    size_t stride;
+    const uint16_t* share;
+    float* out;              // none of the X_j
+    RowNorm norm;
+    float* next;             // optional
+    uint16_t* next_b;        // optional
+    uint32_t count, n, d;
+    float eps;
+};
+void launch_depth_average(const DepthArgs& a, cudaStream_t s);
 struct SideGateArgs {
     const float* x;          // [n][ldx]
     SideTable side;
@@ -335,6 +354,7 @@ struct MixerCache {
     float* ring;
     uint32_t ring_len, channels;
     uint32_t recurrent;  // a recurrence's index among the model's (see RecurrentCache)
+    const float* per_head;  // the mixer's fixed decays or slopes
 };
 // The work between an attention mixer's projections and its attention (k_mixer.cu).
 struct ConvArgs {
@@ -351,7 +371,9 @@ struct ConvArgs {
     uint32_t ldu, taps, ring_len, conv_channels, heads, rot_dims;
     bool write_ring;                      // false: launch_conv_state does it afterwards
     float unit_eps;                       // with unit_qk: q's and k's heads over sqrt(mean square + unit_eps), times a weight (optional)
-    bool unit_qk, neighbours;             // neighbours: see Rotation
+    bool unit_qk, unit_v, neighbours;     // unit_v: v's heads likewise, without a weight; neighbours: see Rotation
+    ValueMix mix;                         // (behind unit_v; without a convolution)
+    float* v_first;                       // [n][kv heads dv]: the values mixed in, which the first layer leaves there
     RowNorm q_norm, k_norm;
     QueryTemperature temp;
 };
@@ -387,15 +409,18 @@ struct ChunkedAttnArgs {
     PagedKv kv;
     const float* gate;                    // optional [n][ldg]: the output is multiplied by sigmoid(gate)
     uint32_t ldg, heads, chunk, window;   // what a position sees (see Attention); both 0: every position before
+    uint32_t keep;                        // with a window: it sees the first `keep` positions as well
     float scale, softcap;                 // softcap: see Attention
+    const float* slopes;                  // optional [heads]: see Attention (not launch_attn_latent)
+    const uint16_t* sink;                 // optional [heads], bf16: see LatentAttention (not launch_attn_chunked)
     float* out;                           // optional [n][heads][dv]
     uint16_t* out_b;                      // optional
 };
 bool chunk_attn_fits(uint32_t dk, uint32_t dv, uint32_t page);  // k_chunk_attn.cu's kernels, bf16 caches; else launch_attn_any
 void launch_attn_chunked(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, cudaStream_t s);
 void launch_attn_any(const ChunkedAttnArgs& a, uint32_t n, bool fp32, cudaStream_t s);
-// What stands between a latent attention's projections (k_latent.cu). From the rows q | c | r of the first one: n(q) for the query
-// projection, and n(c) and r rotated into the cache (kv.dk entries a row).
+// What stands between a latent attention's projections (k_latent.cu). From the rows q | c | r of the first one, c at column key_at:
+// n(q) for the query projection (with q_rank), and n(c) and r rotated into the cache (kv.dk entries a row).
 struct LatentRowsArgs {
     const float* u;                       // [n][ldu]
     RowNorm q_norm, kv_norm;
@@ -404,7 +429,7 @@ struct LatentRowsArgs {
     PagedKv kv;
     float* q_f;                           // optional: [n][q_rank]
     uint16_t* q_b;                        // optional
-    uint32_t ldu, q_rank, kv_rank, rot_dim;
+    uint32_t ldu, q_rank, key_at, kv_rank, rot_dim;
     bool own, neighbours;                 // own: (c ; r) is this layer's to write
     float eps;
 };
@@ -423,6 +448,8 @@ struct LatentQueryArgs {
     float factor;
 };
 void launch_latent_query(const LatentQueryArgs& a, cudaStream_t s);
+// Both in one launch, where the queries come with (c ; r) from the first projection.
+void launch_latent_split(const LatentRowsArgs& r, const LatentQueryArgs& q, bool fp32, cudaStream_t s);
 bool latent_attn_fits(uint32_t kv_rank, uint32_t rot_dim, uint32_t page);  // k_latent_attn.cu's kernels, bf16 caches; else launch_attn_any
 void launch_attn_latent(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t max_keys, uint32_t sm_count, uint32_t keys_per_block, uint32_t* err_flag, cudaStream_t s);
 void launch_mixer_compact(const RunIn* runs, const uint32_t* path, const uint32_t* path_len, const uint32_t* lens, const MixerCache* caches, uint32_t n_runs, uint32_t n_caches,

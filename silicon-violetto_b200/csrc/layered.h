@@ -1,5 +1,5 @@
 // Model folders: decoders whose config.json lists their layers one by one. This file has the mechanisms a layer can hold, each a
-// parameter struct of its own, the list of layer runs, and what the readers of the designs (lonasun.h, leduvik.h, pasovik.h) share: the
+// parameter struct of its own, the list of layer runs, and what the readers of the designs (lonasun.h, leduvik.h, pasovik.h, sopetar.h) share: the
 // tensors' places and the loop over a span of layers. A design's reader fills it; engine_layered.cu runs it.
 #pragma once
 #include <memory>
@@ -10,10 +10,11 @@ namespace vlt {
 
 bool decay_fits(uint32_t rank, uint32_t dim);  // of a TimeMix (k_recurrent.cu)
 
-// Of rows: x / sqrt(mean x^2 + eps), times the weight (as stored, or stored around zero: 1 + w).
+// Of rows: x / sqrt(mean x^2 + eps), times the weight (as stored, or stored around zero: 1 + w). centered: of x less its mean
+// (in front of layers and the head only).
 struct RowNorm {
-    const uint16_t* w = nullptr;
-    bool around_zero = false;
+    const uint16_t *w = nullptr, *b = nullptr;  // b: what is added at the end (optional, with centered)
+    bool around_zero = false, centered = false;
 };
 // y_t = b[c] + sum_j w[c][j] u_(t - taps + 1 + j) per channel.
 struct ShortConv {
@@ -33,19 +34,28 @@ struct QueryTemperature {
     float coef = 0;
     double every = 0;
 };
+// Values v of a layer become (1 - share) v + share v', v' being the same token's in the first layer that takes part.
+struct ValueMix {
+    const uint16_t* share = nullptr;  // one number; none: the layer takes no part
+    bool first = false;
+};
 // Attention over pages of keys. What a position sees of the positions up to its own: those of its own block of `chunk`, or the
-// last `window`, or (both 0) all.
+// last `window` and the sequence's first `keep`, or (both 0) all.
 struct Attention {
-    uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, chunk = 0, window = 0;
+    uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, chunk = 0, window = 0, keep = 0;
     float scale = 1;
     float softcap = 0;       // scores become softcap tanh(score / softcap); 0: they stay
+    std::vector<float> slopes;  // per head (or none): what a score loses per position between the query and its key, behind the cap
     bool unit_qk = false;    // q's and k's heads are divided by their root mean square, ...
     RowNorm q_norm, k_norm;  // ... and multiplied by a weight of one head's size (optional)
+    bool unit_v = false;     // v's heads are divided by their root mean square
+    ValueMix mix;            // behind that
     bool gated = false;      // the output times sigmoid(gate)
     Rotation rot;
     QueryTemperature temp;
     ShortConv conv;  // over q | k | v
     Matrix proj, o;  // proj: the rows of q, k, v and, if gated, the gate stacked
+    uint32_t v_w() const { return kv_heads * vdim; }
     uint32_t qkv_w() const { return (heads + kv_heads) * dim + kv_heads * vdim; }
     uint32_t out_w() const { return heads * vdim; }
 };
@@ -71,17 +81,24 @@ struct TimeMix {
 };
 // Attention whose keys and values are linear in a short normed row c of every position: per head, the key is (W_uk c ; r) with a
 // rotated part r that all heads share, the value W_uv c. Only (c ; r) is kept. W_uk goes onto the queries and W_uv onto the sums of
-// c: the heads are query heads of one kv head whose key is (c ; r) and whose value is c. Queries come from a normed row of their own.
+// c: the heads are query heads of one kv head whose key is (c ; r) and whose value is c. Queries come from a normed row of their own,
+// or (q_rank 0) straight from the layer's.
 struct LatentAttention {
     static constexpr uint32_t OWN = 0xffffffffu;
     uint32_t heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0, q_rank = 0;
+    uint32_t window = 0;      // a position sees the last `window` up to its own; 0: all
     float scale = 1;
     Rotation rot;             // of the rotated parts
     uint32_t kv_from = OWN;   // the layer whose (c ; r) this one reads
-    Matrix in;                // W_dq | W_dkv (unless kv_from) | W_g stacked
+    const uint16_t* sink = nullptr;  // per head (optional): a logit that takes its share of the softmax and has no value
+    bool gate_by_head = false;       // the gate has a row per head, not per output
+    Matrix in;                // W_dq (or W_q) | W_dkv (unless kv_from) | W_g stacked
     Matrix uq, uk_t, uv, o;   // uk_t, uv: per head [kv_rank][dim] and [vdim][kv_rank], stacked
     RowNorm q_norm, kv_norm;
     uint32_t key_w() const { return kv_rank + rot_dim; }
+    uint32_t query_w() const { return heads * (dim + rot_dim); }
+    uint32_t first_w() const { return q_rank ? q_rank : query_w(); }  // rows of `in` in front of W_dkv
+    uint32_t gate_w() const { return gate_by_head ? heads : out_w(); }
     uint32_t out_w() const { return heads * vdim; }
     uint32_t kv_w() const { return kv_from == OWN ? key_w() : 0; }  // rows of W_dkv in `in`
 };
@@ -123,6 +140,7 @@ struct ExpertLayer {
 };
 struct DenseLayer {
     Hidden hidden = Hidden::Relu2;
+    float limit = 0;
     Matrix up, down;
 };
 // n(W_proj (gelu(W_gate x) * e)) onto the stream, e a span of the token's row in the model's side table; gelu by tanh.
@@ -140,6 +158,10 @@ struct FolderLayer {
     DenseLayer dense;
     bool post_norm = false;  // norm1 and norm2 go onto what the mixer and the feed-forward leave; both read the stream itself
     SideInput side;          // (layers with post_norm)
+    bool parallel = false;   // the feed-forward reads norm1's rows, beside the mixer (dense ones; one mixer)
+    // X_0 being the embedding and X_(i + 1) what layer run i leaves: what goes on from this run is the sum over j <= i + 1 of depth[j] X_j
+    // (optional; all layers or none).
+    const uint16_t* depth = nullptr;
 };
 // A layer run: with a loop a layer runs several times, each with a cache of its own.
 struct LayerRun {
@@ -173,7 +195,7 @@ struct LayeredModel {
     const uint16_t* side = nullptr;                         // the layers' side inputs: a row of side_w per token id (optional)
     uint32_t side_w = 0;
     RowNorm final_norm;
-    float logit_scale = 1;
+    float logit_scale = 1, embed_scale = 1;
 
     // A design's reader: its own part of config.json and the tensors it names.
     using Reader = void (*)(LayeredModel&, const Json&, ModelDesc&);
@@ -212,8 +234,13 @@ struct LayeredModel {
         w.zeros(size_t(whole - rows) * k * 2);
         matrix(m, whole, k, offset);
     }
-    // q, k, v and, if gated, g of an attention, and its output matrix.
-    void attention_matrices(Attention& a, const std::string& pre, uint32_t d) {
+    // The bias of a matrix whose last rows may be padding: it is the tensor, or the stack, placed last.
+    void bias(Matrix& m, uint32_t rows, size_t offset) {
+        w.zeros(size_t(m.m - rows) * 2);
+        point(m.bias, offset);
+    }
+    // q, k, v and, if gated, g of an attention, and its output matrix; biased: q, k and v have biases.
+    void attention_matrices(Attention& a, const std::string& pre, uint32_t d, bool biased = false) {
         if (a.kv_heads == 0 || a.heads == 0 || a.heads % a.kv_heads || a.dim == 0 || a.vdim == 0) throw Error(pre + ": the heads do not fit the kv heads");
         const uint32_t qw = a.heads * a.dim, kw = a.kv_heads * a.dim, vw = a.kv_heads * a.vdim;
         const size_t at = w.place(pre + "q", {qw, d});
@@ -221,6 +248,39 @@ struct LayeredModel {
         w.place(pre + "v", {vw, d}, false);
         if (a.gated) w.place(pre + "g", {a.out_w(), d}, false);
         padded(a.proj, qw + kw + vw + (a.gated ? a.out_w() : 0), d, at);
+        matrix(a.o, pre + "o", d, a.out_w());
+        if (!biased) return;
+        const size_t b = w.place(pre + "q.b", {qw});
+        w.place(pre + "k.b", {kw}, false);
+        w.place(pre + "v.b", {vw}, false);
+        bias(a.proj, qw + kw + vw, b);
+    }
+    // Neighbouring pairs of the first rot.dims of `width` dimensions.
+    void neighbours(Rotation& rot, const Json& r, const std::string& pre, uint32_t width) {
+        rot.dims = r.at("dims").count("rot.dims");
+        rot.base = r.at("base").number("rot.base");
+        if (!r["scaling"].is_null()) rot.factor = r["scaling"].at("factor").number("rot.scaling.factor");
+        rot.neighbours = true;
+        if (rot.dims % 2 || rot.dims > width) throw Error(pre + ": rot.dims does not fit the heads");
+        if (!(rot.base > 0) || !(rot.factor > 0)) throw Error(pre + ": rot.base and rot.scaling.factor must be positive");
+        share(rot);
+    }
+    // The sizes of a latent attention (q_rank: if its queries have one) and its rotation.
+    void sizes(LatentAttention& a, const Json& m, const std::string& pre) {
+        a.heads = m.at("heads").count("heads");
+        a.dim = m.at("dim").count("dim");
+        a.rot_dim = m.at("rot_dim").count("rot_dim");
+        a.vdim = m.at("vdim").count("vdim");
+        a.kv_rank = m.at("kv_rank").count("kv_rank");
+        a.scale = float(m.at("scale").number("scale"));
+        if (a.heads == 0 || a.dim == 0 || a.vdim == 0 || a.kv_rank == 0) throw Error(pre + ": a size of 0");
+        neighbours(a.rot, m.at("rot"), pre, a.rot_dim);
+        if (a.rot.dims != a.rot_dim) throw Error(pre + ": rot.dims is not rot_dim");
+    }
+    // What its heads make of the latents, and its output matrix.
+    void latent_matrices(LatentAttention& a, const std::string& pre, uint32_t d) {
+        matrix(a.uk_t, a.heads * a.kv_rank, a.dim, w.place_transposed(pre + "uk", a.heads, a.dim, a.kv_rank));
+        matrix(a.uv, pre + "uv", a.heads * a.vdim, a.kv_rank);
         matrix(a.o, pre + "o", d, a.out_w());
     }
     static void sizes(Attention& a, const Json& m) {

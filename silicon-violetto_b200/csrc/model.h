@@ -5,6 +5,7 @@
 #include "leduvik.h"
 #include "lonasun.h"
 #include "pasovik.h"
+#include "sopetar.h"
 #include "weights.h"
 
 namespace vlt {
@@ -33,7 +34,7 @@ struct Model {
         const std::string path = dir + "/config.json";
         const Json cfg = read_json(path);
         const std::string& arch = cfg.at("architecture").text("architecture");
-        static const struct { const char* name; LayeredModel::Reader read; } registry[] = {{"Lonasun", lonasun::read}, {"Leduvik", leduvik::read}, {"Pasovik", pasovik::read}};
+        static const struct { const char* name; LayeredModel::Reader read; } registry[] = {{"Lonasun", lonasun::read}, {"Leduvik", leduvik::read}, {"Pasovik", pasovik::read}, {"Sopetar", sopetar::read}};
         for (const auto& r : registry) {
             if (arch != r.name) continue;
             layered = LayeredModel::load(r.read, cfg, dir, host_only, md);

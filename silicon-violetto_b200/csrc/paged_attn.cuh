@@ -24,15 +24,19 @@ __device__ __forceinline__ float gated(float y, float gate) { return y / (1.0f +
 
 constexpr uint32_t PAGE_SHIFT = 6, PAGE = 1u << PAGE_SHIFT;
 
-// What token t sees: cached keys [lo, first) and, of its tile of 8 rows that starts at cache position `first`, those `mask`
-// names (its `vis`, less the rows of an earlier chunk or out of the window: the rows of a draft tree may lie on both sides of an edge).
+// What token t sees: cached keys [0, keep) and [lo, first) and, of its tile of 8 rows (token `tile` on) that starts at cache position
+// `first`, those `mask` names (its `vis`, less the rows of an earlier chunk or out of the window: the rows of a draft tree may lie on
+// both sides of an edge).
 struct View {
-    uint32_t slot, lo, first, mask;
+    uint32_t slot, pos, lo, keep, first, mask, tile;
 };
 __device__ __forceinline__ View view_of(const ChunkedAttnArgs& a, uint32_t t) {
     const uint32_t pos = a.meta[2 * t + 1], row = a.tin[2 * t + 1], i = row % 8;
     View v;
     v.slot = a.meta[2 * t];
+    v.pos = pos;
+    v.keep = a.keep;
+    v.tile = t - i;
     v.first = a.meta[2 * (t - row) + 1] + row - i;
     v.lo = a.chunk ? pos / a.chunk * a.chunk : a.window && pos + 1 > a.window ? pos + 1 - a.window : 0;
     v.mask = a.vis[t];
@@ -41,13 +45,32 @@ __device__ __forceinline__ View view_of(const ChunkedAttnArgs& a, uint32_t t) {
         for (uint32_t m = v.mask; m;) {
             const uint32_t j = __ffs(m) - 1;
             m &= m - 1;
-            if (a.meta[2 * (t - i + j) + 1] >= v.lo) seen |= 1u << j;
+            const uint32_t at = a.meta[2 * (v.tile + j) + 1];
+            if (at >= v.lo || at < v.keep) seen |= 1u << j;
         }
         v.mask = seen;
     }
     return v;
 }
-__device__ __forceinline__ bool sees(const View& v, uint32_t key) { return key >= v.lo && (key < v.first || (key - v.first < 32 && ((v.mask >> (key - v.first)) & 1u))); }
+__device__ __forceinline__ bool sees(const View& v, uint32_t key) {
+    return key < v.first ? key >= v.lo || key < v.keep : key - v.first < 32 && ((v.mask >> (key - v.first)) & 1u);
+}
+// How far a seen key lies back. (A draft tree's rows lie in the cache one after the other, but at positions of their own.)
+__device__ __forceinline__ float distance(const ChunkedAttnArgs& a, const View& v, uint32_t key) {
+    return float(int(v.pos) - int(key < v.first ? key : a.meta[2 * (v.tile + key - v.first) + 1]));
+}
+// The tiles of SIZE positions that hold keys seen, of rows whose lowest `lo` is `low`: the first `head` ones with keys kept, then from
+// low's on. Walked by number.
+template <uint32_t SIZE>
+struct Tiles {
+    uint32_t head, skip;
+    __device__ __forceinline__ Tiles(uint32_t low, uint32_t keep) {
+        head = min((keep + SIZE - 1) / SIZE, low / SIZE);
+        skip = low / SIZE - head;
+    }
+    __device__ __forceinline__ uint32_t count(uint32_t end) const { return (end + SIZE - 1) / SIZE - skip; }
+    __device__ __forceinline__ uint32_t at(uint32_t i) const { return i < head ? i : i + skip; }
+};
 // A score times log2(e), soft-capped: cap tanh(s / cap) as cap - 2 cap / (e^(2 s / cap) + 1), whose error is one of the exponential's and
 // the quotient's last bits of the cap. cap: the constant times log2(e); inv: 2 / the constant.
 __device__ __forceinline__ float capped(float s, float cap, float inv) { return cap - __fdividef(2.0f * cap, fast_exp2(s * inv) + 1.0f); }

@@ -10,16 +10,6 @@ namespace vlt {
 
 namespace pasovik {
 
-inline void rotation(LayeredModel& model, const Json& r, const std::string& pre, Rotation& rot, uint32_t width) {
-    rot.dims = r.at("dims").count("rot.dims");
-    rot.base = r.at("base").number("rot.base");
-    if (!r["scaling"].is_null()) rot.factor = r["scaling"].at("factor").number("rot.scaling.factor");
-    rot.neighbours = true;
-    if (rot.dims % 2 || rot.dims > width) throw Error(pre + ": rot.dims does not fit the heads");
-    if (!(rot.base > 0) || !(rot.factor > 0)) throw Error(pre + ": rot.base and rot.scaling.factor must be positive");
-    model.share(rot);
-}
-
 inline void attention(LayeredModel& model, const Json& m, const std::string& pre, Attention& a, uint32_t d) {
     LayeredModel::sizes(a, m);
     a.unit_qk = true;
@@ -27,7 +17,7 @@ inline void attention(LayeredModel& model, const Json& m, const std::string& pre
         a.softcap = float(m["softcap"].number("softcap"));
         if (!(a.softcap > 0)) throw Error(pre + ": softcap must be positive");
     }
-    rotation(model, m.at("rot"), pre, a.rot, a.dim);
+    model.neighbours(a.rot, m.at("rot"), pre, a.dim);
     model.attention_matrices(a, pre, d);
     model.point(a.q_norm.w, pre + "q.norm", {a.dim});
     model.point(a.k_norm.w, pre + "k.norm", {a.dim});
@@ -35,16 +25,9 @@ inline void attention(LayeredModel& model, const Json& m, const std::string& pre
 
 inline void latent_attention(LayeredModel& model, const Json& m, const std::string& pre, uint32_t index, LatentAttention& a, uint32_t d) {
     SafeTensors& w = model.w;
-    a.heads = m.at("heads").count("heads");
-    a.dim = m.at("dim").count("dim");
-    a.rot_dim = m.at("rot_dim").count("rot_dim");
-    a.vdim = m.at("vdim").count("vdim");
-    a.kv_rank = m.at("kv_rank").count("kv_rank");
+    model.sizes(a, m, pre);
     a.q_rank = m.at("q_rank").count("q_rank");
-    a.scale = float(m.at("scale").number("scale"));
-    if (a.heads == 0 || a.dim == 0 || a.vdim == 0 || a.kv_rank == 0 || a.q_rank == 0) throw Error(pre + ": a size of 0");
-    rotation(model, m.at("rot"), pre, a.rot, a.rot_dim);
-    if (a.rot.dims != a.rot_dim) throw Error(pre + ": rot.dims is not rot_dim");
+    if (a.q_rank == 0) throw Error(pre + ": a size of 0");
     if (!m["kv_from"].is_null()) {
         a.kv_from = m["kv_from"].count("kv_from");
         const std::vector<Mixer>* from = a.kv_from < index ? &model.layers[a.kv_from].mix : nullptr;
@@ -59,11 +42,8 @@ inline void latent_attention(LayeredModel& model, const Json& m, const std::stri
     model.padded(a.in, a.q_rank + a.kv_w() + a.out_w(), d, at);
     model.point(a.q_norm.w, pre + "dq.norm", {a.q_rank});
     if (a.kv_w()) model.point(a.kv_norm.w, pre + "dkv.norm", {a.kv_rank});
-    const uint32_t q_w = a.heads * (a.dim + a.rot_dim);
-    model.padded(a.uq, q_w, a.q_rank, w.place(pre + "uq", {q_w, a.q_rank}));
-    model.matrix(a.uk_t, a.heads * a.kv_rank, a.dim, w.place_transposed(pre + "uk", a.heads, a.dim, a.kv_rank));
-    model.matrix(a.uv, pre + "uv", a.heads * a.vdim, a.kv_rank);
-    model.matrix(a.o, pre + "o", d, a.out_w());
+    model.padded(a.uq, a.query_w(), a.q_rank, w.place(pre + "uq", {a.query_w(), a.q_rank}));
+    model.latent_matrices(a, pre, d);
 }
 
 inline void lightning(LayeredModel& model, const Json& m, const std::string& pre, LinearAttention& a, uint32_t d) {

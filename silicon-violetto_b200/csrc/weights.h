@@ -163,6 +163,7 @@ struct SafeTensors {
             if (size && e.nbytes != count * size) throw Error(name + ": its data does not fit its shape");
             total += e.nbytes + 256;
             if (e.shape.size() == 2) total += size_t(128) * e.shape[1] * 2 + size_t(126) * e.shape[0];  // (room for `zeros` and `place_wide`; untouched pages of it cost nothing)
+            if (e.shape.size() == 1) total += 256;
             entries[name] = e;
         }
         buffer.alloc(total + 256, true);  // (filled on the host, then moved to the device in one copy: see to_device)
@@ -186,10 +187,10 @@ struct SafeTensors {
         std::memcpy(buffer.as<uint8_t>() + at, e.data, e.nbytes);
         return at;
     }
-    // Two matrices of one shape with their rows in turn: a, b, a, b, ...
+    // Two matrices of one shape with their rows (two vectors: their entries) in turn: a, b, a, b, ...
     size_t place_pairs(const std::string& a, const std::string& b, const std::vector<uint32_t>& shape, bool fresh = true) {
         const Entry &ea = get(a, shape), &eb = get(b, shape);
-        const size_t row = size_t(shape[1]) * 2, at = room(2 * ea.nbytes, fresh);
+        const size_t row = size_t(shape.size() > 1 ? shape[1] : 1) * 2, at = room(2 * ea.nbytes, fresh);
         uint8_t* dst = buffer.as<uint8_t>() + at;
         for (size_t r = 0; r < shape[0]; r++) {
             std::memcpy(dst + 2 * r * row, ea.data + r * row, row);
@@ -249,10 +250,10 @@ struct SafeTensors {
 };
 
 // engine/src/model.rs:22-47 `Matrix`, `Int8`: [m][k] row-major at `w`; int8 has bf16 scales
-// [m][k / group] at `scales`.
+// [m][k / group] at `scales`; bf16 may have a bias [m], which goes onto its products first thing.
 struct Matrix {
     const uint8_t* w = nullptr;
-    const uint16_t* scales = nullptr;
+    const uint16_t *scales = nullptr, *bias = nullptr;
     uint32_t m = 0, k = 0, group = 0;
     bool int8 = false;
     size_t bytes() const { return int8 ? size_t(m) * k + size_t(2) * m * (k / group) : size_t(2) * m * k; }
