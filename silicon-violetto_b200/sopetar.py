@@ -66,7 +66,9 @@ def random_weights(cfg: dict, seed: int = 0, pool: int = 1 << 22) -> dict:
             v[-1] += 1.0
         elif leaf == "vmix":
             v = 0.4 + 0.1 * v
-        elif leaf != "sink" and name != "embed":
+        elif leaf == "sink":
+            v = 2.0 + v
+        elif name != "embed":
             v = v * (shape[-1] ** -0.5)
         out[name] = to_bf16(v).reshape(shape)
     return out
