@@ -449,14 +449,61 @@ def pasovik_work(size):
     return c, {"pasovik": ours, **leduvik_work(size)[1]}
 
 
+# Layers of real models' sizes, in blocks of latent attention, attention, latent attention; beside each a Pasovik model, the framework's
+# closest other one, of the same width, heads, latents and feed-forwards (without its side inputs), decoding over as many keys as a
+# window here lets a token see.
+SOPETAR_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512), q_rank=1536, ff=5376, window=4096, keep=64, vocab=32768,
+                 blocks=2, ctx=8000),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512), q_rank=1536, ff=9472, window=1024, keep=16, vocab=32768,
+                 blocks=1, ctx=4000),
+}
+
+
+def sopetar_files(size):
+    """A Sopetar model and the Pasovik model beside it (SOPETAR_SIZES), random-init, bf16, written once per box."""
+    from silicon_violetto_b200 import pasovik, sopetar
+    CACHE.mkdir(parents=True, exist_ok=True)
+    c = SOPETAR_SIZES[size]
+    heads = (c["heads"], c["kv_heads"], c["dim"], c["dim"])
+    ours = sopetar.latent(**c["latent"], window=c["window"], base=500000.0, mlp=sopetar.dense(c["ff"]))
+    ours = sopetar.config(c["width"], c["vocab"], [ours, sopetar.attention(*heads, window=c["window"], keep=c["keep"], mlp=sopetar.dense(c["ff"])), ours] * c["blocks"], embed_scale=0.5)
+    other = pasovik.latent(**c["latent"], q_rank=c["q_rank"], base=500000.0, mlp=pasovik.dense(c["ff"]))
+    other = pasovik.config(c["width"], c["vocab"], [other, pasovik.attention(*heads, softcap=50.0, rot_dims=64, base=500000.0, mlp=pasovik.dense(c["ff"])), other] * c["blocks"], side=None)
+    folders = []
+    for module, cfg in ((sopetar, ours), (pasovik, other)):
+        folder = CACHE / f"sopetar_{size}_{cfg['architecture']}"
+        if not (folder / "ok").exists():
+            module.write_model(folder, cfg, module.random_weights(cfg))
+            (folder / "ok").write_text("ok")
+        folders.append(folder)
+    return folders
+
+
+def sopetar_work(size):
+    """What the two models of SOPETAR_SIZES read and compute, for folder_figure."""
+    c = SOPETAR_SIZES[size]
+    d, B, l, W = c["width"], c["blocks"], c["latent"], c["window"]
+    attn_p = (2 * c["heads"] + 2 * c["kv_heads"]) * c["dim"] * d
+    row, q_w, inner = l["kv_rank"] + l["rot_dim"], l["heads"] * (l["dim"] + l["rot_dim"]), l["heads"] * l["vdim"]
+    shared = (row + inner) * d + l["heads"] * l["kv_rank"] * (l["dim"] + l["vdim"])  # W_dkv, W_o, W_uk, W_uv
+    weights = lambda latent_p: B * (attn_p + 2 * latent_p + 3 * 3 * c["ff"] * d)
+
+    def at(latent_p, ctx, keep, pairs):
+        return {"decode_weights": lambda n: weights(latent_p), "prompt_weights": weights(latent_p), "kv": B * 2 * (2 * c["kv_heads"] * c["dim"] * (W + keep) + 2 * row * W), "state": 0, "ctx": ctx,
+                "attention_flops": B * 2.0 * (2 * c["heads"] * c["dim"] + 2 * l["heads"] * (row + l["kv_rank"])) * pairs}  # (as the kernel does them: all heads on the rows)
+    return c, {"sopetar": at((q_w + l["heads"]) * d + shared, c["ctx"], c["keep"], c["ctx"] * W - W * W / 2),
+               "pasovik": at((c["q_rank"] + inner) * d + q_w * c["q_rank"] + shared, W, 0, W * W / 2)}
+
+
 def folder_figure(E, local, c, files, work, steps, stream_counts, hbm_peak, tc_peak):
     """Decoding over a filled context and a prompt of the same length in portions of 512, the folder's model and the plain
     decoder: step times, and per kernel group (time from CUDA events around each group's launches, in steps of their own) the
     fraction of the measured copy bandwidth or bf16 throughput its algorithmic bytes or FLOPs make."""
-    ctx = c["ctx"]
-    out = {"workload": f"layers of width {c['width']}, bf16, random-init; decode at ctx {ctx}, prompts of {ctx} in portions of 512"}
+    out = {"workload": f"layers of width {c['width']}, bf16, random-init; decode at ctx {c['ctx']}, prompts of {c['ctx']} in portions of 512 (a model with a ctx of its own below: at that)"}
     for (name, w), path in zip(work.items(), files):
-        res = out[name] = {}
+        ctx = w.get("ctx", c["ctx"])
+        res = out[name] = {"ctx": ctx}
         for n_s in stream_counts:
             eng = E.Engine(path, E.EngineConfig(max_seqs=n_s, max_step_tokens=max(64, n_s), max_chunk=32, global_kv_tokens=n_s * (ctx + 192), max_seq_len=ctx + 128,
                                                 max_head_rows=max(8, n_s), device_ordinal=local), E.Tuning(spec_policy_off=True))
@@ -559,11 +606,11 @@ def main():
     ap.add_argument("--attn-keys", type=int, default=0, help="keys per attention block (0: the engine's own choice)")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers: a profiler-size case, not a bench value")
     ap.add_argument("--no-limite", action="store_true", help="skip the reference-architecture pass of the extras (it writes a 2 GB file first)")
-    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite, lonasun, leduvik and pasovik")
+    ap.add_argument("--limite-streams", default="1,8,32", help="stream counts of --only limite, lonasun, leduvik, pasovik and sopetar")
     ap.add_argument("--limite-drafter", action="store_true", help="--only limite: with the reference's block drafter loaded (tree drafts of up to 8 rows)")
     ap.add_argument("--limite-int8", action="store_true", help="--only limite: int8 weights in the reference converter's default groups (64; the head 8)")
     ap.add_argument("--limite-keys", type=int, default=0, help="--only limite: keys per attention block (VltTuning.attn_keys_per_cta); 0 = the library's choice")
-    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) 'lonasun', 'leduvik' or 'pasovik' (models of those designs beside others of equal size): run that one pass alone and print its figure (not the bench line)")
+    ap.add_argument("--only", default="", help="'prefill', 'acceptance', 'limite' (the reference's own architecture at its shapes, decoding) 'lonasun', 'leduvik', 'pasovik' or 'sopetar' (models of those designs beside others of equal size): run that one pass alone and print its figure (not the bench line)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank, world, local = int(os.environ.get("RANK", 0)), int(os.environ.get("WORLD_SIZE", 1)), int(os.environ.get("LOCAL_RANK", 0))
@@ -609,10 +656,10 @@ def main():
     solo = lambda: torch.cuda.synchronize(local)
     _package()
     from silicon_violetto_b200 import engine as E
-    if args.only in ("lonasun", "leduvik", "pasovik"):
+    if args.only in ("lonasun", "leduvik", "pasovik", "sopetar"):
         peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
         sizes, files, work = {"lonasun": (LONASUN_SIZES, lonasun_files, lonasun_work), "leduvik": (LEDUVIK_SIZES, leduvik_files, leduvik_work),
-                              "pasovik": (PASOVIK_SIZES, pasovik_files, pasovik_work)}[args.only]
+                              "pasovik": (PASOVIK_SIZES, pasovik_files, pasovik_work), "sopetar": (SOPETAR_SIZES, sopetar_files, sopetar_work)}[args.only]
         figures = {}
         for n in sizes:
             c, w = work(n)
@@ -629,7 +676,7 @@ def main():
         elif args.only == "limite":
             print(json.dumps(limite_figure(E, local, args.ctx, min(args.steps, 30), [int(x) for x in args.limite_streams.split(",")], args.limite_keys, args.limite_drafter, args.limite_int8)))
         else:
-            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite', 'lonasun', 'leduvik' or 'pasovik'")
+            raise SystemExit(f"--only {args.only}: 'prefill', 'acceptance', 'limite', 'lonasun', 'leduvik', 'pasovik' or 'sopetar'")
         return
     total = args.warmup + args.steps + 6
     # The headline pass, on every rank: the int8 target with the chain drafter loaded (1 layer + fc + a head over 16 384 draft

@@ -351,7 +351,7 @@ __global__ void __launch_bounds__(threads_of(CONV_WARPS), CONV_WARPS == 16 ? 1 :
         for (uint32_t j = 0; j < NTOK; j++) {
             const float x = INT8 ? v[j] * scale : v[j] + bias;
             if (EPI == EPI_GLU_CLAMP) {
-                y[j] = clamped_glu(x, __shfl_xor_sync(0xffffffffu, x, 1), m.limit);
+                y[j] = clamped_glu<true>(x, __shfl_xor_sync(0xffffffffu, x, 1), m.limit);
             } else if (PAIRS) {
                 const float other = __shfl_xor_sync(0xffffffffu, x, 1);
                 const float gt = EPI == EPI_GLU ? x : x * inv[j], up = EPI == EPI_GLU ? other : other * inv[j];

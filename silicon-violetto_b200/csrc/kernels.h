@@ -39,10 +39,12 @@ struct QkvEpilogue {
 __device__ __forceinline__ float weight_of(const RowNorm& n, uint32_t i) { return (n.around_zero ? 1.0f : 0.0f) + bf16_to_f32(n.w[i]); }
 
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
+// FAST: by the hardware's exponential and quotient, whose errors are far below a rounding to bf16.
+template <bool FAST = false>
 __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
-    return g * sigmoid_of(1.702f * g) * (u + 1.0f);
+    return g * (FAST ? __fdividef(1.0f, 1.0f + __expf(-1.702f * g)) : sigmoid_of(1.702f * g)) * (u + 1.0f);
 }
 template <uint32_t V>
 __device__ __forceinline__ void weights_of(float (&x)[V], const RowNorm& n, uint32_t i) {

@@ -34,12 +34,15 @@ def lightning(dim, vdim, decay, mlp=None) -> dict:
 
 
 def config(width, vocab, layers, side=32, eps=1e-5) -> dict:
-    return {"architecture": "Pasovik", "width": width, "vocab": vocab, "layers": layers, "norm": {"eps": eps}, "token_side": {"dim": side}}
+    """side: each layer's span of the tokens' side embedding (None: there is none)."""
+    return {"architecture": "Pasovik", "width": width, "vocab": vocab, "layers": layers, "norm": {"eps": eps}, "token_side": side and {"dim": side}}
 
 
 def shapes(cfg: dict) -> dict:
-    d, side = cfg["width"], cfg["token_side"]["dim"]
-    out = {"embed": (cfg["vocab"], d), "side.embed": (cfg["vocab"], side * len(cfg["layers"]))}
+    d, side = cfg["width"], (cfg["token_side"] or {"dim": 0})["dim"]
+    out = {"embed": (cfg["vocab"], d)}
+    if side:
+        out["side.embed"] = (cfg["vocab"], side * len(cfg["layers"]))
     for i, lc in enumerate(cfg["layers"]):
         L, m, f = f"l{i}.", lc["mixer"], lc.get("mlp")
         mx, ml = L + "mix.", L + "mlp."
@@ -63,7 +66,8 @@ def shapes(cfg: dict) -> dict:
                 out.update({ml + p + "gate": (ff, d), ml + p + "up": (ff, d), ml + p + "down": (d, ff)})
             if f["kind"] == "moe":
                 out[ml + "router"] = (f["router"]["experts"], d)
-        out.update({L + "side.gate": (side, d), L + "side.proj": (d, side), L + "side.norm": (d,)})
+        if side:
+            out.update({L + "side.gate": (side, d), L + "side.proj": (d, side), L + "side.norm": (d,)})
     out["final.norm"] = (d,)
     out["head"] = (cfg["vocab"], d)
     return out
