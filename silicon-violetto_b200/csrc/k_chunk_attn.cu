@@ -253,8 +253,8 @@ constexpr uint32_t prefill_stages() { return DK + DV > 128 ? 2 : 3; }
 template <uint32_t DK, uint32_t DV>
 constexpr uint32_t prefill_smem() { return GROUPS * prefill_stages<DK, DV>() * CK * (DK + DV) * 2; }
 
-// grid (chunk tiles, query heads), 256 threads: warp w of a group has rows 16 w .. 16 w + 15 of the tile.
-template <uint32_t DK, uint32_t DV>
+// grid (chunk tiles, query heads), 256 threads: warp w of a group has rows 16 w .. 16 w + 15 of the tile. SLOPES: with a.slopes.
+template <uint32_t DK, uint32_t DV, bool SLOPES>
 __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(const ChunkedAttnArgs a) {
     pdl_start();
     extern __shared__ __align__(1024) uint8_t smem[];
@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
     __syncthreads();
     const Tiles<CK> walk(min(min(lows[0], lows[1]), min(lows[2], lows[3])), a.keep);
     const uint32_t b0 = grp, b1 = walk.count(max(max(ends[0], ends[1]), max(ends[2], ends[3])));
-    const float slope = a.slopes ? a.slopes[h] * LOG2E : 0.0f;
+    const float slope = SLOPES ? a.slopes[h] * LOG2E : 0.0f;
 
     const uint32_t* pages = a.kv.page_table + size_t(v[0].slot) * a.kv.max_pages;
     const uint16_t* K = static_cast<const uint16_t*>(a.kv.k);
@@ -355,7 +355,7 @@ __global__ void __launch_bounds__(GROUPS * WARPS * 32) chunk_prefill_kernel(cons
 #pragma unroll
                     for (int e = 0; e < 4; e++) s[j][e] = capped(s[j][e], cap, cap_inv);
             }
-            if (a.slopes) {
+            if (SLOPES) {
                 const bool tree = key0 + CK > first_min;
 #pragma unroll
                 for (uint32_t j = 0; j < 8; j++)
@@ -475,10 +475,10 @@ void launch(const ChunkedAttnArgs& a, uint32_t n, uint32_t n_ctiles, uint32_t sp
     configured.once([] {
         VLT_CUDA(cudaFuncSetAttribute(chunk_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(dsm)));
         VLT_CUDA(cudaFuncSetAttribute(chunk_decode_kernel<DK, DV>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
-        VLT_CUDA(cudaFuncSetAttribute(chunk_prefill_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(psm)));
+        for (auto f : {chunk_prefill_kernel<DK, DV, false>, chunk_prefill_kernel<DK, DV, true>}) VLT_CUDA(cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, int(psm)));
     });
     if (n_ctiles) {
-        launch_pdl(chunk_prefill_kernel<DK, DV>, dim3(n_ctiles, a.heads), GROUPS * WARPS * 32, psm, s, a);
+        launch_pdl(a.slopes ? chunk_prefill_kernel<DK, DV, true> : chunk_prefill_kernel<DK, DV, false>, dim3(n_ctiles, a.heads), GROUPS * WARPS * 32, psm, s, a);
         return;
     }
     const uint32_t groups = (a.heads / a.kv.n_kv + 7) / 8;
